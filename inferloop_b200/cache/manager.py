@@ -5,7 +5,9 @@ Layers are sorted into *page groups* by what they need (`PagedKVNeed`: kv heads,
 size, window).  A group has its own pool, its own block tables and one device tensor
 `[layers_in_group, 2, pages, kv_heads, page_size, head_dim]`; layer l's keys are
 `storage[l, 0]`, its values `storage[l, 1]` (a group whose values have another head size
-than its keys keeps them in a tensor of their own, `[layers, pages, kv_heads, page_size, v_head_dim]`).  Pages are taken when the step that first
+than its keys keeps them in a tensor of their own, `[layers, pages, kv_heads, page_size, v_head_dim]`).
+A layer may have a second set of pages beside its tokens' (`CacheNeeds.pooled`), in a group whose rows stand
+for `stride` tokens each: such a group needs a page per `page_size * stride` tokens.  Pages are taken when the step that first
 touches them is prepared, all groups or none (the reference grows pages per step,
 all-or-nothing: crates/engine/state/src/logical/reservation.rs:106-158), and given back
 when the request ends (crates/engine/runtime/src/pipeline/lifecycle.rs:242-251) or, in a
@@ -48,6 +50,7 @@ class LayerCache:
     writable: bool
     state: Dict[str, torch.Tensor] = field(default_factory=dict)
     instance: int = 0          # which run of a layer that runs several times (RunEntry.instance)
+    pooled: Optional["LayerCache"] = None      # the layer's second set of pages, whose rows stand for several tokens each
 
 
 @dataclass
@@ -72,8 +75,9 @@ class CacheManager:
                  device: Optional[torch.device] = None,
                  run_order: Optional[Sequence[RunEntry]] = None,
                  model_slots: Sequence[SlotStateNeed] = ()) -> None:
-        """`num_pages`: one number for every page group, or one number per group in the
-        order of :meth:`group_needs` (a group that reads a window needs fewer).
+        """`num_pages`: one number for every page group (pages of tokens: a group whose rows stand for
+        several tokens gets as many pages as the rows of those tokens need), or one number per group in
+        the order of :meth:`group_needs` (a group that reads a window needs fewer).
         `model_slots`: state per request that belongs to no layer (the embedding's), found
         under :meth:`model_state`."""
         if page_size <= 0:
@@ -92,24 +96,24 @@ class CacheManager:
         self._index_in_group: Dict[int, int] = {}
         found: List[Tuple[PagedKVNeed, List[int]]] = []
         for owner in owners:
-            need = self.layer_needs[owner[0]].paged
-            if need is None:
-                continue
-            for gi, (n, layers) in enumerate(found):
-                if n == need:
-                    break
-            else:
-                gi = len(found)
-                found.append((need, []))
-            self._group_of_layer[owner] = gi
-            self._index_in_group[owner] = len(found[gi][1])
-            found[gi][1].append(owner[0])
+            for key, need in ((owner, self.layer_needs[owner[0]].paged), (owner + ("pooled",), self.layer_needs[owner[0]].pooled)):
+                if need is None:
+                    continue
+                for gi, (n, layers) in enumerate(found):
+                    if n == need:
+                        break
+                else:
+                    gi = len(found)
+                    found.append((need, []))
+                self._group_of_layer[key] = gi
+                self._index_in_group[key] = len(found[gi][1])
+                found[gi][1].append(owner[0])
         if isinstance(num_pages, (list, tuple)):
             if len(num_pages) != len(found):
                 raise ValueError(f"{len(num_pages)} pool sizes for {len(found)} page groups")
             pages_of = [int(n) for n in num_pages]
-        else:
-            pages_of = [int(num_pages)] * len(found)
+        else:      # (a group with a row per n tokens: as many tokens, and for every request a page that it does not fill)
+            pages_of = [int(num_pages) if n.stride == 1 else -(-int(num_pages) // n.stride) + max(int(max_requests), 0) for n, _ in found]
         if any(n <= 0 for n in pages_of):
             raise ValueError("a page pool needs at least one page")
         if max_requests <= 0:
@@ -119,7 +123,8 @@ class CacheManager:
         windows = (ctypes.c_int * max(1, len(found)))(*[(-1 if n.window is None else int(n.window)) for n, _ in found])
         h = ctypes.c_void_p()
         sizes = (ctypes.c_int * max(1, len(found)))(*pages_of)
-        rc = self._lib.ilb_ledger_new(len(found), windows, sizes, self.page_size, int(max_requests), ctypes.byref(h))
+        strides = (ctypes.c_int * max(1, len(found)))(*[int(n.stride) for n, _ in found])
+        rc = self._lib.ilb_ledger_new(len(found), windows, strides, sizes, self.page_size, int(max_requests), ctypes.byref(h))
         if rc:
             raise_for(rc)
         self._h = h
@@ -164,15 +169,15 @@ class CacheManager:
         order = list(run_order) if run_order is not None else [RunEntry(i, i) for i in range(len(needs))]
         found: List[Tuple[PagedKVNeed, List[int]]] = []
         for layer, _ in sorted({(e.cache_of, e.instance) for e in order}):
-            need = needs[layer].paged
-            if need is None:
-                continue
-            for n, layers in found:
-                if n == need:
-                    layers.append(layer)
-                    break
-            else:
-                found.append((need, [layer]))
+            for need in (needs[layer].paged, needs[layer].pooled):
+                if need is None:
+                    continue
+                for n, layers in found:
+                    if n == need:
+                        layers.append(layer)
+                        break
+                else:
+                    found.append((need, [layer]))
         return found
 
     @property
@@ -279,19 +284,27 @@ class CacheManager:
 
     def layer_cache(self, entry: RunEntry) -> LayerCache:
         owner = (entry.cache_of, entry.instance)
-        gi = self._group_of_layer.get(owner)
-        k = v = None
-        if gi is not None and self.groups[gi].storage is not None:
-            g = self.groups[gi]
-            s = g.storage[self._index_in_group[owner]]
-            k = s[0]
-            if g.storage_v is not None:
-                v = g.storage_v[self._index_in_group[owner]]
-            elif g.need.value_dim == g.need.head_dim:
-                v = s[1]
+
+        def pages(key):
+            gi, k, v = self._group_of_layer.get(key), None, None
+            if gi is not None and self.groups[gi].storage is not None:
+                g = self.groups[gi]
+                s = g.storage[self._index_in_group[key]]
+                k = s[0]
+                if g.storage_v is not None:
+                    v = g.storage_v[self._index_in_group[key]]
+                elif g.need.value_dim == g.need.head_dim:
+                    v = s[1]
+            return gi, k, v
+
+        gi, k, v = pages(owner)
+        pooled = None
+        if owner + ("pooled",) in self._group_of_layer:
+            pg, pk, pv = pages(owner + ("pooled",))
+            pooled = LayerCache(entry.cache_of, pg, self.page_size, pk, pv, entry.writes_cache, {}, entry.instance)
         state = {need.name: self._slot_state[(owner, need.name)]
                  for need in self._slot_needs.get(owner, ()) if (owner, need.name) in self._slot_state}
-        return LayerCache(entry.cache_of, gi, self.page_size, k, v, entry.writes_cache, state, entry.instance)
+        return LayerCache(entry.cache_of, gi, self.page_size, k, v, entry.writes_cache, state, entry.instance, pooled)
 
     def model_state(self) -> Dict[str, torch.Tensor]:
         """The state per request that belongs to no layer: name -> [slots, *shape]."""
@@ -316,7 +329,7 @@ class CacheManager:
             "live_requests": len(self._live),
             "groups": [{
                 "index": g.index, "layers": list(g.layers), "kv_heads": g.need.kv_heads,
-                "head_dim": g.need.head_dim, "v_head_dim": g.need.value_dim, "window": g.need.window,
+                "head_dim": g.need.head_dim, "v_head_dim": g.need.value_dim, "window": g.need.window, "stride": g.need.stride,
                 "total": g.pool.num_pages, "free": g.pool.num_free,
                 "active": g.pool.num_pages - g.pool.num_free,
                 "allocations": g.pool.allocations, "reuses": g.pool.reuses,

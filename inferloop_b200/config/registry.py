@@ -103,11 +103,13 @@ def default_registry() -> ArchitectureRegistry:
         from ..models.mamevik import ARCHITECTURE as MAMEVIK
         from ..models.dalavik import ARCHITECTURE as DALAVIK
         from ..models.zebivik import ARCHITECTURE as ZEBIVIK
+        from ..models.sapanex import ARCHITECTURE as SAPANEX
         _DEFAULT.register(ARCHITECTURE)
         _DEFAULT.register(SUFOLIX)
         _DEFAULT.register(MAMEVIK)
         _DEFAULT.register(DALAVIK)
         _DEFAULT.register(ZEBIVIK)
+        _DEFAULT.register(SAPANEX)
     return _DEFAULT
 
 

@@ -10,6 +10,10 @@
 // Keys and queries have head size d, values and the output dv (the V cache is
 // [pages, nkv, page_size, dv]).
 //
+// With `pool` = P > 0 (and a window) the token also sees, in the same softmax, one row for each block of P tokens
+// that lies wholly before its window: block b (positions bP .. bP + P - 1) is row b of a second set of pages
+// (`pk_cache`, `pv_cache`, `p_table`), seen if b < floor(lo / P).
+//
 // With `sink` (one learned logit per query head) the softmax's denominator also holds exp(sink):
 // a key that is always seen, has no value, and whose logit is taken as it is (no scale).
 //
@@ -31,7 +35,9 @@ paged_attention_simple_kernel(const TQ* __restrict__ q, TQ* __restrict__ out,
                               const int* __restrict__ positions, const int* __restrict__ seq_of_token,
                               const int* __restrict__ block_table, int max_blocks, int page_size,
                               int num_pages, int window, float scale, int nq, int nkv, int d, int dv,
-                              int q_stride, int out_stride, const float* __restrict__ sink) {
+                              int q_stride, int out_stride, const float* __restrict__ sink,
+                              const TC* __restrict__ pk_cache, const TC* __restrict__ pv_cache, const int* __restrict__ p_table,
+                              int p_num_pages, int pool) {
   ilb::pdl_launch_dependents();
   ilb::pdl_wait();
   __shared__ float qs[kMaxHeadDim];
@@ -44,6 +50,19 @@ paged_attention_simple_kernel(const TQ* __restrict__ q, TQ* __restrict__ out,
   const int seq = seq_of_token[t];
   const int lo = (window > 0 && p + 1 > window) ? p + 1 - window : 0;
   const int* table = block_table + (size_t)seq * max_blocks;
+  const int* ptable = p_table + (size_t)seq * max_blocks;      // (not read without pooled rows)
+  const int n_pooled = pool > 0 ? lo / pool : 0;
+  // key j of the walk: the pooled rows first, then the window's tokens; false: its page is not held
+  auto locate = [&](int j, const TC*& kr, const TC*& vr) {
+    const bool pooled = j < n_pooled;
+    const int row = pooled ? j : lo + j - n_pooled;
+    const int page = (pooled ? ptable : table)[row / page_size];
+    if (page < 0 || page >= (pooled ? p_num_pages : num_pages)) return false;
+    const size_t at = ((size_t)page * nkv + kvh) * page_size + row % page_size;
+    kr = (pooled ? pk_cache : k_cache) + at * d;
+    vr = (pooled ? pv_cache : v_cache) + at * dv;
+    return true;
+  };
 
   for (int i = threadIdx.x; i < d; i += blockDim.x)
     qs[i] = to_float(q[(size_t)t * q_stride + (size_t)h * d + i]);
@@ -54,16 +73,14 @@ paged_attention_simple_kernel(const TQ* __restrict__ q, TQ* __restrict__ out,
 #pragma unroll
   for (int i = 0; i < R; ++i) acc[i] = 0.f;
   float m = -INFINITY, l = 0.f;
-  const int n_keys = p - lo + 1;
+  const int n_keys = n_pooled + p - lo + 1;
   const int n_tiles = (n_keys + 31) / 32;
   for (int tile = warp; tile < n_tiles; tile += kWarps) {
-    const int j = lo + tile * 32 + lane;
-    const bool valid = j <= p;
+    const int j = tile * 32 + lane;
     float s = -INFINITY;
-    if (valid) {
-      const int page = table[j / page_size];
-      if (page >= 0 && page < num_pages) {
-        const TC* kr = k_cache + (((size_t)page * nkv + kvh) * page_size + (j % page_size)) * d;
+    if (j < n_keys) {
+      const TC *kr, *vr;
+      if (locate(j, kr, vr)) {
         float dot = 0.f;
         for (int i = 0; i < d; ++i) dot = fmaf(qs[i], to_float(kr[i]), dot);
         s = dot * scale;
@@ -76,13 +93,11 @@ paged_attention_simple_kernel(const TQ* __restrict__ q, TQ* __restrict__ out,
 #pragma unroll
     for (int i = 0; i < R; ++i) acc[i] *= corr;
     m = m_new;
-    const int count = min(32, p - (lo + tile * 32) + 1);
+    const int count = min(32, n_keys - tile * 32);
     for (int jj = 0; jj < count; ++jj) {
       const float w = __shfl_sync(0xffffffffu, pj, jj);
-      const int key = lo + tile * 32 + jj;
-      const int page = table[key / page_size];
-      if (page < 0 || page >= num_pages) continue;
-      const TC* vr = v_cache + (((size_t)page * nkv + kvh) * page_size + (key % page_size)) * dv;
+      const TC *kr, *vr;
+      if (!locate(tile * 32 + jj, kr, vr)) continue;
 #pragma unroll
       for (int i = 0; i < R; ++i) {
         const int c = lane + 32 * i;
@@ -119,13 +134,16 @@ ILB_EXPORT int ilb_paged_attention_simple(
     const void* q, void* out, int dtype, const void* k_cache, const void* v_cache, int cache_dtype,
     const int* positions, const int* seq_of_token, const int* block_table, int max_blocks,
     int page_size, int num_pages, int window, float scale, int n_tokens, int nq, int nkv, int d, int dv,
-    int q_stride, int out_stride, const float* sink, cudaStream_t stream) {
+    int q_stride, int out_stride, const float* sink, const void* pk_cache, const void* pv_cache, const int* p_table,
+    int p_num_pages, int pool, cudaStream_t stream) {
   ILB_REQUIRE(n_tokens >= 0 && nq > 0 && nkv > 0 && d > 0, "attention: bad sizes");
   ILB_REQUIRE(nq % nkv == 0, "attention: %d query heads are not a multiple of %d kv heads", nq, nkv);
   ILB_REQUIRE(dv > 0 && d <= kMaxHeadDim && dv <= kMaxHeadDim, "attention: head size %d / %d exceeds %d", d, dv, kMaxHeadDim);
   ILB_REQUIRE(nq <= 65535, "attention: too many heads");
   ILB_REQUIRE(page_size > 0 && max_blocks > 0 && num_pages > 0, "attention: bad cache geometry");
   ILB_REQUIRE(window >= 0, "attention: negative window");
+  ILB_REQUIRE(pool == 0 || (pool > 0 && window > 0 && pk_cache != nullptr && pv_cache != nullptr && p_table != nullptr && p_num_pages > 0),
+              "attention: pooled blocks need a window and pages of their own");
   ILB_REQUIRE(q_stride >= nq * d && out_stride >= nq * dv, "attention: strides too small");
   if (n_tokens == 0) return 0;
   dim3 grid(n_tokens, nq);
@@ -133,7 +151,7 @@ ILB_EXPORT int ilb_paged_attention_simple(
   ilb::launch(paged_attention_simple_kernel<TQ, TC>, dim3(grid), dim3(kWarps * 32), 0, stream,                      \
       (const TQ*)q, (TQ*)out, (const TC*)k_cache, (const TC*)v_cache, positions, seq_of_token, \
       block_table, max_blocks, page_size, num_pages, window, scale, nq, nkv, d, dv, q_stride,  \
-      out_stride, sink)
+      out_stride, sink, (const TC*)pk_cache, (const TC*)pv_cache, p_table, p_num_pages, pool)
   if (dtype == kF32 && cache_dtype == kF32) ILB_LAUNCH(float, float);
   else if (dtype == kBF16 && cache_dtype == kBF16) ILB_LAUNCH(__nv_bfloat16, __nv_bfloat16);
   else if (dtype == kF32 && cache_dtype == kBF16) ILB_LAUNCH(float, __nv_bfloat16);

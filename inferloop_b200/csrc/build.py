@@ -46,6 +46,7 @@ MODULES: Dict[str, List[str]] = {
     "sublayer_norm": [],
     "attention_mix": [],
     "recurrent": [],
+    "delta": [],
 }
 
 _LOCK = threading.Lock()

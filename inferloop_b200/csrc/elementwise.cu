@@ -246,10 +246,11 @@ ILB_EXPORT int ilb_gather_rows(const float* x, const int* idx, float* out, int n
 
 // ---------------------------------------------------------------- rotation table
 // cos/sin of pos * inv_freq[i], angle and functions evaluated in 64-bit and rounded once
-// to 32-bit, so the table is as good as a 32-bit number can be at any position.
+// to 32-bit, so the table is as good as a 32-bit number can be at any position.  Both are
+// multiplied by `stretch` (1: the plain rotation).
 __global__ void rope_table_kernel(const int* __restrict__ positions,
                                   const double* __restrict__ inv_freq,
-                                  float2* __restrict__ table, int n_tokens, int half) {
+                                  float2* __restrict__ table, int n_tokens, int half, double stretch) {
   ilb::pdl_launch_dependents();
   ilb::pdl_wait();
   const int i = blockIdx.x * blockDim.x + threadIdx.x;
@@ -258,16 +259,71 @@ __global__ void rope_table_kernel(const int* __restrict__ positions,
   const double angle = (double)positions[t] * inv_freq[f];
   double s, c;
   sincos(angle, &s, &c);
-  table[i] = make_float2((float)c, (float)s);
+  table[i] = make_float2((float)(c * stretch), (float)(s * stretch));
 }
 
 ILB_EXPORT int ilb_rope_table(const int* positions, const double* inv_freq, float* table,
-                              int n_tokens, int half, cudaStream_t stream) {
+                              int n_tokens, int half, double stretch, cudaStream_t stream) {
   ILB_REQUIRE(n_tokens >= 0 && half > 0, "rope_table: bad sizes");
   if (n_tokens == 0) return 0;
   const int n = n_tokens * half;
-  ilb::launch(rope_table_kernel, dim3((n + 127) / 128), dim3(128), 0, stream, positions, inv_freq, (float2*)table, n_tokens, half);
+  ilb::launch(rope_table_kernel, dim3((n + 127) / 128), dim3(128), 0, stream, positions, inv_freq, (float2*)table, n_tokens, half, stretch);
   return check_launch("rope_table");
+}
+
+// ---------------------------------------------------------------- out = f(x), element by element
+// f = tanh, or relu squared; x and out in the same type with row strides of their own (out may be x).
+enum : int { kActTanh = 0, kActRelu2 = 1 };
+__device__ __forceinline__ float act_of(float x, int act) {
+  if (act == kActTanh) return tanhf(x);
+  const float r = fmaxf(x, 0.f);
+  return r * r;
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+act_rows_kernel(const T* x, int ldx, T* out, int ldo, int rows, int width, int act) {
+  ilb::pdl_launch_dependents();
+  ilb::pdl_wait();
+  const size_t n = (size_t)rows * width;
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
+    const size_t r = i / width, c = i % width;
+    out[r * ldo + c] = from_float<T>(act_of(to_float(x[r * ldx + c]), act));
+  }
+}
+
+// Eight bfloat16 elements a thread and access.
+__global__ void __launch_bounds__(256)
+act_rows_vec_kernel(const __nv_bfloat16* x, int ldx, __nv_bfloat16* out, int ldo, int rows, int width8, int act) {
+  ilb::pdl_launch_dependents();
+  ilb::pdl_wait();
+  const size_t n = (size_t)rows * width8;
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
+    const size_t r = i / width8, c = (i % width8) * 8;
+    uint4 v = *reinterpret_cast<const uint4*>(x + r * ldx + c);
+    uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const __nv_bfloat162 p = __floats2bfloat162_rn(act_of(__uint_as_float(w[j] << 16), act), act_of(__uint_as_float(w[j] & 0xFFFF0000u), act));
+      w[j] = *reinterpret_cast<const uint32_t*>(&p);
+    }
+    *reinterpret_cast<uint4*>(out + r * ldo + c) = make_uint4(w[0], w[1], w[2], w[3]);
+  }
+}
+
+ILB_EXPORT int ilb_act_rows(const void* x, int ldx, void* out, int ldo, int dtype, int rows, int width, int act, cudaStream_t stream) {
+  ILB_REQUIRE(rows >= 0 && width > 0 && ldx >= width && ldo >= width, "act_rows: bad sizes");
+  ILB_REQUIRE(act == kActTanh || act == kActRelu2, "act_rows: unknown function %d", act);
+  if (rows == 0) return 0;
+  const bool vec = dtype == kBF16 && width % 8 == 0 && ldx % 8 == 0 && ldo % 8 == 0 && ((uintptr_t)x % 16 == 0) && ((uintptr_t)out % 16 == 0);
+  const size_t n = (size_t)rows * (vec ? width / 8 : width);
+  const int blocks = (int)((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16);
+  if (vec) ilb::launch(act_rows_vec_kernel, dim3(blocks), dim3(256), 0, stream, (const __nv_bfloat16*)x, ldx, (__nv_bfloat16*)out, ldo, rows, width / 8, act);
+  else if (dtype == kF32) ilb::launch(act_rows_kernel<float>, dim3(blocks), dim3(256), 0, stream, (const float*)x, ldx, (float*)out, ldo, rows, width, act);
+  else if (dtype == kBF16)
+    ilb::launch(act_rows_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, (const __nv_bfloat16*)x, ldx, (__nv_bfloat16*)out, ldo, rows, width, act);
+  else return fail("act_rows: unknown dtype %d", dtype);
+  return check_launch("act_rows");
 }
 
 // ---------------------------------------------------------------- x += y (32-bit)

@@ -345,12 +345,24 @@ def latent_write_rot(proj: torch.Tensor, col0: int, rank: int, tail: int, rot: i
 
 
 # --------------------------------------------------------------------------- norm on a sublayer's output
-def cast_zero(x: torch.Tensor, xc: torch.Tensor, y: torch.Tensor) -> None:
-    """xc = x in xc's dtype; y = 0 (x and y 32-bit, all of one shape)."""
+def cast_zero(x: torch.Tensor, xc: torch.Tensor, y: torch.Tensor, keep: float = 0.0) -> None:
+    """xc = x in xc's dtype; y = keep * x (keep 0: zero); x and y 32-bit, all of one shape."""
     _need(x, "cast_zero x", torch.float32); _need(xc, "cast_zero out"); _need(y, "cast_zero y", torch.float32)
     if xc.shape != x.shape or y.shape != x.shape:
         raise KernelError("cast_zero: shapes do not agree")
-    _call("sublayer_norm", "ilb_cast_zero", _ptr(x), _ptr(xc), _i(_code(xc)), _ptr(y), ctypes.c_longlong(x.numel()), _stream(x))
+    _call("sublayer_norm", "ilb_cast_zero", _ptr(x), _ptr(xc), _i(_code(xc)), _ptr(y), ctypes.c_longlong(x.numel()), _f(keep),
+          _stream(x))
+
+
+def sum_norm(y: torch.Tensor, weight: torch.Tensor, eps: float, keep: float, x: Optional[torch.Tensor], xc: torch.Tensor) -> None:
+    """n = y / sqrt(mean(y^2) + eps) * weight; x = n (if given), xc = n in xc's dtype, y = keep * n; y and x 32-bit."""
+    _need(y, "sum_norm y", torch.float32); _need(weight, "sum_norm weight", torch.float32); _need(x, "sum_norm x", torch.float32)
+    _need(xc, "sum_norm out")
+    rows, width = y.shape
+    if weight.numel() != width or xc.shape != y.shape or (x is not None and x.shape != y.shape):
+        raise KernelError("sum_norm: shapes do not agree")
+    _call("sublayer_norm", "ilb_sum_norm", _ptr(y), _ptr(weight), _f(eps), _f(keep), _i(rows), _i(width), _ptr(x), _ptr(xc), _i(_code(xc)),
+          _stream(y))
 
 
 def group_norm_add(y: torch.Tensor, weight: torch.Tensor, eps: float, groups: int, x: Optional[torch.Tensor] = None,
@@ -443,9 +455,11 @@ def silu_rows(x: torch.Tensor, width: int, out: torch.Tensor) -> None:
     _call("recurrent", "ilb_silu_rows", _ptr(x), _i(_code(x)), _i(x.stride(0)), _ptr(out), _i(x.shape[0]), _i(width), _stream(out))
 
 
-def rms_gate(y: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor, scale: float = 1.0) -> None:
-    """out = y / sqrt(mean(y^2) + eps) * weight * sigmoid(gate) * scale over whole rows; y 32-bit, gate [T, >= width]
-    (its first `width` columns) and out [T, width] (rows of any stride) in the compute dtype."""
+def rms_gate(y: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor, scale: float = 1.0,
+             groups: int = 1) -> None:
+    """out = y / sqrt(mean(y^2) + eps) * weight * sigmoid(gate) * scale over whole rows, or over each of `groups` equal parts
+    of them; y 32-bit, gate [T, >= width] (its first `width` columns) and out [T, width] (rows of any stride) in the compute
+    dtype."""
     _need(y, "rms_gate y", torch.float32); _need(gate, "rms_gate gate", contiguous=False); _need(weight, "rms_gate weight", torch.float32)
     _need(out, "rms_gate out", gate.dtype, contiguous=False)
     T, width = y.shape
@@ -453,7 +467,36 @@ def rms_gate(y: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: flo
             or out.stride(1) != 1:
         raise KernelError("rms_gate: shapes do not agree")
     _call("recurrent", "ilb_rms_gate", _ptr(y), _ptr(gate), _i(_code(gate)), _i(gate.stride(0)), _ptr(weight), _ptr(out), _i(out.stride(0)),
-          _i(T), _i(width), _f(eps), _f(scale), _stream(out))
+          _i(T), _i(width), _i(groups), _f(eps), _f(scale), _stream(out))
+
+
+ACTIVATIONS = {"tanh": 0, "relu2": 1}
+
+
+def act_rows(x: torch.Tensor, activation: str, out: torch.Tensor) -> None:
+    """out = tanh(x) or relu(x)^2, element by element; x and out [rows, width] of one dtype, rows of any stride (out may be x)."""
+    _need(x, "act_rows x", contiguous=False); _need(out, "act_rows out", x.dtype, contiguous=False)
+    if x.shape != out.shape or x.stride(1) != 1 or out.stride(1) != 1:
+        raise KernelError("act_rows: shapes do not agree")
+    _call("elementwise", "ilb_act_rows", _ptr(x), _i(x.stride(0)), _ptr(out), _i(out.stride(0)), _i(_code(x)), _i(x.shape[0]), _i(x.shape[1]),
+          _i(ACTIVATIONS[activation]), _stream(out))
+
+
+# --------------------------------------------------------------------------- generalized delta rule
+def delta_scan(proj: torch.Tensor, col_r: int, col_k: int, col_v: int, col_a: int, low: torch.Tensor, w0: torch.Tensor, ab: torch.Tensor,
+               log_decay: float, unit_eps: float, state: torch.Tensor, y: torch.Tensor, step, heads: int, d: int, dv: int) -> None:
+    """S_t = diag(w) S_{t-1} - (g u)(u^T S_{t-1}) + k v^T, y_t = S_t^T r per head over the step's tokens, from and to state
+    [slots, heads, d, dv] (see delta.cu); r, k, a at columns of `proj` (heads * d each), v (heads * dv); `low` [T, heads * d]
+    32-bit: what w0 joins under the decay's sigmoid."""
+    _need(proj, "delta projection", contiguous=False); _need(low, "delta decay input", torch.float32); _need(state, "delta state", torch.float32)
+    _need(y, "delta y", torch.float32); _need(w0, "delta w0", torch.float32); _need(ab, "delta a bias", torch.float32)
+    T = proj.shape[0]
+    if proj.stride(1) != 1 or tuple(low.shape) != (T, heads * d) or tuple(y.shape) != (T, heads * dv) or w0.numel() != heads * d \
+            or ab.numel() != heads * d or tuple(state.shape[1:]) != (heads, d, dv):
+        raise KernelError("delta_scan: shapes do not agree")
+    _call("delta", "ilb_delta_scan", _ptr(proj), _i(_code(proj)), _i(proj.stride(0)), _i(col_r), _i(col_k), _i(col_v), _i(col_a), _ptr(low),
+          _ptr(w0), _ptr(ab), _f(log_decay), _f(unit_eps), _ptr(state), _ptr(y), _ptr(step.cu_q), _ptr(step.slots), _i(step.n_seqs),
+          _i(heads), _i(d), _i(dv), _stream(y))
 
 
 def head_gate(o: torch.Tensor, gate: torch.Tensor, heads: int, scale: float = 1.0, out: Optional[torch.Tensor] = None) -> None:
@@ -657,15 +700,15 @@ def gemm_simt_grouped(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, block
           _i(K), _i(K), _i(N), _ptr(block_group), ctypes.c_longlong(N * K), _stream(out))
 
 
-def rope_table(positions: torch.Tensor, inv_freq: torch.Tensor, out: torch.Tensor) -> None:
-    """out[t, i] = (cos, sin)(positions[t] * inv_freq[i]); inv_freq is 64-bit."""
+def rope_table(positions: torch.Tensor, inv_freq: torch.Tensor, out: torch.Tensor, stretch: float = 1.0) -> None:
+    """out[t, i] = stretch * (cos, sin)(positions[t] * inv_freq[i]); inv_freq is 64-bit."""
     _need(positions, "rope positions", torch.int32); _need(inv_freq, "rope inv_freq", torch.float64)
     _need(out, "rope table", torch.float32)
     T, half = positions.numel(), inv_freq.numel()
     if tuple(out.shape) != (T, half, 2):
         raise KernelError("rope_table: out must be [T, rotary_dim/2, 2]")
     _call("elementwise", "ilb_rope_table", _ptr(positions), _ptr(inv_freq), _ptr(out), _i(T),
-          _i(half), _stream(out))
+          _i(half), ctypes.c_double(float(stretch)), _stream(out))
 
 
 def add_inplace(x: torch.Tensor, y: torch.Tensor) -> None:
@@ -754,11 +797,65 @@ def qk_norm_rope_cache(qkv: torch.Tensor, q_out: torch.Tensor, q_weight: Optiona
           _stream(qkv))
 
 
+def rows_norm_rope_cache(qkv: torch.Tensor, q_out: torch.Tensor, q_weight: torch.Tensor, k_weight: torch.Tensor, eps: float,
+                         rope: Optional[torch.Tensor], rotary_dim: int, v_rope: Optional[torch.Tensor], step, block_table: torch.Tensor,
+                         k_cache: Optional[torch.Tensor], v_cache: Optional[torch.Tensor], nq: int, nkv: int, d: int, dv: int) -> None:
+    """The input stage of an attention that norms queries and keys over all their heads' elements at once: q -> q_out,
+    k and v -> cache pages, the first `rotary_dim` elements of q and k heads turned by `rope` [T, rotary_dim / 2, 2], values
+    turned over their whole size by `v_rope` [T, dv / 2, 2] (either table may be None); see qk_norm_rope.cu."""
+    _need(qkv, "qkv", contiguous=False); _need(q_out, "q_out", qkv.dtype); _need(q_weight, "q norm weight", torch.float32)
+    _need(k_weight, "k norm weight", torch.float32); _need(rope, "rope table", torch.float32); _need(v_rope, "value rope table", torch.float32)
+    _need(k_cache, "k cache", qkv.dtype); _need(v_cache, "v cache", qkv.dtype); _need(block_table, "block table", torch.int32)
+    T = qkv.shape[0]
+    if qkv.stride(1) != 1 or qkv.shape[1] < (nq + nkv) * d + nkv * dv or q_weight.numel() != nq * d or k_weight.numel() != nkv * d \
+            or (rope is not None and tuple(rope.shape) != (T, rotary_dim // 2, 2)) or (v_rope is not None and tuple(v_rope.shape) != (T, dv // 2, 2)):
+        raise KernelError("rows_norm_rope_cache: shapes do not agree")
+    page_size = num_pages = 0
+    if k_cache is not None:
+        num_pages, page_size = k_cache.shape[0], k_cache.shape[2]
+        if tuple(k_cache.shape[1:]) != (nkv, page_size, d) or tuple(v_cache.shape) != (num_pages, nkv, page_size, dv):
+            raise KernelError("rows_norm_rope_cache: cache shapes do not match the heads")
+    _call("qk_norm_rope", "ilb_rows_norm_rope_cache", _ptr(qkv), _ptr(q_out), _i(_code(qkv)), _ptr(q_weight), _ptr(k_weight), _f(eps), _ptr(rope),
+          _i(rotary_dim), _ptr(v_rope), _ptr(step.positions), _ptr(step.seq_of_token), _ptr(block_table), _i(block_table.shape[1]), _i(page_size),
+          _i(num_pages), _ptr(k_cache), _ptr(v_cache), _i(T), _i(nq), _i(nkv), _i(d), _i(dv), _i(qkv.stride(0)), _i(q_out.shape[1]), _stream(qkv))
+
+
+class PooledRows:
+    """What attention over a window sees before it: the means of aligned blocks of `pool` tokens, in pages of their own
+    (`k`, `v` [pages, nkv, page_size, d / dv], block table `table`)."""
+
+    def __init__(self, pool: int, k: torch.Tensor, v: torch.Tensor, table: torch.Tensor) -> None:
+        self.pool, self.k, self.v, self.table = int(pool), k, v, table
+
+
+def pool_means(k_cache: torch.Tensor, v_cache: torch.Tensor, pooled: PooledRows, step, block_table: torch.Tensor) -> None:
+    """The blocks of `pooled.pool` positions that the step's tokens complete: their rows of the pooled pages become the means
+    of the block's cached keys and values."""
+    _need(k_cache, "k cache"); _need(v_cache, "v cache", k_cache.dtype); _need(pooled.k, "pooled keys", k_cache.dtype)
+    _need(pooled.v, "pooled values", k_cache.dtype); _need(block_table, "block table", torch.int32); _need(pooled.table, "pooled block table", torch.int32)
+    num_pages, nkv, page_size, d = k_cache.shape
+    dv = v_cache.shape[3]
+    if tuple(pooled.k.shape[1:]) != (nkv, page_size, d) or tuple(pooled.v.shape[1:]) != (nkv, page_size, dv) or pooled.table.shape != block_table.shape:
+        raise KernelError("pool_means: the pooled pages do not match the cache")
+    _call("qk_norm_rope", "ilb_pool_means", _ptr(k_cache), _ptr(v_cache), _ptr(pooled.k), _ptr(pooled.v), _i(_code(k_cache)), _ptr(step.positions),
+          _ptr(step.seq_of_token), _ptr(block_table), _ptr(pooled.table), _i(block_table.shape[1]), _i(page_size), _i(num_pages),
+          _i(pooled.k.shape[0]), _i(pooled.pool), _i(step.n_tokens), _i(nkv), _i(d), _i(dv), _stream(k_cache))
+
+
+def turn_back(o: torch.Tensor, table: torch.Tensor, heads: int) -> None:
+    """o[t, h] in pairs (i, i + dv / 2) turned by minus the angle of table[t, i], in place; o [T, heads * dv]."""
+    _need(o, "turn_back o"); _need(table, "turn_back table", torch.float32)
+    T, dv = o.shape[0], o.shape[1] // heads
+    if o.shape[1] != heads * dv or tuple(table.shape) != (T, dv // 2, 2):
+        raise KernelError("turn_back: shapes do not agree")
+    _call("qk_norm_rope", "ilb_turn_back", _ptr(o), _i(_code(o)), _ptr(table), _i(T), _i(heads), _i(dv), _stream(o))
+
+
 def paged_attention_simple(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor,
                            v_cache: torch.Tensor, positions: torch.Tensor,
                            seq_of_token: torch.Tensor, block_table: torch.Tensor, window: int,
                            scale: float, nq: int, nkv: int, d: int, dv: Optional[int] = None,
-                           sink: Optional[torch.Tensor] = None) -> None:
+                           sink: Optional[torch.Tensor] = None, pooled: Optional[PooledRows] = None) -> None:
     dv = d if dv is None else int(dv)
     _need(q, "attention q"); _need(out, "attention out", q.dtype); _need(sink, "attention sink", torch.float32)
     if sink is not None and sink.numel() != nq:
@@ -769,11 +866,18 @@ def paged_attention_simple(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Te
     num_pages, nkv_c, page_size, d_c = k_cache.shape
     if (nkv_c, d_c) != (nkv, d) or tuple(v_cache.shape) != (num_pages, nkv, page_size, dv):
         raise KernelError("attention: cache shape does not match the heads")
+    if pooled is not None:
+        _need(pooled.k, "pooled keys", k_cache.dtype); _need(pooled.v, "pooled values", k_cache.dtype); _need(pooled.table, "pooled block table", torch.int32)
+        if not window or tuple(pooled.k.shape[1:]) != (nkv, page_size, d) or tuple(pooled.v.shape) != (pooled.k.shape[0], nkv, page_size, dv) \
+                or pooled.table.shape != block_table.shape:
+            raise KernelError("attention: pooled rows need a window, and pages like the cache's")
     _call("attention_simple", "ilb_paged_attention_simple", _ptr(q), _ptr(out), _i(_code(q)),
           _ptr(k_cache), _ptr(v_cache), _i(_code(k_cache)), _ptr(positions), _ptr(seq_of_token),
           _ptr(block_table), _i(block_table.shape[1]), _i(page_size), _i(num_pages),
           _i(window or 0), _f(scale), _i(q.shape[0]), _i(nq), _i(nkv), _i(d), _i(dv), _i(q.shape[1]),
-          _i(out.shape[1]), _ptr(sink), _stream(q))
+          _i(out.shape[1]), _ptr(sink), _ptr(None if pooled is None else pooled.k), _ptr(None if pooled is None else pooled.v),
+          _ptr(None if pooled is None else pooled.table), _i(0 if pooled is None else pooled.k.shape[0]),
+          _i(0 if pooled is None else pooled.pool), _stream(q))
 
 
 def attention_mixed_heads(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, step,
@@ -1172,18 +1276,19 @@ def attention_decode_fused(qkv, out, q_weight, k_weight, eps, rope_table, k_cach
 def attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
               step, block_table: torch.Tensor, window: int, scale: float, nq: int, nkv: int,
               d: int, workspace=None, decode_chunk: int = DECODE_CHUNK_MIN, dv: Optional[int] = None,
-              sink: Optional[torch.Tensor] = None) -> None:
+              sink: Optional[torch.Tensor] = None, pooled: Optional[PooledRows] = None) -> None:
     """Causal attention of the step's tokens over the cache; picks the kernel: the
     tensor-core kernels for a bfloat16 cache and a head size they are built for (split-KV
     when every sequence brings one token), else the exact kernel.  `sink` [nq] 32-bit: a logit
-    per query head that joins the softmax's denominator (no key, no value, no scale)."""
+    per query head that joins the softmax's denominator (no key, no value, no scale).  `pooled`: rows
+    that stand for whole blocks of tokens before the window, in the same softmax."""
     dv = d if dv is None else int(dv)
     _need(sink, "attention sink", torch.float32)
-    fast = (q.dtype == torch.bfloat16 and k_cache.dtype == torch.bfloat16 and attention_flash_supported(d) and dv == d
+    fast = (pooled is None and q.dtype == torch.bfloat16 and k_cache.dtype == torch.bfloat16 and attention_flash_supported(d) and dv == d
             and workspace is not None and FLASH_ENABLED)
     if not fast:          # the 32-bit path, and values of another head size than the keys'
         paged_attention_simple(q, out, k_cache, v_cache, step.positions, step.seq_of_token,
-                               block_table, window, scale, nq, nkv, d, dv, sink)
+                               block_table, window, scale, nq, nkv, d, dv, sink, pooled)
         return
     G = nq // nkv
     # (the cluster-merged decode kernel takes no sink: single tokens of such layers go to the ticketed split-KV kernel)

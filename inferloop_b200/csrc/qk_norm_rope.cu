@@ -401,4 +401,234 @@ ILB_EXPORT int ilb_qk_norm_rope_cache(
   return check_launch("qk_norm_rope_cache");
 }
 
+// ---------------------------------------------------------------- norms over whole rows, turned values
+// The input stage of an attention whose query norm is taken over ALL query heads' elements at once and its key norm
+// over all key heads' (weights [nq * d] and [nkv * d]), and whose values may be turned too:
+//   q <- turn(q / sqrt(mean(q^2) + eps) * wq),  k likewise,  v <- turn_v(v)
+// turn: the first `rotary_dim` elements of a head in pairs (i, i + rotary_dim / 2) by `rope`; turn_v: all dv elements
+// of a value in pairs (i, i + dv / 2) by `v_rope`.  Either table may be null.
+// A row's units of VEC elements are dealt to gridDim.y blocks; every one of them takes the row's sums itself.
+template <typename T, int VEC> struct RowUnit;
+template <typename T> struct RowUnit<T, 1> {
+  __device__ static __forceinline__ void load(const T* p, float* x) { x[0] = to_float(*p); }
+  __device__ static __forceinline__ void store(T* p, const float* x) { *p = from_float<T>(x[0]); }
+};
+template <> struct RowUnit<__nv_bfloat16, 8> {
+  __device__ static __forceinline__ void load(const __nv_bfloat16* p, float* x) { unpack8(*reinterpret_cast<const uint4*>(p), x); }
+  __device__ static __forceinline__ void store(__nv_bfloat16* p, const float* x) { *reinterpret_cast<uint4*>(p) = pack8(x); }
+};
+
+struct RowsParams {
+  const float* q_weight; const float* k_weight;
+  const float2* rope; const float2* v_rope;
+  const int* positions; const int* seq_of_token; const int* block_table;
+  int max_blocks, page_size, num_pages, nq, nkv, d, dv, rotary_dim, qkv_stride, q_out_stride;
+  float eps;
+};
+
+constexpr int kRowsThreads = 256;
+
+template <typename TQ, typename TC, int VEC>
+__global__ void __launch_bounds__(kRowsThreads)
+rows_norm_rope_kernel(const TQ* __restrict__ qkv, TQ* __restrict__ q_out, TC* __restrict__ k_cache, TC* __restrict__ v_cache,
+                      const RowsParams p) {
+  ilb::pdl_launch_dependents();
+  ilb::pdl_wait();
+  __shared__ float scratch[33];
+  const int t = blockIdx.x;
+  const TQ* row = qkv + (size_t)t * p.qkv_stride;
+  const int nqd = p.nq * p.d, nkd = p.nkv * p.d, nvd = p.nkv * p.dv;
+  float x[VEC], y[VEC];
+  float sums[2] = {0.f, 0.f};
+  for (int e = threadIdx.x * VEC; e < nqd + nkd; e += kRowsThreads * VEC) {
+    RowUnit<TQ, VEC>::load(row + e, x);
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) ss = fmaf(x[i], x[i], ss);
+    sums[e < nqd ? 0 : 1] += ss;
+  }
+  const float inv_q = 1.0f / sqrtf(block_sum(sums[0], scratch) / (float)nqd + p.eps);
+  const float inv_k = 1.0f / sqrtf(block_sum(sums[1], scratch) / (float)nkd + p.eps);
+  // where this token's key and value go
+  long long place = -1;
+  if (k_cache != nullptr) {
+    const int pos = p.positions[t], blk = pos / p.page_size;
+    if (blk >= 0 && blk < p.max_blocks) {
+      const int page = p.block_table[(size_t)p.seq_of_token[t] * p.max_blocks + blk];
+      if (page >= 0 && page < p.num_pages) place = (long long)page * p.nkv * p.page_size + pos % p.page_size;      // never write outside the pool
+    }
+  }
+  const int units = (nqd + nkd + nvd) / VEC;
+  for (int u = blockIdx.y * kRowsThreads + threadIdx.x; u < units; u += gridDim.y * kRowsThreads) {
+    int e = u * VEC;
+    const int kind = e < nqd ? 0 : (e < nqd + nkd ? 1 : 2);
+    if (kind != 0 && place < 0) continue;
+    e -= kind == 0 ? 0 : (kind == 1 ? nqd : nqd + nkd);
+    const int width = kind == 2 ? p.dv : p.d;
+    const int h = e / width, c = e % width;
+    const float2* table = kind == 2 ? p.v_rope : p.rope;
+    const int half = kind == 2 ? p.dv / 2 : p.rotary_dim / 2;
+    const bool pair = table != nullptr && c < 2 * half;
+    if (pair && c >= half) continue;                       // the pair's first member writes both
+    const TQ* src = row + u * VEC;
+    RowUnit<TQ, VEC>::load(src, x);
+    if (pair) RowUnit<TQ, VEC>::load(src + half, y);
+    if (kind != 2) {
+      const float inv = kind == 0 ? inv_q : inv_k;
+      const float* w = (kind == 0 ? p.q_weight : p.k_weight) + e;
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) {
+        x[i] = x[i] * inv * w[i];
+        if (pair) y[i] = y[i] * inv * w[half + i];
+      }
+    }
+    if (pair) {
+      const float2* cs = table + (size_t)t * half + c;
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) {
+        const float a = x[i], b = y[i];
+        const float2 w = cs[i];
+        x[i] = __fsub_rn(__fmul_rn(a, w.x), __fmul_rn(b, w.y));
+        y[i] = __fadd_rn(__fmul_rn(a, w.y), __fmul_rn(b, w.x));
+      }
+    }
+    if (kind == 0) {
+      TQ* dst = q_out + (size_t)t * p.q_out_stride + e;
+      RowUnit<TQ, VEC>::store(dst, x);
+      if (pair) RowUnit<TQ, VEC>::store(dst + half, y);
+    } else {
+      TC* dst = (kind == 1 ? k_cache : v_cache) + ((size_t)place + (size_t)h * p.page_size) * width + c;
+      RowUnit<TC, VEC>::store(dst, x);
+      if (pair) RowUnit<TC, VEC>::store(dst + half, y);
+    }
+  }
+}
+
+ILB_EXPORT int ilb_rows_norm_rope_cache(
+    const void* qkv, void* q_out, int dtype, const float* q_weight, const float* k_weight, float eps, const float* rope,
+    int rotary_dim, const float* v_rope, const int* positions, const int* seq_of_token, const int* block_table, int max_blocks,
+    int page_size, int num_pages, void* k_cache, void* v_cache, int n_tokens, int nq, int nkv, int d, int dv, int qkv_stride,
+    int q_out_stride, cudaStream_t stream) {
+  ILB_REQUIRE(n_tokens >= 0 && nq > 0 && nkv > 0 && d > 0 && dv > 0 && eps > 0.f, "rows_norm_rope: bad sizes");
+  ILB_REQUIRE(q_weight != nullptr && k_weight != nullptr, "rows_norm_rope: the norms' weights are missing");
+  ILB_REQUIRE(rope == nullptr || (rotary_dim > 0 && rotary_dim % 2 == 0 && rotary_dim <= d),
+              "rows_norm_rope: rotary dimension %d must be even and at most the head size %d", rotary_dim, d);
+  ILB_REQUIRE(v_rope == nullptr || dv % 2 == 0, "rows_norm_rope: values of %d elements cannot be turned in pairs", dv);
+  ILB_REQUIRE(qkv_stride >= (nq + nkv) * d + nkv * dv && q_out_stride >= nq * d, "rows_norm_rope: strides too small");
+  ILB_REQUIRE((k_cache == nullptr) == (v_cache == nullptr), "rows_norm_rope: need both caches or none");
+  ILB_REQUIRE(k_cache == nullptr || (page_size > 0 && max_blocks > 0 && num_pages > 0), "rows_norm_rope: bad cache geometry");
+  ILB_REQUIRE(dtype == kF32 || dtype == kBF16, "rows_norm_rope: unknown dtype %d", dtype);
+  if (n_tokens == 0) return 0;
+  const RowsParams p{q_weight, k_weight, (const float2*)rope, (const float2*)v_rope, positions, seq_of_token, block_table, max_blocks,
+                     page_size, num_pages, nq, nkv, d, dv, rope != nullptr ? rotary_dim : 0, qkv_stride, q_out_stride, eps};
+  auto a16 = [](const void* x) { return (uintptr_t)x % 16 == 0; };
+  const bool vec = dtype == kBF16 && d % 8 == 0 && dv % 8 == 0 && (rope == nullptr || rotary_dim % 16 == 0) && (v_rope == nullptr || dv % 16 == 0) &&
+                   qkv_stride % 8 == 0 && q_out_stride % 8 == 0 && a16(qkv) && a16(q_out) && a16(k_cache) && a16(v_cache);
+  const int units = ((nq + nkv) * d + nkv * dv) / (vec ? 8 : 1);
+  int ny = 1;
+  while (n_tokens * ny < 296 && ny * kRowsThreads < units) ++ny;
+  const dim3 grid(n_tokens, ny);
+  if (vec)
+    ilb::launch(rows_norm_rope_kernel<__nv_bfloat16, __nv_bfloat16, 8>, grid, dim3(kRowsThreads), 0, stream, (const __nv_bfloat16*)qkv,
+                (__nv_bfloat16*)q_out, (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, p);
+  else if (dtype == kBF16)
+    ilb::launch(rows_norm_rope_kernel<__nv_bfloat16, __nv_bfloat16, 1>, grid, dim3(kRowsThreads), 0, stream, (const __nv_bfloat16*)qkv,
+                (__nv_bfloat16*)q_out, (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, p);
+  else
+    ilb::launch(rows_norm_rope_kernel<float, float, 1>, grid, dim3(kRowsThreads), 0, stream, (const float*)qkv, (float*)q_out,
+                (float*)k_cache, (float*)v_cache, p);
+  return check_launch("rows_norm_rope_cache");
+}
+
+// ---------------------------------------------------------------- means of blocks of cached rows
+// The token at position p completes block b = p / pool if (p + 1) % pool == 0: row b of the second set of pages becomes the
+// mean (32-bit sum) of the block's `pool` keys and of its values as the cache holds them.  One block of threads a token.
+template <typename T>
+__global__ void __launch_bounds__(256)
+pool_means_kernel(const T* __restrict__ k_cache, const T* __restrict__ v_cache, T* __restrict__ pk_cache, T* __restrict__ pv_cache,
+                  const int* __restrict__ positions, const int* __restrict__ seq_of_token, const int* __restrict__ block_table,
+                  const int* __restrict__ p_table, int max_blocks, int page_size, int num_pages, int p_num_pages, int pool, int nkv,
+                  int d, int dv) {
+  ilb::pdl_launch_dependents();
+  ilb::pdl_wait();
+  const int t = blockIdx.x, pos = positions[t];
+  if ((pos + 1) % pool != 0) return;
+  const int seq = seq_of_token[t], b = pos / pool;
+  if (b / page_size >= max_blocks) return;
+  const int* table = block_table + (size_t)seq * max_blocks;
+  const int p_page = p_table[(size_t)seq * max_blocks + b / page_size];
+  if (p_page < 0 || p_page >= p_num_pages) return;          // never write outside the pool
+  const int e = blockIdx.y * 256 + threadIdx.x;
+  if (e >= nkv * (d + dv)) return;
+  const bool is_k = e < nkv * d;
+  const int width = is_k ? d : dv, h = (is_k ? e : e - nkv * d) / width, c = (is_k ? e : e - nkv * d) % width;
+  const T* src = is_k ? k_cache : v_cache;
+  float sum = 0.f;
+  const int first = b * pool;
+  for (int j0 = 0; j0 < pool; j0 += 8) {                    // eight loads in flight
+    float x[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const int pj = first + j0 + i;
+      x[i] = 0.f;
+      if (j0 + i < pool) {
+        const int page = table[pj / page_size];
+        if (page >= 0 && page < num_pages) x[i] = to_float(src[(((size_t)page * nkv + h) * page_size + pj % page_size) * width + c]);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < 8; ++i) sum += x[i];
+  }
+  (is_k ? pk_cache : pv_cache)[(((size_t)p_page * nkv + h) * page_size + b % page_size) * width + c] = from_float<T>(sum / (float)pool);
+}
+
+ILB_EXPORT int ilb_pool_means(const void* k_cache, const void* v_cache, void* pk_cache, void* pv_cache, int dtype, const int* positions,
+                              const int* seq_of_token, const int* block_table, const int* p_table, int max_blocks, int page_size,
+                              int num_pages, int p_num_pages, int pool, int n_tokens, int nkv, int d, int dv, cudaStream_t stream) {
+  ILB_REQUIRE(n_tokens >= 0 && nkv > 0 && d > 0 && dv > 0 && pool > 0, "pool_means: bad sizes");
+  ILB_REQUIRE(page_size > 0 && max_blocks > 0 && num_pages > 0 && p_num_pages > 0, "pool_means: bad cache geometry");
+  ILB_REQUIRE(k_cache != nullptr && v_cache != nullptr && pk_cache != nullptr && pv_cache != nullptr, "pool_means: a cache is missing");
+  if (n_tokens == 0) return 0;
+  const dim3 grid(n_tokens, (nkv * (d + dv) + 255) / 256);
+#define ILB_PM(T) ilb::launch(pool_means_kernel<T>, grid, dim3(256), 0, stream, (const T*)k_cache, (const T*)v_cache, (T*)pk_cache, (T*)pv_cache, \
+                              positions, seq_of_token, block_table, p_table, max_blocks, page_size, num_pages, p_num_pages, pool, nkv, d, dv)
+  if (dtype == kF32) ILB_PM(float);
+  else if (dtype == kBF16) ILB_PM(__nv_bfloat16);
+  else return fail("pool_means: unknown dtype %d", dtype);
+#undef ILB_PM
+  return check_launch("pool_means");
+}
+
+// ---------------------------------------------------------------- heads turned back, in place
+// o[t, h, :] of `dv` elements in pairs (i, i + dv / 2), turned by minus the angle whose (cos, sin) is table[t, i].
+template <typename T>
+__global__ void __launch_bounds__(256)
+turn_back_kernel(T* __restrict__ o, const float2* __restrict__ table, int n_tokens, int heads, int dv) {
+  ilb::pdl_launch_dependents();
+  ilb::pdl_wait();
+  const int half = dv / 2;
+  const size_t n = (size_t)n_tokens * heads * half;
+  for (size_t i = (size_t)blockIdx.x * 256 + threadIdx.x; i < n; i += (size_t)gridDim.x * 256) {
+    const int m = (int)(i % half);
+    const size_t th = i / half, t = th / heads;
+    T* p = o + th * dv + m;
+    const float a = to_float(p[0]), b = to_float(p[half]);
+    const float2 w = table[t * half + m];
+    p[0] = from_float<T>(__fadd_rn(__fmul_rn(a, w.x), __fmul_rn(b, w.y)));
+    p[half] = from_float<T>(__fsub_rn(__fmul_rn(b, w.x), __fmul_rn(a, w.y)));
+  }
+}
+
+ILB_EXPORT int ilb_turn_back(void* o, int dtype, const float* table, int n_tokens, int heads, int dv, cudaStream_t stream) {
+  ILB_REQUIRE(n_tokens >= 0 && heads > 0 && dv > 0 && dv % 2 == 0 && table != nullptr, "turn_back: bad sizes");
+  if (n_tokens == 0) return 0;
+  const size_t n = (size_t)n_tokens * heads * (dv / 2);
+  const int blocks = (int)((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16);
+  if (dtype == kF32) ilb::launch(turn_back_kernel<float>, dim3(blocks), dim3(256), 0, stream, (float*)o, (const float2*)table, n_tokens, heads, dv);
+  else if (dtype == kBF16)
+    ilb::launch(turn_back_kernel<__nv_bfloat16>, dim3(blocks), dim3(256), 0, stream, (__nv_bfloat16*)o, (const float2*)table, n_tokens, heads, dv);
+  else return fail("turn_back: unknown dtype %d", dtype);
+  return check_launch("turn_back");
+}
+
 ILB_DEFINE_LAST_ERROR()

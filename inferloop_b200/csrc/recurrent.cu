@@ -12,7 +12,8 @@
 //               portions and single tokens run one pass from and to the state slot.
 //   silu_rows   out = silu(x) of the leading columns of a projection, widened to 32-bit: the inputs of a linear
 //               attention whose queries, keys and values pass silu.
-//   rms_gate    out = y / sqrt(mean(y^2) + eps) * w * sigmoid(gate) * scale over a whole row.
+//   rms_gate    out = y / sqrt(mean(y^2) + eps) * w * sigmoid(gate) * scale over a whole row, or over each of `groups`
+//               equal consecutive parts of it (one block a part).
 //   head_gate   dst[t, h, :] = o[t, h, :] * sigmoid(g[t, h]) * scale: one gate a head on an attention's output (in place, or into
 //               the columns of a wider matrix).
 //
@@ -270,9 +271,11 @@ rms_gate_kernel(const float* __restrict__ y, const TI* __restrict__ gate, int ld
   ilb::pdl_launch_dependents();
   ilb::pdl_wait();
   __shared__ float scratch[33];
-  const int t = blockIdx.x;
-  const float* yr = y + (size_t)t * width;
-  const TI* gr = gate + (size_t)t * ld_gate;
+  const int t = blockIdx.x, part = blockIdx.y;              // `width`: elements of a part
+  const float* yr = y + ((size_t)t * gridDim.y + part) * width;
+  const TI* gr = gate + (size_t)t * ld_gate + (size_t)part * width;
+  w += (size_t)part * width;
+  out += (size_t)part * width;
   float ss = 0.f;
   for (int i = threadIdx.x; i < width; i += blockDim.x) ss = fmaf(yr[i], yr[i], ss);
   ss = block_sum(ss, scratch);
@@ -291,11 +294,11 @@ rms_gate_vec_kernel(const float* __restrict__ y, const __nv_bfloat16* __restrict
   ilb::pdl_launch_dependents();
   ilb::pdl_wait();
   __shared__ float scratch[33];
-  const int t = blockIdx.x, n4 = width / 4;
-  const float4* yr = reinterpret_cast<const float4*>(y + (size_t)t * width);
-  const uint2* gr = reinterpret_cast<const uint2*>(gate + (size_t)t * ld_gate);
-  const float4* wr = reinterpret_cast<const float4*>(w);
-  uint2* o = reinterpret_cast<uint2*>(out + (size_t)t * ld_out);
+  const int t = blockIdx.x, part = blockIdx.y, n4 = width / 4;
+  const float4* yr = reinterpret_cast<const float4*>(y + ((size_t)t * gridDim.y + part) * width);
+  const uint2* gr = reinterpret_cast<const uint2*>(gate + (size_t)t * ld_gate + (size_t)part * width);
+  const float4* wr = reinterpret_cast<const float4*>(w + (size_t)part * width);
+  uint2* o = reinterpret_cast<uint2*>(out + (size_t)t * ld_out + (size_t)part * width);
   float4 keep[kGateKeep];
   float ss = 0.f;
 #pragma unroll
@@ -336,22 +339,24 @@ rms_gate_vec_kernel(const float* __restrict__ y, const __nv_bfloat16* __restrict
 // y: [rows, width] 32-bit; gate: [rows, ld_gate] of `dtype` (its first `width` columns from the pointer given);
 // out: [rows, ld_out] of `dtype` (its first `width` columns).
 ILB_EXPORT int ilb_rms_gate(const float* y, const void* gate, int dtype, int ld_gate, const float* w, void* out, int ld_out, int rows,
-                            int width, float eps, float scale, cudaStream_t stream) {
+                            int width, int groups, float eps, float scale, cudaStream_t stream) {
   ILB_REQUIRE(rows >= 0 && width > 0 && ld_gate >= width && ld_out >= width && eps > 0.f, "rms_gate: bad sizes");
+  ILB_REQUIRE(groups > 0 && groups <= 65535 && width % groups == 0, "rms_gate: %d groups do not cut a row of %d", groups, width);
   if (rows == 0) return 0;
-  if (dtype == kBF16 && width % 4 == 0 && ld_gate % 4 == 0 && ld_out % 4 == 0 && ((uintptr_t)y % 16 == 0) && ((uintptr_t)w % 16 == 0) &&
+  const int part = width / groups;
+  if (dtype == kBF16 && part % 4 == 0 && ld_gate % 4 == 0 && ld_out % 4 == 0 && ((uintptr_t)y % 16 == 0) && ((uintptr_t)w % 16 == 0) &&
       ((uintptr_t)gate % 8 == 0) && ((uintptr_t)out % 8 == 0)) {
-    const int per = width / 4, vthreads = per >= 1024 ? 256 : (per >= 256 ? 128 : 64);
-    ilb::launch(rms_gate_vec_kernel, dim3(rows), dim3(vthreads), 0, stream, y, (const __nv_bfloat16*)gate, ld_gate, w, (__nv_bfloat16*)out, ld_out,
-                width, eps, scale);
+    const int per = part / 4, vthreads = per >= 1024 ? 256 : (per >= 256 ? 128 : (per > 32 ? 64 : 32));
+    ilb::launch(rms_gate_vec_kernel, dim3(rows, groups), dim3(vthreads), 0, stream, y, (const __nv_bfloat16*)gate, ld_gate, w, (__nv_bfloat16*)out, ld_out,
+                part, eps, scale);
     return check_launch("rms_gate");
   }
-  const int threads = width >= 1024 ? 256 : (width >= 256 ? 128 : 64);
+  const int threads = part >= 1024 ? 256 : (part >= 256 ? 128 : 64);
   if (dtype == kF32)
-    ilb::launch(rms_gate_kernel<float>, dim3(rows), dim3(threads), 0, stream, y, (const float*)gate, ld_gate, w, (float*)out, ld_out, width, eps, scale);
+    ilb::launch(rms_gate_kernel<float>, dim3(rows, groups), dim3(threads), 0, stream, y, (const float*)gate, ld_gate, w, (float*)out, ld_out, part, eps, scale);
   else if (dtype == kBF16)
-    ilb::launch(rms_gate_kernel<__nv_bfloat16>, dim3(rows), dim3(threads), 0, stream, y, (const __nv_bfloat16*)gate, ld_gate, w,
-                (__nv_bfloat16*)out, ld_out, width, eps, scale);
+    ilb::launch(rms_gate_kernel<__nv_bfloat16>, dim3(rows, groups), dim3(threads), 0, stream, y, (const __nv_bfloat16*)gate, ld_gate, w,
+                (__nv_bfloat16*)out, ld_out, part, eps, scale);
   else return fail("rms_gate: unknown dtype %d", dtype);
   return check_launch("rms_gate");
 }

@@ -1,12 +1,14 @@
 // A block that norms what a sublayer GIVES instead of what it reads:  x <- x + gn(sublayer(x)) * g.
 //
-//   cast_zero        xc = x in the compute dtype (what the sublayer reads), y = 0 (what it adds into)
+//   cast_zero        xc = x in the compute dtype (what the sublayer reads), y = keep * x (what it adds into; keep 0: zero)
 //   group_norm_add   y is cut into `groups` equal consecutive parts, each divided by its own
 //                    sqrt(mean(part^2) + eps), the whole multiplied by g; then either
 //                      x += that; xc = x in the compute dtype; y = 0     (between two sublayers, one launch), or
 //                      out = that                                        (a plain grouped norm, the model's last one)
 //   gated_rows       out[t, k] = gelu_tanh(a[t, k]) * table[token[t], col0 + k]: a gate on a slice of a
 //                    per-token row of a table
+//
+//   sum_norm         the other arrangement, x <- norm(keep * x + sublayer(x)) * g: y already holds the sum (below)
 //
 // Everything is 32-bit but what is stored in the compute dtype.  One block a token row.  The sum of squares of a
 // part is taken by a fixed set of warps over fixed ranges and added in a fixed order: a row's result depends on
@@ -22,19 +24,20 @@ constexpr int kMaxGroups = 64;
 
 template <typename TO>
 __global__ void __launch_bounds__(kNormThreads)
-cast_zero_kernel(const float* __restrict__ x, TO* __restrict__ xc, float* __restrict__ y, size_t n) {
+cast_zero_kernel(const float* __restrict__ x, TO* __restrict__ xc, float* __restrict__ y, size_t n, float keep) {
   ilb::pdl_launch_dependents();
   ilb::pdl_wait();
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
-    xc[i] = from_float<TO>(x[i]);
-    y[i] = 0.f;
+    const float v = x[i];
+    xc[i] = from_float<TO>(v);
+    y[i] = keep == 0.f ? 0.f : keep * v;
   }
 }
 
 // Four elements a thread and access.
 template <typename TO>
 __global__ void __launch_bounds__(kNormThreads)
-cast_zero_vec_kernel(const float4* __restrict__ x, TO* __restrict__ xc, float4* __restrict__ y, size_t n4) {
+cast_zero_vec_kernel(const float4* __restrict__ x, TO* __restrict__ xc, float4* __restrict__ y, size_t n4, float keep) {
   ilb::pdl_launch_dependents();
   ilb::pdl_wait();
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n4; i += (size_t)gridDim.x * blockDim.x) {
@@ -48,11 +51,11 @@ cast_zero_vec_kernel(const float4* __restrict__ x, TO* __restrict__ xc, float4* 
       pk.y = *reinterpret_cast<uint32_t*>(&hi);
       reinterpret_cast<uint2*>(xc)[i] = pk;
     }
-    y[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    y[i] = keep == 0.f ? make_float4(0.f, 0.f, 0.f, 0.f) : make_float4(keep * v.x, keep * v.y, keep * v.z, keep * v.w);
   }
 }
 
-ILB_EXPORT int ilb_cast_zero(const float* x, void* xc, int dtype, float* y, long long n, cudaStream_t stream) {
+ILB_EXPORT int ilb_cast_zero(const float* x, void* xc, int dtype, float* y, long long n, float keep, cudaStream_t stream) {
   ILB_REQUIRE(n >= 0, "cast_zero: bad size");
   ILB_REQUIRE(dtype == kF32 || dtype == kBF16, "cast_zero: unknown dtype %d", dtype);
   if (n == 0) return 0;
@@ -61,11 +64,11 @@ ILB_EXPORT int ilb_cast_zero(const float* x, void* xc, int dtype, float* y, long
   long long blocks = (units + kNormThreads - 1) / kNormThreads;
   if (blocks > 148 * 16) blocks = 148 * 16;
   if (vec) {
-    if (dtype == kF32) ilb::launch(cast_zero_vec_kernel<float>, dim3((int)blocks), dim3(kNormThreads), 0, stream, (const float4*)x, (float*)xc, (float4*)y, (size_t)units);
-    else ilb::launch(cast_zero_vec_kernel<__nv_bfloat16>, dim3((int)blocks), dim3(kNormThreads), 0, stream, (const float4*)x, (__nv_bfloat16*)xc, (float4*)y, (size_t)units);
+    if (dtype == kF32) ilb::launch(cast_zero_vec_kernel<float>, dim3((int)blocks), dim3(kNormThreads), 0, stream, (const float4*)x, (float*)xc, (float4*)y, (size_t)units, keep);
+    else ilb::launch(cast_zero_vec_kernel<__nv_bfloat16>, dim3((int)blocks), dim3(kNormThreads), 0, stream, (const float4*)x, (__nv_bfloat16*)xc, (float4*)y, (size_t)units, keep);
   } else {
-    if (dtype == kF32) ilb::launch(cast_zero_kernel<float>, dim3((int)blocks), dim3(kNormThreads), 0, stream, x, (float*)xc, y, (size_t)n);
-    else ilb::launch(cast_zero_kernel<__nv_bfloat16>, dim3((int)blocks), dim3(kNormThreads), 0, stream, x, (__nv_bfloat16*)xc, y, (size_t)n);
+    if (dtype == kF32) ilb::launch(cast_zero_kernel<float>, dim3((int)blocks), dim3(kNormThreads), 0, stream, x, (float*)xc, y, (size_t)n, keep);
+    else ilb::launch(cast_zero_kernel<__nv_bfloat16>, dim3((int)blocks), dim3(kNormThreads), 0, stream, x, (__nv_bfloat16*)xc, y, (size_t)n, keep);
   }
   return check_launch("cast_zero");
 }
@@ -160,6 +163,92 @@ ILB_EXPORT int ilb_group_norm_add(float* y, int ldy, const float* w, float eps, 
   else { if (vec) ILB_GN(float, true); else ILB_GN(float, false); }
 #undef ILB_GN
   return check_launch("group_norm_add");
+}
+
+// ---------------------------------------------------------------- the norm of a sum
+// y holds keep * x + sublayer(x) when this runs:  x = y / sqrt(mean(y^2) + eps) * w,  xc = x in the compute dtype,
+// y = keep * x: the stream, the next sublayer's input and what that sublayer adds into, from one read of the sum.
+// One block a row; up to kSumKeep vectors a thread stay in registers between the sum and the writes.
+constexpr int kSumKeep = 4;
+
+template <typename TO>
+__device__ __forceinline__ void store4(TO* p, float4 r) {
+  if constexpr (sizeof(TO) == 4) {
+    *reinterpret_cast<float4*>(p) = r;
+  } else {
+    __nv_bfloat162 lo = __floats2bfloat162_rn(r.x, r.y), hi = __floats2bfloat162_rn(r.z, r.w);
+    uint2 pk;
+    pk.x = *reinterpret_cast<uint32_t*>(&lo);
+    pk.y = *reinterpret_cast<uint32_t*>(&hi);
+    *reinterpret_cast<uint2*>(p) = pk;
+  }
+}
+
+template <typename TO, bool kVec>
+__global__ void __launch_bounds__(kNormThreads)
+sum_norm_kernel(float* __restrict__ y, const float* __restrict__ w, float eps, float keep, int width, float* __restrict__ x, TO* __restrict__ xc) {
+  ilb::pdl_launch_dependents();
+  ilb::pdl_wait();
+  __shared__ float scratch[33];
+  float* row = y + (size_t)blockIdx.x * width;
+  float* xr = x != nullptr ? x + (size_t)blockIdx.x * width : nullptr;
+  TO* o = xc + (size_t)blockIdx.x * width;
+  float ss = 0.f;
+  if constexpr (kVec) {
+    const int n4 = width / 4;
+    float4 v[kSumKeep];
+#pragma unroll
+    for (int j = 0; j < kSumKeep; ++j) {
+      const int i = threadIdx.x + j * kNormThreads;
+      if (i < n4) {
+        v[j] = reinterpret_cast<const float4*>(row)[i];
+        ss = fmaf(v[j].x, v[j].x, ss); ss = fmaf(v[j].y, v[j].y, ss); ss = fmaf(v[j].z, v[j].z, ss); ss = fmaf(v[j].w, v[j].w, ss);
+      }
+    }
+    for (int i = threadIdx.x + kSumKeep * kNormThreads; i < n4; i += kNormThreads) {
+      const float4 t = reinterpret_cast<const float4*>(row)[i];
+      ss = fmaf(t.x, t.x, ss); ss = fmaf(t.y, t.y, ss); ss = fmaf(t.z, t.z, ss); ss = fmaf(t.w, t.w, ss);
+    }
+    ss = block_sum(ss, scratch);
+    const float inv = 1.0f / sqrtf(ss / (float)width + eps);
+    auto write = [&](int i, const float4 t) {
+      const float4 g = reinterpret_cast<const float4*>(w)[i];
+      const float4 r = make_float4(t.x * inv * g.x, t.y * inv * g.y, t.z * inv * g.z, t.w * inv * g.w);
+      if (xr != nullptr) reinterpret_cast<float4*>(xr)[i] = r;
+      store4<TO>(o + 4 * i, r);
+      reinterpret_cast<float4*>(row)[i] = make_float4(keep * r.x, keep * r.y, keep * r.z, keep * r.w);
+    };
+#pragma unroll
+    for (int j = 0; j < kSumKeep; ++j) {
+      const int i = threadIdx.x + j * kNormThreads;
+      if (i < n4) write(i, v[j]);
+    }
+    for (int i = threadIdx.x + kSumKeep * kNormThreads; i < n4; i += kNormThreads) write(i, reinterpret_cast<const float4*>(row)[i]);
+  } else {
+    for (int i = threadIdx.x; i < width; i += kNormThreads) ss = fmaf(row[i], row[i], ss);
+    ss = block_sum(ss, scratch);
+    const float inv = 1.0f / sqrtf(ss / (float)width + eps);
+    for (int i = threadIdx.x; i < width; i += kNormThreads) {
+      const float r = row[i] * inv * w[i];
+      if (xr != nullptr) xr[i] = r;
+      o[i] = from_float<TO>(r);
+      row[i] = keep * r;
+    }
+  }
+}
+
+// y, x: [rows, width] 32-bit (x may be null: only the copy and the next sum are written); xc: [rows, width] of `dtype`.
+ILB_EXPORT int ilb_sum_norm(float* y, const float* w, float eps, float keep, int rows, int width, float* x, void* xc, int dtype,
+                            cudaStream_t stream) {
+  ILB_REQUIRE(rows >= 0 && width > 0 && eps > 0.f && xc != nullptr, "sum_norm: bad sizes");
+  ILB_REQUIRE(dtype == kF32 || dtype == kBF16, "sum_norm: unknown dtype %d", dtype);
+  if (rows == 0) return 0;
+  const bool vec = width % 4 == 0 && ((uintptr_t)y % 16 == 0) && ((uintptr_t)w % 16 == 0) && ((uintptr_t)x % 16 == 0) && ((uintptr_t)xc % 16 == 0);
+#define ILB_SN(TO, V) ilb::launch(sum_norm_kernel<TO, V>, dim3(rows), dim3(kNormThreads), 0, stream, y, w, eps, keep, width, x, (TO*)xc)
+  if (dtype == kBF16) { if (vec) ILB_SN(__nv_bfloat16, true); else ILB_SN(__nv_bfloat16, false); }
+  else { if (vec) ILB_SN(float, true); else ILB_SN(float, false); }
+#undef ILB_SN
+  return check_launch("sum_norm");
 }
 
 __device__ __forceinline__ float gelu_tanh(float z) {

@@ -135,8 +135,9 @@ class Engine:
         # window, the largest step's own tokens and a page of slack.  Every group gets room
         # for the same number of such requests; no set of requests can use more than
         # max_num_seqs of them.
-        per_request = [-(-(want if g.need.window is None else min(want, g.need.window + int(step_tokens) + self.block_size))
-                         // self.block_size) + (0 if g.need.window is None else 1) for g in groups]
+        # (A group whose rows stand for several tokens: a row per `stride` of them.)
+        per_request = [max(1, -(-(want if g.need.window is None else min(want, g.need.window + int(step_tokens) + self.block_size))
+                                // g.need.stride // self.block_size)) + (0 if g.need.window is None else 1) for g in groups]
         bytes_per_request = sum(n * g.page_bytes(element) for n, g in zip(per_request, groups))
         requests = min(max(budget, 0) / bytes_per_request, float(max(max_num_seqs, 1)))
         pages = [int(requests * n) for n in per_request]

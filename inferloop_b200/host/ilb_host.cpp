@@ -478,9 +478,10 @@ struct Slots {
 // ------------------------------------------------------------------ ledger
 struct Group {
   int window;                                   // keys a token may look back over, or -1 for all
+  int stride;                                   // tokens that one row of a page stands for (1: a row per token; n: a row per n tokens, once all n are there)
   Pool pool;
   std::unordered_map<long long, std::vector<int>> tables;
-  Group(int w, int pages) : window(w), pool(pages) {}
+  Group(int w, int s, int pages) : window(w), stride(s), pool(pages) {}
 };
 
 struct Ledger {
@@ -492,17 +493,18 @@ struct Ledger {
 
   // Every group has a pool of its own size: a group whose layers read a window of the keys
   // needs fewer pages than one that keeps them all.
-  Ledger(int n_groups, const int* windows, const int* num_pages, int page_size_, int max_requests)
+  Ledger(int n_groups, const int* windows, const int* strides, const int* num_pages, int page_size_, int max_requests)
       : page_size(page_size_), slots(max_requests) {
     groups.reserve((size_t)n_groups);
-    for (int g = 0; g < n_groups; ++g) groups.emplace_back(windows[g], num_pages[g]);
+    for (int g = 0; g < n_groups; ++g) groups.emplace_back(windows[g], strides[g], num_pages[g]);
   }
-  long long blocks_for(long long tokens) const { return (tokens + page_size - 1) / page_size; }
+  // Pages that the rows of so many tokens fill.
+  long long blocks_for(const Group& g, long long tokens) const { return (tokens / g.stride + page_size - 1) / page_size; }
   // Blocks below this index hold only keys that no present or future token reads.
   long long first_needed_block(const Group& g, long long first_query_pos) const {
     if (g.window < 0) return 0;
     const long long oldest = std::max(0ll, first_query_pos - g.window + 1);
-    return oldest / page_size;
+    return oldest / g.stride / page_size;
   }
   int pages_needed(long long req, long long new_length, int* out) const {
     auto it = length.find(req);
@@ -511,7 +513,7 @@ struct Ledger {
     for (size_t gi = 0; gi < groups.size(); ++gi) {
       const Group& g = groups[gi];
       const std::vector<int>& table = g.tables.at(req);
-      const long long want = blocks_for(new_length);
+      const long long want = blocks_for(g, new_length);
       const long long first = std::min<long long>(first_needed_block(g, cur), (long long)table.size());
       long long releasable = 0;
       for (long long b = 0; b < first; ++b) releasable += table[(size_t)b] >= 0;
@@ -536,17 +538,16 @@ struct Ledger {
         window_pages_released += (long long)gone.size();
       }
     }
-    const long long want = blocks_for(new_length);
     for (size_t gi = 0; gi < groups.size(); ++gi) {
       const Group& g = groups[gi];
-      const long long extra = want - (long long)g.tables.at(req).size();
+      const long long extra = blocks_for(g, new_length) - (long long)g.tables.at(req).size();
       if (extra > (long long)g.pool.free_.size())
         return fail(kOutOfPages, "request %lld needs %lld more pages in group %zu, %zu free of %d", req, extra, gi,
                     g.pool.free_.size(), g.pool.num_pages);
     }
     for (Group& g : groups) {
       std::vector<int>& table = g.tables[req];
-      const long long extra = want - (long long)table.size();
+      const long long extra = blocks_for(g, new_length) - (long long)table.size();
       if (extra > 0) {
         const size_t old = table.size();
         table.resize(old + (size_t)extra);
@@ -559,9 +560,8 @@ struct Ledger {
   int commit(long long req, long long new_length) {
     auto it = length.find(req);
     if (it == length.end()) return fail(kInvalid, "request %lld is not live", req);
-    const long long want = blocks_for(new_length);
     for (size_t gi = 0; gi < groups.size(); ++gi)
-      if ((long long)groups[gi].tables.at(req).size() < want)
+      if ((long long)groups[gi].tables.at(req).size() < blocks_for(groups[gi], new_length))
         return fail(kLedger, "request %lld commits %lld tokens but holds %zu blocks in group %zu", req, new_length,
                     groups[gi].tables.at(req).size(), gi);
     if (new_length < it->second) return fail(kInvalid, "commit cannot shrink a request");
@@ -690,15 +690,16 @@ ILB_API int ilb_slots_num_free(void* h) { return (int)static_cast<Slots*>(h)->fr
 ILB_API int ilb_slots_check(void* h) { return static_cast<Slots*>(h)->check(); }
 
 // ------------------------------------------------------------------ ledger, C interface
-// num_pages: one entry per group.
-ILB_API int ilb_ledger_new(int n_groups, const int* windows, const int* num_pages, int page_size, int max_requests, void** out) {
+// num_pages, strides: one entry per group.
+ILB_API int ilb_ledger_new(int n_groups, const int* windows, const int* strides, const int* num_pages, int page_size, int max_requests,
+                           void** out) {
   *out = nullptr;
   if (page_size <= 0) return fail(kInvalid, "page_size must be positive");
   if (n_groups < 0) return fail(kInvalid, "a negative number of page groups");
   for (int g = 0; g < n_groups; ++g)
-    if (num_pages[g] <= 0) return fail(kInvalid, "a page pool needs at least one page");
+    if (num_pages[g] <= 0 || strides[g] <= 0) return fail(kInvalid, "a page pool needs at least one page and a positive stride");
   if (max_requests <= 0) return fail(kInvalid, "a slot pool needs at least one slot");
-  *out = new Ledger(n_groups, windows, num_pages, page_size, max_requests);
+  *out = new Ledger(n_groups, windows, strides, num_pages, page_size, max_requests);
   return kOk;
 }
 ILB_API void ilb_ledger_free(void* h) { delete static_cast<Ledger*>(h); }
@@ -783,7 +784,7 @@ ILB_API int ilb_step_fits(void* h, int n, const long long* req, const int* n_tok
       if (rc) return rc;
       for (size_t g = 0; g < need.size(); ++g) need[g] += per[g];
     } else {
-      for (size_t g = 0; g < need.size(); ++g) need[g] += l->blocks_for(n_tok[i]);
+      for (size_t g = 0; g < need.size(); ++g) need[g] += l->blocks_for(l->groups[g], n_tok[i]);
     }
   }
   for (size_t g = 0; g < need.size(); ++g)
@@ -950,7 +951,7 @@ struct Sched {
       l->pages_needed(id, new_len, per.data());
       for (size_t g = 0; g < need.size(); ++g) need[g] = per[g];
     } else {
-      for (size_t g = 0; g < need.size(); ++g) need[g] = l->blocks_for(new_len);
+      for (size_t g = 0; g < need.size(); ++g) need[g] = l->blocks_for(l->groups[g], new_len);
     }
   }
   void held(long long id, std::vector<long long>& out) const {
@@ -1021,7 +1022,7 @@ struct Sched {
           room = -1;
           for (size_t g = 0; g < G; ++g) {
             const long long have = live(id) ? (long long)l->groups[g].tables.at(id).size() : 0;
-            const long long r = (have + free_[g]) * l->page_size;
+            const long long r = ((have + free_[g]) * l->page_size + 1) * l->groups[g].stride - 1;
             room = room < 0 ? r : std::min(room, r);
           }
         }
@@ -1103,11 +1104,10 @@ ILB_API int ilb_sched_add(void* h, long long id, long long prompt_len, long long
     // reserved tokens = prompt + max_new_tokens must fit the context (crates/engine/workloads/src/native.rs:91-111)
     return fail(kInvalid, "request #%lld: prompt %lld + max_new_tokens %lld exceeds max_model_len %lld", id, prompt_len, max_new,
                 s->max_model_len);
-  const long long pages = s->l->blocks_for(total);
   for (size_t g = 0; g < s->l->groups.size(); ++g) {
     const Group& grp = s->l->groups[g];
-    long long reach = pages;
-    if (grp.window >= 0) reach = std::min(pages, s->l->blocks_for(grp.window + s->chunk) + 1);
+    long long reach = s->l->blocks_for(grp, total);
+    if (grp.window >= 0) reach = std::min(reach, s->l->blocks_for(grp, grp.window + s->chunk) + 1);
     if (reach > grp.pool.num_pages)
       return fail(kCapacity, "request #%lld needs %lld pages of group %zu, the pool has %d", id, reach, g, grp.pool.num_pages);
   }

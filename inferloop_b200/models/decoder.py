@@ -76,7 +76,7 @@ class DecoderModel:
         # Every declared tensor is read once by a step, except the token table, of which a step
         # reads one row per token (unless it is also the output matrix).
         self._weight_bytes = sum(tensors[d.name].numel() * tensors[d.name].element_size() for d in self.declare_weights()
-                                 if d.name != s.embedding_name or s.head_name is None)
+                                 if d.name in tensors and (d.name != s.embedding_name or s.head_name is None))
 
     def cache_needs(self) -> List[CacheNeeds]:
         return [b.cache_needs() for b in self.blocks]

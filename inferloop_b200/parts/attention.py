@@ -17,7 +17,8 @@ What a description may vary beyond that (all spec parameters, the defaults give 
 above): `v_head_dim` (values of another head size than queries and keys), `bias` = True /
 False / "qkv" (no bias on the output projection), `qk_norm` = True (weight [head_dim]) or
 "unweighted" (q and k divided by their root mean square), `qk_norm_after_rotation`,
-`scale` (the multiplier of q.k), a position kind whose pairs are interleaved, tensor names
+"rows" (weights [num_heads * head_dim] and [num_kv_heads * head_dim]: q's norm over all its heads' elements at once, and
+k's), `scale` (the multiplier of q.k), a position kind whose pairs are interleaved, tensor names
 (`names`: pairs (role, name under the prefix)), and `value_mix` = "first" | "mixed": the first
 such layer of a model keeps its values of the step's tokens, every later one caches
 (1 - lambda) v + lambda v_first with its own learned scalar lambda.
@@ -28,6 +29,12 @@ csrc/attention_mix.cu): `query_temperature` = (coef, every): q at position i is 
 1 + coef ln(floor((i + 1) / every) + 1); `softcap` = c: s <- c tanh(s / c); `distance_bias`: s <- s -
 r1_h ln(1 + r2_h (i - j)) with two learned vectors; `head_mix`: s_h <- sum_g M[h, g] s_g with a learned
 [heads, heads] matrix; in that order.  `sink`: a learned logit per head joins the softmax's denominator.
+
+`value_position`: a position encoding (half-split, over the whole value) by which a value is turned at its own position
+before it is cached; the head's output is turned back by the query's position.  `pool` = P (with a window): beside the
+window's tokens a position sees, in the same softmax, the mean key and the mean value of each aligned block of P tokens that
+lies wholly before its window.  The means are rows of a second set of pages (one row per P tokens), made as soon as a block's
+last token is cached; the tokens' own pages go when both the window and their block are done with them.
 
 `output_gate` = "head": head h's output is multiplied by sigmoid((W_g x)_h), one number a head from a matrix
 [heads, hidden] whose rows ride behind q|k|v in the one projection.  `out_scale`: a constant on the whole mixer's
@@ -63,9 +70,10 @@ class GQAttention(Mixer):
             raise ValueError(f"{self.nq} query heads are not a multiple of {self.nkv} kv heads")
         self.dv = int(spec.get("v_head_dim") or self.d)
         qk_norm = spec.get("qk_norm", False)
-        if qk_norm not in (False, True, "unweighted"):
-            raise ValueError(f"qk_norm must be False, True or 'unweighted', found {qk_norm!r}")
+        if qk_norm not in (False, True, "unweighted", "rows"):
+            raise ValueError(f"qk_norm must be False, True, 'unweighted' or 'rows', found {qk_norm!r}")
         self.qk_norm = qk_norm is True                       # with a weight per head element
+        self.qk_norm_rows = qk_norm == "rows"                # over all heads' elements at once
         self.qk_norm_unweighted = qk_norm == "unweighted"
         self.qk_norm_after = bool(spec.get("qk_norm_after_rotation", False))
         self.qk_norm_eps = float(spec.get("qk_norm_eps", 1e-6))
@@ -100,7 +108,19 @@ class GQAttention(Mixer):
         self.shaped = bool(self.temp_coef or self.softcap or self.distance_bias or self.head_mix)
         if self.shaped and self.value_mix is not None:
             raise ValueError("attention: reshaped scores and mixed values are not served together")
+        self.pool = int(spec.get("pool") or 0)
+        if self.pool and not self.window:
+            raise ValueError("attention: pooled blocks lie before a window, and there is none")
         self.position = registry.build("position", spec["position"], ctx)
+        value_position = spec.get("value_position")
+        self.value_position = registry.build("position", value_position, ctx) if value_position is not None else None
+        if self.value_position is not None and getattr(self.value_position, "interleaved", False):
+            raise ValueError("attention: values are turned in pairs (i, i + half)")
+        if (self.value_position is not None or self.pool) and not self.qk_norm_rows:
+            raise ValueError("attention: turned values and pooled blocks are served with norms over whole rows (qk_norm='rows')")
+        if self.qk_norm_rows and (self.shaped or self.value_mix is not None or self.has_sink or self.qk_norm_after
+                                  or getattr(self.position, "interleaved", False)):
+            raise ValueError("attention: norms over whole rows are served before a half-split rotation, with a plain softmax and unmixed values")
         self.rotary_dim = int(spec["position"].get("rotary_dim", 0))
         p = prefix
         names = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight",
@@ -129,9 +149,10 @@ class GQAttention(Mixer):
                     WeightDecl(n["vb"], (self.nkv * dv,), "vector", "bias")]
         if self.out_bias:
             out.append(WeightDecl(n["ob"], (H,), "vector", "bias"))
-        if self.qk_norm:
-            out += [WeightDecl(n["qn"], (d,), "vector", "norm"),
-                    WeightDecl(n["kn"], (d,), "vector", "norm")]
+        if self.qk_norm or self.qk_norm_rows:
+            per_q, per_k = (self.nq * d, self.nkv * d) if self.qk_norm_rows else (d, d)
+            out += [WeightDecl(n["qn"], (per_q,), "vector", "norm"),
+                    WeightDecl(n["kn"], (per_k,), "vector", "norm")]
         if self.distance_bias:
             out += [WeightDecl(n["r1"], (self.nq,), "vector", "positive"), WeightDecl(n["r2"], (self.nq,), "vector", "positive")]
         if self.head_mix:
@@ -163,7 +184,7 @@ class GQAttention(Mixer):
             self.b_o = (tensors[n["ob"]] * self.out_scale).contiguous() if self.out_scale != 1.0 else tensors[n["ob"]].contiguous()
         if self.value_mix == "mixed":
             self.v_lambda = tensors[n["vmix"]].reshape(1).contiguous()
-        if self.qk_norm:
+        if self.qk_norm or self.qk_norm_rows:
             self.q_norm = tensors[n["qn"]].contiguous()
             self.k_norm = tensors[n["kn"]].contiguous()
         if self.distance_bias:
@@ -174,7 +195,12 @@ class GQAttention(Mixer):
             self.sink = tensors[n["sink"]].contiguous()
 
     def cache_needs(self) -> CacheNeeds:
-        return CacheNeeds(paged=PagedKVNeed(self.nkv, self.d, self.window, self.dv if self.dv != self.d else None))
+        v_dim = self.dv if self.dv != self.d else None
+        if not self.pool:
+            return CacheNeeds(paged=PagedKVNeed(self.nkv, self.d, self.window, v_dim))
+        # a token is read while it is in the window, and until its block is complete
+        return CacheNeeds(paged=PagedKVNeed(self.nkv, self.d, max(self.window, self.pool), v_dim),
+                          pooled=PagedKVNeed(self.nkv, self.d, None, v_dim, self.pool))
 
     def scratch_bytes(self, tokens: int) -> int:
         size = torch.empty((), dtype=self.ctx.dtype).element_size()
@@ -217,6 +243,9 @@ class GQAttention(Mixer):
         table = step.block_tables[cache.group]
         ops.scope("attention.position_table")
         rope = self.position.table(step)
+        if self.qk_norm_rows:
+            self._forward_rows(qkv, rope, table, step, cache, gate_col0, residual, out)
+            return
         v_first = None
         if self.value_mix is not None:
             # the step's tokens' values of the first layer that mixes: kept by it, read by the later ones
@@ -257,6 +286,30 @@ class GQAttention(Mixer):
         else:
             ops.attention(q, o, cache.k, cache.v, step, table, self.window or 0, self.scale,
                           self.nq, self.nkv, self.d, workspace=ws, decode_chunk=self.decode_chunk, dv=self.dv, sink=self.sink)
+        self._finish(o, qkv, gate_col0, residual, out)
+
+    def _forward_rows(self, qkv, rope, table, step, cache, gate_col0, residual, out) -> None:
+        """The layer with norms over whole rows: input stage, means of the blocks this step completes, attention, the
+        heads' outputs turned back."""
+        T, ws, dt = qkv.shape[0], self.ctx.workspace, self.ctx.dtype
+        v_rope = self.value_position.table(step) if self.value_position is not None else None
+        q = ws.buffer("attn.q", (T, self.nq * self.d), dt)
+        ops.scope("attention.qk_norm_rotation_cache_write")
+        ops.rows_norm_rope_cache(qkv, q, self.q_norm, self.k_norm, self.qk_norm_eps, rope, self.rotary_dim, v_rope, step, table,
+                                 cache.k if cache.writable else None, cache.v if cache.writable else None, self.nq, self.nkv, self.d, self.dv)
+        pooled = None
+        if self.pool:
+            pooled = ops.PooledRows(self.pool, cache.pooled.k, cache.pooled.v, step.block_tables[cache.pooled.group])
+            if cache.writable:
+                ops.scope("attention.block_means")
+                ops.pool_means(cache.k, cache.v, pooled, step, table)
+        o = ws.buffer("attn.o", (T, self.nq * self.dv), dt)
+        ops.scope("attention.attention")
+        ops.attention(q, o, cache.k, cache.v, step, table, self.window or 0, self.scale, self.nq, self.nkv, self.d, workspace=ws,
+                      decode_chunk=self.decode_chunk, dv=self.dv, pooled=pooled)
+        if v_rope is not None:
+            ops.scope("attention.turn_back")
+            ops.turn_back(o, v_rope, self.nq)
         self._finish(o, qkv, gate_col0, residual, out)
 
     def _finish(self, o: torch.Tensor, qkv: torch.Tensor, gate_col0: int, residual: torch.Tensor, out: Optional[torch.Tensor]) -> None:

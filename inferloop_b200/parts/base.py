@@ -90,6 +90,7 @@ class PagedKVNeed:
     head_dim: int
     window: Optional[int] = None     # None: all keys are kept; n: only the last n are read
     v_head_dim: Optional[int] = None  # head size of the values when it is not the keys'; 0: the cached vector is all there is
+    stride: int = 1                  # tokens that one cached row stands for: n keeps a row per n tokens, once all n are there
 
     @property
     def value_dim(self) -> int:
@@ -108,6 +109,7 @@ class SlotStateNeed:
 class CacheNeeds:
     paged: Optional[PagedKVNeed] = None
     slots: Tuple[SlotStateNeed, ...] = ()
+    pooled: Optional[PagedKVNeed] = None     # a second set of pages of the layer: rows that stand for `stride` tokens each
 
 
 class Part:

@@ -10,7 +10,11 @@ that buffer, adds it to the stream, hands the next sublayer its input and zeroes
 
 Norms on both sides (`sandwich`): h += m * norm1b(mixer(norm1(h))); h += m * norm2b(ffn(norm2(h))) with a constant
 multiplier m on what joins the stream.  The norms are element-wise (Dynamic Tanh), so the norm on a sublayer's
-output, the sum into the stream and the norm in front of the next sublayer are one launch."""
+output, the sum into the stream and the norm in front of the next sublayer are one launch.
+
+Norm of the sum (`sum_norm`): h = norm1(a h + mixer(h)); h = norm2(a h + ffn(h)) with a constant multiplier a on the stream.
+The sublayers read the stream as it is and add into a 32-bit buffer that already holds a h; one kernel norms the buffer,
+writes the new stream and its copy for the next sublayer, and leaves a times the new stream in the buffer."""
 from __future__ import annotations
 
 from typing import List, Mapping
@@ -244,6 +248,70 @@ class SandwichBlock(Block):
             memo[self.PREPARED] = (y.data_ptr(), tuple(hidden.shape), id(nxt) if nxt is not None else None)
 
 
+class SumNormBlock(Block):
+    """spec: hidden_size; alpha (the stream's multiplier); tensor-name pieces mixer_prefix, ffn_prefix, mixer_norm, ffn_norm
+    (under the layer prefix).  The layer's norm must be a plain RMS norm."""
+
+    PREPARED = "sum_norm.prepared"          # memo key: (stream, copy, buffer, shape, alpha) that the block before left ready
+
+    def __init__(self, spec, ctx, prefix: str = "", layer=None) -> None:
+        super().__init__(spec, ctx, prefix)
+        self.hidden = int(spec["hidden_size"])
+        self.alpha = float(spec["alpha"])
+        self.norm1 = registry.build_norm(layer.norm, ctx, prefix + spec.get("mixer_norm", "norm1"), width=self.hidden)
+        self.norm2 = registry.build_norm(layer.norm, ctx, prefix + spec.get("ffn_norm", "norm2"), width=self.hidden)
+        self.mixer = registry.build("mixer", layer.mixer, ctx, prefix + spec.get("mixer_prefix", "mix."))
+        self.ffn = registry.build("feed_forward", layer.feed_forward, ctx, prefix + spec.get("ffn_prefix", "mlp."))
+        self.has_ffn = not getattr(self.ffn, "absent", False)
+        for n in (self.norm1, self.norm2):
+            if not isinstance(n, RMSNorm) or n.groups != 1:
+                raise ValueError("sum_norm: the norm of a sum must be an RMS norm over the whole row")
+
+    @property
+    def graph_safe(self) -> bool:
+        return bool(self.mixer.graph_safe and (not self.has_ffn or self.ffn.graph_safe))
+
+    def declare_weights(self) -> List[WeightDecl]:
+        second = self.norm2.declare_weights()
+        if not self.has_ffn:          # the absent sublayer's norm may be stored; it is not read
+            second = [WeightDecl(d.name, d.shape, d.role, d.init, d.root, True) for d in second]
+        return self.norm1.declare_weights() + self.mixer.declare_weights() + second + self.ffn.declare_weights()
+
+    def bind(self, tensors: Mapping[str, torch.Tensor]) -> None:
+        for part in (self.norm1, self.mixer) + ((self.norm2, self.ffn) if self.has_ffn else ()):
+            part.bind(tensors)
+
+    def cache_needs(self) -> CacheNeeds:
+        return self.mixer.cache_needs()
+
+    def scratch_bytes(self, tokens: int) -> int:
+        size = torch.empty((), dtype=self.ctx.dtype).element_size()
+        return tokens * self.hidden * (size + 4) + max(self.mixer.scratch_bytes(tokens), self.ffn.scratch_bytes(tokens) if self.has_ffn else 0)
+
+    def forward(self, hidden: torch.Tensor, step, cache) -> None:
+        ws = self.ctx.workspace
+        x = ws.buffer("block.normed", hidden.shape, self.ctx.dtype)          # what a sublayer reads
+        y = ws.buffer("block.sublayer_out", hidden.shape, torch.float32)     # alpha * stream, which it adds into
+        memo = getattr(step, "memo", None)
+        prepared = (hidden.data_ptr(), x.data_ptr(), y.data_ptr(), tuple(hidden.shape), self.alpha)
+        if memo is None or memo.pop(self.PREPARED, None) != prepared:
+            ops.scope("norm")
+            ops.cast_zero(hidden, x, y, self.alpha)
+        ops.scope("mixer")
+        self.mixer.forward(x, y, step, cache)
+        ops.scope("norm")
+        # (between the two sublayers only the copy and the next sum are read)
+        ops.sum_norm(y, self.norm1.weight, self.norm1.eps, self.alpha, None if self.has_ffn else hidden, x)
+        if self.has_ffn:
+            ops.scope("feed_forward")
+            self.ffn.forward(x, y, step)
+            ops.scope("norm")
+            ops.sum_norm(y, self.norm2.weight, self.norm2.eps, self.alpha, hidden, x)
+        if memo is not None:
+            memo[self.PREPARED] = prepared
+
+
 registry.register("block", "pre_norm", PreNormBlock)
+registry.register("block", "sum_norm", SumNormBlock)
 registry.register("block", "sandwich", SandwichBlock)
 registry.register("block", "output_norm", OutputNormBlock)

@@ -103,6 +103,46 @@ class SwiGLU(FeedForward):
         linear(act, self.w_down, residual, accumulate=accumulate)
 
 
+class TwoMatrixFeedForward(FeedForward):
+    """residual += W_down f(W_up x), f = `activation` ("relu2": relu squared, "tanh"), element by element.  spec:
+    hidden_size, intermediate_size, activation, names ((role "up" | "down", name under the prefix), ...)."""
+    graph_safe = True
+
+    def __init__(self, spec, ctx, prefix: str = "") -> None:
+        super().__init__(spec, ctx, prefix)
+        self.hidden = int(spec["hidden_size"])
+        self.inter = int(spec["intermediate_size"])
+        self.activation = str(spec["activation"])
+        if self.activation not in ops.ACTIVATIONS:
+            raise ValueError(f"two-matrix feed-forward: unknown activation {self.activation!r}")
+        names = {"up": "up_proj.weight", "down": "down_proj.weight"}
+        for role, name in spec.get("names", ()):
+            if role not in names:
+                raise ValueError(f"two-matrix feed-forward has no tensor role {role!r}")
+            names[role] = name
+        self.names = {k: prefix + v for k, v in names.items()}
+        self.w_up = self.w_down = None
+
+    def declare_weights(self) -> List[WeightDecl]:
+        return [WeightDecl(self.names["up"], (self.inter, self.hidden)), WeightDecl(self.names["down"], (self.hidden, self.inter))]
+
+    def bind(self, tensors: Mapping[str, torch.Tensor]) -> None:
+        self.w_up = tensors[self.names["up"]].contiguous()
+        self.w_down = tensors[self.names["down"]].contiguous()
+
+    def scratch_bytes(self, tokens: int) -> int:
+        return tokens * self.inter * torch.empty((), dtype=self.ctx.dtype).element_size()
+
+    def forward(self, x: torch.Tensor, residual: torch.Tensor, step, accumulate: bool = True) -> None:
+        act = self.ctx.workspace.buffer("mlp.act", (x.shape[0], self.inter), self.ctx.dtype)
+        ops.scope("feed_forward.up")
+        linear(x, self.w_up, act)
+        ops.scope("feed_forward.activation")
+        ops.act_rows(act, self.activation, act)
+        ops.scope("feed_forward.down")
+        linear(act, self.w_down, residual, accumulate=accumulate)
+
+
 class NoFeedForward(FeedForward):
     """A layer that has only its mixer: blocks skip the feed-forward's norm and sublayer."""
     graph_safe = True
@@ -113,4 +153,5 @@ class NoFeedForward(FeedForward):
 
 
 register("feed_forward", "swiglu", SwiGLU)
+register("feed_forward", "two_matrix", TwoMatrixFeedForward)
 register("feed_forward", "none", NoFeedForward)

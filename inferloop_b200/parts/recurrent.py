@@ -18,6 +18,14 @@ constant `out_scale`, and projected.  State per request: S [heads, dim, vdim] in
 state-space layer's scan with a stored decay and unit step sizes (csrc/ssm.cu, `fixed`), so long portions run in
 chunks side by side.
 
+`general_delta` (a delta rule with a decay and a removal rate per key channel): r, k, v, a, g = projections of h,
+w = exp(-c sigmoid(W_2 tanh(W_1 h) + w0)), a = sigmoid(a + ab), u = k / sqrt(sum(k^2) + unit_eps) per head,
+
+    S_t = diag(w) S_{t-1} - (a u)(u^T S_{t-1}) + k v^T,   o_t = S_t^T r
+
+each head's o is RMS-normed by itself, the heads together are multiplied by a weight and by sigmoid(g), and projected.  State
+per request: S [heads, dim, vdim] in 32-bit.  All projections of h are one product; the kernels are csrc/delta.cu.
+
 `parallel`: several mixers read the same input and add into the same output, each with its own tensors under its
 own prefix, its own cache (at most one of them paged) and its own constant on its output.
 """
@@ -29,7 +37,7 @@ from typing import List, Mapping
 import torch
 
 from ..csrc import ops
-from ..weights.decl import WeightDecl
+from ..weights.decl import FreeDim, WeightDecl
 from . import registry
 from .base import CacheNeeds, Mixer, SlotStateNeed
 from .linear import linear
@@ -203,6 +211,81 @@ class DecayedLinearAttention(Mixer):
             linear(gated, self.w_o, residual, accumulate=True)
 
 
+class GeneralDelta(Mixer):
+    """spec: hidden_size, heads, head_dim, v_head_dim (default head_dim), eps, log_decay (c), unit_eps, rank (what random
+    weights get as the inner size of the decay's map; a stored model's tensors decide it), names."""
+    graph_safe = True
+
+    def __init__(self, spec, ctx, prefix: str = "") -> None:
+        super().__init__(spec, ctx, prefix)
+        self.hidden = int(spec["hidden_size"])
+        self.heads = int(spec["heads"])
+        self.d = int(spec["head_dim"])
+        self.dv = int(spec.get("v_head_dim") or self.d)
+        self.eps = float(spec["eps"])
+        self.log_decay = float(spec["log_decay"])
+        self.unit_eps = float(spec["unit_eps"])
+        self.rank = int(spec.get("rank") or self.d)
+        self.inner_k, self.inner_v = self.heads * self.d, self.heads * self.dv
+        self.names = _names({"r": "r", "k": "k", "v": "v", "g": "g", "a": "a", "ab": "a.b", "w1": "w1", "w2": "w2", "w0": "w0",
+                             "norm": "norm", "o": "o"}, spec, prefix, "the delta rule")
+        # columns of the one projection: r | k | a | v | g | the decay map's inner row (padded to a multiple of eight)
+        self.col_k, self.col_a, self.col_v = self.inner_k, 2 * self.inner_k, 3 * self.inner_k
+        self.col_g = self.col_v + self.inner_v
+        self.col_low = self.col_g + self.inner_v
+        self.w_in = self.w2 = self.w0 = self.ab = self.norm_w = self.w_o = None
+
+    def declare_weights(self) -> List[WeightDecl]:
+        n, H = self.names, self.hidden
+        rank = FreeDim(self.rank, n["w1"])
+        return [WeightDecl(n["r"], (self.inner_k, H)), WeightDecl(n["k"], (self.inner_k, H)), WeightDecl(n["v"], (self.inner_v, H)),
+                WeightDecl(n["g"], (self.inner_v, H)), WeightDecl(n["a"], (self.inner_k, H)), WeightDecl(n["ab"], (self.inner_k,), "vector", "bias"),
+                WeightDecl(n["w1"], (rank, H)), WeightDecl(n["w2"], (self.inner_k, rank)), WeightDecl(n["w0"], (self.inner_k,), "vector", "bias"),
+                WeightDecl(n["norm"], (self.inner_v,), "vector", "norm"), WeightDecl(n["o"], (H, self.inner_v))]
+
+    def bind(self, tensors: Mapping[str, torch.Tensor]) -> None:
+        n = self.names
+        w1, w2 = tensors[n["w1"]], tensors[n["w2"]]
+        if w1.shape[0] != w2.shape[1]:
+            raise ValueError(f"{n['w1']} and {n['w2']} do not meet: {tuple(w1.shape)} and {tuple(w2.shape)}")
+        self.rank = w1.shape[0]
+        pad = -self.rank % 8
+        rows = [tensors[n[k]] for k in ("r", "k", "a", "v", "g")] + [w1, w1.new_zeros(pad, self.hidden)]
+        self.w_in = torch.cat(rows, dim=0).contiguous()
+        self.w2 = torch.cat([w2, w2.new_zeros(self.inner_k, pad)], dim=1).contiguous()
+        self.w0, self.ab = tensors[n["w0"]].contiguous(), tensors[n["ab"]].contiguous()
+        self.norm_w = tensors[n["norm"]].contiguous()
+        self.w_o = tensors[n["o"]].contiguous()
+
+    def cache_needs(self) -> CacheNeeds:
+        return CacheNeeds(slots=(SlotStateNeed("state", (self.heads, self.d, self.dv), torch.float32),))
+
+    def scratch_bytes(self, tokens: int) -> int:
+        size = torch.empty((), dtype=self.ctx.dtype).element_size()
+        wide = -(-self.rank // 8) * 8
+        return tokens * ((self.col_low + 2 * wide + self.inner_v) * size + (self.inner_k + self.inner_v) * 4)
+
+    def forward(self, x: torch.Tensor, residual: torch.Tensor, step, cache) -> None:
+        T, ws, dt = x.shape[0], self.ctx.workspace, self.ctx.dtype
+        proj = ws.buffer("delta.proj", (T, self.w_in.shape[0]), dt)
+        ops.scope("delta.in_projection")
+        linear(x, self.w_in, proj)
+        ops.scope("delta.decay_map")
+        low = ws.buffer("delta.low", (T, self.w2.shape[1]), dt)
+        ops.act_rows(proj[:, self.col_low:], "tanh", low)
+        decay = ws.buffer("delta.decay", (T, self.inner_k), torch.float32)
+        linear(low, self.w2, decay)
+        ops.scope("delta.scan")
+        y = ws.buffer("delta.y", (T, self.inner_v), torch.float32)
+        ops.delta_scan(proj, 0, self.col_k, self.col_v, self.col_a, decay, self.w0, self.ab, self.log_decay, self.unit_eps,
+                       cache.state["state"], y, step, self.heads, self.d, self.dv)
+        ops.scope("delta.norm_gate")
+        gated = ws.buffer("delta.gated", (T, self.inner_v), dt)
+        ops.rms_gate(y, proj[:, self.col_g:], self.norm_w, self.eps, gated, groups=self.heads)
+        ops.scope("delta.out_projection")
+        linear(gated, self.w_o, residual, accumulate=True)
+
+
 class ParallelMixers(Mixer):
     """spec: `branches` = ((sub-prefix, PartSpec of role mixer), ...).  Every branch reads the block's input and adds
     into the block's output; a branch's constant on its output is its own parameter (`out_scale`).  Branches that start
@@ -300,4 +383,5 @@ class ParallelMixers(Mixer):
 
 registry.register("mixer", "gated_linear_recurrence", GatedLinearRecurrence)
 registry.register("mixer", "decayed_linear_attention", DecayedLinearAttention)
+registry.register("mixer", "general_delta", GeneralDelta)
 registry.register("mixer", "parallel", ParallelMixers)

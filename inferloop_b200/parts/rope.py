@@ -12,6 +12,11 @@ step that has the same constants.
 `scaling` = (factor, low, high, original) rescales the frequencies by wavelength, as Llama 3.1 does: with
 wavelength l = 2 pi / f, f is kept where l < original / high, divided by `factor` where l > original / low, and in
 between becomes (1 - s) f / factor + s f with s = (original / l - low) / (high - low).
+
+`ramp` = (factor, original, fast, slow) blends along the pair's number instead, as YaRN does: with
+place(t) = rd ln(original / (2 pi t)) / (2 ln theta), the pair whose wave turns t times over `original` positions,
+lo = max(floor(place(fast)), 0), hi = min(ceil(place(slow)), rd - 1) and r_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1),
+the frequency is (f / factor) r_i + f (1 - r_i), and cos and sin are both multiplied by 0.1 ln(factor) + 1.
 """
 from __future__ import annotations
 
@@ -41,11 +46,26 @@ class RopeNeox(PositionEncoding):
             factor, low, high, original = self.scaling
             if factor <= 0 or original <= 0 or low <= 0 or high <= low:
                 raise ValueError(f"rope scaling {self.scaling}: factor, low and original must be positive and high above low")
+        ramp = spec.get("ramp")
+        self.ramp = None if ramp is None else tuple(float(v) for v in ramp)
+        if self.ramp is not None:
+            if self.scaling is not None:
+                raise ValueError("rope: frequencies are rescaled by wavelength or along a ramp, not both")
+            if min(self.ramp) <= 0 or self.theta == 1.0:
+                raise ValueError(f"rope ramp {self.ramp}: all four must be positive, and the base not one")
+        self.stretch = 1.0 if self.ramp is None else 0.1 * math.log(self.ramp[0]) + 1.0      # what cos and sin are multiplied by
         self._inv_freq: Optional[torch.Tensor] = None
 
     @property
     def key(self):
-        return ("rope", self.theta, self.rotary_dim, self.scaling)
+        return ("rope", self.theta, self.rotary_dim, self.scaling, self.ramp)
+
+    def _blended(self, i: int, f: float) -> float:
+        factor, original, fast, slow = self.ramp
+        place = lambda turns: self.rotary_dim * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(self.theta))
+        lo, hi = max(math.floor(place(fast)), 0), min(math.ceil(place(slow)), self.rotary_dim - 1)
+        r = min(max((i - lo) / max(hi - lo, 0.001), 0.0), 1.0)
+        return f / factor * r + f * (1.0 - r)
 
     def _scaled(self, f: float) -> float:
         if self.scaling is None:
@@ -63,6 +83,8 @@ class RopeNeox(PositionEncoding):
         if self._inv_freq is None:
             half = self.rotary_dim // 2
             host = [self._scaled(self.theta ** (-(2.0 * i) / self.rotary_dim)) for i in range(half)]
+            if self.ramp is not None:
+                host = [self._blended(i, f) for i, f in enumerate(host)]
             self._inv_freq = torch.tensor(host, dtype=torch.float64, device=self.ctx.device)
         return self._inv_freq
 
@@ -71,8 +93,8 @@ class RopeNeox(PositionEncoding):
         if cached is None:
             half = self.rotary_dim // 2
             cached = self.ctx.workspace.buffer(
-                f"rope_table/{self.theta}/{self.rotary_dim}/{self.scaling}", (step.n_tokens, half, 2), torch.float32)
-            ops.rope_table(step.positions, self.inv_freq(), cached)
+                f"rope_table/{self.theta}/{self.rotary_dim}/{self.scaling}/{self.ramp}", (step.n_tokens, half, 2), torch.float32)
+            ops.rope_table(step.positions, self.inv_freq(), cached, self.stretch)
             step.position_tables[self.key] = cached
         return cached
 

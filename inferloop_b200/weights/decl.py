@@ -5,9 +5,34 @@ from dataclasses import dataclass
 from typing import Tuple
 
 
+class FreeDim(int):
+    """A dimension that the configuration does not give: the stored tensor decides it.  All dimensions of one
+    `name` must agree within a model; the number itself is what random weights are made with."""
+
+    name: str
+
+    def __new__(cls, size: int, name: str) -> "FreeDim":
+        self = super().__new__(cls, size)
+        self.name = name
+        return self
+
+
+def shapes_agree(declared, stored, found) -> bool:
+    """Whether a stored shape is the declared one.  `found` remembers what each free dimension turned out to be."""
+    if len(declared) != len(stored):
+        return False
+    for d, s in zip(declared, stored):
+        if isinstance(d, FreeDim):
+            if s <= 0 or found.setdefault(d.name, int(s)) != s:
+                return False
+        elif d != s:
+            return False
+    return True
+
+
 @dataclass(frozen=True)
 class WeightDecl:
-    """One tensor a part needs, by name.
+    """One tensor a part needs, by name.  A dimension of `shape` may be a :class:`FreeDim`.
 
     role:  "matrix" and "table" follow the engine's compute dtype (bfloat16, or float32
            on the 32-bit path); "vector" (norm weights, biases) is held in float32, which

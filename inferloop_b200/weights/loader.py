@@ -15,7 +15,7 @@ from typing import Callable, Dict, Iterable, List, Mapping, Optional, Sequence, 
 
 import torch
 
-from .decl import WeightDecl
+from .decl import WeightDecl, shapes_agree
 from .safetensors_io import TensorSource
 
 _FLOAT = ("F32", "BF16", "F16", "F64")
@@ -85,11 +85,11 @@ def load_weights(folder: str, decls: Sequence[WeightDecl], prefixes: Sequence[st
         full = {(d.name if d.root else prefix + d.name): d for d in decls}
         missing = [n for n, d in full.items() if n not in source.where and not d.optional]
         unexpected = sorted(n for n in stored if n not in full)
-        wrong_shape, wrong_dtype = [], []
+        wrong_shape, wrong_dtype, free = [], [], {}
         for n, d in full.items():
             if n in source.where:
                 e = source.entry(n)
-                if tuple(e.shape) != tuple(d.shape):
+                if not shapes_agree(d.shape, e.shape, free):
                     wrong_shape.append((n, tuple(d.shape), tuple(e.shape)))
                 ok = _INT if d.role == "int" else _FLOAT
                 if e.dtype not in ok:
