@@ -31,6 +31,10 @@
 //            and patches them into the tile in shared memory.  The producer warp then reads
 //            nothing that the preceding kernel writes and starts its stream before the
 //            dependency wait.
+//   pooled   (kMode 2) a window with pooled blocks before it: the tiles of a second set of pages (row b =
+//            the mean of block b of `pool` positions) come first in the deal, then the window's;
+//            values may have another head size (DV) than keys, q comes ready, and with `turn` the
+//            merged row is turned back in pairs (i, i + DV / 2) as it is written.
 // Every mbarrier wait is bounded; on expiry a flag is raised and the CTA leaves (or, in the
 // form with cluster barriers, still walks to them), so nobody is left waiting.  No multicast.
 //
@@ -86,6 +90,9 @@ struct Params {
   // v_first [tokens][nkv * D]; 2: they become (1 - lambda) v + lambda v_first before they are cached.
   int mode, rotary_dim, v_mode;
   __nv_bfloat16* v_first; const float* v_lambda;
+  // kMode 2: block table and pages of the pooled rows, tokens a row stands for, (cos, sin) [tokens][DV / 2] or null
+  const int* p_table; int p_num_pages, pool;
+  const float2* turn;
 };
 
 constexpr int kPairsInterleaved = 1, kNormAfterRotation = 2, kNormUnweighted = 4;
@@ -115,8 +122,8 @@ struct RowState {
 // 16 keys (rows row0 .. row0 + 15 of the tile's K and V slices, the first being key
 // `key0`) against the warp's 16 query rows.  live[r]: row g + 8r is a head of the group;
 // keys outside [lo, hi) are not seen.
-template <int D>
-__device__ __forceinline__ void tile_step(RowState<D>& st, const uint32_t (&q)[D / 16][4], uint32_t ks, uint32_t vs,
+template <int D, int DV>
+__device__ __forceinline__ void tile_step(RowState<DV>& st, const uint32_t (&q)[D / 16][4], uint32_t ks, uint32_t vs,
                                           int row0, int key0, const bool (&live)[2], int lo, int hi, float scale_log2,
                                           int lane) {
   constexpr uint32_t kSlice = kKeys * 128;           // bytes of one 64-wide slice of a tile
@@ -170,7 +177,7 @@ __device__ __forceinline__ void tile_step(RowState<D>& st, const uint32_t (&q)[D
 #pragma unroll
   for (int r = 0; r < 2; ++r) st.l[r] = st.l[r] * corr[r] + sum[r];
 #pragma unroll
-  for (int i = 0; i < D / 8; ++i) {
+  for (int i = 0; i < DV / 8; ++i) {
     st.o[i][0] *= corr[0]; st.o[i][1] *= corr[0];
     st.o[i][2] *= corr[1]; st.o[i][3] *= corr[1];
   }
@@ -180,7 +187,7 @@ __device__ __forceinline__ void tile_step(RowState<D>& st, const uint32_t (&q)[D
   a[2] = pack_bf16(s[1][0], s[1][1]);
   a[3] = pack_bf16(s[1][2], s[1][3]);
 #pragma unroll
-  for (int nd = 0; nd < D / 16; ++nd) {
+  for (int nd = 0; nd < DV / 16; ++nd) {
     uint32_t r0, r1, r2, r3;
     const int col = nd * 16 + (lane >> 4) * 8;
     ldmatrix_x4_trans(swz(vs + (col >> 6) * kSlice, row0 + (lane & 7) + ((lane >> 3) & 1) * 8, (col & 63) >> 3), r0, r1, r2, r3);
@@ -474,15 +481,20 @@ __device__ __forceinline__ void patch_new_key_variant(uint32_t ks, uint32_t vs, 
   __syncwarp();
 }
 
-template <int D, int kStages, bool kVariant>
+// kMode: 0 the stock input stage (or none), 1 its variants, 2 pooled blocks before a window.
+template <int D, int DV, int kStages, int kMode>
 __global__ void __launch_bounds__(kThreads)
 decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
-              const __grid_constant__ CUtensorMap map_k_run, const __grid_constant__ CUtensorMap map_v_run, const Params p) {
-  constexpr int kSlices = D / 64;
+              const __grid_constant__ CUtensorMap map_k_run, const __grid_constant__ CUtensorMap map_v_run,
+              const __grid_constant__ CUtensorMap map_pk, const __grid_constant__ CUtensorMap map_pv, const Params p) {
+  constexpr bool kVariant = kMode == 1, kPool = kMode == 2;
+  static_assert(kPool || D == DV, "values of another head size come with the pooled form");
+  constexpr int kSlices = D / 64, kSlicesV = DV / 64;
   constexpr uint32_t kSlice = kKeys * 128;                 // bytes: one slice of one tensor of a tile
   constexpr uint32_t kTensor = kSlices * kSlice;           // K (or V) of a tile
-  constexpr uint32_t kStage = 2 * kTensor;
-  constexpr int kRec = D + 2;                              // O row, then max and sum
+  constexpr uint32_t kTensorV = kSlicesV * kSlice;
+  constexpr uint32_t kStage = kTensor + kTensorV;
+  constexpr int kRec = DV + 2;                             // O row, then max and sum
   static_assert(kConsumers * 16 * kRec * 4 <= kStages * (int)kStage, "records must fit the tile ring");
 
   extern __shared__ __align__(1024) uint8_t smem_raw[];
@@ -492,8 +504,8 @@ decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + kStages * kStage);
   const uint32_t full0 = smem_u32(bars), empty0 = full0 + 8 * kStages;
   volatile int* failed = reinterpret_cast<volatile int*>(bars + 2 * kStages);
-  // Records that the cluster sends here: [source CTA][row of this CTA][D + 4] (O, max, sum)
-  constexpr int kRecIn = D + 4;
+  // Records that the cluster sends here: [source CTA][row of this CTA][DV + 4] (O, max, sum)
+  constexpr int kRecIn = DV + 4;
   const uint32_t inbox_bar = smem_u32(bars + 2 * kStages + 1);
   float* inbox = reinterpret_cast<float*>(bars + 2 * kStages + 2);
 
@@ -515,7 +527,7 @@ decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__
     if (push) mbar_init(inbox_bar, 1);
     *failed = 0;
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
-    if (push && rows_mine > 0) mbar_expect_tx(inbox_bar, (uint32_t)(rows_mine * p.split * (D * 4 + 8)));
+    if (push && rows_mine > 0) mbar_expect_tx(inbox_bar, (uint32_t)(rows_mine * p.split * (DV * 4 + 8)));
   }
   if (push) cluster_sync_all();          // every owner's mbarrier is ready before anything is sent to it
   else __syncthreads();
@@ -535,19 +547,36 @@ decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__
   const int lo = (p.window > 0 && pos + 1 > p.window) ? pos + 1 - p.window : 0;
   const int hi = pos + 1;
   const int kSplit = p.split;
-  const int all_tiles = (hi + kKeys - 1) / kKeys - lo / kKeys;
+  const int n_pooled = kPool ? lo / p.pool : 0, pool_tiles = (n_pooled + kKeys - 1) / kKeys;      // pooled rows this token sees, and their tiles
+  const int all_tiles = pool_tiles + (hi + kKeys - 1) / kKeys - lo / kKeys;
   // the clusters that take part for this sequence, and this one's run of tiles
   int chunks_on = all_tiles / (kSplit * kChunkTiles);
   chunks_on = chunks_on < 1 ? 1 : (chunks_on > p.chunks ? p.chunks : chunks_on);
   if (chunk >= chunks_on) return;                          // (the whole cluster: nothing has been sent yet)
   const int per_chunk = (all_tiles + chunks_on - 1) / chunks_on;
-  const int first_tile = lo / kKeys + chunk * per_chunk;
+  const int deal0 = chunk * per_chunk;                     // this cluster's first tile, of all of them
+  const int first_tile = lo / kKeys + deal0 - pool_tiles;
   const int n_tiles = min(per_chunk, all_tiles - chunk * per_chunk);
   const int n_my = rank < n_tiles ? (n_tiles - rank + kSplit - 1) / kSplit : 0;
   const int* table = p.block_table + (size_t)seq * p.max_blocks;
   const int rows16 = (G + 15) / 16 * 16;
   const int n_passes = rows16 / 16;
-  auto key_of = [&](int j) { return (first_tile + rank + j * kSplit) * kKeys; };
+  auto in_pool = [&](int j) { return kPool && deal0 + rank + j * kSplit < pool_tiles; };      // this CTA's tile j holds pooled rows
+  auto key_of = [&](int j) { return ((in_pool(j) ? deal0 : first_tile) + rank + j * kSplit) * kKeys; };
+  const float2* turn = kPool && p.turn != nullptr ? p.turn + (size_t)tok * (DV / 2) : nullptr;
+  // Writes element pairs (m, m + DV / 2) of a head's row, turned back, from what `value(c)` gives for column c.
+  auto emit_pair = [&](int head, int m, auto&& value) {
+    float a = value(m), b = value(m + DV / 2);
+    if (turn != nullptr) {
+      const float2 w = __ldg(turn + m);
+      const float t = fmaf(b, w.y, a * w.x);
+      b = fmaf(-a, w.y, b * w.x);
+      a = t;
+    }
+    __nv_bfloat16* dst = p.out + (size_t)tok * p.out_stride + (size_t)head * DV + m;
+    dst[0] = __float2bfloat16_rn(a);
+    dst[DV / 2] = __float2bfloat16_rn(b);
+  };
 
   for (int pass = 0; pass < n_passes; ++pass) {            // 16 query heads of the group at a time
     const int rb = pass * 16;
@@ -558,9 +587,15 @@ decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__
       const int parts = kKeys / box_keys;
       const int per_tensor = kSlices * parts;
       const int b = lane;
-      const bool has_box = b < 2 * per_tensor;
-      const int which = b / per_tensor, rem = b % per_tensor, slice = rem / parts, part = rem % parts;
+      const bool has_box = b < per_tensor + kSlicesV * parts;
+      const int which = b / per_tensor > 0 ? 1 : 0, rem = b - which * per_tensor, slice = rem / parts, part = rem % parts;
       auto lookup = [&](int j) {                           // page of this lane's box of tile j, or one past the tensor
+        if (in_pool(j)) {
+          const int row = key_of(j) + part * box_keys, blk = row / p.page_size;
+          int pg = -1;
+          if (has_box && j < n_my && row < n_pooled && blk < p.max_blocks) pg = __ldg(p.p_table + (size_t)seq * p.max_blocks + blk);
+          return pg >= 0 && pg < p.p_num_pages ? pg : p.p_num_pages;
+        }
         int page = p.num_pages;
         if (has_box && j < n_my) {
           const int key = key_of(j) + part * box_keys;
@@ -591,14 +626,15 @@ decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__
           // The TMA unit's time per box hardly depends on its size: two 16-key pages that
           // follow one another in the pool come as one box.
           const int page_nb = __shfl_down_sync(0xffffffffu, pg[i], 1);
-          const bool run = has_box && parts == 2 && part == 0 && pg[i] + 1 < p.num_pages && page_nb == pg[i] + 1;
+          const bool pooled = in_pool(j);
+          const bool run = has_box && parts == 2 && part == 0 && pg[i] + 1 < p.num_pages && page_nb == pg[i] + 1 && !pooled;
           const bool covered = __shfl_up_sync(0xffffffffu, run ? 1 : 0, 1) != 0 && part == 1;
           if (run)
             tma_load_4d(base + s * kStage + which * kTensor + slice * kSlice, which == 0 ? &map_k_run : &map_v_run,
                         full0 + 8 * s, slice * 64, 0, kvh, pg[i]);
           else if (has_box && !covered)
             tma_load_4d(base + s * kStage + which * kTensor + slice * kSlice + part * box_keys * 128,
-                        which == 0 ? &map_k : &map_v, full0 + 8 * s, slice * 64, (key_of(j) + part * box_keys) % p.page_size,
+                        pooled ? (which == 0 ? &map_pk : &map_pv) : (which == 0 ? &map_k : &map_v), full0 + 8 * s, slice * 64, (key_of(j) + part * box_keys) % p.page_size,
                         kvh, pg[i]);
           pg[i] = lookup(j + kAhead);
         }
@@ -607,13 +643,13 @@ decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__
     } else {
       // ------------------------------------------------------------ consumers
       const int g = lane >> 2, t = lane & 3;
-      RowState<D> st;
+      RowState<DV> st;
       st.init();
       bool live[2];
       uint32_t q[D / 16][4];
 #pragma unroll
       for (int r = 0; r < 2; ++r) live[r] = rb + g + 8 * r < G;
-      if (p.qkv != nullptr) {
+      if (!kPool && p.qkv != nullptr) {
         const __nv_bfloat16* base_q = p.qkv + (size_t)tok * p.qkv_stride + (size_t)(kvh * G + rb) * D;
         if constexpr (kVariant)
           load_q_variant<D>(q, live[0] ? base_q + (size_t)g * D : nullptr, live[1] ? base_q + (size_t)(g + 8) * D : nullptr,
@@ -639,7 +675,8 @@ decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__
         ok = mbar_wait(full0 + 8 * s, (it / kStages) & 1);
         if (!ok) break;
         const int key0 = key_of(j) + warp * 16;
-        if (p.qkv != nullptr && p.k_write != nullptr && pos >= key0 && pos < key0 + 16) {
+        const int see_lo = in_pool(j) ? 0 : lo, see_hi = in_pool(j) ? n_pooled : hi;
+        if constexpr (!kPool) if (p.qkv != nullptr && p.k_write != nullptr && pos >= key0 && pos < key0 + 16) {
           // this warp's slice of this tile holds the step's own position: its key and value
           // are not in the cache yet (the tile came with whatever the page held there)
           const __nv_bfloat16* row = p.qkv + (size_t)tok * p.qkv_stride;
@@ -661,8 +698,8 @@ decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__
           // TMA will write this stage again later: order these ordinary stores before it
           asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
         }
-        if (key0 < hi)
-          tile_step<D>(st, q, base + s * kStage, base + s * kStage + kTensor, warp * 16, key0, live, lo, hi, p.scale_log2, lane);
+        if (key0 < see_hi)
+          tile_step<D, DV>(st, q, base + s * kStage, base + s * kStage + kTensor, warp * 16, key0, live, see_lo, see_hi, p.scale_log2, lane);
         __syncwarp();
         if (lane == 0) mbar_arrive(empty0 + 8 * s);
       }
@@ -679,24 +716,24 @@ decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__
           l += __shfl_xor_sync(0xffffffffu, l, 2);
           l2[r] = l;
         }
-        constexpr int kDump = D / 2 + 4;                     // floats a lane leaves: O fragments, two maxima, two sums
+        constexpr int kDump = DV / 2 + 4;                    // floats a lane leaves: O fragments, two maxima, two sums
         float* dump = reinterpret_cast<float*>(smem);        // [kDump][32]
         static_assert(kDump * 32 * 4 <= kStages * (int)kStage, "a warp's fragments must fit the tile ring");
         asm volatile("bar.sync 1, %0;" ::"n"(kConsumers * 32) : "memory");
         if (warp == 1) {
 #pragma unroll
-          for (int i = 0; i < D / 8; ++i)
+          for (int i = 0; i < DV / 8; ++i)
 #pragma unroll
             for (int c = 0; c < 4; ++c) dump[(i * 4 + c) * 32 + lane] = st.o[i][c];
 #pragma unroll
-          for (int r = 0; r < 2; ++r) { dump[(D / 2 + r) * 32 + lane] = st.m[r]; dump[(D / 2 + 2 + r) * 32 + lane] = l2[r]; }
+          for (int r = 0; r < 2; ++r) { dump[(DV / 2 + r) * 32 + lane] = st.m[r]; dump[(DV / 2 + 2 + r) * 32 + lane] = l2[r]; }
         }
         asm volatile("bar.sync 1, %0;" ::"n"(kConsumers * 32) : "memory");
         if (warp == 0) {
           float f0[2], f1[2];
 #pragma unroll
           for (int r = 0; r < 2; ++r) {
-            const float m1 = dump[(D / 2 + r) * 32 + lane], l1 = dump[(D / 2 + 2 + r) * 32 + lane];
+            const float m1 = dump[(DV / 2 + r) * 32 + lane], l1 = dump[(DV / 2 + 2 + r) * 32 + lane];
             const float m = fmaxf(st.m[r], m1);
             f0[r] = st.m[r] == -INFINITY ? 0.f : exp2f(st.m[r] - m);
             f1[r] = m1 == -INFINITY ? 0.f : exp2f(m1 - m);
@@ -704,7 +741,7 @@ decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__
             l2[r] = l2[r] * f0[r] + l1 * f1[r];
           }
 #pragma unroll
-          for (int i = 0; i < D / 8; ++i)
+          for (int i = 0; i < DV / 8; ++i)
 #pragma unroll
             for (int c = 0; c < 4; ++c) st.o[i][c] = st.o[i][c] * f0[c >> 1] + dump[(i * 4 + c) * 32 + lane] * f1[c >> 1];
           // Row g + 8r goes to CTA (row % S), place row / S.  A lane holds pairs of columns;
@@ -718,7 +755,7 @@ decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__
             const uint32_t at = smem_u32(inbox) + 4u * (uint32_t)((me * rows_cap + row / kSplit) * kRecIn);
             const uint32_t dst = peer_addr(at, owner), bar = peer_addr(inbox_bar, owner);
 #pragma unroll
-            for (int i0 = 0; i0 < D / 8; i0 += 2) {
+            for (int i0 = 0; i0 < DV / 8; i0 += 2) {
               const float ax = st.o[i0][2 * r], ay = st.o[i0][2 * r + 1], bx = st.o[i0 + 1][2 * r], by = st.o[i0 + 1][2 * r + 1];
               const float rx = __shfl_xor_sync(0xffffffffu, odd ? ax : bx, 1), ry = __shfl_xor_sync(0xffffffffu, odd ? ay : by, 1);
               if (live[r]) {
@@ -726,7 +763,7 @@ decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__
                 else st_peer_v4(dst + 4u * (uint32_t)((i0 + 1) * 8 + 2 * (t - 1)), bar, rx, ry, bx, by);
               }
             }
-            if (live[r] && t == 0) st_peer_v2(dst + 4u * (uint32_t)D, bar, st.m[r], l2[r]);
+            if (live[r] && t == 0) st_peer_v2(dst + 4u * (uint32_t)DV, bar, st.m[r], l2[r]);
           }
         }
       } else {
@@ -739,8 +776,8 @@ decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__
         l += __shfl_xor_sync(0xffffffffu, l, 2);
         float* row = rec + ((size_t)warp * 16 + g + 8 * r) * kRec;
 #pragma unroll
-        for (int i = 0; i < D / 8; ++i) { row[i * 8 + 2 * t] = st.o[i][2 * r]; row[i * 8 + 2 * t + 1] = st.o[i][2 * r + 1]; }
-        if (t == 0) { row[D] = st.m[r]; row[D + 1] = l; }
+        for (int i = 0; i < DV / 8; ++i) { row[i * 8 + 2 * t] = st.o[i][2 * r]; row[i * 8 + 2 * t + 1] = st.o[i][2 * r + 1]; }
+        if (t == 0) { row[DV] = st.m[r]; row[DV + 1] = l; }
       }
       }
     }
@@ -749,26 +786,42 @@ decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__
       if (rows_mine > 0) {
         if (!mbar_wait(inbox_bar, 0)) { *failed = 1; if (p.error_flag) *p.error_flag = 1; return; }
         const int n_rec = kSplit;
-        for (int e = threadIdx.x; e < rows_mine * D; e += kThreads) {
-          const int slot = e / D, c = e % D, row = slot * kSplit + rank;
+        auto merged = [&](int slot, int c, float& m_all, float& l_all) {
           const float* first = inbox + (size_t)slot * kRecIn;
-          float m_all = -INFINITY;
-          for (int i = 0; i < n_rec; ++i) m_all = fmaxf(m_all, first[(size_t)i * rows_cap * kRecIn + D]);
-          float l_all = 0.f, o = 0.f;
+          m_all = -INFINITY;
+          for (int i = 0; i < n_rec; ++i) m_all = fmaxf(m_all, first[(size_t)i * rows_cap * kRecIn + DV]);
+          float o = 0.f;
+          l_all = 0.f;
           for (int i = 0; i < n_rec; ++i) {
             const float* rcd = first + (size_t)i * rows_cap * kRecIn;
-            const float m = rcd[D];
+            const float m = rcd[DV];
             const float f = (m == -INFINITY) ? 0.f : exp2f(m - m_all);
-            l_all += rcd[D + 1] * f;
+            l_all += rcd[DV + 1] * f;
             o += rcd[c] * f;
           }
+          return o;
+        };
+        if (kPool && chunks_on == 1) {
+          for (int e = threadIdx.x; e < rows_mine * (DV / 2); e += kThreads) {
+            const int slot = e / (DV / 2);
+            emit_pair(kvh * G + slot * kSplit + rank, e % (DV / 2), [&](int c) {
+              float m_all, l_all;
+              const float o = merged(slot, c, m_all, l_all);
+              return l_all > 0.f ? o / l_all : 0.f;
+            });
+          }
+        } else
+        for (int e = threadIdx.x; e < rows_mine * DV; e += kThreads) {
+          const int slot = e / DV, c = e % DV, row = slot * kSplit + rank;
+          float m_all, l_all;
+          const float o = merged(slot, c, m_all, l_all);
           if (chunks_on == 1) {
-            p.out[(size_t)tok * p.out_stride + (size_t)(kvh * G + row) * D + c] = __float2bfloat16_rn(l_all > 0.f ? o / l_all : 0.f);
+            p.out[(size_t)tok * p.out_stride + (size_t)(kvh * G + row) * DV + c] = __float2bfloat16_rn(l_all > 0.f ? o / l_all : 0.f);
           } else {
             // this cluster's record of the row, for the owner that comes last
-            float* rcd = p.scratch + ((((size_t)seq * p.nkv + kvh) * p.chunks + chunk) * 16 + row) * (D + 2);
+            float* rcd = p.scratch + ((((size_t)seq * p.nkv + kvh) * p.chunks + chunk) * 16 + row) * (DV + 2);
             rcd[c] = o;
-            if (c == 0) { rcd[D] = m_all; rcd[D + 1] = l_all; }
+            if (c == 0) { rcd[DV] = m_all; rcd[DV + 1] = l_all; }
           }
         }
         if (chunks_on > 1) {
@@ -787,20 +840,30 @@ decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__
           __syncthreads();
           if (last_ticket) {
             __threadfence();
-            const float* base_rec = p.scratch + (((size_t)seq * p.nkv + kvh) * p.chunks) * 16 * (D + 2);
-            for (int e = threadIdx.x; e < rows_mine * D; e += kThreads) {
-              const int c = e % D, row = (e / D) * kSplit + rank;
+            const float* base_rec = p.scratch + (((size_t)seq * p.nkv + kvh) * p.chunks) * 16 * (DV + 2);
+            auto total = [&](int row, int c) {
               float m_all = -INFINITY;
-              for (int z = 0; z < chunks_on; ++z) m_all = fmaxf(m_all, __ldcg(base_rec + ((size_t)z * 16 + row) * (D + 2) + D));
+              for (int z = 0; z < chunks_on; ++z) m_all = fmaxf(m_all, __ldcg(base_rec + ((size_t)z * 16 + row) * (DV + 2) + DV));
               float l_all = 0.f, o = 0.f;
               for (int z = 0; z < chunks_on; ++z) {
-                const float* rcd = base_rec + ((size_t)z * 16 + row) * (D + 2);
-                const float m = __ldcg(rcd + D);
+                const float* rcd = base_rec + ((size_t)z * 16 + row) * (DV + 2);
+                const float m = __ldcg(rcd + DV);
                 const float f = (m == -INFINITY) ? 0.f : exp2f(m - m_all);
-                l_all += __ldcg(rcd + D + 1) * f;
+                l_all += __ldcg(rcd + DV + 1) * f;
                 o += __ldcg(rcd + c) * f;
               }
-              p.out[(size_t)tok * p.out_stride + (size_t)(kvh * G + row) * D + c] = __float2bfloat16_rn(l_all > 0.f ? o / l_all : 0.f);
+              return l_all > 0.f ? o / l_all : 0.f;
+            };
+            if constexpr (kPool) {
+              for (int e = threadIdx.x; e < rows_mine * (DV / 2); e += kThreads) {
+                const int row = e / (DV / 2) * kSplit + rank;
+                emit_pair(kvh * G + row, e % (DV / 2), [&](int c) { return total(row, c); });
+              }
+            } else {
+              for (int e = threadIdx.x; e < rows_mine * DV; e += kThreads) {
+                const int c = e % DV, row = (e / DV) * kSplit + rank;
+                p.out[(size_t)tok * p.out_stride + (size_t)(kvh * G + row) * DV + c] = __float2bfloat16_rn(total(row, c));
+              }
             }
           }
         }
@@ -812,15 +875,14 @@ decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__
     const int live_rows = min(16, G - rb);
     const uint32_t rec_addr = smem_u32(rec);
     const int n_rec = kSplit * kConsumers;
-    for (int e = rank * kThreads + threadIdx.x; e < live_rows * D; e += kSplit * kThreads) {
-      const int row = e / D, c = e % D;
+    auto total = [&](int row, int c) {
       auto rec_of = [&](int i) { return rec_addr + (uint32_t)(((i % kConsumers) * 16 + row) * kRec) * 4u; };
       float m_all = -INFINITY;
       for (int i0 = 0; i0 < n_rec; i0 += 8) {                // the records' maxima, eight loads in flight
         float m[8];
 #pragma unroll
         for (int i = 0; i < 8; ++i)
-          m[i] = i0 + i < n_rec ? ld_peer_f32(rec_of(i0 + i) + D * 4u, (uint32_t)((i0 + i) / kConsumers)) : -INFINITY;
+          m[i] = i0 + i < n_rec ? ld_peer_f32(rec_of(i0 + i) + DV * 4u, (uint32_t)((i0 + i) / kConsumers)) : -INFINITY;
 #pragma unroll
         for (int i = 0; i < 8; ++i) m_all = fmaxf(m_all, m[i]);
       }
@@ -831,8 +893,8 @@ decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__
         for (int i = 0; i < 8; ++i) {
           const bool on = i0 + i < n_rec;
           const uint32_t a = rec_of(on ? i0 + i : 0), peer = (uint32_t)((on ? i0 + i : 0) / kConsumers);
-          m[i] = on ? ld_peer_f32(a + D * 4u, peer) : -INFINITY;
-          l[i] = on ? ld_peer_f32(a + (D + 1) * 4u, peer) : 0.f;
+          m[i] = on ? ld_peer_f32(a + DV * 4u, peer) : -INFINITY;
+          l[i] = on ? ld_peer_f32(a + (DV + 1) * 4u, peer) : 0.f;
           v[i] = on ? ld_peer_f32(a + (uint32_t)c * 4u, peer) : 0.f;
         }
 #pragma unroll
@@ -842,7 +904,18 @@ decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__
           o += v[i] * f;
         }
       }
-      p.out[(size_t)tok * p.out_stride + (size_t)(kvh * G + rb + row) * D + c] = __float2bfloat16_rn(l_all > 0.f ? o / l_all : 0.f);
+      return l_all > 0.f ? o / l_all : 0.f;
+    };
+    if constexpr (kPool) {
+      for (int e = rank * kThreads + threadIdx.x; e < live_rows * (DV / 2); e += kSplit * kThreads) {
+        const int row = e / (DV / 2);
+        emit_pair(kvh * G + rb + row, e % (DV / 2), [&](int c) { return total(row, c); });
+      }
+    } else {
+      for (int e = rank * kThreads + threadIdx.x; e < live_rows * DV; e += kSplit * kThreads) {
+        const int row = e / DV, c = e % DV;
+        p.out[(size_t)tok * p.out_stride + (size_t)(kvh * G + rb + row) * DV + c] = __float2bfloat16_rn(total(row, c));
+      }
     }
     cluster_sync_all();                                    // the records stay until every peer has read them
     // the next pass's TMA writes land where ordinary stores and loads have just been
@@ -890,32 +963,32 @@ int cache_map(CUtensorMap* out, const void* ptr, int d, int page_size, int nkv, 
 }
 
 // Ring, alignment slack, barriers and the flag; the records that a cluster sends to this CTA follow.
-template <int D, int STAGES>
-constexpr size_t ring_bytes() { return (size_t)STAGES * 2 * (D / 64) * kKeys * 128 + 1024 + (2 * STAGES + 2) * 8; }
+template <int D, int DV, int STAGES>
+constexpr size_t ring_bytes() { return (size_t)STAGES * (D / 64 + DV / 64) * kKeys * 128 + 1024 + (2 * STAGES + 2) * 8; }
 
 // Rows of a group of `group` query heads that one CTA of a cluster of `split` owns at most,
 // and the bytes of the records sent to it (none when the records stay where they are).
 inline int rows_cap_of(int group, int split) { return (split > 1 && group <= 16) ? (group + split - 1) / split : 0; }
 inline size_t inbox_bytes(int d, int group, int split) { return (size_t)split * rows_cap_of(group, split) * (d + 4) * 4; }
 
-template <int D, int STAGES, bool V = false>
+template <int D, int DV, int STAGES, int V>
 int configure() {
   static OncePerDevice once;
   if (once.first()) {
-    constexpr size_t smem = ring_bytes<D, STAGES>() + (size_t)2 * kMaxSplit * (D + 4) * 4;   // the most a launch asks for
+    constexpr size_t smem = ring_bytes<D, DV, STAGES>() + (size_t)2 * kMaxSplit * (DV + 4) * 4;   // the most a launch asks for
     static_assert(smem <= 227 * 1024, "tile ring does not fit shared memory");
-    cudaError_t e = cudaFuncSetAttribute(decode_kernel<D, STAGES, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(decode_kernel<D, DV, STAGES, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) once.forget();
     if (e != cudaSuccess) return fail("attention decode: cannot reserve %zu bytes of shared memory", smem);
-    cudaFuncSetAttribute(decode_kernel<D, STAGES, V>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
-    cudaFuncSetAttribute(decode_kernel<D, STAGES, V>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
+    cudaFuncSetAttribute(decode_kernel<D, DV, STAGES, V>, cudaFuncAttributePreferredSharedMemoryCarveout, cudaSharedmemCarveoutMaxShared);
+    cudaFuncSetAttribute(decode_kernel<D, DV, STAGES, V>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1);
   }
   return 0;
 }
 
 // Clusters of `split` CTAs of this kernel, each with `extra` more bytes of shared memory, that
 // the device holds at a time (0 if it cannot tell or cannot run them).
-template <int D, int STAGES, bool V = false>
+template <int D, int DV, int STAGES, int V>
 int active_clusters(int split, size_t extra) {
   static std::unordered_map<long long, int> cache;
   static std::mutex mu;
@@ -924,27 +997,27 @@ int active_clusters(int split, size_t extra) {
   std::lock_guard<std::mutex> g(mu);
   auto it = cache.find(key);
   if (it != cache.end()) return it->second;
-  if (configure<D, STAGES, V>()) return 0;
+  if (configure<D, DV, STAGES, V>()) return 0;
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(split, 64, 8);
   cfg.blockDim = dim3(kThreads);
-  cfg.dynamicSmemBytes = ring_bytes<D, STAGES>() + extra;
+  cfg.dynamicSmemBytes = ring_bytes<D, DV, STAGES>() + extra;
   cudaLaunchAttribute attr[1];
   attr[0].id = cudaLaunchAttributeClusterDimension;
   attr[0].val.clusterDim.x = (unsigned)split; attr[0].val.clusterDim.y = 1; attr[0].val.clusterDim.z = 1;
   cfg.attrs = attr; cfg.numAttrs = 1;
   int n = 0;
-  if (cudaOccupancyMaxActiveClusters(&n, decode_kernel<D, STAGES, V>, &cfg) != cudaSuccess) { cudaGetLastError(); n = 0; }
+  if (cudaOccupancyMaxActiveClusters(&n, decode_kernel<D, DV, STAGES, V>, &cfg) != cudaSuccess) { cudaGetLastError(); n = 0; }
   if (n < 0) n = 0;
   cache.emplace(key, n);
   return n;
 }
 
-template <int D, int STAGES, bool V = false>
-int launch(const CUtensorMap (&m)[4], const Params& p, size_t extra, cudaStream_t stream) {
-  if (configure<D, STAGES, V>()) return -1;
-  ilb::launch_cluster(decode_kernel<D, STAGES, V>, dim3(p.split, p.nkv, p.n_seqs * p.chunks), dim3(kThreads), ring_bytes<D, STAGES>() + extra, stream,
-                      p.split, m[0], m[1], m[2], m[3], p);
+template <int D, int DV, int STAGES, int V>
+int launch(const CUtensorMap (&m)[6], const Params& p, size_t extra, cudaStream_t stream) {
+  if (configure<D, DV, STAGES, V>()) return -1;
+  ilb::launch_cluster(decode_kernel<D, DV, STAGES, V>, dim3(p.split, p.nkv, p.n_seqs * p.chunks), dim3(kThreads), ring_bytes<D, DV, STAGES>() + extra, stream,
+                      p.split, m[0], m[1], m[2], m[3], m[4], m[5], p);
   return check_launch("attention decode");
 }
 
@@ -955,43 +1028,43 @@ constexpr int kMaxChunks = 8;
 // `long_context`: the step's longest sequence is long enough for several clusters per
 // (sequence, kv head) to pay; the launch is then shaped for the most CTAs at work, not for the
 // widest cluster.
-template <int D, bool V = false>
+template <int D, int DV = D, int V = 0>
 void plan_for(int n_seqs, int nq, int nkv, int long_context, int& split, int& stages, int& chunks) {
   const long long pairs = (long long)n_seqs * nkv;
   const int group = nq / nkv;
   split = kMaxSplit;
-  while (split > 1 && active_clusters<D, 3, V>(split, inbox_bytes(D, group, split)) < pairs) split /= 2;
+  while (split > 1 && active_clusters<D, DV, 3, V>(split, inbox_bytes(DV, group, split)) < pairs) split /= 2;
   chunks = 1;
   if (long_context && split > 1 && group <= 16) {
     long long best = 0;
     int best_split = split;
     for (int s = split; s >= 2; s /= 2) {
-      long long c = active_clusters<D, 3, V>(s, inbox_bytes(D, group, s)) / pairs;
+      long long c = active_clusters<D, DV, 3, V>(s, inbox_bytes(DV, group, s)) / pairs;
       c = c > kMaxChunks ? kMaxChunks : c;
       if (c * s > best) { best = c * s; best_split = s; chunks = (int)c; }
     }
     split = best_split;
   }
-  const size_t extra = inbox_bytes(D, group, split);
+  const size_t extra = inbox_bytes(DV, group, split);
   const long long clusters = pairs * chunks;
-  stages = active_clusters<D, 12, V>(split, extra) >= clusters ? 12 : active_clusters<D, 6, V>(split, extra) >= clusters ? 6 : 3;
+  stages = active_clusters<D, DV, 12, V>(split, extra) >= clusters ? 12 : active_clusters<D, DV, 6, V>(split, extra) >= clusters ? 6 : 3;
 }
 
-template <int D, bool V = false>
-int launch_for(const CUtensorMap (&m)[4], Params& p, int long_context, long long scratch_floats, long long n_counters, cudaStream_t stream) {
+template <int D, int DV = D, int V = 0>
+int launch_for(const CUtensorMap (&m)[6], Params& p, int long_context, long long scratch_floats, long long n_counters, cudaStream_t stream) {
   int stages = 3;
-  plan_for<D, V>(p.n_seqs, p.nq, p.nkv, long_context, p.split, stages, p.chunks);
+  plan_for<D, DV, V>(p.n_seqs, p.nq, p.nkv, long_context, p.split, stages, p.chunks);
   const int group = p.nq / p.nkv;
   if (p.chunks > 1) {
-    const long long need_f = (long long)p.n_seqs * p.nkv * p.chunks * 16 * (D + 2), need_c = (long long)p.n_seqs * p.nkv * 16;
+    const long long need_f = (long long)p.n_seqs * p.nkv * p.chunks * 16 * (DV + 2), need_c = (long long)p.n_seqs * p.nkv * 16;
     if (p.scratch == nullptr || p.counters == nullptr || need_f > scratch_floats || need_c > n_counters)
-      plan_for<D, V>(p.n_seqs, p.nq, p.nkv, 0, p.split, stages, p.chunks);       // no room for the records: one cluster each
+      plan_for<D, DV, V>(p.n_seqs, p.nq, p.nkv, 0, p.split, stages, p.chunks);       // no room for the records: one cluster each
   }
   p.rows_cap = rows_cap_of(group, p.split);
-  const size_t extra = inbox_bytes(D, group, p.split);
-  if (stages == 12) return launch<D, 12, V>(m, p, extra, stream);
-  if (stages == 6) return launch<D, 6, V>(m, p, extra, stream);
-  return launch<D, 3, V>(m, p, extra, stream);
+  const size_t extra = inbox_bytes(DV, group, p.split);
+  if (stages == 12) return launch<D, DV, 12, V>(m, p, extra, stream);
+  if (stages == 6) return launch<D, DV, 6, V>(m, p, extra, stream);
+  return launch<D, DV, 3, V>(m, p, extra, stream);
 }
 
 }  // namespace
@@ -1037,12 +1110,13 @@ int decode_common(const void* q, const void* qkv, int qkv_stride, const float* q
                 ((uintptr_t)rope % 8 == 0) && eps > 0.f, "attention decode: bad fused inputs");
   else
     ILB_REQUIRE(q_stride % 2 == 0 && ((uintptr_t)q % 4 == 0), "attention decode: misaligned operands");
-  CUtensorMap m[4];                      // K, V, and the same with boxes of two pages
+  CUtensorMap m[6];                      // K, V, the same with boxes of two pages, (pooled rows' K and V)
   const int run = page_size < kKeys ? kKeys / page_size : 1;
   if (cache_map(&m[0], k_cache, d, page_size, nkv, num_pages, 1)) return -1;
   if (cache_map(&m[1], v_cache, d, page_size, nkv, num_pages, 1)) return -1;
   if (cache_map(&m[2], k_cache, d, page_size, nkv, num_pages, run)) return -1;
   if (cache_map(&m[3], v_cache, d, page_size, nkv, num_pages, run)) return -1;
+  m[4] = m[0]; m[5] = m[1];
   Params p{};
   p.q = (const __nv_bfloat16*)q; p.out = (__nv_bfloat16*)out;
   p.positions = positions; p.cu_q = cu_q; p.block_table = block_table; p.error_flag = error_flag;
@@ -1057,8 +1131,8 @@ int decode_common(const void* q, const void* qkv, int qkv_stride, const float* q
   p.v_write = (qkv != nullptr && write_kv) ? (__nv_bfloat16*)const_cast<void*>(v_cache) : nullptr;
   p.chunks = 1; p.scratch = scratch; p.counters = counters;
   if (p.mode != 0 || p.v_mode != 0)        // the input stage's variants are a kernel of their own: the stock one stays as it was
-    return d == 64 ? launch_for<64, true>(m, p, long_context, scratch_floats, n_counters, stream)
-                   : launch_for<128, true>(m, p, long_context, scratch_floats, n_counters, stream);
+    return d == 64 ? launch_for<64, 64, 1>(m, p, long_context, scratch_floats, n_counters, stream)
+                   : launch_for<128, 128, 1>(m, p, long_context, scratch_floats, n_counters, stream);
   return d == 64 ? launch_for<64>(m, p, long_context, scratch_floats, n_counters, stream)
                  : launch_for<128>(m, p, long_context, scratch_floats, n_counters, stream);
 }
@@ -1099,6 +1173,38 @@ ILB_EXPORT int ilb_attention_decode_fused(const void* qkv, int qkv_stride, const
   return decode_common(nullptr, qkv, qkv_stride, q_weight, k_weight, eps, rope, in, write_kv, out, k_cache, v_cache, positions,
                        cu_q, block_table, max_blocks, page_size, num_pages, window, scale, n_seqs, nq, nkv, d, 0, out_stride,
                        long_context, scratch, scratch_floats, counters, n_counters, error_flag, stream);
+}
+
+// A window with pooled blocks before it (kMode 2): q ready in its own matrix, the step's keys and values already cached, the
+// pooled rows in pages of their own; out [tokens, nq * dv], turned back by `turn` [tokens][dv / 2][2] if that is not null.
+ILB_EXPORT int ilb_attention_decode_pooled(const void* q, void* out, const void* k_cache, const void* v_cache, const void* pk_cache,
+                                           const void* pv_cache, const int* positions, const int* cu_q, const int* block_table,
+                                           const int* p_table, int max_blocks, int page_size, int num_pages, int p_num_pages, int window,
+                                           int pool, float scale, int n_seqs, int nq, int nkv, int d, int dv, int q_stride, int out_stride,
+                                           const float* turn, int long_context, float* scratch, long long scratch_floats, int* counters,
+                                           long long n_counters, int* error_flag, cudaStream_t stream) {
+  ILB_REQUIRE(ilb_attention_decode_tma_supported(nq, nkv, d, page_size) && (dv == 64 || dv == 128) && dv <= d,
+              "attention decode: heads %d/%d, head sizes %d / %d, page size %d are not built", nq, nkv, d, dv, page_size);
+  ILB_REQUIRE(n_seqs > 0 && n_seqs <= 65535 && nkv <= 65535 && max_blocks > 0 && num_pages > 0 && p_num_pages > 0 && window > 0 && pool > 0,
+              "attention decode: bad sizes");
+  for (const void* ptr : {k_cache, v_cache, pk_cache, pv_cache}) ILB_REQUIRE(ptr != nullptr && (uintptr_t)ptr % 16 == 0, "attention decode: misaligned cache");
+  ILB_REQUIRE(q_stride % 2 == 0 && ((uintptr_t)q % 4 == 0) && ((uintptr_t)turn % 8 == 0), "attention decode: misaligned operands");
+  CUtensorMap m[6];
+  const int run = page_size < kKeys ? kKeys / page_size : 1;
+  if (cache_map(&m[0], k_cache, d, page_size, nkv, num_pages, 1) || cache_map(&m[1], v_cache, dv, page_size, nkv, num_pages, 1) ||
+      cache_map(&m[2], k_cache, d, page_size, nkv, num_pages, run) || cache_map(&m[3], v_cache, dv, page_size, nkv, num_pages, run) ||
+      cache_map(&m[4], pk_cache, d, page_size, nkv, p_num_pages, 1) || cache_map(&m[5], pv_cache, dv, page_size, nkv, p_num_pages, 1)) return -1;
+  Params p{};
+  p.q = (const __nv_bfloat16*)q; p.out = (__nv_bfloat16*)out;
+  p.positions = positions; p.cu_q = cu_q; p.block_table = block_table; p.error_flag = error_flag;
+  p.max_blocks = max_blocks; p.n_seqs = n_seqs; p.nq = nq; p.nkv = nkv; p.window = window;
+  p.q_stride = q_stride; p.out_stride = out_stride; p.page_size = page_size; p.num_pages = num_pages;
+  p.split = 1; p.scale_log2 = scale * kLog2e;
+  p.chunks = 1; p.scratch = scratch; p.counters = counters;
+  p.p_table = p_table; p.p_num_pages = p_num_pages; p.pool = pool; p.turn = (const float2*)turn;
+  if (d == 64) return launch_for<64, 64, 2>(m, p, long_context, scratch_floats, n_counters, stream);
+  if (dv == 64) return launch_for<128, 64, 2>(m, p, long_context, scratch_floats, n_counters, stream);
+  return launch_for<128, 128, 2>(m, p, long_context, scratch_floats, n_counters, stream);
 }
 
 ILB_DEFINE_LAST_ERROR()

@@ -29,6 +29,12 @@
 // Every mbarrier wait is bounded; on expiry a flag is raised, the CTA drains and frees its
 // tensor memory.  No cluster, no multicast.
 //
+// POOL: a window with pooled blocks before it.  The walk then starts with tiles of a second set
+// of pages (row b = the mean of block b of `pool` positions; a row of the CTA sees the blocks that
+// lie wholly before its window) and goes on with the window's tiles; values may have another
+// head size (DV) than keys, and with `turn` every head's output is turned back in pairs
+// (i, i + DV / 2) by its position's angle as it is written.
+//
 // Reference counterparts: the query-tile prefill kernel on MMAs
 // (crates/backend/cuda-kernels/src/tile/attention/resident_attention_prefill_kernels.rs:378-469)
 // and the CuTe-generated sm_100a artifact that the reference ships for another geometry only
@@ -139,6 +145,8 @@ struct Params {
   int* error_flag;
   int max_blocks, n_seqs, nq, nkv, window, out_stride, page_size, num_pages;
   float scale_log2;
+  const int* p_table; int p_num_pages, pool;      // POOL: block table and pages of the pooled rows, tokens a row stands for
+  const float2* turn;                             // POOL: [tokens][DV / 2] (cos, sin), or null
   int skip_single;       // sequences that bring one token are somebody else's (the decode kernel's)
   const float* sink;     // [nq] or null: a logit per query head that joins the softmax's denominator unscaled, without a value
 };
@@ -154,12 +162,15 @@ struct Params {
 //   every K and V tile that comes in; tensor memory holds one S buffer and O per block (4 x
 //   128 columns), scores are issued one tile ahead, and while one block's warps work on a
 //   tile the tensor core works for the other block.
-template <int D, int QB>
+template <int D, int DV, int QB, bool POOL>
 __global__ void __launch_bounds__(64 + 256 * QB)
 prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                   const __grid_constant__ CUtensorMap map_v, const __grid_constant__ CUtensorMap map_k_run,
-                  const __grid_constant__ CUtensorMap map_v_run, const Params p) {
+                  const __grid_constant__ CUtensorMap map_v_run, const __grid_constant__ CUtensorMap map_pk,
+                  const __grid_constant__ CUtensorMap map_pv, const Params p) {
+  static_assert(POOL || D == DV, "values of another head size come with the pooled form");
   constexpr int kChunks = D / 64;                       // 64-wide slices of the head
+  constexpr int kChunksV = DV / 64;                     // of the values'
   constexpr uint32_t kSlice = kRows * 128;              // bytes of a [128][64] bf16 slice
   constexpr uint32_t kQBytes = kChunks * kSlice;        // one row block of Q
   // A K or V tile lies as [group of 8 keys][slice of the head][8 keys][64]: a page of the
@@ -171,8 +182,9 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
   // 2 % slower than slice-major tiles were; choosing between the two per stage cost the
   // issuing thread more than that.)
   constexpr uint32_t kKBytes = kChunks * kSlice;
-  constexpr uint32_t kVBytes = kChunks * kSlice;
+  constexpr uint32_t kVBytes = kChunksV * kSlice;
   constexpr uint32_t kGroup = kChunks * 1024;           // bytes from one group of 8 keys to the next
+  constexpr uint32_t kGroupV = kChunksV * 1024;
   constexpr int kStagesK = stages_k(D, QB), kStagesV = stages_v(D, QB);
   constexpr int KS = kKeys;                             // keys of a score tile
   constexpr int SUB = kKeys / KS;                       // score tiles per K / V tile
@@ -219,7 +231,13 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
   const int pos_first = p.positions[tok0 + t_first], pos_last = p.positions[tok0 + t_last];
   const int key_lo = (p.window > 0 && pos_first + 1 > p.window) ? pos_first + 1 - p.window : 0;
   const int first_tile = key_lo / kKeys;
-  const int n_tiles = pos_last / kKeys - first_tile + 1;      // both blocks walk all of them; what a row may not see is masked
+  // pooled rows that the CTA's last row sees (earlier rows see no more), and their tiles: they come first
+  int n_pooled = 0, pool_tiles = 0;
+  if constexpr (POOL) {
+    n_pooled = pos_last + 1 > p.window ? (pos_last + 1 - p.window) / p.pool : 0;
+    pool_tiles = (n_pooled + kKeys - 1) / kKeys;
+  }
+  const int n_tiles = pool_tiles + pos_last / kKeys - first_tile + 1;      // both blocks walk all of them; what a row may not see is masked
   const int* table = p.block_table + (size_t)seq * p.max_blocks;
 
   if (threadIdx.x == 0) {
@@ -264,15 +282,21 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
     const int pages_per_tile = kKeys / p.page_size;
     const int box_page = lane & 15;                       // lanes 0-15 bring K pages, 16-31 V pages
     const bool has_box = box_page < pages_per_tile;
-    const uint32_t page_bytes = (uint32_t)p.page_size * D * 2;
+    const uint32_t page_bytes = (uint32_t)p.page_size * D * 2, page_bytes_v = (uint32_t)p.page_size * DV * 2;
     const int groups_per_page = p.page_size / 8;
     const int run_boxes = pages_per_tile > 1 ? 2 : 1;     // a run of pages comes as two boxes side by side (one, if the tile is one page)
 
     bool ok = true;
     auto lookup = [&](int j) {                            // page of this lane's box of tile j
+      if (POOL && j < pool_tiles) {
+        const int blk = j * pages_per_tile + box_page;
+        int pg = -1;
+        if (has_box && blk < p.max_blocks && blk * p.page_size < n_pooled) pg = __ldg(p.p_table + (size_t)seq * p.max_blocks + blk);
+        return pg >= 0 && pg < p.p_num_pages ? pg : p.p_num_pages;
+      }
       int page = p.num_pages;                             // outside the tensor: TMA fills zeros
       if (has_box && j < n_tiles) {
-        const int key0 = (first_tile + j) * kKeys;
+        const int key0 = (first_tile + j - pool_tiles) * kKeys;
         const int blk = key0 / p.page_size + box_page;
         const int pg = blk < p.max_blocks ? __ldg(table + blk) : -1;
         if (pg >= 0 && pg < p.num_pages && key0 + box_page * p.page_size <= pos_last) page = pg;
@@ -300,8 +324,9 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
         const int page = page_k;
         page_k = lookup(jk + 1);                            // in flight while this tile's boxes are issued
         const int first_page = __shfl_sync(0xffffffffu, page, 0);
+        const bool pooled = POOL && jk < pool_tiles;
         const bool run = __all_sync(0xffffffffu, !has_box || page == first_page + box_page) &&
-                         first_page + pages_per_tile <= p.num_pages;
+                         first_page + pages_per_tile <= p.num_pages && !pooled;
         if (lane == 0) mbar_expect_tx(k_full + 8 * s, kKBytes);
         __syncwarp();
         if (run) {
@@ -309,7 +334,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
             tma_load_5d(k_s + s * kKBytes + lane * (kKBytes / 2), &map_k_run, k_full + 8 * s, 0, 0, 0, kvh * groups_per_page,
                         first_page + lane * (pages_per_tile / 2));
         } else if (has_box && lane < 16)
-          tma_load_5d(k_s + s * kKBytes + box_page * page_bytes, &map_k, k_full + 8 * s, 0, 0, 0, 0, page * p.nkv + kvh);
+          tma_load_5d(k_s + s * kKBytes + box_page * page_bytes, pooled ? &map_pk : &map_k, k_full + 8 * s, 0, 0, 0, 0, page * p.nkv + kvh);
         ++jk;
       }
       if (free_v) {
@@ -317,8 +342,9 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
         const int page = page_v;
         page_v = lookup(jv + 1);
         const int first_page = __shfl_sync(0xffffffffu, page, 0);
+        const bool pooled = POOL && jv < pool_tiles;
         const bool run = __all_sync(0xffffffffu, !has_box || page == first_page + box_page) &&
-                         first_page + pages_per_tile <= p.num_pages;
+                         first_page + pages_per_tile <= p.num_pages && !pooled;
         if (lane == 0) mbar_expect_tx(v_full + 8 * sv, kVBytes);
         __syncwarp();
         if (run) {
@@ -326,7 +352,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
             tma_load_5d(v_s + sv * kVBytes + (lane - 16) * (kVBytes / 2), &map_v_run, v_full + 8 * sv, 0, 0, 0, kvh * groups_per_page,
                         first_page + (lane - 16) * (pages_per_tile / 2));
         } else if (has_box && lane >= 16)
-          tma_load_5d(v_s + sv * kVBytes + box_page * page_bytes, &map_v, v_full + 8 * sv, 0, 0, 0, 0, page * p.nkv + kvh);
+          tma_load_5d(v_s + sv * kVBytes + box_page * page_bytes_v, pooled ? &map_pv : &map_v, v_full + 8 * sv, 0, 0, 0, 0, page * p.nkv + kvh);
         ++jv;
       }
       if (free_k || free_v) idle = 0;
@@ -339,7 +365,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
     // the operands could stay in uniform registers, was measured and was slower.)
     if (lane == 0) {
       constexpr uint32_t idesc_s = instr_desc(kRows, KS, 0);
-      constexpr uint32_t idesc_o = instr_desc(kRows, D, 1);
+      constexpr uint32_t idesc_o = instr_desc(kRows, DV, 1);
       bool ok = mbar_wait(q_full, 0);
       // scores of (block q, score tile u) = Q_q K^T over the tile's KS keys, into their S buffer
       auto issue_s = [&](int q, int u) {
@@ -393,7 +419,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
           const uint32_t p_t = s_cols(q, u);       // P: KS / 2 columns, two bfloat16 of consecutive keys each
 #pragma unroll
           for (int k = 0; k < KS / 16; ++k)   // 16 keys a step: 8 columns of P, two 8-key groups of V
-            mma_bf16_ts(tmem_o + (uint32_t)q * 128u, p_t + 8 * k, desc_mn_major(v_s + sv * kVBytes + (h * (KS / 16) + k) * 2 * kGroup, 1024, kGroup),
+            mma_bf16_ts(tmem_o + (uint32_t)q * 128u, p_t + 8 * k, desc_mn_major(v_s + sv * kVBytes + (h * (KS / 16) + k) * 2 * kGroupV, 1024, kGroupV),
                         idesc_o, (u > 0 || k > 0) ? 1u : 0u);
           tcgen05_commit(o_done + 8 * q);
           pv_issued[q] = u + 1;
@@ -427,7 +453,8 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
     const int head = kvh * G + row % G;
     const int pos = live ? p.positions[tok0 + tl] : -1;
     const int lo = (live && p.window > 0 && pos + 1 > p.window) ? pos + 1 - p.window : 0;
-    constexpr int kOCols = D / 2;                      // columns of O this thread owns
+    const int row_pooled = POOL ? lo / p.pool : 0;     // pooled rows this row sees
+    constexpr int kOCols = DV / 2;                     // columns of O this thread owns
     float m_used = -1e30f, l = 0.f;
     bool ok = true;
     auto block_sync = [&]() {                           // the 256 threads of this row block
@@ -435,7 +462,9 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
       else asm volatile("bar.sync 2, 256;" ::: "memory");
     };
     for (int u = 0; u < n_sub; ++u) {
-      const int key0 = first_tile * kKeys + u * KS + half * E;
+      const bool in_pool = POOL && u < pool_tiles * SUB;
+      const int key0 = (in_pool ? 0 : (first_tile - pool_tiles) * kKeys) + u * KS + half * E;
+      const int see_lo = in_pool ? 0 : lo, see_hi = in_pool ? row_pooled - 1 : pos;      // what this row sees of the tile's set of keys
       const int t = s_buf(q, u);
       const uint32_t s_t = s_cols(q, u) + lane_addr;     // this row of the S buffer
       // `ok` only ever changes through waits that all 256 threads of the block share, so they
@@ -450,12 +479,12 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
       // raw scores stay in v (the scale is positive and folds into the exponent's multiply-add);
       // keys this row may not see become -inf; the maximum is taken in log2 units, in four
       // chains so that no instruction waits for the one before it
-      const bool all_visible = key0 + E - 1 <= pos && key0 >= lo;
+      const bool all_visible = key0 + E - 1 <= see_hi && key0 >= see_lo;
       if (!all_visible) {
 #pragma unroll
         for (int c = 0; c < E; ++c) {
           const int key = key0 + c;
-          v[c] = (key <= pos && key >= lo) ? v[c] : -INFINITY;
+          v[c] = (key <= see_hi && key >= see_lo) ? v[c] : -INFINITY;
         }
       }
       float m4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
@@ -520,11 +549,24 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
     if (p.sink != nullptr && live && l > 0.f) l += exp2f(p.sink[head] * kLog2e - m_used);
     if (ok) {
       const float inv = l > 0.f ? 1.f / l : 0.f;
-      __nv_bfloat16* dst = p.out + (size_t)(tok0 + (live ? tl : 0)) * p.out_stride + (size_t)head * D + half * kOCols;
+      __nv_bfloat16* dst = p.out + (size_t)(tok0 + (live ? tl : 0)) * p.out_stride + (size_t)head * DV + half * kOCols;
 #pragma unroll 1
       for (int c0 = 0; c0 < kOCols; c0 += 32) {
         float o[32];
         tmem_load_32(o_t + half * kOCols + c0, o);       // collective: every lane of the warp takes part
+        if constexpr (POOL) {
+          if (p.turn != nullptr) {                         // the pair's other member is the other thread's column
+            float w[32];
+            tmem_load_32(o_t + (half ^ 1) * kOCols + c0, w);
+            const float4* cs = reinterpret_cast<const float4*>(p.turn + (size_t)(tok0 + (live ? tl : 0)) * kOCols + c0);
+#pragma unroll
+            for (int c = 0; c < 16; ++c) {
+              const float4 a = __ldg(cs + c);              // (cos, sin) of two pairs
+              o[2 * c] = half == 0 ? fmaf(w[2 * c], a.y, o[2 * c] * a.x) : fmaf(-w[2 * c], a.y, o[2 * c] * a.x);
+              o[2 * c + 1] = half == 0 ? fmaf(w[2 * c + 1], a.w, o[2 * c + 1] * a.z) : fmaf(-w[2 * c + 1], a.w, o[2 * c + 1] * a.z);
+            }
+          }
+        }
         if (live) {
 #pragma unroll
           for (int g = 0; g < 4; ++g) {
@@ -562,21 +604,22 @@ int encode(CUtensorMap* out, const void* ptr, int rank, const cuuint64_t* dims, 
   return 0;
 }
 
-template <int D, int QB>
-int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const CUtensorMap& mkr,
-           const CUtensorMap& mvr, const Params& p, int n_tiles, cudaStream_t stream) {
-  constexpr int kChunks = D / 64;
+struct Maps { CUtensorMap q, k, v, k_run, v_run, pk, pv; };
+
+template <int D, int DV, int QB, bool POOL>
+int launch(const Maps& m, const Params& p, int n_tiles, cudaStream_t stream) {
   constexpr int kStagesK = stages_k(D, QB), kStagesV = stages_v(D, QB);
-  constexpr size_t smem = (size_t)kChunks * kRows * 128 * (QB + kStagesK + kStagesV) + 1024 +
+  constexpr size_t smem = (size_t)kRows * 128 * (D / 64 * (QB + kStagesK) + DV / 64 * kStagesV) + 1024 +
                           (1 + 2 * kStagesK + 2 * kStagesV + 10 + 2) * 8 + (size_t)QB * 768 * 4;
   static_assert(smem <= 227 * 1024, "tiles do not fit shared memory");
   static OncePerDevice once;
   if (once.first()) {
-    cudaError_t e = cudaFuncSetAttribute(prefill_tc_kernel<D, QB>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    cudaError_t e = cudaFuncSetAttribute(prefill_tc_kernel<D, DV, QB, POOL>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) once.forget();
     if (e != cudaSuccess) return fail("attention (tensor cores): cannot reserve %zu bytes of shared memory", smem);
   }
-  ilb::launch(prefill_tc_kernel<D, QB>, dim3(p.nkv, n_tiles), dim3(64 + 256 * QB), smem, stream, mq, mk, mv, mkr, mvr, p);
+  ilb::launch(prefill_tc_kernel<D, DV, QB, POOL>, dim3(p.nkv, n_tiles), dim3(64 + 256 * QB), smem, stream, m.q, m.k, m.v, m.k_run, m.v_run,
+              m.pk, m.pv, p);
   return check_launch("attention prefill (tensor cores)");
 }
 
@@ -594,11 +637,15 @@ ILB_EXPORT int ilb_attention_tc_supported(int nq, int nkv, int d, int page_size)
 // portions); n_tiles = sum over sequences of ceil(q_len / (row_blocks * floor(128 / G))),
 // without the sequences of one token if skip_single is set (their rows of `out` are then
 // left alone).
+// With pool > 0 (and a window): pk_cache, pv_cache, p_table, p_num_pages are the pooled rows' pages, dv the values' head
+// size, turn [tokens][dv / 2][2] what the output is turned back by (or null).
 ILB_EXPORT int ilb_attention_prefill_tc(const void* q, void* out, const void* k_cache, const void* v_cache,
                                         const int* positions, const int* cu_q, const int* block_table,
                                         int max_blocks, int page_size, int num_pages, int window, float scale,
                                         int n_tokens, int n_seqs, int n_tiles, int row_blocks, int skip_single, int nq, int nkv, int d,
-                                        int q_stride, int out_stride, int* error_flag, const float* sink, cudaStream_t stream) {
+                                        int dv, int q_stride, int out_stride, int* error_flag, const float* sink, const void* pk_cache,
+                                        const void* pv_cache, const int* p_table, int p_num_pages, int pool, const float* turn,
+                                        cudaStream_t stream) {
   ILB_REQUIRE(row_blocks == 1 || row_blocks == 2, "attention (tensor cores): %d row blocks per CTA (1 or 2)", row_blocks);
   ILB_REQUIRE(ilb_attention_tc_supported(nq, nkv, d, page_size),
               "attention (tensor cores): heads %d/%d, head size %d, page size %d are not built", nq, nkv, d, page_size);
@@ -607,38 +654,57 @@ ILB_EXPORT int ilb_attention_prefill_tc(const void* q, void* out, const void* k_
   ILB_REQUIRE(q_stride % 8 == 0 && out_stride % 8 == 0 && ((uintptr_t)q % 16 == 0) && ((uintptr_t)out % 16 == 0) &&
               ((uintptr_t)k_cache % 16 == 0) && ((uintptr_t)v_cache % 16 == 0), "attention (tensor cores): misaligned operands");
   const int G = nq / nkv;
-  CUtensorMap mq, mk, mv, mkr, mvr;
+  Maps m;
   {   // q as (d, heads, tokens); a box is 64 x G x floor(128/G) = the rows of a tile, one slice of the head
     const cuuint64_t dims[3] = {(cuuint64_t)d, (cuuint64_t)nq, (cuuint64_t)n_tokens};
     const cuuint64_t strides[2] = {(cuuint64_t)d * 2, (cuuint64_t)q_stride * 2};
     const cuuint32_t box[3] = {64, (cuuint32_t)G, (cuuint32_t)(kRows / G)};
-    if (encode(&mq, q, 3, dims, strides, box, "q")) return -1;
+    if (encode(&m.q, q, 3, dims, strides, box, "q")) return -1;
   }
-  {   // The cache [page][kv head][key][d] as (64 of d, key in its group of 8, slice of the head,
-      // group in the page, page x kv head): a box is the whole page of one head and lands as
-      // [group][slice][8 keys][64], the operand layout with its groups 1 or 2 KB apart.
-      // (The strides are not ascending: the encoder takes that; the coordinates are all zero
-      // but the last, so every copy starts on a 16-byte boundary.)
-    const cuuint64_t slices = (cuuint64_t)d / 64, groups = (cuuint64_t)page_size / 8;
-    const cuuint64_t dims[5] = {64, 8, slices, groups, (cuuint64_t)num_pages * nkv};
-    const cuuint64_t strides[4] = {(cuuint64_t)d * 2, 128, (cuuint64_t)d * 2 * 8, (cuuint64_t)d * 2 * page_size};
+  // The cache [page][kv head][key][d] as (64 of d, key in its group of 8, slice of the head,
+  // group in the page, page x kv head): a box is the whole page of one head and lands as
+  // [group][slice][8 keys][64], the operand layout with its groups 1 or 2 KB apart.
+  // (The strides are not ascending: the encoder takes that; the coordinates are all zero
+  // but the last, so every copy starts on a 16-byte boundary.)
+  auto page_map = [&](CUtensorMap* out_map, const void* ptr, int hd, int pages, const char* what) {
+    const cuuint64_t slices = (cuuint64_t)hd / 64, groups = (cuuint64_t)page_size / 8;
+    const cuuint64_t dims[5] = {64, 8, slices, groups, (cuuint64_t)pages * nkv};
+    const cuuint64_t strides[4] = {(cuuint64_t)hd * 2, 128, (cuuint64_t)hd * 2 * 8, (cuuint64_t)hd * 2 * page_size};
     const cuuint32_t box[5] = {64, 8, (cuuint32_t)slices, (cuuint32_t)groups, 1};
-    if (encode(&mk, k_cache, 5, dims, strides, box, "k cache")) return -1;
-    if (encode(&mv, v_cache, 5, dims, strides, box, "v cache")) return -1;
-    // the same with (group in the page, kv head) as one dimension and the page as the last: a
-    // box spans half the pages of a 128-key tile when their numbers follow one another
+    return encode(out_map, ptr, 5, dims, strides, box, what);
+  };
+  // the same with (group in the page, kv head) as one dimension and the page as the last: a
+  // box spans half the pages of a 128-key tile when their numbers follow one another
+  auto run_map = [&](CUtensorMap* out_map, const void* ptr, int hd, const char* what) {
+    const cuuint64_t slices = (cuuint64_t)hd / 64, groups = (cuuint64_t)page_size / 8;
     const cuuint64_t rdims[5] = {64, 8, slices, groups * nkv, (cuuint64_t)num_pages};
-    const cuuint64_t rstrides[4] = {(cuuint64_t)d * 2, 128, (cuuint64_t)d * 2 * 8, (cuuint64_t)d * 2 * page_size * nkv};
+    const cuuint64_t rstrides[4] = {(cuuint64_t)hd * 2, 128, (cuuint64_t)hd * 2 * 8, (cuuint64_t)hd * 2 * page_size * nkv};
     const int pages_per_tile = kKeys / page_size;
     const cuuint32_t run[5] = {64, 8, (cuuint32_t)slices, (cuuint32_t)groups, (cuuint32_t)(pages_per_tile > 1 ? pages_per_tile / 2 : 1)};
-    if (encode(&mkr, k_cache, 5, rdims, rstrides, run, "k cache (page run)")) return -1;
-    if (encode(&mvr, v_cache, 5, rdims, rstrides, run, "v cache (page run)")) return -1;
-  }
+    return encode(out_map, ptr, 5, rdims, rstrides, run, what);
+  };
+  if (page_map(&m.k, k_cache, d, num_pages, "k cache") || page_map(&m.v, v_cache, dv, num_pages, "v cache") ||
+      run_map(&m.k_run, k_cache, d, "k cache (page run)") || run_map(&m.v_run, v_cache, dv, "v cache (page run)")) return -1;
+  m.pk = m.k; m.pv = m.v;
   Params p{(__nv_bfloat16*)out, positions, cu_q, block_table, error_flag, max_blocks, n_seqs, nq, nkv, window,
-           out_stride, page_size, num_pages, scale * kLog2e, skip_single ? 1 : 0, sink};
+           out_stride, page_size, num_pages, scale * kLog2e, p_table, p_num_pages, pool, (const float2*)turn, skip_single ? 1 : 0, sink};
+  if (pool > 0) {
+    ILB_REQUIRE(window > 0 && sink == nullptr && pk_cache != nullptr && pv_cache != nullptr && p_table != nullptr && p_num_pages > 0 &&
+                ((uintptr_t)pk_cache % 16 == 0) && ((uintptr_t)pv_cache % 16 == 0) && ((uintptr_t)turn % 16 == 0),
+                "attention (tensor cores): pooled blocks need a window, no sink, and aligned pages of their own");
+    if (page_map(&m.pk, pk_cache, d, p_num_pages, "pooled keys") || page_map(&m.pv, pv_cache, dv, p_num_pages, "pooled values")) return -1;
+#define ILB_POOLED(D, DV) \
+    if (d == D && dv == DV) return row_blocks == 2 ? launch<D, DV, 2, true>(m, p, n_tiles, stream) : launch<D, DV, 1, true>(m, p, n_tiles, stream)
+    ILB_POOLED(64, 64);
+    ILB_POOLED(128, 64);
+    ILB_POOLED(128, 128);
+#undef ILB_POOLED
+    return fail("attention (tensor cores): pooled blocks with head sizes %d / %d are not built", d, dv);
+  }
+  ILB_REQUIRE(dv == d && turn == nullptr, "attention (tensor cores): values of another head size, or turned ones, come with pooled blocks");
   if (row_blocks == 2)
-    return d == 64 ? launch<64, 2>(mq, mk, mv, mkr, mvr, p, n_tiles, stream) : launch<128, 2>(mq, mk, mv, mkr, mvr, p, n_tiles, stream);
-  return d == 64 ? launch<64, 1>(mq, mk, mv, mkr, mvr, p, n_tiles, stream) : launch<128, 1>(mq, mk, mv, mkr, mvr, p, n_tiles, stream);
+    return d == 64 ? launch<64, 64, 2, false>(m, p, n_tiles, stream) : launch<128, 128, 2, false>(m, p, n_tiles, stream);
+  return d == 64 ? launch<64, 64, 1, false>(m, p, n_tiles, stream) : launch<128, 128, 1, false>(m, p, n_tiles, stream);
 }
 
 ILB_DEFINE_LAST_ERROR()

@@ -77,6 +77,12 @@ __device__ __forceinline__ float gate_mul(const P& p, float g, float u) {
   return __fdividef(g, 1.0f + __expf(-p.act_sharp * g)) * (u + p.act_offset);
 }
 
+// A plain bfloat16 result passed through relu squared (Params::relu2).
+__device__ __forceinline__ float relu2_if(int on, float v) {
+  const float r = fmaxf(v, 0.f);
+  return on ? r * r : v;
+}
+
 // K-major operand tile in shared memory, 128-byte swizzle: rows of 128 bytes, 8-row
 // groups 1024 bytes apart.
 __device__ __forceinline__ uint64_t smem_desc(uint32_t addr) {
@@ -105,6 +111,7 @@ struct Params {
   int cluster;               // > 1: a tile's K ranges belong to the CTAs of one cluster, added through their shared memory
   int tma_out;               // many tokens: the result leaves through shared memory and TMA stores (adds, when accumulating)
   int red_out;               // few tokens, accumulating: the K ranges of a tile are separate CTAs whose shares meet in memory (red.add)
+  int relu2;                 // a plain bfloat16 result leaves as relu(result)^2
   int gate_relu;             // the gated epilogue's activation: 0 silu, 1 relu, 2 the clamped unit with the constants below
   float act_limit, act_sharp, act_offset;
 };
@@ -450,7 +457,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
           for (int j = 0; j < 4; ++j) {
             const int m = y0 + cg * 4 + j;
             if (m < p.M && n < n_end) {
-              const float val = sw ? gate_mul(p, acc[j], up[j]) : acc[j] + bv + old[j];
+              const float val = sw ? gate_mul(p, acc[j], up[j]) : relu2_if(p.relu2, acc[j] + bv + old[j]);
               const size_t o = (size_t)m * p.ldo + n;
               if (p.out_f32) ((float*)p.out)[o] = val; else ((__nv_bfloat16*)p.out)[o] = __float2bfloat16_rn(val);
             }
@@ -636,6 +643,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
 #pragma unroll
                   for (int c = 0; c < 32; ++c) v[c] += (y0 + c0 + 32 * half + c < p.N) ? p.bias[y0 + c0 + 32 * half + c] : 0.f;
                 }
+                if (p.relu2) {
+#pragma unroll
+                  for (int c = 0; c < 32; ++c) v[c] = relu2_if(1, v[c]);
+                }
 #pragma unroll
                 for (int j = 0; j < 4; ++j) piece[4 * half + j] = pack8(v + 8 * j);
               }
@@ -736,7 +747,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
                 const int m = y0 + c0 + c;
                 if (m < p.M) {
                   const size_t o = (size_t)m * p.ldo + xr;
-                  const float r = v[c] + bv;
+                  const float r = relu2_if(p.relu2, v[c] + bv);
                   if (p.out_f32) ((float*)p.out)[o] = r;
                   else ((__nv_bfloat16*)p.out)[o] = __float2bfloat16_rn(r);
                 }
@@ -752,6 +763,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
               if (p.bias) {
 #pragma unroll
                 for (int c = 0; c < CH; ++c) v[c] += p.bias[n0 + c];
+              }
+              if (p.relu2) {
+#pragma unroll
+                for (int c = 0; c < CH; ++c) v[c] = relu2_if(1, v[c]);
               }
               if (p.out_f32) {
                 float4* dst = reinterpret_cast<float4*>((float*)p.out + o);
@@ -784,7 +799,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
                 const int n = y0 + c0 + c;
                 if (n < p.N) {
                   const size_t o = (size_t)xr * p.ldo + n;
-                  float r = v[c] + (p.bias ? p.bias[n] : 0.f);
+                  float r = relu2_if(p.relu2, v[c] + (p.bias ? p.bias[n] : 0.f));
                   if (p.out_f32) {
                     float* dst = (float*)p.out + o;
                     if (p.epilogue == kAccumulate) r += *dst;
@@ -859,7 +874,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant_
           const int c = cb + j * cstep, m = y0 + c;
           if (c < BN && m < p.M && n < n_end) {
             const float g = acc[j];
-            const float v = sw ? gate_mul(p, g, up[j]) : g + bv + old[j];
+            const float v = sw ? gate_mul(p, g, up[j]) : relu2_if(p.relu2, g + bv + old[j]);
             const size_t o = (size_t)m * p.ldo + n;
             if (p.out_f32) ((float*)p.out)[o] = v; else ((__nv_bfloat16*)p.out)[o] = __float2bfloat16_rn(v);
           }
@@ -907,6 +922,7 @@ struct PairParams {
   int n_whole, rest, split;  // tiles that are one item each; tiles cut into `split` K ranges
   int n_items;               // n_whole + rest * split
   int epilogue, out_f32;
+  int relu2;                 // a plain bfloat16 result leaves as relu(result)^2
   int gate_relu;             // the gated epilogue's activation: 0 silu, 1 relu, 2 the clamped unit with the constants below
   float act_limit, act_sharp, act_offset;
 };
@@ -1113,6 +1129,10 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constan
             if (p.bias) {
 #pragma unroll
               for (int c = 0; c < 32; ++c) v[c] += (y0 + c0 + 32 * half + c < p.N) ? p.bias[y0 + c0 + 32 * half + c] : 0.f;
+            }
+            if (p.relu2) {
+#pragma unroll
+              for (int c = 0; c < 32; ++c) v[c] = relu2_if(1, v[c]);
             }
 #pragma unroll
             for (int j = 0; j < 4; ++j) piece[4 * half + j] = pack8(v + 8 * j);
@@ -1575,6 +1595,10 @@ ILB_EXPORT int ilb_gemm_tc(const void* A, const void* W, const float* bias, void
               "gemm_tc: K (%d) and the leading dimensions (%d, %d) must be multiples of 8", K, lda, ldw);
   ILB_REQUIRE(((uintptr_t)A % 16 == 0) && ((uintptr_t)W % 16 == 0), "gemm_tc: operands must be 16-byte aligned");
   // 3 from the caller: the gated epilogue with relu as the gate's activation (else silu); 4: the clamped gated unit
+  // 5: a plain product whose bfloat16 result leaves as relu(result)^2
+  const int relu2 = accumulate == 5 ? 1 : 0;
+  if (relu2) accumulate = kStore;
+  ILB_REQUIRE(!relu2 || !out_f32, "gemm_tc: relu squared belongs to a bfloat16 result");
   const int gate_relu = accumulate == 3 ? 1 : (accumulate == 4 ? 2 : 0);
   if (gate_relu) accumulate = kSwiGLU;
   ILB_REQUIRE(gate_relu != 2 || act_limit > 0.f, "gemm_tc: the clamped unit needs a positive limit");
@@ -1594,6 +1618,7 @@ ILB_EXPORT int ilb_gemm_tc(const void* A, const void* W, const float* bias, void
   p.k_blocks = (K + kBlockK - 1) / kBlockK;
   p.epilogue = accumulate;
   p.out_f32 = out_f32;
+  p.relu2 = relu2;
   p.gate_relu = gate_relu; p.act_limit = act_limit; p.act_sharp = act_sharp; p.act_offset = act_offset;
 
   Plan plan{};
@@ -1609,7 +1634,7 @@ ILB_EXPORT int ilb_gemm_tc(const void* A, const void* W, const float* bias, void
       q.bias = bias; q.error_flag = error_flag; q.M = M; q.N = N;
       q.tiles_m = (M + 2 * kTileX - 1) / (2 * kTileX);
       q.k_blocks = p.k_blocks; q.n_whole = pp.n_whole; q.rest = pp.rest; q.split = pp.split; q.n_items = (int)pp.items;
-      q.epilogue = accumulate; q.out_f32 = out_f32; q.gate_relu = gate_relu;
+      q.epilogue = accumulate; q.out_f32 = out_f32; q.gate_relu = gate_relu; q.relu2 = relu2;
       q.act_limit = act_limit; q.act_sharp = act_sharp; q.act_offset = act_offset;
       CUtensorMap mx, my, mo;
       if (make_map(&mx, A, M, K, lda, kTileX)) return -1;

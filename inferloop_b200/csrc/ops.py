@@ -484,7 +484,8 @@ def act_rows(x: torch.Tensor, activation: str, out: torch.Tensor) -> None:
 
 # --------------------------------------------------------------------------- generalized delta rule
 def delta_scan(proj: torch.Tensor, col_r: int, col_k: int, col_v: int, col_a: int, low: torch.Tensor, w0: torch.Tensor, ab: torch.Tensor,
-               log_decay: float, unit_eps: float, state: torch.Tensor, y: torch.Tensor, step, heads: int, d: int, dv: int) -> None:
+               log_decay: float, unit_eps: float, state: torch.Tensor, y: torch.Tensor, step, heads: int, d: int, dv: int,
+               workspace=None) -> None:
     """S_t = diag(w) S_{t-1} - (g u)(u^T S_{t-1}) + k v^T, y_t = S_t^T r per head over the step's tokens, from and to state
     [slots, heads, d, dv] (see delta.cu); r, k, a at columns of `proj` (heads * d each), v (heads * dv); `low` [T, heads * d]
     32-bit: what w0 joins under the decay's sigmoid."""
@@ -799,10 +800,14 @@ def qk_norm_rope_cache(qkv: torch.Tensor, q_out: torch.Tensor, q_weight: Optiona
 
 def rows_norm_rope_cache(qkv: torch.Tensor, q_out: torch.Tensor, q_weight: torch.Tensor, k_weight: torch.Tensor, eps: float,
                          rope: Optional[torch.Tensor], rotary_dim: int, v_rope: Optional[torch.Tensor], step, block_table: torch.Tensor,
-                         k_cache: Optional[torch.Tensor], v_cache: Optional[torch.Tensor], nq: int, nkv: int, d: int, dv: int) -> None:
+                         k_cache: Optional[torch.Tensor], v_cache: Optional[torch.Tensor], nq: int, nkv: int, d: int, dv: int,
+                         pooled: Optional["PooledRows"] = None) -> None:
     """The input stage of an attention that norms queries and keys over all their heads' elements at once: q -> q_out,
     k and v -> cache pages, the first `rotary_dim` elements of q and k heads turned by `rope` [T, rotary_dim / 2, 2], values
-    turned over their whole size by `v_rope` [T, dv / 2, 2] (either table may be None); see qk_norm_rope.cu."""
+    turned over their whole size by `v_rope` [T, dv / 2, 2] (either table may be None); see qk_norm_rope.cu.  With `pooled`
+    (a step of single tokens): the blocks these tokens complete also get their means (what `pool_means` does)."""
+    if pooled is not None and not step.decode_only:
+        raise KernelError("rows_norm_rope_cache: block means inside the input stage are for steps of single tokens")
     _need(qkv, "qkv", contiguous=False); _need(q_out, "q_out", qkv.dtype); _need(q_weight, "q norm weight", torch.float32)
     _need(k_weight, "k norm weight", torch.float32); _need(rope, "rope table", torch.float32); _need(v_rope, "value rope table", torch.float32)
     _need(k_cache, "k cache", qkv.dtype); _need(v_cache, "v cache", qkv.dtype); _need(block_table, "block table", torch.int32)
@@ -817,7 +822,9 @@ def rows_norm_rope_cache(qkv: torch.Tensor, q_out: torch.Tensor, q_weight: torch
             raise KernelError("rows_norm_rope_cache: cache shapes do not match the heads")
     _call("qk_norm_rope", "ilb_rows_norm_rope_cache", _ptr(qkv), _ptr(q_out), _i(_code(qkv)), _ptr(q_weight), _ptr(k_weight), _f(eps), _ptr(rope),
           _i(rotary_dim), _ptr(v_rope), _ptr(step.positions), _ptr(step.seq_of_token), _ptr(block_table), _i(block_table.shape[1]), _i(page_size),
-          _i(num_pages), _ptr(k_cache), _ptr(v_cache), _i(T), _i(nq), _i(nkv), _i(d), _i(dv), _i(qkv.stride(0)), _i(q_out.shape[1]), _stream(qkv))
+          _i(num_pages), _ptr(k_cache), _ptr(v_cache), _i(T), _i(nq), _i(nkv), _i(d), _i(dv), _i(qkv.stride(0)), _i(q_out.shape[1]),
+          _ptr(None if pooled is None else pooled.k), _ptr(None if pooled is None else pooled.v), _ptr(None if pooled is None else pooled.table),
+          _i(0 if pooled is None else pooled.k.shape[0]), _i(0 if pooled is None else pooled.pool), _stream(qkv))
 
 
 class PooledRows:
@@ -1036,11 +1043,14 @@ def gemm_tc_eligible(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> boo
 
 
 def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[torch.Tensor] = None,
-            accumulate: bool = False, max_ctas: int = 0, swiglu: bool = False, gate: str = "silu", glu=None) -> None:
+            accumulate: bool = False, max_ctas: int = 0, swiglu: bool = False, gate: str = "silu", glu=None, relu2: bool = False) -> None:
     """out (+)= a @ w.T (+ bias) on tcgen05 tensor cores (see gemm_tcgen05.cu).  With
     `swiglu`, `w` holds blocks of 64 gate rows followed by their 64 up rows and `out` is
     [M, N/2] = act(gate) * up, act = `gate` ("silu" or "relu"); or, with `glu` = (limit, sharpness, up_offset), the
-    clamped unit a(min(gate, limit)) * (clamp(up, -limit, limit) + up_offset), a(g) = g * sigmoid(sharpness * g)."""
+    clamped unit a(min(gate, limit)) * (clamp(up, -limit, limit) + up_offset), a(g) = g * sigmoid(sharpness * g).
+    With `relu2` a bfloat16 `out` receives relu(result)^2."""
+    if relu2 and (swiglu or accumulate or out.dtype != torch.bfloat16):
+        raise KernelError("gemm: relu squared belongs to a plain product with a bfloat16 result")
     if gate not in ("silu", "relu"):
         raise KernelError(f"gemm: the gated epilogue has no activation {gate!r}")
     if glu is not None and (not swiglu or float(glu[0]) <= 0):
@@ -1055,7 +1065,7 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[
     if accumulate and (out.dtype != torch.float32 or swiglu):
         raise KernelError("gemm: accumulation needs a 32-bit output and no SwiGLU epilogue")
     st = _tc_state(a.device)
-    mode = (4 if glu is not None else 3 if gate == "relu" else 2) if swiglu else (1 if accumulate else 0)
+    mode = (4 if glu is not None else 3 if gate == "relu" else 2) if swiglu else (1 if accumulate else 5 if relu2 else 0)
     limit, sharp, offset = glu if glu is not None else (0.0, 1.0, 0.0)
     _call("gemm_tcgen05", "ilb_gemm_tc", _ptr(a), _ptr(w), _ptr(bias), _ptr(out),
           _i(1 if out.dtype == torch.float32 else 0), _i(M), _i(N), _i(K), _i(a.stride(0)), _i(w.stride(0)),
@@ -1165,7 +1175,8 @@ def attention_prefill_tc(q, out, k_cache, v_cache, positions, cu_q, block_table,
     _call("attention_tc", "ilb_attention_prefill_tc", _ptr(q), _ptr(out), _ptr(k_cache), _ptr(v_cache),
           _ptr(positions), _ptr(cu_q), _ptr(block_table), _i(block_table.shape[1]), _i(page_size),
           _i(num_pages), _i(window or 0), _f(scale), _i(q.shape[0]), _i(n_seqs), _i(n_tiles), _i(row_blocks), _i(1 if skip_single else 0), _i(nq), _i(nkv),
-          _i(d), _i(q.shape[1]), _i(out.shape[1]), _ptr(st.error), _ptr(sink), _stream(q))
+          _i(d), _i(d), _i(q.shape[1]), _i(out.shape[1]), _ptr(st.error), _ptr(sink), _ptr(None), _ptr(None), _ptr(None), _i(0), _i(0), _ptr(None),
+          _stream(q))
 
 
 def attention_prefill(q, out, k_cache, v_cache, positions, cu_q, block_table, window, scale, n_seqs,
@@ -1276,14 +1287,22 @@ def attention_decode_fused(qkv, out, q_weight, k_weight, eps, rope_table, k_cach
 def attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor,
               step, block_table: torch.Tensor, window: int, scale: float, nq: int, nkv: int,
               d: int, workspace=None, decode_chunk: int = DECODE_CHUNK_MIN, dv: Optional[int] = None,
-              sink: Optional[torch.Tensor] = None, pooled: Optional[PooledRows] = None) -> None:
+              sink: Optional[torch.Tensor] = None, pooled: Optional[PooledRows] = None, turn: Optional[torch.Tensor] = None) -> None:
     """Causal attention of the step's tokens over the cache; picks the kernel: the
     tensor-core kernels for a bfloat16 cache and a head size they are built for (split-KV
     when every sequence brings one token), else the exact kernel.  `sink` [nq] 32-bit: a logit
     per query head that joins the softmax's denominator (no key, no value, no scale).  `pooled`: rows
-    that stand for whole blocks of tokens before the window, in the same softmax."""
+    that stand for whole blocks of tokens before the window, in the same softmax.  `turn` [T, dv / 2, 2]: the heads'
+    outputs are turned back by these angles (see `turn_back`)."""
     dv = d if dv is None else int(dv)
     _need(sink, "attention sink", torch.float32)
+    if pooled is not None and attention_pooled_supported(q.dtype, k_cache.dtype, nq, nkv, d, dv, k_cache.shape[2], scale) and sink is None:
+        attention_pooled(q, out, k_cache, v_cache, step, block_table, window, scale, nq, nkv, d, dv, pooled, turn)
+        return
+    if turn is not None:
+        attention(q, out, k_cache, v_cache, step, block_table, window, scale, nq, nkv, d, workspace, decode_chunk, dv, sink, pooled)
+        turn_back(out, turn, nq)
+        return
     fast = (pooled is None and q.dtype == torch.bfloat16 and k_cache.dtype == torch.bfloat16 and attention_flash_supported(d) and dv == d
             and workspace is not None and FLASH_ENABLED)
     if not fast:          # the 32-bit path, and values of another head size than the keys'
@@ -1329,6 +1348,50 @@ def attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache
         n_tiles = sum(-(-n * G // 64) for n in step.h_q_len)
         attention_prefill(q, out, k_cache, v_cache, step.positions, step.cu_q, block_table, window, scale,
                           step.n_seqs, n_tiles, nq, nkv, d, sink)
+
+
+def attention_pooled_supported(dtype: torch.dtype, cache_dtype: torch.dtype, nq: int, nkv: int, d: int, dv: int, page_size: int,
+                               scale: float) -> bool:
+    """Whether a window with pooled blocks runs on the tensor-core kernels (else the exact kernel)."""
+    return (FLASH_ENABLED and TC_ATTENTION_ENABLED and dtype == torch.bfloat16 and cache_dtype == torch.bfloat16 and scale > 0
+            and (d, dv) in ((64, 64), (128, 64), (128, 128)) and attention_tc_supported(nq, nkv, d, page_size))
+
+
+def attention_pooled(q, out, k_cache, v_cache, step, block_table, window, scale, nq, nkv, d, dv, pooled: PooledRows, turn=None) -> None:
+    """Attention over a window and the pooled blocks before it on the tensor-core kernels: single tokens on the TMA decode
+    kernel, portions on the tcgen05 prefill kernel."""
+    for t, w in ((q, "q"), (out, "out"), (k_cache, "k cache"), (v_cache, "v cache"), (pooled.k, "pooled keys"), (pooled.v, "pooled values")):
+        _need(t, "attention " + w, torch.bfloat16)
+    _need(turn, "attention turn table", torch.float32); _need(pooled.table, "pooled block table", torch.int32)
+    num_pages, _, page_size, _ = k_cache.shape
+    if tuple(k_cache.shape[1:]) != (nkv, page_size, d) or tuple(v_cache.shape) != (num_pages, nkv, page_size, dv) \
+            or tuple(pooled.k.shape[1:]) != (nkv, page_size, d) or tuple(pooled.v.shape) != (pooled.k.shape[0], nkv, page_size, dv) \
+            or pooled.table.shape != block_table.shape or (turn is not None and tuple(turn.shape) != (q.shape[0], dv // 2, 2)) or not window:
+        raise KernelError("attention: pooled rows need a window, and pages like the cache's")
+    st = _tc_state(q.device)
+    lens, kv_lens = step.h_q_len, step.h_kv_len
+    singles = step.decode_only or (MIXED_SPLIT_ENABLED and 1 in lens)
+    if singles:
+        # what a token sees at most: its window, and the blocks before it
+        seen = max(min(n, window) + max(0, n - window) // pooled.pool for n in kv_lens)
+        _call("attention_decode", "ilb_attention_decode_pooled", _ptr(q), _ptr(out), _ptr(k_cache), _ptr(v_cache), _ptr(pooled.k), _ptr(pooled.v),
+              _ptr(step.positions), _ptr(step.cu_q), _ptr(block_table), _ptr(pooled.table), _i(block_table.shape[1]), _i(page_size),
+              _i(num_pages), _i(pooled.k.shape[0]), _i(window), _i(pooled.pool), _f(scale), _i(step.n_seqs), _i(nq), _i(nkv), _i(d), _i(dv),
+              _i(q.shape[1]), _i(out.shape[1]), _ptr(turn), _i(1 if step.decode_only and seen >= DECODE_LONG_CONTEXT else 0), _ptr(st.attn_scratch),
+              ctypes.c_longlong(st.attn_scratch.numel()), _ptr(st.attn_counters), ctypes.c_longlong(st.attn_counters.numel()), _ptr(st.error),
+              _stream(q))
+        if step.decode_only:
+            return
+        lens = [n for n in lens if n > 1]
+    per_block = 128 // (nq // nkv)
+    n_one = sum(-(-n // per_block) for n in lens)
+    n_two = sum(-(-n // (2 * per_block)) for n in lens)
+    blocks = TC_ATTENTION_ROW_BLOCKS or tc_row_blocks(n_one * nkv, n_two * nkv, _sm_count(q.device), False)
+    _call("attention_tc", "ilb_attention_prefill_tc", _ptr(q), _ptr(out), _ptr(k_cache), _ptr(v_cache), _ptr(step.positions), _ptr(step.cu_q),
+          _ptr(block_table), _i(block_table.shape[1]), _i(page_size), _i(num_pages), _i(window), _f(scale), _i(q.shape[0]), _i(step.n_seqs),
+          _i(n_two if blocks == 2 else n_one), _i(blocks), _i(1 if singles else 0), _i(nq), _i(nkv), _i(d), _i(dv), _i(q.shape[1]),
+          _i(out.shape[1]), _ptr(st.error), _ptr(None), _ptr(pooled.k), _ptr(pooled.v), _ptr(pooled.table), _i(pooled.k.shape[0]),
+          _i(pooled.pool), _ptr(turn), _stream(q))
 
 
 def tc_row_blocks(ctas_one: int, ctas_two: int, sms: int, behind_cache: bool) -> int:

@@ -408,6 +408,8 @@ ILB_EXPORT int ilb_qk_norm_rope_cache(
 // turn: the first `rotary_dim` elements of a head in pairs (i, i + rotary_dim / 2) by `rope`; turn_v: all dv elements
 // of a value in pairs (i, i + dv / 2) by `v_rope`.  Either table may be null.
 // A row's units of VEC elements are dealt to gridDim.y blocks; every one of them takes the row's sums itself.
+// POOL (steps of single tokens only): a token that completes a block of `pool` positions also writes the block's mean key
+// and value (its own and the ones before it in the cache) to row pos / pool of the pooled pages; see pool_means below.
 template <typename T, int VEC> struct RowUnit;
 template <typename T> struct RowUnit<T, 1> {
   __device__ static __forceinline__ void load(const T* p, float* x) { x[0] = to_float(*p); }
@@ -424,13 +426,14 @@ struct RowsParams {
   const int* positions; const int* seq_of_token; const int* block_table;
   int max_blocks, page_size, num_pages, nq, nkv, d, dv, rotary_dim, qkv_stride, q_out_stride;
   float eps;
+  const int* p_table; int p_num_pages, pool;
 };
 
 constexpr int kRowsThreads = 256;
 
-template <typename TQ, typename TC, int VEC>
+template <typename TQ, typename TC, int VEC, bool POOL>
 __global__ void __launch_bounds__(kRowsThreads)
-rows_norm_rope_kernel(const TQ* __restrict__ qkv, TQ* __restrict__ q_out, TC* __restrict__ k_cache, TC* __restrict__ v_cache,
+rows_norm_rope_kernel(const TQ* __restrict__ qkv, TQ* __restrict__ q_out, TC* k_cache, TC* v_cache, TC* pk_cache, TC* pv_cache,
                       const RowsParams p) {
   ilb::pdl_launch_dependents();
   ilb::pdl_wait();
@@ -456,6 +459,19 @@ rows_norm_rope_kernel(const TQ* __restrict__ qkv, TQ* __restrict__ q_out, TC* __
     if (blk >= 0 && blk < p.max_blocks) {
       const int page = p.block_table[(size_t)p.seq_of_token[t] * p.max_blocks + blk];
       if (page >= 0 && page < p.num_pages) place = (long long)page * p.nkv * p.page_size + pos % p.page_size;      // never write outside the pool
+    }
+  }
+  long long pooled_place = -1;                             // where the block's mean goes, if this token completes one
+  int first = 0, pos = 0;
+  if constexpr (POOL) {
+    pos = p.positions[t];
+    if (place >= 0 && (pos + 1) % p.pool == 0) {
+      const int b = pos / p.pool;
+      first = b * p.pool;
+      if (b / p.page_size < p.max_blocks) {
+        const int page = p.p_table[(size_t)p.seq_of_token[t] * p.max_blocks + b / p.page_size];
+        if (page >= 0 && page < p.p_num_pages) pooled_place = (long long)page * p.nkv * p.page_size + b % p.page_size;
+      }
     }
   }
   const int units = (nqd + nkd + nvd) / VEC;
@@ -497,9 +513,44 @@ rows_norm_rope_kernel(const TQ* __restrict__ qkv, TQ* __restrict__ q_out, TC* __
       RowUnit<TQ, VEC>::store(dst, x);
       if (pair) RowUnit<TQ, VEC>::store(dst + half, y);
     } else {
-      TC* dst = (kind == 1 ? k_cache : v_cache) + ((size_t)place + (size_t)h * p.page_size) * width + c;
+      TC* cache = kind == 1 ? k_cache : v_cache;
+      TC* dst = cache + ((size_t)place + (size_t)h * p.page_size) * width + c;
       RowUnit<TC, VEC>::store(dst, x);
       if (pair) RowUnit<TC, VEC>::store(dst + half, y);
+      if constexpr (POOL) {
+        if (pooled_place >= 0) {
+          const int* table = p.block_table + (size_t)p.seq_of_token[t] * p.max_blocks;
+          TC* mean = (kind == 1 ? pk_cache : pv_cache) + ((size_t)pooled_place + (size_t)h * p.page_size) * width + c;
+          for (int member = 0; member < (pair ? 2 : 1); ++member) {
+            const int off = member * half;
+            float sum[VEC], own[VEC];
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) { sum[i] = 0.f; own[i] = to_float(from_float<TC>(member ? y[i] : x[i])); }
+            constexpr int kFlight = 4;                     // rows whose loads are in flight together
+            for (int j0 = first; j0 < pos; j0 += kFlight) {
+              float r[kFlight][VEC];
+#pragma unroll
+              for (int f = 0; f < kFlight; ++f) {
+                const int j = j0 + f;
+                const int page = j < pos ? table[j / p.page_size] : -1;
+                if (page >= 0 && page < p.num_pages)
+                  RowUnit<TC, VEC>::load(cache + (((size_t)page * p.nkv + h) * p.page_size + j % p.page_size) * width + c + off, r[f]);
+                else {
+#pragma unroll
+                  for (int i = 0; i < VEC; ++i) r[f][i] = 0.f;
+                }
+              }
+#pragma unroll
+              for (int f = 0; f < kFlight; ++f)
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) sum[i] += r[f][i];
+            }
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) sum[i] = (sum[i] + own[i]) / (float)p.pool;
+            RowUnit<TC, VEC>::store(mean + off, sum);
+          }
+        }
+      }
     }
   }
 }
@@ -508,7 +559,7 @@ ILB_EXPORT int ilb_rows_norm_rope_cache(
     const void* qkv, void* q_out, int dtype, const float* q_weight, const float* k_weight, float eps, const float* rope,
     int rotary_dim, const float* v_rope, const int* positions, const int* seq_of_token, const int* block_table, int max_blocks,
     int page_size, int num_pages, void* k_cache, void* v_cache, int n_tokens, int nq, int nkv, int d, int dv, int qkv_stride,
-    int q_out_stride, cudaStream_t stream) {
+    int q_out_stride, void* pk_cache, void* pv_cache, const int* p_table, int p_num_pages, int pool, cudaStream_t stream) {
   ILB_REQUIRE(n_tokens >= 0 && nq > 0 && nkv > 0 && d > 0 && dv > 0 && eps > 0.f, "rows_norm_rope: bad sizes");
   ILB_REQUIRE(q_weight != nullptr && k_weight != nullptr, "rows_norm_rope: the norms' weights are missing");
   ILB_REQUIRE(rope == nullptr || (rotary_dim > 0 && rotary_dim % 2 == 0 && rotary_dim <= d),
@@ -518,25 +569,24 @@ ILB_EXPORT int ilb_rows_norm_rope_cache(
   ILB_REQUIRE((k_cache == nullptr) == (v_cache == nullptr), "rows_norm_rope: need both caches or none");
   ILB_REQUIRE(k_cache == nullptr || (page_size > 0 && max_blocks > 0 && num_pages > 0), "rows_norm_rope: bad cache geometry");
   ILB_REQUIRE(dtype == kF32 || dtype == kBF16, "rows_norm_rope: unknown dtype %d", dtype);
+  ILB_REQUIRE(pool == 0 || (pool > 0 && k_cache != nullptr && pk_cache != nullptr && pv_cache != nullptr && p_table != nullptr && p_num_pages > 0),
+              "rows_norm_rope: pooled rows need both sets of pages");
   if (n_tokens == 0) return 0;
   const RowsParams p{q_weight, k_weight, (const float2*)rope, (const float2*)v_rope, positions, seq_of_token, block_table, max_blocks,
-                     page_size, num_pages, nq, nkv, d, dv, rope != nullptr ? rotary_dim : 0, qkv_stride, q_out_stride, eps};
+                     page_size, num_pages, nq, nkv, d, dv, rope != nullptr ? rotary_dim : 0, qkv_stride, q_out_stride, eps, p_table, p_num_pages, pool};
   auto a16 = [](const void* x) { return (uintptr_t)x % 16 == 0; };
   const bool vec = dtype == kBF16 && d % 8 == 0 && dv % 8 == 0 && (rope == nullptr || rotary_dim % 16 == 0) && (v_rope == nullptr || dv % 16 == 0) &&
-                   qkv_stride % 8 == 0 && q_out_stride % 8 == 0 && a16(qkv) && a16(q_out) && a16(k_cache) && a16(v_cache);
+                   qkv_stride % 8 == 0 && q_out_stride % 8 == 0 && a16(qkv) && a16(q_out) && a16(k_cache) && a16(v_cache) && a16(pk_cache) && a16(pv_cache);
   const int units = ((nq + nkv) * d + nkv * dv) / (vec ? 8 : 1);
   int ny = 1;
   while (n_tokens * ny < 296 && ny * kRowsThreads < units) ++ny;
   const dim3 grid(n_tokens, ny);
-  if (vec)
-    ilb::launch(rows_norm_rope_kernel<__nv_bfloat16, __nv_bfloat16, 8>, grid, dim3(kRowsThreads), 0, stream, (const __nv_bfloat16*)qkv,
-                (__nv_bfloat16*)q_out, (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, p);
-  else if (dtype == kBF16)
-    ilb::launch(rows_norm_rope_kernel<__nv_bfloat16, __nv_bfloat16, 1>, grid, dim3(kRowsThreads), 0, stream, (const __nv_bfloat16*)qkv,
-                (__nv_bfloat16*)q_out, (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, p);
-  else
-    ilb::launch(rows_norm_rope_kernel<float, float, 1>, grid, dim3(kRowsThreads), 0, stream, (const float*)qkv, (float*)q_out,
-                (float*)k_cache, (float*)v_cache, p);
+#define ILB_ROWS(T, V, POOL) ilb::launch(rows_norm_rope_kernel<T, T, V, POOL>, grid, dim3(kRowsThreads), 0, stream, (const T*)qkv, (T*)q_out, \
+                                         (T*)k_cache, (T*)v_cache, (T*)pk_cache, (T*)pv_cache, p)
+  if (vec) { if (pool) ILB_ROWS(__nv_bfloat16, 8, true); else ILB_ROWS(__nv_bfloat16, 8, false); }
+  else if (dtype == kBF16) { if (pool) ILB_ROWS(__nv_bfloat16, 1, true); else ILB_ROWS(__nv_bfloat16, 1, false); }
+  else { if (pool) ILB_ROWS(float, 1, true); else ILB_ROWS(float, 1, false); }
+#undef ILB_ROWS
   return check_launch("rows_norm_rope_cache");
 }
 

@@ -295,21 +295,21 @@ class GQAttention(Mixer):
         v_rope = self.value_position.table(step) if self.value_position is not None else None
         q = ws.buffer("attn.q", (T, self.nq * self.d), dt)
         ops.scope("attention.qk_norm_rotation_cache_write")
-        ops.rows_norm_rope_cache(qkv, q, self.q_norm, self.k_norm, self.qk_norm_eps, rope, self.rotary_dim, v_rope, step, table,
-                                 cache.k if cache.writable else None, cache.v if cache.writable else None, self.nq, self.nkv, self.d, self.dv)
         pooled = None
         if self.pool:
             pooled = ops.PooledRows(self.pool, cache.pooled.k, cache.pooled.v, step.block_tables[cache.pooled.group])
-            if cache.writable:
-                ops.scope("attention.block_means")
-                ops.pool_means(cache.k, cache.v, pooled, step, table)
+        # (a step of single tokens: a block's other rows are cached already, and the input stage makes its mean too)
+        inside = pooled is not None and cache.writable and step.decode_only
+        ops.rows_norm_rope_cache(qkv, q, self.q_norm, self.k_norm, self.qk_norm_eps, rope, self.rotary_dim, v_rope, step, table,
+                                 cache.k if cache.writable else None, cache.v if cache.writable else None, self.nq, self.nkv, self.d, self.dv,
+                                 pooled=pooled if inside else None)
+        if pooled is not None and cache.writable and not inside:
+            ops.scope("attention.block_means")
+            ops.pool_means(cache.k, cache.v, pooled, step, table)
         o = ws.buffer("attn.o", (T, self.nq * self.dv), dt)
         ops.scope("attention.attention")
         ops.attention(q, o, cache.k, cache.v, step, table, self.window or 0, self.scale, self.nq, self.nkv, self.d, workspace=ws,
-                      decode_chunk=self.decode_chunk, dv=self.dv, pooled=pooled)
-        if v_rope is not None:
-            ops.scope("attention.turn_back")
-            ops.turn_back(o, v_rope, self.nq)
+                      decode_chunk=self.decode_chunk, dv=self.dv, pooled=pooled, turn=v_rope)
         self._finish(o, qkv, gate_col0, residual, out)
 
     def _finish(self, o: torch.Tensor, qkv: torch.Tensor, gate_col0: int, residual: torch.Tensor, out: Optional[torch.Tensor]) -> None:

@@ -136,9 +136,12 @@ class TwoMatrixFeedForward(FeedForward):
     def forward(self, x: torch.Tensor, residual: torch.Tensor, step, accumulate: bool = True) -> None:
         act = self.ctx.workspace.buffer("mlp.act", (x.shape[0], self.inter), self.ctx.dtype)
         ops.scope("feed_forward.up")
-        linear(x, self.w_up, act)
-        ops.scope("feed_forward.activation")
-        ops.act_rows(act, self.activation, act)
+        if self.activation == "relu2" and act.dtype == torch.bfloat16 and ops.gemm_tc_eligible(x, self.w_up, act):
+            ops.gemm_tc(x, self.w_up, act, relu2=True)      # (squared in the product's epilogue, before the one rounding)
+        else:
+            linear(x, self.w_up, act)
+            ops.scope("feed_forward.activation")
+            ops.act_rows(act, self.activation, act)
         ops.scope("feed_forward.down")
         linear(act, self.w_down, residual, accumulate=accumulate)
 

@@ -16,8 +16,8 @@ from inferloop_b200.parts.base import CacheNeeds, PagedKVNeed
 class FakeRunner:
     device = None
 
-    def __init__(self, vocab=50, page_size=4, num_pages=16, max_requests=8, max_positions=512, window=None):
-        needs = [CacheNeeds(paged=PagedKVNeed(1, 16, None)), CacheNeeds(paged=PagedKVNeed(1, 16, window))]
+    def __init__(self, vocab=50, page_size=4, num_pages=16, max_requests=8, max_positions=512, window=None, needs=None):
+        needs = needs or [CacheNeeds(paged=PagedKVNeed(1, 16, None)), CacheNeeds(paged=PagedKVNeed(1, 16, window))]
         self.cache = CacheManager(needs, page_size, num_pages, max_requests)
         self.spec = SimpleNamespace(vocab_size=vocab, max_positions=max_positions)
         self.history = {}

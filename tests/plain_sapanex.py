@@ -98,15 +98,17 @@ def attention(w, p, m, h, eps):
     q = (rms(h @ w[p + "q"].T, eps) * w[p + "q.norm"]).view(T, H, d)
     k = (rms(h @ w[p + "k"].T, eps) * w[p + "k.norm"]).view(T, G, d)
     v = (h @ w[p + "v"].T).view(T, G, dv)
-    rot = m["rot"]
-    freq, stretch = frequencies(rot["base"], int(rot["dims"]), rot.get("scaling"))
-    vfreq, _ = frequencies(rot["base"], dv)
-    q, k = turn(q, positions, freq, stretch), turn(k, positions, freq, stretch)
-    v = turn(v, positions, vfreq)
+    rot = m.get("rot")
+    if rot is not None:
+        freq, stretch = frequencies(rot["base"], int(rot["dims"]), rot.get("scaling"))
+        vfreq, _ = frequencies(rot["base"], dv)
+        q, k = turn(q, positions, freq, stretch), turn(k, positions, freq, stretch)
+        v = turn(v, positions, vfreq)
     mask = m.get("mask")
     o = pooled_window_attention(q, k, v, float(m["scale"]), None if mask is None else int(mask["size"]),
                                 None if mask is None else int(mask["pool"]))
-    o = turn(o, positions, vfreq, sign=-1.0)
+    if rot is not None:
+        o = turn(o, positions, vfreq, sign=-1.0)
     return o.reshape(T, H * dv) @ w[p + "o"].T
 
 
