@@ -249,8 +249,39 @@ def zebivik_numbers(cfg: dict):
             "state_bytes_per_seq": state}
 
 
+def sapanex_numbers(cfg: dict):
+    """The same for a Sapanex configuration.  A token of a windowed layer sees at most its window and a row per block before
+    it: the window's rows count as state of the sequence (read by a decode step), the blocks' as bytes per token of context,
+    and a pair's flops, which do not grow with the context but for the blocks, as parameters a token touches."""
+    W, V, L = cfg["width"], cfg["vocab"], len(cfg["layers"])
+    params, kv, attn, state = 0, 0, 0, 0
+    for layer in cfg["layers"]:
+        m, f = layer["mixer"], layer["mlp"]
+        if layer["type"] == "attention":
+            H, G, row = m["heads"], m["kv_heads"], m["kv_heads"] * (m["dim"] + m["vdim"]) * 2
+            params += ((H + G) * m["dim"] + G * m["vdim"] + H * m["vdim"]) * W
+            mask = m.get("mask")
+            if mask is None:
+                kv += row
+                attn += 2 * H * (m["dim"] + m["vdim"])
+            else:
+                state += mask["size"] * row
+                kv += row / mask["pool"]
+                params += H * (m["dim"] + m["vdim"]) * mask["size"]
+        else:
+            inner = m["heads"] * m["dim"]
+            params += 6 * inner * W + m["dim"] * (inner + W)
+            state += 2 * 4 * inner * m["dim"]
+        if f is not None:
+            params += 2 * W * f["ff"]
+    return {"layer_params": params / L, "head_params": V * W, "kv_bytes_per_token": kv, "attn_flops_per_pair": attn, "layers": L,
+            "state_bytes_per_seq": state}
+
+
 def model_numbers(cfg: dict):
     """Parameters the matrix products of one token touch, and bytes of cache per token."""
+    if cfg.get("architecture") == "Sapanex":
+        return sapanex_numbers(cfg)
     if cfg.get("architecture") == "Zebivik":
         return zebivik_numbers(cfg)
     if cfg.get("architecture") == "Dalavik":
@@ -995,6 +1026,61 @@ def run_zebivik(args) -> dict:
     return out
 
 
+# ----------------------------------------------------------------------------- the Sapanex decoder beside Sufolix and Mamevik
+def sapanex_config(kind: str, layers: int, width: int, vocab: int, ff: int) -> dict:
+    """`kind`: "attention" (every layer attends over a window and the pooled blocks before it), "delta" (every layer is a
+    generalized delta rule) or "mixed" (three recurrent layers, one attention layer, in turn)."""
+    att = {"type": "attention", "mixer": {"heads": 16, "kv_heads": 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5,
+                                          "rot": {"base": 500000.0, "dims": 64, "scaling": {"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}},
+                                          "mask": {"size": 1024, "pool": 64}}}
+    rec = {"type": "general_delta", "mixer": {"heads": width // 128, "dim": 128}}
+    pick = {"attention": lambda i: att, "delta": lambda i: rec, "mixed": lambda i: att if i % 4 == 3 else rec}[kind]
+    return {"architecture": "Sapanex", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "postln_alpha": 2.0,
+            "layers": [dict(pick(i), mlp={"kind": "dense", "ff": ff}) for i in range(layers)]}
+
+
+def run_sapanex(args) -> dict:
+    """Decode and prefill of the Sapanex decoder at layer sizes of a real model (windowed attention with pooled blocks, delta
+    rules, both in turn), beside the closest models the engine has at the same width and layers: the Sufolix decoder with a
+    dense feed-forward of as many parameters (the attention layers' relative) and the Mamevik decoder with state-space
+    recurrences of as many state elements (the recurrent layers' relative; its feed-forward is routed)."""
+    import torch
+    L, W, V, FF = args.layers if args.layers != FULL_LAYERS else 8, 2048, 32768, 8192
+    which = ["attention", "delta", "mixed"] if args.sapanex == "all" else [args.sapanex]
+    out = {"metric": "sapanex_vs_sufolix_and_mamevik_equal_size", "unit": "tokens/s", "n_gpus": 1, "dtype": "bf16", "data": "synthetic",
+           "steps": args.steps, "warmup": args.warmup, "batch": args.batch, "peaks": peaks(), "cases": {}}
+    arms = {kind: sapanex_config(kind, L, W, V, FF * 3 // 2) for kind in which}
+    arms["sufolix"] = sufolix_config("dense", L, W, 16, 4, 128, FF, 0, 0, 0, 0, V, 1)
+    arms["sufolix"].pop("streams")
+    arms["mamevik"] = mamevik_config("ssd", L, W, V, 16, 2, 1408)
+    for arm, cfg in arms.items():
+        pages = (args.batch * (PROMPT_LEN + args.steps + args.warmup + 64) + PREFILL_LEN) // PAGE + 64
+        bench = Bench(cfg, SEED, pages, max(args.batch, 8), 8192, PREFILL_LEN)
+        with ClockSampler() as clocks:
+            tps, ms, kernels, ctx = bench.decode_device(args.batch, args.steps, args.warmup, arm, PROMPT_LEN)
+        routed = sum(1 for l in cfg["layers"] if l["mlp"] is not None and l["mlp"]["kind"] == "moe")
+        touched = bench.weight_bytes - routed * 3 * W * 1408 * 2 * max(0, 16 - min(16, args.batch * 2))
+        step_bytes = touched + args.batch * (ctx * bench.nums["kv_bytes_per_token"] + bench.nums.get("state_bytes_per_seq", 0))
+        r = {"decode_tokens_per_s": round(tps, 1), "decode_ms_per_step": round(ms, 4), "kernels_per_step": kernels,
+             "decode_frac_of_hbm": round(step_bytes / (ms / 1e3) / 1e9 / bench.pk["hbm_gbs"], 4),
+             "weights_gb": round(bench.weight_bytes / 1e9, 3), "clocks": clocks.summary(),
+             "prefill": bench.prefill_timed(PREFILL_LEN, 3, PREFILL_SAMPLES)}
+        if args.breakdown:
+            r["breakdown"] = bench.breakdown(args.batch, PROMPT_LEN, PREFILL_LEN)
+        out["cases"][arm] = r
+        del bench
+        torch.cuda.empty_cache()
+    out["sizes"] = {"layers": L, "width": W, "vocab": V, "ff": FF * 3 // 2,
+                    "mixers": {kind: sorted({json.dumps(l["mixer"], sort_keys=True) for l in arms[kind]["layers"]}) for kind in which}}
+    for kind in which:
+        c = out["cases"][kind]
+        for other in ("sufolix", "mamevik"):
+            base = out["cases"][other]
+            c[f"decode_ms_per_step_over_{other}"] = round(c["decode_ms_per_step"] / base["decode_ms_per_step"], 4)
+            c[f"prefill_ms_over_{other}"] = round(c["prefill"]["ms"] / base["prefill"]["ms"], 4)
+    return out
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1017,6 +1103,8 @@ def main() -> int:
                     help="the Dalavik decoder beside a Sufolix model with a dense feed-forward of equal size (decode, prefill, op classes with --breakdown)")
     ap.add_argument("--zebivik", nargs="?", const="all", default=None, choices=["all", "parallel", "rglru", "mixed"],
                     help="the Zebivik decoder beside a Mamevik and a Sufolix model of equal size (decode, prefill, op classes with --breakdown)")
+    ap.add_argument("--sapanex", nargs="?", const="all", default=None, choices=["all", "attention", "delta", "mixed"],
+                    help="the Sapanex decoder beside a Sufolix and a Mamevik model of equal size (decode, prefill, op classes with --breakdown)")
     args = ap.parse_args()
 
     if args.impl == "reference":
@@ -1046,6 +1134,9 @@ def main() -> int:
         return 0
     if args.zebivik:
         print(json.dumps(run_zebivik(args)))
+        return 0
+    if args.sapanex:
+        print(json.dumps(run_sapanex(args)))
         return 0
     result = {"8b": run_8b, "14b-mixed": run_14b_mixed, "32b-long": run_32b_long}[args.config](args)
     print(json.dumps(result))

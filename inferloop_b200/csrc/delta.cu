@@ -12,7 +12,21 @@
 //   delta_scan   token by token, any sizes up to 256 rows.  A block owns 16 columns of a head's state of one sequence in
 //                registers: eight threads a column, a warp four columns; the read-out u^T S and the output r^T S are sums
 //                over the eight threads of a column.  The tokens' channel vectors are made 16 tokens at a time in shared
-//                memory.
+//                memory.  For short portions, and sizes that the two below do not take.
+//   delta_prep, delta_chunks
+//                long portions, 16 tokens at a time.  Inside a chunk let D_t be the product of the decays up to token t
+//                (D_0 = 1 before the first) and S~_t = S_t / D_t.  With
+//                    p_t = D_{t-1} u_t,   q_t = g_t u_t / D_t,   m_t = k_t / D_t,   s_t = D_t r_t
+//                the recurrence reads  S~_t = S~_{t-1} - q_t z_t^T + m_t v_t^T,  z_t = S~_{t-1}^T p_t,  o_t = S~_t^T s_t, so
+//                    z_t = S_0^T p_t + sum_{j<t} ((p_t.m_j) v_j - (p_t.q_j) z_j)
+//                which is a triangular system over the chunk's tokens.  Its solution is linear in the chunk's incoming
+//                state: Z = W S_0 + U, O = X S_0 + Y, with W, U, X, Y from the tokens alone.  delta_prep makes those (and
+//                D_16 q_t, D_16 m_t, D_16) for every chunk and head side by side; delta_chunks walks a sequence's chunks with
+//                a block per head and 16 columns of the state in registers: two thin products with the state, then
+//                    S_16 = D_16 S_0 + sum_t (D_16 m_t) v_t^T - (D_16 q_t) z_t^T.
+//                Decays of at least exp(-log_decay) a token keep every scale of a chunk within exp(16 log_decay).
+//   delta_step   single tokens, everything between the projections of a layer: the low-rank map, the decay, the recurrence,
+//                the norm of each head and the output gate; a block per (head, sequence) with the whole state in registers.
 //
 // Everything is 32-bit; the projections come in the compute dtype.  A sequence whose slot is negative (a dummy row that
 // pads a recorded launch) starts from zero and stores nothing.
@@ -198,6 +212,553 @@ ILB_EXPORT int ilb_delta_scan(const void* proj, int dtype, int ld, int col_r, in
   if (q == 2) return scan_launch<__nv_bfloat16, 2>(p, stream);
   if (q == 4) return scan_launch<__nv_bfloat16, 4>(p, stream);
   return scan_launch<__nv_bfloat16, 8>(p, stream);
+}
+
+// ---------------------------------------------------------------- chunks
+constexpr int kChunk = 16;
+
+// Floats of one (chunk, head) in scratch: W, X, D q, D m [16][KP], D [KP], then U, Y, V [16][DP]; KP rows, DP columns, padded.
+__host__ __device__ __forceinline__ long long chunk_floats(int KP, int DP) { return (long long)4 * kChunk * KP + KP + (long long)3 * kChunk * DP; }
+__host__ __device__ __forceinline__ int padded_cols(int dv) { return (dv + kCols - 1) / kCols * kCols; }
+static inline int rows_per_thread(int d) { return d <= 64 ? 2 : (d <= 128 ? 4 : 8); }
+
+// which sequence, and which of its chunks, block `b` works on; false: none
+__device__ __forceinline__ bool find_chunk(const int* __restrict__ cu_q, int n_seqs, int b, int& seq, int& index) {
+  for (seq = 0; seq < n_seqs; ++seq) {
+    const int n = (cu_q[seq + 1] - cu_q[seq] + kChunk - 1) / kChunk;
+    if (b < n) { index = b; return true; }
+    b -= n;
+  }
+  return false;
+}
+
+constexpr int kPrepThreads = 128;
+
+static inline size_t prep_smem_floats(int KP, int DP) { return (size_t)4 * kChunk * (KP + 4) + (size_t)kChunk * DP + 4 * kChunk * kChunk; }
+
+template <typename TI>
+__global__ void __launch_bounds__(kPrepThreads, 4)
+delta_prep_kernel(const DeltaParams p, float* __restrict__ scratch, int KP) {
+  ilb::pdl_launch_dependents();
+  ilb::pdl_wait();
+  constexpr bool FAST = sizeof(TI) == 2;
+  extern __shared__ __align__(16) float sm[];
+  const int DP = padded_cols(p.dv), ld = KP + 4;
+  float* P = sm;                                         // [16][ld] each
+  float* R = P + kChunk * ld;
+  float* Qv = R + kChunk * ld;
+  float* M = Qv + kChunk * ld;
+  float* V = M + kChunk * ld;                            // [16][DP]
+  float* A = V + kChunk * DP;                            // [16][16] each: p.q, p.m (j < t), s.q, s.m (j <= t); zero elsewhere
+  float* B = A + kChunk * kChunk;
+  float* C = B + kChunk * kChunk;
+  float* E = C + kChunk * kChunk;
+  __shared__ float inv_norm[kChunk];
+  int seq, ci;
+  if (!find_chunk(p.cu_q, p.n_seqs, blockIdx.x, seq, ci)) return;
+  const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int tok0 = p.cu_q[seq] + ci * kChunk, ts = min(kChunk, p.cu_q[seq + 1] - tok0);
+  const int inner_k = p.heads * p.d;
+  const TI* proj = reinterpret_cast<const TI*>(p.proj);
+  float* out = scratch + ((size_t)blockIdx.x * p.heads + h) * chunk_floats(KP, DP);
+  float* outW = out; float* outX = outW + kChunk * KP; float* outQ = outX + kChunk * KP; float* outM = outQ + kChunk * KP;
+  float* outD = outM + kChunk * KP; float* outU = outD + KP; float* outY = outU + kChunk * DP; float* outV = outY + kChunk * DP;
+
+  for (int n = tid; n < KP; n += kPrepThreads) {
+#pragma unroll
+    for (int t = 0; t < kChunk; ++t)
+      M[t * ld + n] = (n < p.d && t < ts) ? to_float(proj[(size_t)(tok0 + t) * p.ld + p.col_k + h * p.d + n]) : 0.f;
+  }
+  for (int c = tid; c < DP; c += kPrepThreads) {
+#pragma unroll
+    for (int t = 0; t < kChunk; ++t) {
+      const float v = (c < p.dv && t < ts) ? to_float(proj[(size_t)(tok0 + t) * p.ld + p.col_v + h * p.dv + c]) : 0.f;
+      V[t * DP + c] = v;
+      outV[t * DP + c] = v;
+    }
+  }
+  __syncthreads();
+  for (int t = warp; t < kChunk; t += kPrepThreads / 32) {
+    float ss = 0.f;
+    for (int n = lane; n < KP; n += 32) ss = fmaf(M[t * ld + n], M[t * ld + n], ss);
+    ss = warp_sum(ss);
+    if (lane == 0) inv_norm[t] = 1.0f / sqrtf(ss + p.unit_eps);
+  }
+  __syncthreads();
+  for (int n = tid; n < KP; n += kPrepThreads) {
+    const bool live = n < p.d;
+    const int ch = h * p.d + (live ? n : 0);
+    const float w0 = p.w0[ch], ab = p.ab[ch];
+    float r[kChunk], a[kChunk], l[kChunk];
+#pragma unroll
+    for (int t = 0; t < kChunk; ++t) {                   // all loads in flight together
+      const bool on = live && t < ts;
+      const TI* row = proj + (size_t)(tok0 + (on ? t : 0)) * p.ld;
+      r[t] = on ? to_float(row[p.col_r + ch]) : 0.f;
+      a[t] = to_float(row[p.col_a + ch]);
+      l[t] = p.low[(size_t)(tok0 + (on ? t : 0)) * inner_k + ch];
+    }
+    float D = 1.f;
+#pragma unroll
+    for (int t = 0; t < kChunk; ++t) {
+      const bool on = live && t < ts;
+      const float k = M[t * ld + n], u = k * inv_norm[t];
+      const float w = on ? exp_t<FAST>(-p.log_decay * sigmoid_t<FAST>(l[t] + w0)) : 1.f;
+      const float g = on ? sigmoid_t<FAST>(a[t] + ab) : 0.f;
+      P[t * ld + n] = D * u;
+      D *= w;
+      const float inv = 1.0f / D;
+      Qv[t * ld + n] = g * u * inv;
+      M[t * ld + n] = k * inv;
+      R[t * ld + n] = D * r[t];
+    }
+    outD[n] = D;
+#pragma unroll
+    for (int t = 0; t < kChunk; ++t) {
+      outQ[t * KP + n] = Qv[t * ld + n] * D;
+      outM[t * KP + n] = M[t * ld + n] * D;
+    }
+  }
+  __syncthreads();
+  {   // rows of P and R against rows of Q and M: a thread takes four rows and one column of both
+    const int j = tid & 15, rg = tid >> 4;               // rows 4 (rg & 3) .. + 3 of P (rg < 4) or of R
+    const float* rows = (rg < 4 ? P : R) + (size_t)(rg & 3) * 4 * ld;
+    float x[4] = {0.f, 0.f, 0.f, 0.f}, y[4] = {0.f, 0.f, 0.f, 0.f};
+    for (int n = 0; n < KP; n += 4) {
+      const float4 q = *reinterpret_cast<const float4*>(Qv + j * ld + n), m = *reinterpret_cast<const float4*>(M + j * ld + n);
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const float4 v = *reinterpret_cast<const float4*>(rows + i * ld + n);
+        x[i] = fmaf(v.x, q.x, x[i]); x[i] = fmaf(v.y, q.y, x[i]); x[i] = fmaf(v.z, q.z, x[i]); x[i] = fmaf(v.w, q.w, x[i]);
+        y[i] = fmaf(v.x, m.x, y[i]); y[i] = fmaf(v.y, m.y, y[i]); y[i] = fmaf(v.z, m.z, y[i]); y[i] = fmaf(v.w, m.w, y[i]);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int t = 4 * (rg & 3) + i;
+      const bool keep = rg < 4 ? j < t : j <= t;
+      (rg < 4 ? A : C)[t * kChunk + j] = keep ? x[i] : 0.f;
+      (rg < 4 ? B : E)[t * kChunk + j] = keep ? y[i] : 0.f;
+    }
+  }
+  __syncthreads();
+  // Row t of a 16 x 16 matrix from shared memory, its first `n` elements.  (The fence keeps the compiler from holding whole
+  // matrices in registers across the columns' loop.)
+  auto row16 = [&](const float* m, int t, int n, float (&r)[kChunk]) {
+    asm volatile("" ::: "memory");
+#pragma unroll
+    for (int j = 0; j < kChunk / 4; ++j) {
+      if (4 * j < n) {
+        const float4 v = *reinterpret_cast<const float4*>(m + t * kChunk + 4 * j);
+        r[4 * j] = v.x; r[4 * j + 1] = v.y; r[4 * j + 2] = v.z; r[4 * j + 3] = v.w;
+      }
+    }
+  };
+  for (int n = tid; n < KP; n += kPrepThreads) {         // W = (I + A)^-1 P,  X = R - C W, column by column
+    float w[kChunk];
+#pragma unroll
+    for (int t = 0; t < kChunk; ++t) {
+      float v = P[t * ld + n], x = R[t * ld + n], a[kChunk], c[kChunk];
+      row16(A, t, t, a);
+      row16(C, t, t + 1, c);
+#pragma unroll
+      for (int j = 0; j < t; ++j) { v = fmaf(-a[j], w[j], v); x = fmaf(-c[j], w[j], x); }
+      w[t] = v;
+      outW[t * KP + n] = v;
+      outX[t * KP + n] = fmaf(-c[t], v, x);
+    }
+  }
+  for (int c0 = tid; c0 < DP; c0 += kPrepThreads) {      // U = (I + A)^-1 B V,  Y = E V - C U
+    float u[kChunk], v[kChunk];
+#pragma unroll
+    for (int t = 0; t < kChunk; ++t) v[t] = V[t * DP + c0];
+#pragma unroll
+    for (int t = 0; t < kChunk; ++t) {
+      float s = 0.f, y = 0.f, a[kChunk], b[kChunk];
+      row16(A, t, t, a);
+      row16(B, t, t, b);
+#pragma unroll
+      for (int j = 0; j < t; ++j) { s = fmaf(b[j], v[j], s); s = fmaf(-a[j], u[j], s); }
+      u[t] = s;
+      outU[t * DP + c0] = s;
+      row16(E, t, t + 1, a);
+      row16(C, t, t + 1, b);
+#pragma unroll
+      for (int j = 0; j <= t; ++j) { y = fmaf(a[j], v[j], y); y = fmaf(-b[j], u[j], y); }
+      outY[t * DP + c0] = y;
+    }
+  }
+}
+
+__device__ __forceinline__ void delta_cp_async_16(float* dst, const float* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+
+static inline size_t chunks_smem_floats(int KP) {
+  return 2 * ((size_t)4 * kChunk * KP + KP + 3 * kChunk * kCols) + (size_t)4 * 2 * kChunk * kCols + kChunk * kCols;
+}
+
+// RQ: rows of the state a thread holds (of 32 RQ), times four columns.  Thread (warp, lane): rows (8 warp + lane / 4) RQ ..,
+// columns 4 (lane % 4) .. of the block's 16.
+template <int RQ>
+__global__ void __launch_bounds__(kScanThreads)
+delta_chunks_kernel(const DeltaParams p, const float* __restrict__ scratch) {
+  ilb::pdl_launch_dependents();
+  ilb::pdl_wait();
+  constexpr int KP = 32 * RQ;
+  constexpr int kVecs = 4 * kChunk * KP, kBuf = kVecs + KP + 3 * kChunk * kCols;      // floats of one buffer
+  extern __shared__ __align__(16) float sm[];
+  float* red = sm + 2 * kBuf;                            // [4 warps][32][kCols]: sums over a warp's rows, of W S then X S
+  float* zs = red + 4 * 2 * kChunk * kCols;              // [16][kCols]
+  const int h = blockIdx.x, cb = blockIdx.y, c0 = cb * kCols, seq = blockIdx.z;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, cg = lane & 3, rl = lane >> 2, rg = warp * 8 + rl;
+  const int DP = padded_cols(p.dv);
+  const int tok0 = p.cu_q[seq], q_len = p.cu_q[seq + 1] - tok0, n_chunks = (q_len + kChunk - 1) / kChunk;
+  if (n_chunks == 0) return;
+  int first = 0;
+  for (int s = 0; s < seq; ++s) first += (p.cu_q[s + 1] - p.cu_q[s] + kChunk - 1) / kChunk;
+  const int slot = p.slots[seq];
+  float* own = slot >= 0 ? p.state + ((size_t)slot * p.heads + h) * p.d * p.dv : nullptr;
+  const int inner_v = p.heads * p.dv;
+  const long long per = chunk_floats(KP, DP);
+
+  auto issue = [&](int ci) {
+    const float* src = scratch + ((size_t)(first + ci) * p.heads + h) * per;
+    float* dst = sm + (ci & 1) * kBuf;
+    for (int i = tid; i < (kVecs + KP) / 4; i += kScanThreads) delta_cp_async_16(dst + 4 * i, src + 4 * i);
+    const float* cols = src + kVecs + KP + c0;           // U, Y, V: this block's 16 columns of each
+    for (int i = tid; i < 3 * kChunk * kCols / 4; i += kScanThreads)
+      delta_cp_async_16(dst + kVecs + KP + 4 * i, cols + (size_t)(i / (kCols / 4)) * DP + (i % (kCols / 4)) * 4);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  issue(0);
+  float S[RQ][4];
+#pragma unroll
+  for (int i = 0; i < RQ; ++i)
+#pragma unroll
+    for (int c = 0; c < 4; ++c) {
+      const int n = rg * RQ + i, col = c0 + 4 * cg + c;
+      S[i][c] = (own != nullptr && n < p.d && col < p.dv) ? own[(size_t)n * p.dv + col] : 0.f;
+    }
+  // RQ consecutive floats of row `row` at this thread's rows
+  auto rows_at = [&](const float* row, float (&v)[RQ]) {
+    if constexpr (RQ == 2) {
+      const float2 a = *reinterpret_cast<const float2*>(row + rg * RQ);
+      v[0] = a.x; v[1] = a.y;
+    } else {
+#pragma unroll
+      for (int i = 0; i < RQ / 4; ++i) {
+        const float4 a = *reinterpret_cast<const float4*>(row + rg * RQ + 4 * i);
+        v[4 * i] = a.x; v[4 * i + 1] = a.y; v[4 * i + 2] = a.z; v[4 * i + 3] = a.w;
+      }
+    }
+  };
+  for (int ci = 0; ci < n_chunks; ++ci) {
+    if (ci + 1 < n_chunks) {
+      issue(ci + 1);
+      asm volatile("cp.async.wait_group 1;" ::: "memory");
+    } else {
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+    }
+    __syncthreads();
+    const float* buf = sm + (ci & 1) * kBuf;
+    const float* Dv = buf + kVecs;
+    const float* Us = Dv + KP;                           // [16][kCols] each: U, Y, V
+    // products of the 32 rows of W and X with the state, eight rows at a time; their sums over the warp's rows are dealt
+    // out so that lane group rl ends with row 8 g + rl
+#pragma unroll 1
+    for (int g = 0; g < 4; ++g) {
+      float acc[8][4];
+#pragma unroll
+      for (int v = 0; v < 8; ++v) {
+        float w[RQ];
+        rows_at(buf + (g * 8 + v) * KP, w);
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          float s = w[0] * S[0][c];
+#pragma unroll
+          for (int i = 1; i < RQ; ++i) s = fmaf(w[i], S[i][c], s);
+          acc[v][c] = s;
+        }
+      }
+      float a4[4][4], a2[2][4], a1[4];
+      const bool hi4 = rl & 4, hi2 = rl & 2, hi1 = rl & 1;
+#pragma unroll
+      for (int v = 0; v < 4; ++v)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          const float give = hi4 ? acc[v][c] : acc[v + 4][c], have = hi4 ? acc[v + 4][c] : acc[v][c];
+          a4[v][c] = have + __shfl_xor_sync(0xffffffffu, give, 16);
+        }
+#pragma unroll
+      for (int v = 0; v < 2; ++v)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) {
+          const float give = hi2 ? a4[v][c] : a4[v + 2][c], have = hi2 ? a4[v + 2][c] : a4[v][c];
+          a2[v][c] = have + __shfl_xor_sync(0xffffffffu, give, 8);
+        }
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        const float give = hi1 ? a2[0][c] : a2[1][c], have = hi1 ? a2[1][c] : a2[0][c];
+        a1[c] = have + __shfl_xor_sync(0xffffffffu, give, 4);
+      }
+      *reinterpret_cast<float4*>(red + ((warp * 2 * kChunk) + g * 8 + rl) * kCols + 4 * cg) = make_float4(a1[0], a1[1], a1[2], a1[3]);
+    }
+    __syncthreads();
+    {
+      const int v = tid >> 2, c4 = (tid & 3) * 4;        // row of W (v < 16) or of X
+      float4 s = *reinterpret_cast<const float4*>(Us + v * kCols + c4);       // U's rows, then Y's
+#pragma unroll
+      for (int w = 0; w < 4; ++w) {
+        const float4 a = *reinterpret_cast<const float4*>(red + (w * 2 * kChunk + v) * kCols + c4);
+        s.x += a.x; s.y += a.y; s.z += a.z; s.w += a.w;
+      }
+      if (v < kChunk) {
+        *reinterpret_cast<float4*>(zs + v * kCols + c4) = s;
+      } else {
+        const int t = ci * kChunk + v - kChunk, col = c0 + c4;
+        if (t < q_len) {
+          float* dst = p.y + (size_t)(tok0 + t) * inner_v + (size_t)h * p.dv + col;
+          if (col + 3 < p.dv && (inner_v & 3) == 0 && (p.dv & 3) == 0) *reinterpret_cast<float4*>(dst) = s;
+          else {
+            const float e[4] = {s.x, s.y, s.z, s.w};
+#pragma unroll
+            for (int c = 0; c < 4; ++c) if (col + c < p.dv) dst[c] = e[c];
+          }
+        }
+      }
+    }
+    __syncthreads();
+    {
+      float d[RQ];
+      rows_at(Dv, d);
+#pragma unroll
+      for (int i = 0; i < RQ; ++i)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) S[i][c] *= d[i];
+      const float* Qs = buf + 2 * kChunk * KP;
+      const float* Ms = Qs + kChunk * KP;
+      const float* Vs = Us + 2 * kChunk * kCols;
+#pragma unroll 8
+      for (int t = 0; t < kChunk; ++t) {
+        float q[RQ], m[RQ];
+        rows_at(Qs + t * KP, q);
+        rows_at(Ms + t * KP, m);
+        const float4 z = *reinterpret_cast<const float4*>(zs + t * kCols + 4 * cg);
+        const float4 v = *reinterpret_cast<const float4*>(Vs + t * kCols + 4 * cg);
+#pragma unroll
+        for (int i = 0; i < RQ; ++i) {
+          S[i][0] = fmaf(m[i], v.x, fmaf(-q[i], z.x, S[i][0])); S[i][1] = fmaf(m[i], v.y, fmaf(-q[i], z.y, S[i][1]));
+          S[i][2] = fmaf(m[i], v.z, fmaf(-q[i], z.z, S[i][2])); S[i][3] = fmaf(m[i], v.w, fmaf(-q[i], z.w, S[i][3]));
+        }
+      }
+    }
+    __syncthreads();                                     // everyone is done with this buffer and with zs
+  }
+  if (own != nullptr) {
+#pragma unroll
+    for (int i = 0; i < RQ; ++i)
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        const int n = rg * RQ + i, col = c0 + 4 * cg + c;
+        if (n < p.d && col < p.dv) own[(size_t)n * p.dv + col] = S[i][c];
+      }
+  }
+}
+
+// Floats of scratch that `n_blocks` chunks need.
+ILB_EXPORT long long ilb_delta_chunk_floats(int n_blocks, int heads, int d, int dv) {
+  return (long long)n_blocks * heads * chunk_floats(32 * rows_per_thread(d), padded_cols(dv));
+}
+
+template <int RQ>
+static int chunks_launch(const DeltaParams& p, const float* scratch, cudaStream_t stream) {
+  const size_t smem = sizeof(float) * chunks_smem_floats(32 * RQ);
+  static OncePerDevice once;
+  if (once.first() && cudaFuncSetAttribute(delta_chunks_kernel<RQ>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+    once.forget();
+    return fail("delta_chunks: cannot reserve %zu bytes of shared memory", smem);
+  }
+  ilb::launch(delta_chunks_kernel<RQ>, dim3(p.heads, padded_cols(p.dv) / kCols, p.n_seqs), dim3(kScanThreads), smem, stream, p, scratch);
+  return check_launch("delta_chunks");
+}
+
+template <typename TI>
+static int prep_launch(const DeltaParams& p, float* scratch, int n_blocks, cudaStream_t stream) {
+  const int KP = 32 * rows_per_thread(p.d);
+  const size_t smem = sizeof(float) * prep_smem_floats(KP, padded_cols(p.dv));
+  ILB_REQUIRE(smem <= 200 * 1024, "delta_prep: states of %d x %d do not fit the block's shared memory", p.d, p.dv);
+  static OncePerDevice once;
+  if (once.first() && cudaFuncSetAttribute(delta_prep_kernel<TI>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess) {
+    once.forget();
+    return fail("delta_prep: cannot reserve shared memory");
+  }
+  ilb::launch(delta_prep_kernel<TI>, dim3(n_blocks, p.heads), dim3(kPrepThreads), smem, stream, p, scratch, KP);
+  return check_launch("delta_prep");
+}
+
+// As ilb_delta_scan, 16 tokens at a time; n_blocks = the sum over the sequences of ceil(tokens / 16), scratch of
+// ilb_delta_chunk_floats(n_blocks, ...) floats on a 16-byte boundary.
+ILB_EXPORT int ilb_delta_chunks(const void* proj, int dtype, int ld, int col_r, int col_k, int col_v, int col_a, const float* low,
+                                const float* w0, const float* ab, float log_decay, float unit_eps, float* state, float* y,
+                                const int* cu_q, const int* slots, int n_seqs, int heads, int d, int dv, float* scratch,
+                                long long scratch_floats, int n_blocks, cudaStream_t stream) {
+  const DeltaParams p{proj, ld, col_r, col_k, col_v, col_a, low, w0, ab, state, y, cu_q, slots, n_seqs, heads, d, dv, log_decay, unit_eps};
+  if (int rc = check_sizes(p, dtype)) return rc;
+  ILB_REQUIRE(log_decay >= 0.f && log_decay * kChunk <= 40.f, "delta_chunks: a decay of exp(-%f) a token leaves a chunk's range", (double)log_decay);
+  ILB_REQUIRE(scratch != nullptr && (uintptr_t)scratch % 16 == 0 && ilb_delta_chunk_floats(n_blocks, heads, d, dv) <= scratch_floats,
+              "delta_chunks: scratch too small");
+  ILB_REQUIRE(heads <= 65535, "delta_chunks: too many heads");
+  if (n_seqs == 0 || n_blocks <= 0) return 0;
+  if (int rc = dtype == kF32 ? prep_launch<float>(p, scratch, n_blocks, stream) : prep_launch<__nv_bfloat16>(p, scratch, n_blocks, stream)) return rc;
+  const int rq = rows_per_thread(d);
+  return rq == 2 ? chunks_launch<2>(p, scratch, stream) : rq == 4 ? chunks_launch<4>(p, scratch, stream) : chunks_launch<8>(p, scratch, stream);
+}
+
+// ---------------------------------------------------------------- single tokens
+struct StepParams {
+  DeltaParams a;
+  int col_low, rank, ld_w2;          // the low-rank map's inner row in proj, its size, the row stride of w2 [heads * d][ld_w2]
+  const void* w2;
+  int col_g;                         // the output gate's columns in proj (heads * dv)
+  const float* norm_w; float eps;    // [heads * dv]
+  void* out; int ld_out;             // [sequences' tokens, heads * dv] of the compute dtype
+};
+
+constexpr int kStepThreads = 256;
+constexpr int kStepWarps = kStepThreads / 32;
+constexpr int kMaxRank = 512;
+
+// A block per (head, sequence): warp w holds rows w, w + 8, ... of the state, lane l columns 4 l .. 4 l + 3 (dv <= 128, a
+// multiple of four; d <= 128).
+template <typename TI>
+__global__ void __launch_bounds__(kStepThreads)
+delta_step_kernel(const StepParams q) {
+  ilb::pdl_launch_dependents();
+  ilb::pdl_wait();
+  constexpr bool FAST = sizeof(TI) == 2;
+  constexpr int kRows = 128 / kStepWarps;
+  const DeltaParams& p = q.a;
+  __shared__ float low[kMaxRank];
+  __shared__ float Us[128], Ws[128], Gs[128], Ks[128], Rs[128];
+  __shared__ float4 red[kStepWarps][32];
+  __shared__ float scratch[33];
+  const int h = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int t = p.cu_q[seq];
+  if (p.cu_q[seq + 1] - t != 1) return;                  // single tokens only
+  const int slot = p.slots[seq];
+  float* own = slot >= 0 ? p.state + ((size_t)slot * p.heads + h) * p.d * p.dv : nullptr;
+  const bool cols = 4 * lane < p.dv;
+  float4 S[kRows];
+#pragma unroll
+  for (int i = 0; i < kRows; ++i) {                      // the whole state's loads go out first
+    const int n = warp + kStepWarps * i;
+    S[i] = (own != nullptr && cols && n < p.d) ? *reinterpret_cast<const float4*>(own + (size_t)n * p.dv + 4 * lane) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  const TI* row = reinterpret_cast<const TI*>(p.proj) + (size_t)t * p.ld;
+  for (int i = tid; i < q.rank; i += kStepThreads) low[i] = tanhf(to_float(row[q.col_low + i]));
+  float kk = 0.f;
+  if (tid < 128) {
+    kk = tid < p.d ? to_float(row[p.col_k + h * p.d + tid]) : 0.f;
+    Ks[tid] = kk;
+    Rs[tid] = tid < p.d ? to_float(row[p.col_r + h * p.d + tid]) : 0.f;
+  }
+  const float inv = 1.0f / sqrtf(block_sum(kk * kk, scratch) + p.unit_eps);      // (its barriers also publish low, Ks, Rs)
+  {   // two threads a channel: the map's row, then decay and removal rate
+    const int n = tid >> 1, half = tid & 1;
+    const int ch = h * p.d + (n < p.d ? n : 0);
+    const TI* w2 = reinterpret_cast<const TI*>(q.w2) + (size_t)ch * q.ld_w2;
+    float s = 0.f;
+    if constexpr (FAST) {                                // (rows are padded to multiples of eight and start on 16-byte boundaries)
+      for (int i = half * 8; i < q.rank; i += 16) {
+        const uint4 v = *reinterpret_cast<const uint4*>(w2 + i);
+        const uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+          if (i + 2 * j < q.rank) s = fmaf(__uint_as_float(w[j] << 16), low[i + 2 * j], s);
+          if (i + 2 * j + 1 < q.rank) s = fmaf(__uint_as_float(w[j] & 0xFFFF0000u), low[i + 2 * j + 1], s);
+        }
+      }
+    } else {
+      for (int i = half; i < q.rank; i += 2) s = fmaf(to_float(w2[i]), low[i], s);
+    }
+    s += __shfl_xor_sync(0xffffffffu, s, 1);
+    if (half == 0) {
+      const bool on = n < p.d;
+      const float u = Ks[n] * inv;
+      Us[n] = u;
+      Ws[n] = on ? exp_t<FAST>(-p.log_decay * sigmoid_t<FAST>(s + p.w0[ch])) : 0.f;
+      Gs[n] = on ? -sigmoid_t<FAST>(to_float(row[p.col_a + ch]) + p.ab[ch]) * u : 0.f;
+    }
+  }
+  const float4 v = [&]() {
+    float e[4];
+#pragma unroll
+    for (int c = 0; c < 4; ++c) e[c] = cols ? to_float(row[p.col_v + h * p.dv + 4 * lane + c]) : 0.f;
+    return make_float4(e[0], e[1], e[2], e[3]);
+  }();
+  __syncthreads();
+  auto total = [&](float4 part) {                        // sum over the warps, the same in every warp
+    red[warp][lane] = part;
+    __syncthreads();
+    float4 s = red[0][lane];
+#pragma unroll
+    for (int w = 1; w < kStepWarps; ++w) { const float4 a = red[w][lane]; s.x += a.x; s.y += a.y; s.z += a.z; s.w += a.w; }
+    __syncthreads();
+    return s;
+  };
+  float4 part = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int i = 0; i < kRows; ++i) {
+    const float u = Us[warp + kStepWarps * i];
+    part.x = fmaf(u, S[i].x, part.x); part.y = fmaf(u, S[i].y, part.y); part.z = fmaf(u, S[i].z, part.z); part.w = fmaf(u, S[i].w, part.w);
+  }
+  const float4 z = total(part);
+  part = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int i = 0; i < kRows; ++i) {
+    const int n = warp + kStepWarps * i;
+    const float w = Ws[n], g = Gs[n], k = Ks[n], r = Rs[n];
+    S[i].x = fmaf(w, S[i].x, fmaf(g, z.x, k * v.x)); S[i].y = fmaf(w, S[i].y, fmaf(g, z.y, k * v.y));
+    S[i].z = fmaf(w, S[i].z, fmaf(g, z.z, k * v.z)); S[i].w = fmaf(w, S[i].w, fmaf(g, z.w, k * v.w));
+    part.x = fmaf(r, S[i].x, part.x); part.y = fmaf(r, S[i].y, part.y); part.z = fmaf(r, S[i].z, part.z); part.w = fmaf(r, S[i].w, part.w);
+    if (own != nullptr && cols && n < p.d) *reinterpret_cast<float4*>(own + (size_t)n * p.dv + 4 * lane) = S[i];
+  }
+  const float4 o = total(part);
+  if (warp == 0) {
+    const float ss = warp_sum(o.x * o.x + o.y * o.y + o.z * o.z + o.w * o.w);
+    const float f = 1.0f / sqrtf(ss / (float)p.dv + q.eps);
+    if (cols) {
+      const float e[4] = {o.x, o.y, o.z, o.w};
+      TI* dst = reinterpret_cast<TI*>(q.out) + (size_t)t * q.ld_out + h * p.dv + 4 * lane;
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        const int at = h * p.dv + 4 * lane + c;
+        dst[c] = from_float<TI>(e[c] * f * q.norm_w[at] * sigmoid_t<false>(to_float(row[q.col_g + at])));
+      }
+    }
+  }
+}
+
+ILB_EXPORT int ilb_delta_step_supported(int d, int dv, int rank) { return (d <= 128 && dv <= 128 && dv % 4 == 0 && rank <= kMaxRank) ? 1 : 0; }
+
+// Single tokens from the layer's projections to what its output product reads: proj [T, ld] holds r, k, a, v, the gate and the
+// map's inner row; w2 [heads * d, ld_w2] of the same dtype; out [T, ld_out].
+ILB_EXPORT int ilb_delta_step(const void* proj, int dtype, int ld, int col_r, int col_k, int col_v, int col_a, int col_g, int col_low,
+                              int rank, const void* w2, int ld_w2, const float* w0, const float* ab, float log_decay, float unit_eps,
+                              const float* norm_w, float eps, float* state, void* out, int ld_out, const int* cu_q, const int* slots,
+                              int n_seqs, int heads, int d, int dv, cudaStream_t stream) {
+  const DeltaParams p{proj, ld, col_r, col_k, col_v, col_a, w0, w0, ab, state, state, cu_q, slots, n_seqs, heads, d, dv, log_decay, unit_eps};
+  if (int rc = check_sizes(p, dtype)) return rc;
+  ILB_REQUIRE(ilb_delta_step_supported(d, dv, rank) && rank > 0, "delta_step: states of %d x %d with a map of %d are not built", d, dv, rank);
+  ILB_REQUIRE(w2 != nullptr && norm_w != nullptr && out != nullptr && eps > 0.f && col_g >= 0 && col_low >= 0 && ld >= col_g + heads * dv &&
+              ld >= col_low + rank && ld_w2 >= (rank + 7) / 8 * 8 && ld_w2 % 8 == 0 && ((uintptr_t)w2 % 16 == 0) && ((uintptr_t)state % 16 == 0) &&
+              ld_out >= heads * dv, "delta_step: bad inputs");
+  if (n_seqs == 0) return 0;
+  const StepParams q{p, col_low, rank, ld_w2, w2, col_g, norm_w, eps, out, ld_out};
+  if (dtype == kF32) ilb::launch(delta_step_kernel<float>, dim3(heads, n_seqs), dim3(kStepThreads), 0, stream, q);
+  else ilb::launch(delta_step_kernel<__nv_bfloat16>, dim3(heads, n_seqs), dim3(kStepThreads), 0, stream, q);
+  return check_launch("delta_step");
 }
 
 ILB_DEFINE_LAST_ERROR()

@@ -483,21 +483,64 @@ def act_rows(x: torch.Tensor, activation: str, out: torch.Tensor) -> None:
 
 
 # --------------------------------------------------------------------------- generalized delta rule
+DELTA_CHUNK = 16           # tokens a chunk of a long portion's delta rule holds
+DELTA_CHUNK_FROM = 32      # portions from this many tokens on run in chunks
+
+
 def delta_scan(proj: torch.Tensor, col_r: int, col_k: int, col_v: int, col_a: int, low: torch.Tensor, w0: torch.Tensor, ab: torch.Tensor,
                log_decay: float, unit_eps: float, state: torch.Tensor, y: torch.Tensor, step, heads: int, d: int, dv: int,
-               workspace=None) -> None:
+               workspace=None, chunks: Optional[bool] = None) -> None:
     """S_t = diag(w) S_{t-1} - (g u)(u^T S_{t-1}) + k v^T, y_t = S_t^T r per head over the step's tokens, from and to state
     [slots, heads, d, dv] (see delta.cu); r, k, a at columns of `proj` (heads * d each), v (heads * dv); `low` [T, heads * d]
-    32-bit: what w0 joins under the decay's sigmoid."""
+    32-bit: what w0 joins under the decay's sigmoid.  `chunks`: whether the portions run 16 tokens at a time (None: by the
+    longest portion)."""
     _need(proj, "delta projection", contiguous=False); _need(low, "delta decay input", torch.float32); _need(state, "delta state", torch.float32)
     _need(y, "delta y", torch.float32); _need(w0, "delta w0", torch.float32); _need(ab, "delta a bias", torch.float32)
     T = proj.shape[0]
     if proj.stride(1) != 1 or tuple(low.shape) != (T, heads * d) or tuple(y.shape) != (T, heads * dv) or w0.numel() != heads * d \
             or ab.numel() != heads * d or tuple(state.shape[1:]) != (heads, d, dv):
         raise KernelError("delta_scan: shapes do not agree")
+    if chunks is None:
+        chunks = step.max_q_len >= DELTA_CHUNK_FROM and workspace is not None and log_decay * DELTA_CHUNK <= 40.0
+    if chunks:
+        n_blocks = sum(-(-n // DELTA_CHUNK) for n in step.h_q_len) + (step.n_seqs - len(step.h_q_len))
+        scratch = workspace.buffer("delta.chunks", (delta_chunk_floats(n_blocks, heads, d, dv),), torch.float32)
+        _call("delta", "ilb_delta_chunks", _ptr(proj), _i(_code(proj)), _i(proj.stride(0)), _i(col_r), _i(col_k), _i(col_v), _i(col_a), _ptr(low),
+              _ptr(w0), _ptr(ab), _f(log_decay), _f(unit_eps), _ptr(state), _ptr(y), _ptr(step.cu_q), _ptr(step.slots), _i(step.n_seqs),
+              _i(heads), _i(d), _i(dv), _ptr(scratch), ctypes.c_longlong(scratch.numel()), _i(n_blocks), _stream(y))
+        return
     _call("delta", "ilb_delta_scan", _ptr(proj), _i(_code(proj)), _i(proj.stride(0)), _i(col_r), _i(col_k), _i(col_v), _i(col_a), _ptr(low),
           _ptr(w0), _ptr(ab), _f(log_decay), _f(unit_eps), _ptr(state), _ptr(y), _ptr(step.cu_q), _ptr(step.slots), _i(step.n_seqs),
           _i(heads), _i(d), _i(dv), _stream(y))
+
+
+def delta_chunk_floats(n_blocks: int, heads: int, d: int, dv: int) -> int:
+    """32-bit elements of scratch that so many chunks of 16 tokens need (the layout is delta.cu's)."""
+    rows = 64 if d <= 64 else 128 if d <= 128 else 256
+    cols = -(-dv // 16) * 16
+    return n_blocks * heads * (4 * DELTA_CHUNK * rows + rows + 3 * DELTA_CHUNK * cols)
+
+
+def delta_step_supported(d: int, dv: int, rank: int) -> bool:
+    """Sizes of the kernel that takes single tokens from the projections to the output product's input."""
+    return d <= 128 and dv <= 128 and dv % 4 == 0 and rank <= 512
+
+
+def delta_step(proj: torch.Tensor, col_r: int, col_k: int, col_v: int, col_a: int, col_g: int, col_low: int, rank: int, w2: torch.Tensor,
+               w0: torch.Tensor, ab: torch.Tensor, log_decay: float, unit_eps: float, norm_w: torch.Tensor, eps: float, state: torch.Tensor,
+               out: torch.Tensor, step, heads: int, d: int, dv: int) -> None:
+    """A step of single tokens: the decay's low-rank map (tanh of `rank` columns of `proj` times w2), the delta rule, the RMS norm
+    of each head and the output gate, in one launch; out [T, heads * dv] in proj's dtype."""
+    _need(proj, "delta projection", contiguous=False); _need(w2, "delta w2", proj.dtype); _need(w0, "delta w0", torch.float32)
+    _need(ab, "delta a bias", torch.float32); _need(norm_w, "delta norm weight", torch.float32); _need(state, "delta state", torch.float32)
+    _need(out, "delta out", proj.dtype)
+    T = proj.shape[0]
+    if proj.stride(1) != 1 or w2.shape[0] != heads * d or w2.shape[1] < rank or tuple(out.shape) != (T, heads * dv) or w0.numel() != heads * d \
+            or ab.numel() != heads * d or norm_w.numel() != heads * dv or tuple(state.shape[1:]) != (heads, d, dv) or T != step.n_seqs:
+        raise KernelError("delta_step: shapes do not agree")
+    _call("delta", "ilb_delta_step", _ptr(proj), _i(_code(proj)), _i(proj.stride(0)), _i(col_r), _i(col_k), _i(col_v), _i(col_a), _i(col_g),
+          _i(col_low), _i(rank), _ptr(w2), _i(w2.shape[1]), _ptr(w0), _ptr(ab), _f(log_decay), _f(unit_eps), _ptr(norm_w), _f(eps), _ptr(state),
+          _ptr(out), _i(out.shape[1]), _ptr(step.cu_q), _ptr(step.slots), _i(step.n_seqs), _i(heads), _i(d), _i(dv), _stream(out))
 
 
 def head_gate(o: torch.Tensor, gate: torch.Tensor, heads: int, scale: float = 1.0, out: Optional[torch.Tensor] = None) -> None:
@@ -844,9 +887,12 @@ def pool_means(k_cache: torch.Tensor, v_cache: torch.Tensor, pooled: PooledRows,
     dv = v_cache.shape[3]
     if tuple(pooled.k.shape[1:]) != (nkv, page_size, d) or tuple(pooled.v.shape[1:]) != (nkv, page_size, dv) or pooled.table.shape != block_table.shape:
         raise KernelError("pool_means: the pooled pages do not match the cache")
+    done = sum(n // pooled.pool - (n - m) // pooled.pool for m, n in zip(step.h_q_len, step.h_kv_len))      # blocks that end in this step
+    if done == 0:
+        return
     _call("qk_norm_rope", "ilb_pool_means", _ptr(k_cache), _ptr(v_cache), _ptr(pooled.k), _ptr(pooled.v), _i(_code(k_cache)), _ptr(step.positions),
-          _ptr(step.seq_of_token), _ptr(block_table), _ptr(pooled.table), _i(block_table.shape[1]), _i(page_size), _i(num_pages),
-          _i(pooled.k.shape[0]), _i(pooled.pool), _i(step.n_tokens), _i(nkv), _i(d), _i(dv), _stream(k_cache))
+          _ptr(step.cu_q), _i(step.n_seqs), _ptr(block_table), _ptr(pooled.table), _i(block_table.shape[1]), _i(page_size), _i(num_pages),
+          _i(pooled.k.shape[0]), _i(pooled.pool), _i(done), _i(nkv), _i(d), _i(dv), _stream(k_cache))
 
 
 def turn_back(o: torch.Tensor, table: torch.Tensor, heads: int) -> None:

@@ -592,58 +592,89 @@ ILB_EXPORT int ilb_rows_norm_rope_cache(
 
 // ---------------------------------------------------------------- means of blocks of cached rows
 // The token at position p completes block b = p / pool if (p + 1) % pool == 0: row b of the second set of pages becomes the
-// mean (32-bit sum) of the block's `pool` keys and of its values as the cache holds them.  One block of threads a token.
-template <typename T>
-__global__ void __launch_bounds__(256)
+// mean (32-bit sum) of the block's `pool` keys and of its values as the cache holds them.  One block of threads per block of
+// positions that the step completes (and slice of the channels); eight groups of threads share a block's rows.
+constexpr int kMeanRows = 8, kMeanCols = 32;
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(kMeanRows * kMeanCols)
 pool_means_kernel(const T* __restrict__ k_cache, const T* __restrict__ v_cache, T* __restrict__ pk_cache, T* __restrict__ pv_cache,
-                  const int* __restrict__ positions, const int* __restrict__ seq_of_token, const int* __restrict__ block_table,
+                  const int* __restrict__ positions, const int* __restrict__ cu_q, int n_seqs, const int* __restrict__ block_table,
                   const int* __restrict__ p_table, int max_blocks, int page_size, int num_pages, int p_num_pages, int pool, int nkv,
                   int d, int dv) {
   ilb::pdl_launch_dependents();
   ilb::pdl_wait();
-  const int t = blockIdx.x, pos = positions[t];
-  if ((pos + 1) % pool != 0) return;
-  const int seq = seq_of_token[t], b = pos / pool;
-  if (b / page_size >= max_blocks) return;
+  __shared__ float part[kMeanRows][kMeanCols * VEC];
+  int seq = 0, left = blockIdx.x, b = -1;
+  for (; seq < n_seqs; ++seq) {
+    const int n = cu_q[seq + 1] - cu_q[seq];
+    if (n <= 0) continue;
+    const int p0 = positions[cu_q[seq]], done = (p0 + n) / pool - p0 / pool;      // blocks whose last position lies in this step
+    if (left < done) { b = p0 / pool + left; break; }
+    left -= done;
+  }
+  if (b < 0 || b / page_size >= max_blocks) return;
   const int* table = block_table + (size_t)seq * max_blocks;
   const int p_page = p_table[(size_t)seq * max_blocks + b / page_size];
   if (p_page < 0 || p_page >= p_num_pages) return;          // never write outside the pool
-  const int e = blockIdx.y * 256 + threadIdx.x;
-  if (e >= nkv * (d + dv)) return;
-  const bool is_k = e < nkv * d;
+  const int col = threadIdx.x % kMeanCols, grp = threadIdx.x / kMeanCols;
+  const int e = (blockIdx.y * kMeanCols + col) * VEC;
+  const bool live = e < nkv * (d + dv), is_k = e < nkv * d;
   const int width = is_k ? d : dv, h = (is_k ? e : e - nkv * d) / width, c = (is_k ? e : e - nkv * d) % width;
   const T* src = is_k ? k_cache : v_cache;
-  float sum = 0.f;
-  const int first = b * pool;
-  for (int j0 = 0; j0 < pool; j0 += 8) {                    // eight loads in flight
-    float x[8];
+  float sum[VEC];
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      const int pj = first + j0 + i;
-      x[i] = 0.f;
-      if (j0 + i < pool) {
-        const int page = table[pj / page_size];
-        if (page >= 0 && page < num_pages) x[i] = to_float(src[(((size_t)page * nkv + h) * page_size + pj % page_size) * width + c]);
+  for (int i = 0; i < VEC; ++i) sum[i] = 0.f;
+  if (live) {
+    for (int j0 = grp; j0 < pool; j0 += 4 * kMeanRows) {    // four rows in flight
+      float x[4][VEC];
+#pragma unroll
+      for (int f = 0; f < 4; ++f) {
+        const int j = j0 + f * kMeanRows, pj = b * pool + j;
+        const int page = j < pool ? table[pj / page_size] : -1;
+        if (page >= 0 && page < num_pages) RowUnit<T, VEC>::load(src + (((size_t)page * nkv + h) * page_size + pj % page_size) * width + c, x[f]);
+        else {
+#pragma unroll
+          for (int i = 0; i < VEC; ++i) x[f][i] = 0.f;
+        }
       }
-    }
 #pragma unroll
-    for (int i = 0; i < 8; ++i) sum += x[i];
+      for (int f = 0; f < 4; ++f)
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) sum[i] += x[f][i];
+    }
   }
-  (is_k ? pk_cache : pv_cache)[(((size_t)p_page * nkv + h) * page_size + b % page_size) * width + c] = from_float<T>(sum / (float)pool);
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) part[grp][col * VEC + i] = sum[i];
+  __syncthreads();
+  if (grp != 0 || !live) return;
+#pragma unroll
+  for (int i = 0; i < VEC; ++i) {
+    float s = 0.f;
+#pragma unroll
+    for (int g = 0; g < kMeanRows; ++g) s += part[g][col * VEC + i];
+    sum[i] = s / (float)pool;
+  }
+  RowUnit<T, VEC>::store((is_k ? pk_cache : pv_cache) + (((size_t)p_page * nkv + h) * page_size + b % page_size) * width + c, sum);
 }
 
+// n_done: blocks of positions that the step's tokens complete, over all sequences.
 ILB_EXPORT int ilb_pool_means(const void* k_cache, const void* v_cache, void* pk_cache, void* pv_cache, int dtype, const int* positions,
-                              const int* seq_of_token, const int* block_table, const int* p_table, int max_blocks, int page_size,
-                              int num_pages, int p_num_pages, int pool, int n_tokens, int nkv, int d, int dv, cudaStream_t stream) {
-  ILB_REQUIRE(n_tokens >= 0 && nkv > 0 && d > 0 && dv > 0 && pool > 0, "pool_means: bad sizes");
+                              const int* cu_q, int n_seqs, const int* block_table, const int* p_table, int max_blocks, int page_size,
+                              int num_pages, int p_num_pages, int pool, int n_done, int nkv, int d, int dv, cudaStream_t stream) {
+  ILB_REQUIRE(n_done >= 0 && n_seqs > 0 && nkv > 0 && d > 0 && dv > 0 && pool > 0, "pool_means: bad sizes");
   ILB_REQUIRE(page_size > 0 && max_blocks > 0 && num_pages > 0 && p_num_pages > 0, "pool_means: bad cache geometry");
   ILB_REQUIRE(k_cache != nullptr && v_cache != nullptr && pk_cache != nullptr && pv_cache != nullptr, "pool_means: a cache is missing");
-  if (n_tokens == 0) return 0;
-  const dim3 grid(n_tokens, (nkv * (d + dv) + 255) / 256);
-#define ILB_PM(T) ilb::launch(pool_means_kernel<T>, grid, dim3(256), 0, stream, (const T*)k_cache, (const T*)v_cache, (T*)pk_cache, (T*)pv_cache, \
-                              positions, seq_of_token, block_table, p_table, max_blocks, page_size, num_pages, p_num_pages, pool, nkv, d, dv)
-  if (dtype == kF32) ILB_PM(float);
-  else if (dtype == kBF16) ILB_PM(__nv_bfloat16);
+  if (n_done == 0) return 0;
+  auto a16 = [](const void* x) { return (uintptr_t)x % 16 == 0; };
+  const bool vec = dtype == kBF16 && d % 8 == 0 && dv % 8 == 0 && a16(k_cache) && a16(v_cache) && a16(pk_cache) && a16(pv_cache);
+  const int per = kMeanCols * (vec ? 8 : 1);
+  const dim3 grid(n_done, (nkv * (d + dv) + per - 1) / per);
+#define ILB_PM(T, V) ilb::launch(pool_means_kernel<T, V>, grid, dim3(kMeanRows * kMeanCols), 0, stream, (const T*)k_cache, (const T*)v_cache, \
+                                 (T*)pk_cache, (T*)pv_cache, positions, cu_q, n_seqs, block_table, p_table, max_blocks, page_size, num_pages, \
+                                 p_num_pages, pool, nkv, d, dv)
+  if (dtype == kF32) ILB_PM(float, 1);
+  else if (dtype == kBF16) { if (vec) ILB_PM(__nv_bfloat16, 8); else ILB_PM(__nv_bfloat16, 1); }
   else return fail("pool_means: unknown dtype %d", dtype);
 #undef ILB_PM
   return check_launch("pool_means");

@@ -336,6 +336,50 @@ rms_gate_vec_kernel(const float* __restrict__ y, const __nv_bfloat16* __restrict
   for (int i = threadIdx.x + kGateKeep * blockDim.x; i < n4; i += blockDim.x) write(i, yr[i]);
 }
 
+// Narrow parts (up to 1,024 elements): a warp a part, several parts a block; a lane keeps up to eight vectors between the
+// sum and the write.
+constexpr int kPartWarps = 8, kPartKeep = 8;
+
+__global__ void __launch_bounds__(kPartWarps * 32)
+rms_gate_parts_kernel(const float* __restrict__ y, const __nv_bfloat16* __restrict__ gate, int ld_gate, const float* __restrict__ w,
+                      __nv_bfloat16* __restrict__ out, int ld_out, int rows, int groups, int part_width, float eps, float scale) {
+  ilb::pdl_launch_dependents();
+  ilb::pdl_wait();
+  const long long id = (long long)blockIdx.x * kPartWarps + (threadIdx.x >> 5);
+  if (id >= (long long)rows * groups) return;
+  const int lane = threadIdx.x & 31, part = (int)(id % groups), n4 = part_width / 4;
+  const size_t t = id / groups;
+  const float4* yr = reinterpret_cast<const float4*>(y + (t * groups + part) * part_width);
+  const uint2* gr = reinterpret_cast<const uint2*>(gate + t * ld_gate + (size_t)part * part_width);
+  const float4* wr = reinterpret_cast<const float4*>(w + (size_t)part * part_width);
+  uint2* o = reinterpret_cast<uint2*>(out + t * ld_out + (size_t)part * part_width);
+  float4 keep[kPartKeep];
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < kPartKeep; ++j) {
+    const int i = lane + 32 * j;
+    if (i < n4) {
+      keep[j] = yr[i];
+      ss = fmaf(keep[j].x, keep[j].x, ss); ss = fmaf(keep[j].y, keep[j].y, ss);
+      ss = fmaf(keep[j].z, keep[j].z, ss); ss = fmaf(keep[j].w, keep[j].w, ss);
+    }
+  }
+  const float inv = scale / sqrtf(warp_sum(ss) / (float)part_width + eps);
+#pragma unroll
+  for (int j = 0; j < kPartKeep; ++j) {
+    const int i = lane + 32 * j;
+    if (i < n4) {
+      const uint2 g = gr[i];
+      const float4 wv = wr[i], v = keep[j];
+      const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x * inv * wv.x * sigmoid_f(__uint_as_float(g.x << 16)),
+                                                      v.y * inv * wv.y * sigmoid_f(__uint_as_float(g.x & 0xFFFF0000u)));
+      const __nv_bfloat162 hi = __floats2bfloat162_rn(v.z * inv * wv.z * sigmoid_f(__uint_as_float(g.y << 16)),
+                                                      v.w * inv * wv.w * sigmoid_f(__uint_as_float(g.y & 0xFFFF0000u)));
+      o[i] = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+    }
+  }
+}
+
 // y: [rows, width] 32-bit; gate: [rows, ld_gate] of `dtype` (its first `width` columns from the pointer given);
 // out: [rows, ld_out] of `dtype` (its first `width` columns).
 ILB_EXPORT int ilb_rms_gate(const float* y, const void* gate, int dtype, int ld_gate, const float* w, void* out, int ld_out, int rows,
@@ -346,6 +390,12 @@ ILB_EXPORT int ilb_rms_gate(const float* y, const void* gate, int dtype, int ld_
   const int part = width / groups;
   if (dtype == kBF16 && part % 4 == 0 && ld_gate % 4 == 0 && ld_out % 4 == 0 && ((uintptr_t)y % 16 == 0) && ((uintptr_t)w % 16 == 0) &&
       ((uintptr_t)gate % 8 == 0) && ((uintptr_t)out % 8 == 0)) {
+    if (groups > 1 && part <= 4 * 32 * kPartKeep) {
+      const long long blocks = ((long long)rows * groups + kPartWarps - 1) / kPartWarps;
+      ilb::launch(rms_gate_parts_kernel, dim3((unsigned)blocks), dim3(kPartWarps * 32), 0, stream, y, (const __nv_bfloat16*)gate, ld_gate, w,
+                  (__nv_bfloat16*)out, ld_out, rows, groups, part, eps, scale);
+      return check_launch("rms_gate");
+    }
     const int per = part / 4, vthreads = per >= 1024 ? 256 : (per >= 256 ? 128 : (per > 32 ? 64 : 32));
     ilb::launch(rms_gate_vec_kernel, dim3(rows, groups), dim3(vthreads), 0, stream, y, (const __nv_bfloat16*)gate, ld_gate, w, (__nv_bfloat16*)out, ld_out,
                 part, eps, scale);

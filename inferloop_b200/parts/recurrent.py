@@ -263,13 +263,22 @@ class GeneralDelta(Mixer):
     def scratch_bytes(self, tokens: int) -> int:
         size = torch.empty((), dtype=self.ctx.dtype).element_size()
         wide = -(-self.rank // 8) * 8
-        return tokens * ((self.col_low + 2 * wide + self.inner_v) * size + (self.inner_k + self.inner_v) * 4)
+        chunks = ops.delta_chunk_floats(-(-tokens // ops.DELTA_CHUNK) + 1, self.heads, self.d, self.dv) * 4
+        return tokens * ((self.col_low + 2 * wide + self.inner_v) * size + (self.inner_k + self.inner_v) * 4) + chunks
 
     def forward(self, x: torch.Tensor, residual: torch.Tensor, step, cache) -> None:
         T, ws, dt = x.shape[0], self.ctx.workspace, self.ctx.dtype
         proj = ws.buffer("delta.proj", (T, self.w_in.shape[0]), dt)
         ops.scope("delta.in_projection")
         linear(x, self.w_in, proj)
+        gated = ws.buffer("delta.gated", (T, self.inner_v), dt)
+        if step.decode_only and ops.delta_step_supported(self.d, self.dv, self.rank):
+            ops.scope("delta.step (decay map, recurrence, norm and gate inside)")
+            ops.delta_step(proj, 0, self.col_k, self.col_v, self.col_a, self.col_g, self.col_low, self.rank, self.w2, self.w0, self.ab,
+                           self.log_decay, self.unit_eps, self.norm_w, self.eps, cache.state["state"], gated, step, self.heads, self.d, self.dv)
+            ops.scope("delta.out_projection")
+            linear(gated, self.w_o, residual, accumulate=True)
+            return
         ops.scope("delta.decay_map")
         low = ws.buffer("delta.low", (T, self.w2.shape[1]), dt)
         ops.act_rows(proj[:, self.col_low:], "tanh", low)
@@ -278,9 +287,8 @@ class GeneralDelta(Mixer):
         ops.scope("delta.scan")
         y = ws.buffer("delta.y", (T, self.inner_v), torch.float32)
         ops.delta_scan(proj, 0, self.col_k, self.col_v, self.col_a, decay, self.w0, self.ab, self.log_decay, self.unit_eps,
-                       cache.state["state"], y, step, self.heads, self.d, self.dv)
+                       cache.state["state"], y, step, self.heads, self.d, self.dv, workspace=ws)
         ops.scope("delta.norm_gate")
-        gated = ws.buffer("delta.gated", (T, self.inner_v), dt)
         ops.rms_gate(y, proj[:, self.col_g:], self.norm_w, self.eps, gated, groups=self.heads)
         ops.scope("delta.out_projection")
         linear(gated, self.w_o, residual, accumulate=True)

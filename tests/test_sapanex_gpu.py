@@ -117,7 +117,7 @@ def test_mixed_batches_with_pages_and_slots_used_again(root, name, dtype):
     pool that cannot hold all of them: what ends gives its pages (of both kinds) and its slot to the next.  Every row
     equals the request alone."""
     lens = {"a": 97, "b": 5, "c": 124, "d": 21, "e": 110, "f": 2, "g": 83}
-    toks = {k: tokens_for(name, n, 10 + i) for i, (k, n) in enumerate(lens.items())}
+    toks = {k: tokens_for(name, n, 50 + i) for i, (k, n) in enumerate(lens.items())}
     ref = {k: reference(root, name, dtype, v) for k, v in toks.items()}
     page = cases.CASES[name][2]
     pages = sum(-(-n // page) for n in (97, 124, 110, 21)) + 1
@@ -694,3 +694,44 @@ def test_the_delta_rule_whole_and_in_portions(heads, d, dv, dtype):
     ops.delta_scan(proj[1][:1].to(DEV), 0, wk, 3 * wk, 2 * wk, f32(low[1][:1]), f32(w0), f32(ab), log_decay, unit_eps, state, y, step, heads, d, dv, workspace=ws)
     assert torch.equal(state, before)
     assert (y.double().cpu() - ref[1][0][:1]).abs().max() <= 2e-5 * ref[1][0].abs().max()
+
+
+@pytest.mark.parametrize("heads,d,dv,rank", [(2, 64, 64, 24), (3, 128, 128, 5), (1, 128, 64, 200), (4, 10, 12, 1), (2, 48, 48, 16), (5, 100, 4, 33)])
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_single_tokens_of_the_delta_rule_in_one_launch(heads, d, dv, rank, dtype):
+    """The low-rank map, decay, recurrence, norm of each head and gate of several sequences' single tokens, step after step, from
+    states that are not zero; a dummy row beside them; slots of others are left alone."""
+    from inferloop_b200.csrc import ops
+    g = torch.Generator().manual_seed(heads * d + rank)
+    wk, wv = heads * d, heads * dv
+    pad = -rank % 8
+    log_decay, unit_eps, eps = 0.6, 1e-6, 1e-5
+    w2 = torch.zeros(wk, rank + pad)
+    w2[:, :rank] = torch.randn(wk, rank, generator=g) / math.sqrt(rank)
+    w2 = w2.to(dtype)
+    w0, ab, norm = torch.linspace(-9.0, 2.0, wk), torch.linspace(-3.0, 3.0, wk).flip(0), 1 + 0.2 * torch.randn(wv, generator=g)
+    state = torch.randn(6, heads, d, dv, generator=g)
+    ref_state = {0: state[4].double(), 1: state[1].double(), 3: state[5].double()}
+    dev = f32(state)
+    slots = [4, 1, -1, 5]
+    n = len(slots)
+    for _ in range(5):
+        proj = torch.randn(n, 3 * wk + 2 * wv + rank + pad, generator=g).to(dtype)
+        out = torch.full((n, wv), 9.0, dtype=dtype, device=DEV)
+        step = FakeStep([1] * n, [3, 7, 0, 9], slots)
+        ops.delta_step(proj.to(DEV), 0, wk, 3 * wk, 2 * wk, 3 * wk + wv, 3 * wk + 2 * wv, rank, w2.to(DEV), f32(w0), f32(ab), log_decay, unit_eps, f32(norm),
+                       eps, dev, out, step, heads, d, dv)
+        x = proj.double()
+        decay = torch.exp(-log_decay * torch.sigmoid(torch.tanh(x[:, 3 * wk + 2 * wv:3 * wk + 2 * wv + rank]) @ w2.double()[:, :rank].T + w0.double()))
+        removal = torch.sigmoid(x[:, 2 * wk:3 * wk] + ab.double())
+        for i in range(n):
+            one = lambda t, s: t[i].reshape(1, heads, s)
+            o, S = plain.delta_rule(one(decay, d), one(removal, d), one(x[:, wk:2 * wk], d), one(x[:, 3 * wk:3 * wk + wv], dv), one(x[:, :wk], d), ref_state.get(i))
+            want = plain.rms(o, eps).reshape(wv) * norm.double() * torch.sigmoid(x[i, 3 * wk + wv:3 * wk + 2 * wv])
+            assert (out[i].double().cpu() - want).abs().max() <= (2e-5 if dtype == torch.float32 else 2.0 ** -7) * want.abs().max()
+            if i in ref_state:
+                ref_state[i] = S
+    for i, s in ((0, 4), (1, 1), (3, 5)):
+        assert (dev[s].double().cpu() - ref_state[i]).abs().max() <= 2e-5 * ref_state[i].abs().max()
+    for s in (0, 2, 3):
+        assert torch.equal(dev[s].cpu(), state[s])
