@@ -217,10 +217,33 @@ ILB_EXPORT int ilb_delta_scan(const void* proj, int dtype, int ld, int col_r, in
 // ---------------------------------------------------------------- chunks
 constexpr int kChunk = 16;
 
-// Floats of one (chunk, head) in scratch: W, X, D q, D m [16][KP], D [KP], then U, Y, V [16][DP]; KP rows, DP columns, padded.
+// Two 32-bit numbers side by side and the arithmetic on both at once (IEEE, as the scalar instructions).
+__device__ __forceinline__ uint64_t pack2(float lo, float hi) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+  return r;
+}
+__device__ __forceinline__ void unpack2(uint64_t v, float& lo, float& hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v)); }
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ float sum2(uint64_t v) {
+  float lo, hi;
+  unpack2(v, lo, hi);
+  return lo + hi;
+}
+
+// Floats of one (chunk, head) in scratch: W, X, - D q, D m [16][KP], D [KP], then U, Y, V [16][DP]; KP rows, DP columns, padded.
 __host__ __device__ __forceinline__ long long chunk_floats(int KP, int DP) { return (long long)4 * kChunk * KP + KP + (long long)3 * kChunk * DP; }
 __host__ __device__ __forceinline__ int padded_cols(int dv) { return (dv + kCols - 1) / kCols * kCols; }
-static inline int rows_per_thread(int d) { return d <= 64 ? 2 : (d <= 128 ? 4 : 8); }
+static inline int padded_rows(int d) { return d <= 64 ? 64 : (d <= 128 ? 128 : 256); }
 
 // which sequence, and which of its chunks, block `b` works on; false: none
 __device__ __forceinline__ bool find_chunk(const int* __restrict__ cu_q, int n_seqs, int b, int& seq, int& index) {
@@ -239,7 +262,6 @@ static inline size_t prep_smem_floats(int KP, int DP) { return (size_t)4 * kChun
 template <typename TI>
 __global__ void __launch_bounds__(kPrepThreads, 4)
 delta_prep_kernel(const DeltaParams p, float* __restrict__ scratch, int KP) {
-  ilb::pdl_launch_dependents();
   ilb::pdl_wait();
   constexpr bool FAST = sizeof(TI) == 2;
   extern __shared__ __align__(16) float sm[];
@@ -249,10 +271,8 @@ delta_prep_kernel(const DeltaParams p, float* __restrict__ scratch, int KP) {
   float* Qv = R + kChunk * ld;
   float* M = Qv + kChunk * ld;
   float* V = M + kChunk * ld;                            // [16][DP]
-  float* A = V + kChunk * DP;                            // [16][16] each: p.q, p.m (j < t), s.q, s.m (j <= t); zero elsewhere
-  float* B = A + kChunk * kChunk;
-  float* C = B + kChunk * kChunk;
-  float* E = C + kChunk * kChunk;
+  float* AC = V + kChunk * DP;                           // [16][16][2]: - p.q (j < t), - s.q (j <= t); zero elsewhere
+  float* BE = AC + 2 * kChunk * kChunk;                  //              p.m (j < t), s.m (j <= t)
   __shared__ float inv_norm[kChunk];
   int seq, ci;
   if (!find_chunk(p.cu_q, p.n_seqs, blockIdx.x, seq, ci)) return;
@@ -307,7 +327,7 @@ delta_prep_kernel(const DeltaParams p, float* __restrict__ scratch, int KP) {
       const float g = on ? sigmoid_t<FAST>(a[t] + ab) : 0.f;
       P[t * ld + n] = D * u;
       D *= w;
-      const float inv = 1.0f / D;
+      const float inv = FAST ? __fdividef(1.0f, D) : 1.0f / D;
       Qv[t * ld + n] = g * u * inv;
       M[t * ld + n] = k * inv;
       R[t * ld + n] = D * r[t];
@@ -315,7 +335,7 @@ delta_prep_kernel(const DeltaParams p, float* __restrict__ scratch, int KP) {
     outD[n] = D;
 #pragma unroll
     for (int t = 0; t < kChunk; ++t) {
-      outQ[t * KP + n] = Qv[t * ld + n] * D;
+      outQ[t * KP + n] = -Qv[t * ld + n] * D;
       outM[t * KP + n] = M[t * ld + n] * D;
     }
   }
@@ -323,34 +343,37 @@ delta_prep_kernel(const DeltaParams p, float* __restrict__ scratch, int KP) {
   {   // rows of P and R against rows of Q and M: a thread takes four rows and one column of both
     const int j = tid & 15, rg = tid >> 4;               // rows 4 (rg & 3) .. + 3 of P (rg < 4) or of R
     const float* rows = (rg < 4 ? P : R) + (size_t)(rg & 3) * 4 * ld;
-    float x[4] = {0.f, 0.f, 0.f, 0.f}, y[4] = {0.f, 0.f, 0.f, 0.f};
+    uint64_t x2[4], y2[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) { x2[i] = 0; y2[i] = 0; }
+#pragma unroll 4
     for (int n = 0; n < KP; n += 4) {
-      const float4 q = *reinterpret_cast<const float4*>(Qv + j * ld + n), m = *reinterpret_cast<const float4*>(M + j * ld + n);
+      const ulonglong2 q = *reinterpret_cast<const ulonglong2*>(Qv + j * ld + n), m = *reinterpret_cast<const ulonglong2*>(M + j * ld + n);
 #pragma unroll
       for (int i = 0; i < 4; ++i) {
-        const float4 v = *reinterpret_cast<const float4*>(rows + i * ld + n);
-        x[i] = fmaf(v.x, q.x, x[i]); x[i] = fmaf(v.y, q.y, x[i]); x[i] = fmaf(v.z, q.z, x[i]); x[i] = fmaf(v.w, q.w, x[i]);
-        y[i] = fmaf(v.x, m.x, y[i]); y[i] = fmaf(v.y, m.y, y[i]); y[i] = fmaf(v.z, m.z, y[i]); y[i] = fmaf(v.w, m.w, y[i]);
+        const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(rows + i * ld + n);
+        x2[i] = fma2(v.y, q.y, fma2(v.x, q.x, x2[i]));
+        y2[i] = fma2(v.y, m.y, fma2(v.x, m.x, y2[i]));
       }
     }
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int t = 4 * (rg & 3) + i;
       const bool keep = rg < 4 ? j < t : j <= t;
-      (rg < 4 ? A : C)[t * kChunk + j] = keep ? x[i] : 0.f;
-      (rg < 4 ? B : E)[t * kChunk + j] = keep ? y[i] : 0.f;
+      AC[(t * kChunk + j) * 2 + (rg < 4 ? 0 : 1)] = keep ? -sum2(x2[i]) : 0.f;
+      BE[(t * kChunk + j) * 2 + (rg < 4 ? 0 : 1)] = keep ? sum2(y2[i]) : 0.f;
     }
   }
   __syncthreads();
-  // Row t of a 16 x 16 matrix from shared memory, its first `n` elements.  (The fence keeps the compiler from holding whole
-  // matrices in registers across the columns' loop.)
-  auto row16 = [&](const float* m, int t, int n, float (&r)[kChunk]) {
+  // The pairs of row t, columns 0 .. t, from shared memory.  (The fence keeps the compiler from holding whole matrices in
+  // registers across the columns' loop.)
+  auto pairs = [&](const float* m, int t, uint64_t (&r)[kChunk]) {
     asm volatile("" ::: "memory");
 #pragma unroll
-    for (int j = 0; j < kChunk / 4; ++j) {
-      if (4 * j < n) {
-        const float4 v = *reinterpret_cast<const float4*>(m + t * kChunk + 4 * j);
-        r[4 * j] = v.x; r[4 * j + 1] = v.y; r[4 * j + 2] = v.z; r[4 * j + 3] = v.w;
+    for (int j = 0; j < kChunk; j += 2) {
+      if (j <= t) {
+        const ulonglong2 v = *reinterpret_cast<const ulonglong2*>(m + (t * kChunk + j) * 2);
+        r[j] = v.x; r[j + 1] = v.y;
       }
     }
   };
@@ -358,14 +381,15 @@ delta_prep_kernel(const DeltaParams p, float* __restrict__ scratch, int KP) {
     float w[kChunk];
 #pragma unroll
     for (int t = 0; t < kChunk; ++t) {
-      float v = P[t * ld + n], x = R[t * ld + n], a[kChunk], c[kChunk];
-      row16(A, t, t, a);
-      row16(C, t, t + 1, c);
+      uint64_t ac[kChunk], vx = pack2(P[t * ld + n], R[t * ld + n]);
+      pairs(AC, t, ac);
 #pragma unroll
-      for (int j = 0; j < t; ++j) { v = fmaf(-a[j], w[j], v); x = fmaf(-c[j], w[j], x); }
-      w[t] = v;
-      outW[t * KP + n] = v;
-      outX[t * KP + n] = fmaf(-c[t], v, x);
+      for (int j = 0; j < t; ++j) vx = fma2(ac[j], pack2(w[j], w[j]), vx);
+      float c, zero, x;
+      unpack2(ac[t], zero, c);
+      unpack2(vx, w[t], x);
+      outW[t * KP + n] = w[t];
+      outX[t * KP + n] = fmaf(c, w[t], x);
     }
   }
   for (int c0 = tid; c0 < DP; c0 += kPrepThreads) {      // U = (I + A)^-1 B V,  Y = E V - C U
@@ -374,83 +398,80 @@ delta_prep_kernel(const DeltaParams p, float* __restrict__ scratch, int KP) {
     for (int t = 0; t < kChunk; ++t) v[t] = V[t * DP + c0];
 #pragma unroll
     for (int t = 0; t < kChunk; ++t) {
-      float s = 0.f, y = 0.f, a[kChunk], b[kChunk];
-      row16(A, t, t, a);
-      row16(B, t, t, b);
+      uint64_t ac[kChunk], be[kChunk], sy = 0;
+      pairs(AC, t, ac);
+      pairs(BE, t, be);
 #pragma unroll
-      for (int j = 0; j < t; ++j) { s = fmaf(b[j], v[j], s); s = fmaf(-a[j], u[j], s); }
-      u[t] = s;
-      outU[t * DP + c0] = s;
-      row16(E, t, t + 1, a);
-      row16(C, t, t + 1, b);
-#pragma unroll
-      for (int j = 0; j <= t; ++j) { y = fmaf(a[j], v[j], y); y = fmaf(-b[j], u[j], y); }
-      outY[t * DP + c0] = y;
+      for (int j = 0; j < t; ++j) sy = fma2(ac[j], pack2(u[j], u[j]), fma2(be[j], pack2(v[j], v[j]), sy));
+      float c, e, zero, y;
+      unpack2(ac[t], zero, c);
+      unpack2(be[t], zero, e);
+      unpack2(sy, u[t], y);
+      outU[t * DP + c0] = u[t];
+      outY[t * DP + c0] = fmaf(c, u[t], fmaf(e, v[t], y));
     }
   }
+  ilb::pdl_launch_dependents();                          // (the blocks of delta_chunks are few and large: they start when these are done)
 }
 
 __device__ __forceinline__ void delta_cp_async_16(float* dst, const float* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
 
+constexpr int kChunkThreads = 256;
+constexpr int kChunkWarps = kChunkThreads / 32;
+
 static inline size_t chunks_smem_floats(int KP) {
-  return 2 * ((size_t)4 * kChunk * KP + KP + 3 * kChunk * kCols) + (size_t)4 * 2 * kChunk * kCols + kChunk * kCols;
+  return 2 * ((size_t)4 * kChunk * KP + KP + 3 * kChunk * kCols) + (size_t)kChunkWarps * 2 * kChunk * kCols + kChunk * kCols;
 }
 
-// RQ: rows of the state a thread holds (of 32 RQ), times four columns.  Thread (warp, lane): rows (8 warp + lane / 4) RQ ..,
-// columns 4 (lane % 4) .. of the block's 16.
-template <int RQ>
-__global__ void __launch_bounds__(kScanThreads)
+// RH: rows of the state a thread holds (of 16 RH), in pairs, for one column.  Thread (warp, lane): rows (2 warp + lane / 16) RH
+// .., column lane % 16 of the block's 16.
+template <int RH>
+__global__ void __launch_bounds__(kChunkThreads)
 delta_chunks_kernel(const DeltaParams p, const float* __restrict__ scratch) {
   ilb::pdl_launch_dependents();
   ilb::pdl_wait();
-  constexpr int KP = 32 * RQ;
+  constexpr int KP = 16 * RH, PH = RH / 2;
   constexpr int kVecs = 4 * kChunk * KP, kBuf = kVecs + KP + 3 * kChunk * kCols;      // floats of one buffer
   extern __shared__ __align__(16) float sm[];
-  float* red = sm + 2 * kBuf;                            // [4 warps][32][kCols]: sums over a warp's rows, of W S then X S
-  float* zs = red + 4 * 2 * kChunk * kCols;              // [16][kCols]
-  const int h = blockIdx.x, cb = blockIdx.y, c0 = cb * kCols, seq = blockIdx.z;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, cg = lane & 3, rl = lane >> 2, rg = warp * 8 + rl;
+  float* red = sm + 2 * kBuf;                            // [warps][32][kCols]: sums over a warp's rows, of W S then X S
+  float* zs = red + kChunkWarps * 2 * kChunk * kCols;    // [16][kCols]
+  const int h = blockIdx.x, c0 = blockIdx.y * kCols, seq = blockIdx.z;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, cl = lane & 15, r0 = (2 * warp + (lane >> 4)) * RH;
   const int DP = padded_cols(p.dv);
   const int tok0 = p.cu_q[seq], q_len = p.cu_q[seq + 1] - tok0, n_chunks = (q_len + kChunk - 1) / kChunk;
   if (n_chunks == 0) return;
   int first = 0;
-  for (int s = 0; s < seq; ++s) first += (p.cu_q[s + 1] - p.cu_q[s] + kChunk - 1) / kChunk;
+  for (int i = 0; i < seq; ++i) first += (p.cu_q[i + 1] - p.cu_q[i] + kChunk - 1) / kChunk;
   const int slot = p.slots[seq];
   float* own = slot >= 0 ? p.state + ((size_t)slot * p.heads + h) * p.d * p.dv : nullptr;
-  const int inner_v = p.heads * p.dv;
+  const int inner_v = p.heads * p.dv, col = c0 + cl;
   const long long per = chunk_floats(KP, DP);
 
   auto issue = [&](int ci) {
     const float* src = scratch + ((size_t)(first + ci) * p.heads + h) * per;
     float* dst = sm + (ci & 1) * kBuf;
-    for (int i = tid; i < (kVecs + KP) / 4; i += kScanThreads) delta_cp_async_16(dst + 4 * i, src + 4 * i);
+    for (int i = tid; i < (kVecs + KP) / 4; i += kChunkThreads) delta_cp_async_16(dst + 4 * i, src + 4 * i);
     const float* cols = src + kVecs + KP + c0;           // U, Y, V: this block's 16 columns of each
-    for (int i = tid; i < 3 * kChunk * kCols / 4; i += kScanThreads)
+    for (int i = tid; i < 3 * kChunk * kCols / 4; i += kChunkThreads)
       delta_cp_async_16(dst + kVecs + KP + 4 * i, cols + (size_t)(i / (kCols / 4)) * DP + (i % (kCols / 4)) * 4);
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   issue(0);
-  float S[RQ][4];
+  uint64_t S[PH];                                        // rows r0 + 2 i, r0 + 2 i + 1 of this thread's column
 #pragma unroll
-  for (int i = 0; i < RQ; ++i)
+  for (int i = 0; i < PH; ++i) {
+    const int n = r0 + 2 * i;
+    const bool in = own != nullptr && col < p.dv;
+    S[i] = pack2((in && n < p.d) ? own[(size_t)n * p.dv + col] : 0.f, (in && n + 1 < p.d) ? own[(size_t)(n + 1) * p.dv + col] : 0.f);
+  }
+  // this thread's rows of a vector over the state's rows
+  auto rows_at = [&](const float* vec, uint64_t (&v)[PH]) {
 #pragma unroll
-    for (int c = 0; c < 4; ++c) {
-      const int n = rg * RQ + i, col = c0 + 4 * cg + c;
-      S[i][c] = (own != nullptr && n < p.d && col < p.dv) ? own[(size_t)n * p.dv + col] : 0.f;
-    }
-  // RQ consecutive floats of row `row` at this thread's rows
-  auto rows_at = [&](const float* row, float (&v)[RQ]) {
-    if constexpr (RQ == 2) {
-      const float2 a = *reinterpret_cast<const float2*>(row + rg * RQ);
-      v[0] = a.x; v[1] = a.y;
-    } else {
-#pragma unroll
-      for (int i = 0; i < RQ / 4; ++i) {
-        const float4 a = *reinterpret_cast<const float4*>(row + rg * RQ + 4 * i);
-        v[4 * i] = a.x; v[4 * i + 1] = a.y; v[4 * i + 2] = a.z; v[4 * i + 3] = a.w;
-      }
+    for (int i = 0; i < PH / 2; ++i) {
+      const ulonglong2 a = *reinterpret_cast<const ulonglong2*>(vec + r0 + 4 * i);
+      v[2 * i] = a.x; v[2 * i + 1] = a.y;
     }
   };
   for (int ci = 0; ci < n_chunks; ++ci) {
@@ -462,130 +483,95 @@ delta_chunks_kernel(const DeltaParams p, const float* __restrict__ scratch) {
     }
     __syncthreads();
     const float* buf = sm + (ci & 1) * kBuf;
-    const float* Dv = buf + kVecs;
-    const float* Us = Dv + KP;                           // [16][kCols] each: U, Y, V
-    // products of the 32 rows of W and X with the state, eight rows at a time; their sums over the warp's rows are dealt
-    // out so that lane group rl ends with row 8 g + rl
-#pragma unroll 1
-    for (int g = 0; g < 4; ++g) {
-      float acc[8][4];
+    const float* Us = buf + kVecs + KP;                  // [16][kCols] each: U, Y, V
+    // the 32 rows of W and X times the state: sums over the thread's rows, then over the warp's two row groups
+#pragma unroll 8
+    for (int v = 0; v < 2 * kChunk; v += 2) {            // two rows at a time: the two row groups end with one each
+      uint64_t w[PH], x[PH];
+      rows_at(buf + v * KP, w);
+      rows_at(buf + (v + 1) * KP, x);
+      uint64_t a = mul2(w[0], S[0]), b = mul2(x[0], S[0]);
 #pragma unroll
-      for (int v = 0; v < 8; ++v) {
-        float w[RQ];
-        rows_at(buf + (g * 8 + v) * KP, w);
-#pragma unroll
-        for (int c = 0; c < 4; ++c) {
-          float s = w[0] * S[0][c];
-#pragma unroll
-          for (int i = 1; i < RQ; ++i) s = fmaf(w[i], S[i][c], s);
-          acc[v][c] = s;
-        }
-      }
-      float a4[4][4], a2[2][4], a1[4];
-      const bool hi4 = rl & 4, hi2 = rl & 2, hi1 = rl & 1;
-#pragma unroll
-      for (int v = 0; v < 4; ++v)
-#pragma unroll
-        for (int c = 0; c < 4; ++c) {
-          const float give = hi4 ? acc[v][c] : acc[v + 4][c], have = hi4 ? acc[v + 4][c] : acc[v][c];
-          a4[v][c] = have + __shfl_xor_sync(0xffffffffu, give, 16);
-        }
-#pragma unroll
-      for (int v = 0; v < 2; ++v)
-#pragma unroll
-        for (int c = 0; c < 4; ++c) {
-          const float give = hi2 ? a4[v][c] : a4[v + 2][c], have = hi2 ? a4[v + 2][c] : a4[v][c];
-          a2[v][c] = have + __shfl_xor_sync(0xffffffffu, give, 8);
-        }
-#pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        const float give = hi1 ? a2[0][c] : a2[1][c], have = hi1 ? a2[1][c] : a2[0][c];
-        a1[c] = have + __shfl_xor_sync(0xffffffffu, give, 4);
-      }
-      *reinterpret_cast<float4*>(red + ((warp * 2 * kChunk) + g * 8 + rl) * kCols + 4 * cg) = make_float4(a1[0], a1[1], a1[2], a1[3]);
+      for (int i = 1; i < PH; ++i) { a = fma2(w[i], S[i], a); b = fma2(x[i], S[i], b); }
+      const float fa = sum2(a), fb = sum2(b);
+      const bool upper = lane & 16;
+      const float sum = (upper ? fb : fa) + __shfl_xor_sync(0xffffffffu, upper ? fa : fb, 16);
+      red[(warp * 2 * kChunk + v + (lane >> 4)) * kCols + cl] = sum;
     }
     __syncthreads();
     {
-      const int v = tid >> 2, c4 = (tid & 3) * 4;        // row of W (v < 16) or of X
-      float4 s = *reinterpret_cast<const float4*>(Us + v * kCols + c4);       // U's rows, then Y's
+      const int v = tid >> 3, c2 = (tid & 7) * 2;        // row of W (v < 16) or of X
+      float2 s = *reinterpret_cast<const float2*>(Us + v * kCols + c2);       // U's rows, then Y's
 #pragma unroll
-      for (int w = 0; w < 4; ++w) {
-        const float4 a = *reinterpret_cast<const float4*>(red + (w * 2 * kChunk + v) * kCols + c4);
-        s.x += a.x; s.y += a.y; s.z += a.z; s.w += a.w;
+      for (int w = 0; w < kChunkWarps; ++w) {
+        const float2 a = *reinterpret_cast<const float2*>(red + (w * 2 * kChunk + v) * kCols + c2);
+        s.x += a.x; s.y += a.y;
       }
       if (v < kChunk) {
-        *reinterpret_cast<float4*>(zs + v * kCols + c4) = s;
+        *reinterpret_cast<float2*>(zs + v * kCols + c2) = s;
       } else {
-        const int t = ci * kChunk + v - kChunk, col = c0 + c4;
+        const int t = ci * kChunk + v - kChunk;
         if (t < q_len) {
-          float* dst = p.y + (size_t)(tok0 + t) * inner_v + (size_t)h * p.dv + col;
-          if (col + 3 < p.dv && (inner_v & 3) == 0 && (p.dv & 3) == 0) *reinterpret_cast<float4*>(dst) = s;
-          else {
-            const float e[4] = {s.x, s.y, s.z, s.w};
-#pragma unroll
-            for (int c = 0; c < 4; ++c) if (col + c < p.dv) dst[c] = e[c];
-          }
+          float* dst = p.y + (size_t)(tok0 + t) * inner_v + (size_t)h * p.dv + c0 + c2;
+          if (c0 + c2 < p.dv) dst[0] = s.x;
+          if (c0 + c2 + 1 < p.dv) dst[1] = s.y;
         }
       }
     }
     __syncthreads();
     {
-      float d[RQ];
-      rows_at(Dv, d);
+      uint64_t d[PH];
+      rows_at(buf + kVecs, d);
 #pragma unroll
-      for (int i = 0; i < RQ; ++i)
-#pragma unroll
-        for (int c = 0; c < 4; ++c) S[i][c] *= d[i];
-      const float* Qs = buf + 2 * kChunk * KP;
+      for (int i = 0; i < PH; ++i) S[i] = mul2(d[i], S[i]);
+      const float* Qs = buf + 2 * kChunk * KP;           // - D q
       const float* Ms = Qs + kChunk * KP;
       const float* Vs = Us + 2 * kChunk * kCols;
 #pragma unroll 8
       for (int t = 0; t < kChunk; ++t) {
-        float q[RQ], m[RQ];
+        uint64_t q[PH], m[PH];
         rows_at(Qs + t * KP, q);
         rows_at(Ms + t * KP, m);
-        const float4 z = *reinterpret_cast<const float4*>(zs + t * kCols + 4 * cg);
-        const float4 v = *reinterpret_cast<const float4*>(Vs + t * kCols + 4 * cg);
+        const float zf = zs[t * kCols + cl], vf = Vs[t * kCols + cl];
+        const uint64_t z = pack2(zf, zf), v = pack2(vf, vf);
 #pragma unroll
-        for (int i = 0; i < RQ; ++i) {
-          S[i][0] = fmaf(m[i], v.x, fmaf(-q[i], z.x, S[i][0])); S[i][1] = fmaf(m[i], v.y, fmaf(-q[i], z.y, S[i][1]));
-          S[i][2] = fmaf(m[i], v.z, fmaf(-q[i], z.z, S[i][2])); S[i][3] = fmaf(m[i], v.w, fmaf(-q[i], z.w, S[i][3]));
-        }
+        for (int i = 0; i < PH; ++i) S[i] = fma2(m[i], v, fma2(q[i], z, S[i]));
       }
     }
     __syncthreads();                                     // everyone is done with this buffer and with zs
   }
-  if (own != nullptr) {
+  if (own != nullptr && col < p.dv) {
 #pragma unroll
-    for (int i = 0; i < RQ; ++i)
-#pragma unroll
-      for (int c = 0; c < 4; ++c) {
-        const int n = rg * RQ + i, col = c0 + 4 * cg + c;
-        if (n < p.d && col < p.dv) own[(size_t)n * p.dv + col] = S[i][c];
-      }
+    for (int i = 0; i < PH; ++i) {
+      const int n = r0 + 2 * i;
+      float lo, hi;
+      unpack2(S[i], lo, hi);
+      if (n < p.d) own[(size_t)n * p.dv + col] = lo;
+      if (n + 1 < p.d) own[(size_t)(n + 1) * p.dv + col] = hi;
+    }
   }
 }
 
 // Floats of scratch that `n_blocks` chunks need.
 ILB_EXPORT long long ilb_delta_chunk_floats(int n_blocks, int heads, int d, int dv) {
-  return (long long)n_blocks * heads * chunk_floats(32 * rows_per_thread(d), padded_cols(dv));
+  return (long long)n_blocks * heads * chunk_floats(padded_rows(d), padded_cols(dv));
 }
 
-template <int RQ>
+template <int RH>
 static int chunks_launch(const DeltaParams& p, const float* scratch, cudaStream_t stream) {
-  const size_t smem = sizeof(float) * chunks_smem_floats(32 * RQ);
+  const size_t smem = sizeof(float) * chunks_smem_floats(16 * RH);
   static OncePerDevice once;
-  if (once.first() && cudaFuncSetAttribute(delta_chunks_kernel<RQ>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+  if (once.first() && cudaFuncSetAttribute(delta_chunks_kernel<RH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
     once.forget();
     return fail("delta_chunks: cannot reserve %zu bytes of shared memory", smem);
   }
-  ilb::launch(delta_chunks_kernel<RQ>, dim3(p.heads, padded_cols(p.dv) / kCols, p.n_seqs), dim3(kScanThreads), smem, stream, p, scratch);
+  ilb::launch(delta_chunks_kernel<RH>, dim3(p.heads, padded_cols(p.dv) / kCols, p.n_seqs), dim3(kChunkThreads), smem, stream, p, scratch);
   return check_launch("delta_chunks");
 }
 
 template <typename TI>
 static int prep_launch(const DeltaParams& p, float* scratch, int n_blocks, cudaStream_t stream) {
-  const int KP = 32 * rows_per_thread(p.d);
+  const int KP = padded_rows(p.d);
   const size_t smem = sizeof(float) * prep_smem_floats(KP, padded_cols(p.dv));
   ILB_REQUIRE(smem <= 200 * 1024, "delta_prep: states of %d x %d do not fit the block's shared memory", p.d, p.dv);
   static OncePerDevice once;
@@ -611,8 +597,8 @@ ILB_EXPORT int ilb_delta_chunks(const void* proj, int dtype, int ld, int col_r, 
   ILB_REQUIRE(heads <= 65535, "delta_chunks: too many heads");
   if (n_seqs == 0 || n_blocks <= 0) return 0;
   if (int rc = dtype == kF32 ? prep_launch<float>(p, scratch, n_blocks, stream) : prep_launch<__nv_bfloat16>(p, scratch, n_blocks, stream)) return rc;
-  const int rq = rows_per_thread(d);
-  return rq == 2 ? chunks_launch<2>(p, scratch, stream) : rq == 4 ? chunks_launch<4>(p, scratch, stream) : chunks_launch<8>(p, scratch, stream);
+  const int rows = padded_rows(d);
+  return rows == 64 ? chunks_launch<4>(p, scratch, stream) : rows == 128 ? chunks_launch<8>(p, scratch, stream) : chunks_launch<16>(p, scratch, stream);
 }
 
 // ---------------------------------------------------------------- single tokens
