@@ -32,6 +32,7 @@
 // pads a recorded launch) starts from zero and stores nothing.
 #include <math.h>
 #include "common.cuh"
+#include "sm100.cuh"
 
 using namespace ilb;
 
@@ -242,6 +243,15 @@ __device__ __forceinline__ float sum2(uint64_t v) {
 
 // Floats of one (chunk, head) in scratch: W, X, - D q, D m [16][KP], D [KP], then U, Y, V [16][DP]; KP rows, DP columns, padded.
 __host__ __device__ __forceinline__ long long chunk_floats(int KP, int DP) { return (long long)4 * kChunk * KP + KP + (long long)3 * kChunk * DP; }
+// The tensor-core form keeps W, X, D m, - D q as three bfloat16 pieces each (x = hi + mid + lo exactly), in the order in which the
+// lanes of a warp hold the operands of mma.m16n8k16, 16 bytes a lane:
+//   per 16 rows of the state: W, X (A operands, 16 tokens x 16 rows), pieces hi mid lo each       6 x 512 bytes
+//   then per 16 rows:         D m, - D q (B operands, 16 tokens x 2 x 8 rows), hi mid lo each      6 x 512 bytes
+//   then D [KP], U, Y [16][DP] in 32-bit, and per 16 columns V transposed (A operand, 16 columns x 16 tokens; exact)   512 bytes
+constexpr int kFragFloats = 128;                         // 512 bytes
+__host__ __device__ __forceinline__ long long chunk_floats_mma(int KP, int DP) {
+  return (long long)(KP / 16) * 12 * kFragFloats + KP + (long long)2 * kChunk * DP + (long long)(DP / 16) * kFragFloats;
+}
 __host__ __device__ __forceinline__ int padded_cols(int dv) { return (dv + kCols - 1) / kCols * kCols; }
 static inline int padded_rows(int d) { return d <= 64 ? 64 : (d <= 128 ? 128 : 256); }
 
@@ -253,6 +263,15 @@ __device__ __forceinline__ bool find_chunk(const int* __restrict__ cu_q, int n_s
     b -= n;
   }
   return false;
+}
+
+// (x, y) = hi + mid + lo exactly, each a pair of bfloat16.
+__device__ __forceinline__ void split3(float x, float y, uint32_t& hi, uint32_t& mid, uint32_t& lo) {
+  hi = pack_bf16(x, y);
+  x -= __uint_as_float(hi << 16); y -= __uint_as_float(hi & 0xFFFF0000u);
+  mid = pack_bf16(x, y);
+  x -= __uint_as_float(mid << 16); y -= __uint_as_float(mid & 0xFFFF0000u);
+  lo = pack_bf16(x, y);
 }
 
 constexpr int kPrepThreads = 128;
@@ -273,17 +292,34 @@ delta_prep_kernel(const DeltaParams p, float* __restrict__ scratch, int KP) {
   float* V = M + kChunk * ld;                            // [16][DP]
   float* AC = V + kChunk * DP;                           // [16][16][2]: - p.q (j < t), - s.q (j <= t); zero elsewhere
   float* BE = AC + 2 * kChunk * kChunk;                  //              p.m (j < t), s.m (j <= t)
-  __shared__ float inv_norm[kChunk];
+  __shared__ float inv_norm[kChunk], Ds[256];
   int seq, ci;
   if (!find_chunk(p.cu_q, p.n_seqs, blockIdx.x, seq, ci)) return;
   const int h = blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int tok0 = p.cu_q[seq] + ci * kChunk, ts = min(kChunk, p.cu_q[seq + 1] - tok0);
   const int inner_k = p.heads * p.d;
   const TI* proj = reinterpret_cast<const TI*>(p.proj);
-  float* out = scratch + ((size_t)blockIdx.x * p.heads + h) * chunk_floats(KP, DP);
+  // FAST: the tensor-core form's layout, else the plain one
+  float* out = scratch + ((size_t)blockIdx.x * p.heads + h) * (FAST ? chunk_floats_mma(KP, DP) : chunk_floats(KP, DP));
   float* outW = out; float* outX = outW + kChunk * KP; float* outQ = outX + kChunk * KP; float* outM = outQ + kChunk * KP;
-  float* outD = outM + kChunk * KP; float* outU = outD + KP; float* outY = outU + kChunk * DP; float* outV = outY + kChunk * DP;
+  float* outD = FAST ? out + (KP / 16) * 12 * kFragFloats : outM + kChunk * KP;
+  float* outU = outD + KP; float* outY = outU + kChunk * DP; float* outV = outY + kChunk * DP;
 
+  // the raw inputs of a channel, all in flight together; this thread's first channel's before anything is waited for
+  TI r_raw[kChunk], a_raw[kChunk];
+  float l_raw[kChunk];
+  auto fetch = [&](int n) {
+    const int ch = h * p.d + (n < p.d ? n : 0);
+#pragma unroll
+    for (int t = 0; t < kChunk; ++t) {
+      const int tt = tok0 + (t < ts ? t : 0);
+      const TI* row = proj + (size_t)tt * p.ld;
+      r_raw[t] = row[p.col_r + ch];
+      a_raw[t] = row[p.col_a + ch];
+      l_raw[t] = p.low[(size_t)tt * inner_k + ch];
+    }
+  };
+  fetch(tid);
   for (int n = tid; n < KP; n += kPrepThreads) {
 #pragma unroll
     for (int t = 0; t < kChunk; ++t)
@@ -294,7 +330,7 @@ delta_prep_kernel(const DeltaParams p, float* __restrict__ scratch, int KP) {
     for (int t = 0; t < kChunk; ++t) {
       const float v = (c < p.dv && t < ts) ? to_float(proj[(size_t)(tok0 + t) * p.ld + p.col_v + h * p.dv + c]) : 0.f;
       V[t * DP + c] = v;
-      outV[t * DP + c] = v;
+      if constexpr (!FAST) outV[t * DP + c] = v;
     }
   }
   __syncthreads();
@@ -309,35 +345,23 @@ delta_prep_kernel(const DeltaParams p, float* __restrict__ scratch, int KP) {
     const bool live = n < p.d;
     const int ch = h * p.d + (live ? n : 0);
     const float w0 = p.w0[ch], ab = p.ab[ch];
-    float r[kChunk], a[kChunk], l[kChunk];
-#pragma unroll
-    for (int t = 0; t < kChunk; ++t) {                   // all loads in flight together
-      const bool on = live && t < ts;
-      const TI* row = proj + (size_t)(tok0 + (on ? t : 0)) * p.ld;
-      r[t] = on ? to_float(row[p.col_r + ch]) : 0.f;
-      a[t] = to_float(row[p.col_a + ch]);
-      l[t] = p.low[(size_t)(tok0 + (on ? t : 0)) * inner_k + ch];
-    }
+    if (n != tid) fetch(n);
     float D = 1.f;
 #pragma unroll
     for (int t = 0; t < kChunk; ++t) {
       const bool on = live && t < ts;
       const float k = M[t * ld + n], u = k * inv_norm[t];
-      const float w = on ? exp_t<FAST>(-p.log_decay * sigmoid_t<FAST>(l[t] + w0)) : 1.f;
-      const float g = on ? sigmoid_t<FAST>(a[t] + ab) : 0.f;
+      const float w = on ? exp_t<FAST>(-p.log_decay * sigmoid_t<FAST>(l_raw[t] + w0)) : 1.f;
+      const float g = on ? sigmoid_t<FAST>(to_float(a_raw[t]) + ab) : 0.f;
       P[t * ld + n] = D * u;
       D *= w;
       const float inv = FAST ? __fdividef(1.0f, D) : 1.0f / D;
       Qv[t * ld + n] = g * u * inv;
       M[t * ld + n] = k * inv;
-      R[t * ld + n] = D * r[t];
+      R[t * ld + n] = on ? D * to_float(r_raw[t]) : 0.f;
     }
     outD[n] = D;
-#pragma unroll
-    for (int t = 0; t < kChunk; ++t) {
-      outQ[t * KP + n] = -Qv[t * ld + n] * D;
-      outM[t * KP + n] = M[t * ld + n] * D;
-    }
+    Ds[n] = D;
   }
   __syncthreads();
   {   // rows of P and R against rows of Q and M: a thread takes four rows and one column of both
@@ -388,8 +412,15 @@ delta_prep_kernel(const DeltaParams p, float* __restrict__ scratch, int KP) {
       float c, zero, x;
       unpack2(ac[t], zero, c);
       unpack2(vx, w[t], x);
-      outW[t * KP + n] = w[t];
-      outX[t * KP + n] = fmaf(c, w[t], x);
+      x = fmaf(c, w[t], x);
+      if constexpr (FAST) { P[t * ld + n] = w[t]; R[t * ld + n] = x; }      // (this thread's own column: nobody else reads it any more)
+      else { outW[t * KP + n] = w[t]; outX[t * KP + n] = x; }
+    }
+    const float D = Ds[n];
+#pragma unroll
+    for (int t = 0; t < kChunk; ++t) {
+      if constexpr (FAST) { Qv[t * ld + n] *= -D; M[t * ld + n] *= D; }
+      else { outQ[t * KP + n] = -Qv[t * ld + n] * D; outM[t * KP + n] = M[t * ld + n] * D; }
     }
   }
   for (int c0 = tid; c0 < DP; c0 += kPrepThreads) {      // U = (I + A)^-1 B V,  Y = E V - C U
@@ -409,6 +440,46 @@ delta_prep_kernel(const DeltaParams p, float* __restrict__ scratch, int KP) {
       unpack2(sy, u[t], y);
       outU[t * DP + c0] = u[t];
       outY[t * DP + c0] = fmaf(c, u[t], fmaf(e, v[t], y));
+    }
+  }
+  if constexpr (FAST) {
+    __syncthreads();
+    uint4* frag = reinterpret_cast<uint4*>(out);
+    // eight values of a lane, cut into three pieces, 16 bytes each
+    auto emit = [&](size_t at, const float (&x)[8]) {
+      uint32_t hi[4], mid[4], lo[4];
+#pragma unroll
+      for (int i = 0; i < 4; ++i) split3(x[2 * i], x[2 * i + 1], hi[i], mid[i], lo[i]);
+      frag[at] = make_uint4(hi[0], hi[1], hi[2], hi[3]);
+      frag[at + 32] = make_uint4(mid[0], mid[1], mid[2], mid[3]);
+      frag[at + 64] = make_uint4(lo[0], lo[1], lo[2], lo[3]);
+    };
+    const int slices = KP / 16;
+    for (int i = tid; i < slices * 4 * 32; i += kPrepThreads) {
+      const int ln = i & 31, what = (i >> 5) & 3, ks = i >> 7, g = ln >> 2, t4 = ln & 3;
+      float x[8];
+      if (what < 2) {                                    // A operand: rows are tokens g and g + 8, columns the state's rows
+        const float* m = (what == 0 ? P : R) + ks * 16 + 2 * t4;
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          x[e] = m[g * ld + e]; x[2 + e] = m[(g + 8) * ld + e]; x[4 + e] = m[g * ld + 8 + e]; x[6 + e] = m[(g + 8) * ld + 8 + e];
+        }
+        emit((size_t)((ks * 2 + what) * 3) * 32 + ln, x);
+      } else {                                           // B operand: rows are tokens, columns the state's rows g and g + 8
+        const float* m = (what == 2 ? M : Qv) + ks * 16 + g;
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          x[e] = m[(2 * t4 + e) * ld]; x[2 + e] = m[(2 * t4 + 8 + e) * ld]; x[4 + e] = m[(2 * t4 + e) * ld + 8]; x[6 + e] = m[(2 * t4 + 8 + e) * ld + 8];
+        }
+        emit((size_t)(slices * 6 + (ks * 2 + what - 2) * 3) * 32 + ln, x);
+      }
+    }
+    uint4* vfrag = reinterpret_cast<uint4*>(outY + kChunk * DP);
+    for (int i = tid; i < DP / 16 * 32; i += kPrepThreads) {
+      const int ln = i & 31, g = ln >> 2, t4 = ln & 3;
+      const float* m = V + (i >> 5) * 16 + g;
+      vfrag[i] = make_uint4(pack_bf16(m[2 * t4 * DP], m[(2 * t4 + 1) * DP]), pack_bf16(m[2 * t4 * DP + 8], m[(2 * t4 + 1) * DP + 8]),
+                            pack_bf16(m[(2 * t4 + 8) * DP], m[(2 * t4 + 9) * DP]), pack_bf16(m[(2 * t4 + 8) * DP + 8], m[(2 * t4 + 9) * DP + 8]));
     }
   }
   ilb::pdl_launch_dependents();                          // (the blocks of delta_chunks are few and large: they start when these are done)
@@ -552,9 +623,200 @@ delta_chunks_kernel(const DeltaParams p, const float* __restrict__ scratch) {
   }
 }
 
+// The same walk on the tensor cores (mma.sync m16n8k16, 32-bit accumulation), for projections stored in bfloat16: every 32-bit
+// operand is three exact bfloat16 pieces, and of the nine products of two such operands the six that reach 32-bit precision
+// are added, smallest first.  A warp owns 16 rows of the state and the block's 16 columns, transposed in the layout of an
+// accumulator, which is the layout of the operand that the two thin products read; the sums over the warps meet in shared
+// memory.  What a chunk adds to the state is formed apart and joins it with one rounding.
+template <int KP>
+__global__ void __launch_bounds__(KP * 2)
+delta_chunks_mma_kernel(const DeltaParams p, const float* __restrict__ scratch) {
+  ilb::pdl_launch_dependents();
+  ilb::pdl_wait();
+  constexpr int kWarps = KP / 16, kLd = 24;              // kLd: floats from one row of a warp's sums to the next
+  extern __shared__ __align__(16) float sm[];
+  float* red = sm;                                       // [warps][32][kLd]
+  float* zs = red + kWarps * 2 * kChunk * kLd;           // [16][kCols + 1]
+  constexpr int kZ = kCols + 1;
+  const int h = blockIdx.x, cb = blockIdx.y, c0 = cb * kCols, seq = blockIdx.z;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
+  const int DP = padded_cols(p.dv);
+  const int tok0 = p.cu_q[seq], q_len = p.cu_q[seq + 1] - tok0, n_chunks = (q_len + kChunk - 1) / kChunk;
+  if (n_chunks == 0) return;
+  int first = 0;
+  for (int i = 0; i < seq; ++i) first += (p.cu_q[i + 1] - p.cu_q[i] + kChunk - 1) / kChunk;
+  const int slot = p.slots[seq];
+  float* own = slot >= 0 ? p.state + ((size_t)slot * p.heads + h) * p.d * p.dv : nullptr;
+  const int inner_v = p.heads * p.dv;
+  const size_t per = (size_t)p.heads * chunk_floats_mma(KP, DP);        // from one chunk to the next
+  const float* src = scratch + ((size_t)first * p.heads + h) * chunk_floats_mma(KP, DP);
+
+  uint4 A[6], B[6], V;                                   // W hi mid lo, X hi mid lo;  D m hi mid lo, - D q hi mid lo
+  float2 D[2];
+  auto load_a = [&](const float* at) {
+    const uint4* f = reinterpret_cast<const uint4*>(at) + (size_t)warp * 6 * 32 + lane;
+#pragma unroll
+    for (int i = 0; i < 6; ++i) A[i] = __ldg(f + 32 * i);
+  };
+  auto load_b = [&](const float* at) {
+    const uint4* f = reinterpret_cast<const uint4*>(at) + (size_t)(kWarps * 6 + warp * 6) * 32 + lane;
+#pragma unroll
+    for (int i = 0; i < 6; ++i) B[i] = __ldg(f + 32 * i);
+    const float* d = at + kWarps * 12 * kFragFloats;
+    D[0] = *reinterpret_cast<const float2*>(d + warp * 16 + 2 * t4);
+    D[1] = *reinterpret_cast<const float2*>(d + warp * 16 + 8 + 2 * t4);
+    V = __ldg(reinterpret_cast<const uint4*>(d + KP + 2 * kChunk * DP) + cb * 32 + lane);
+  };
+  // this thread's elements of U and Y: pairs of columns, dealt out by number
+  constexpr int kAdd = (2 * kChunk * 8 + KP * 2 - 1) / (KP * 2);
+  float2 add[kAdd];
+  auto load_uy = [&](const float* at) {
+    const float* uy = at + kWarps * 12 * kFragFloats + KP + c0;
+#pragma unroll
+    for (int i = 0; i < kAdd; ++i) {
+      const int e = tid + i * KP * 2;
+      if (e < 2 * kChunk * 8) add[i] = *reinterpret_cast<const float2*>(uy + (size_t)(e >> 3) * DP + (e & 7) * 2);
+    }
+  };
+  // The chunks two and three ahead are asked into L2, each block of a head its share of the lines.
+  const int lines = (int)((chunk_floats_mma(KP, DP) * 4 + 127) / 128), share = (lines + (int)gridDim.y - 1) / (int)gridDim.y;
+  auto ahead = [&](int ci) {
+    if (ci >= n_chunks) return;
+    const char* at = reinterpret_cast<const char*>(scratch + (size_t)first * per + (size_t)ci * per + (size_t)h * chunk_floats_mma(KP, DP));
+    for (int i = tid; i < share; i += KP * 2) {
+      const int line = cb * share + i;
+      if (line < lines) asm volatile("prefetch.global.L2 [%0];" ::"l"(at + (size_t)line * 128));
+    }
+  };
+  load_a(src);
+  load_b(src);
+  load_uy(src);
+  ahead(1);
+  ahead(2);
+  // S[j][0, 1]: rows 16 warp + 8 j + 2 t4 (+ 1), column g; [2, 3]: column g + 8
+  float S[2][4];
+#pragma unroll
+  for (int j = 0; j < 2; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int n = warp * 16 + 8 * j + 2 * t4 + (e & 1), col = c0 + g + 8 * (e >> 1);
+      S[j][e] = (own != nullptr && n < p.d && col < p.dv) ? own[(size_t)n * p.dv + col] : 0.f;
+    }
+  auto mma = [&](float (&c)[4], const uint4& a, uint32_t b0, uint32_t b1) {
+    const uint32_t aa[4] = {a.x, a.y, a.z, a.w};
+    mma_16816(c, aa, b0, b1);
+  };
+  for (int ci = 0; ci < n_chunks; ++ci, src += per) {
+    {
+      uint32_t b[3][2][2];                               // pieces of the state: [piece][columns 8 jj + g][rows 2 t4, 2 t4 + 8]
+#pragma unroll
+      for (int jj = 0; jj < 2; ++jj)
+#pragma unroll
+        for (int j = 0; j < 2; ++j) split3(S[j][2 * jj], S[j][2 * jj + 1], b[0][jj][j], b[1][jj][j], b[2][jj][j]);
+#pragma unroll
+      for (int m = 0; m < 2; ++m)
+#pragma unroll
+        for (int jj = 0; jj < 2; ++jj) {
+          float c[4] = {0.f, 0.f, 0.f, 0.f}, f[4] = {0.f, 0.f, 0.f, 0.f};
+          mma(c, A[3 * m + 2], b[0][jj][0], b[0][jj][1]);
+          mma(f, A[3 * m], b[1][jj][0], b[1][jj][1]);
+          mma(c, A[3 * m], b[2][jj][0], b[2][jj][1]);
+          mma(f, A[3 * m], b[0][jj][0], b[0][jj][1]);
+          mma(c, A[3 * m + 1], b[1][jj][0], b[1][jj][1]);
+          mma(c, A[3 * m + 1], b[0][jj][0], b[0][jj][1]);
+#pragma unroll
+          for (int e = 0; e < 4; ++e) c[e] += f[e];
+          float* r = red + (size_t)(warp * 2 * kChunk + m * kChunk + g) * kLd + 8 * jj + 2 * t4;
+          *reinterpret_cast<float2*>(r) = make_float2(c[0], c[1]);
+          *reinterpret_cast<float2*>(r + 8 * kLd) = make_float2(c[2], c[3]);
+        }
+    }
+    const bool more = ci + 1 < n_chunks;
+    if (more) load_a(src + per);
+    ahead(ci + 3);
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < kAdd; ++i) {
+      const int e = tid + i * KP * 2;
+      if (e < 2 * kChunk * 8) {
+        const int v = e >> 3, c2 = (e & 7) * 2;          // row of W (v < 16) or of X
+        float2 s = add[i];
+#pragma unroll
+        for (int w = 0; w < kWarps; ++w) {
+          const float2 a = *reinterpret_cast<const float2*>(red + (size_t)(w * 2 * kChunk + v) * kLd + c2);
+          s.x += a.x; s.y += a.y;
+        }
+        if (v < kChunk) {
+          zs[v * kZ + c2] = s.x; zs[v * kZ + c2 + 1] = s.y;
+        } else {
+          const int t = ci * kChunk + v - kChunk;
+          if (t < q_len) {
+            float* dst = p.y + (size_t)(tok0 + t) * inner_v + (size_t)h * p.dv + c0 + c2;
+            if (c0 + c2 < p.dv) dst[0] = s.x;
+            if (c0 + c2 + 1 < p.dv) dst[1] = s.y;
+          }
+        }
+      }
+    }
+    if (more) load_uy(src + per);
+    __syncthreads();
+    {
+      uint4 z[3];                                        // pieces of Z transposed: columns g, g + 8, tokens 2 t4 (+ 1), + 8
+      const float* zr = zs + 2 * t4 * kZ + g;
+      split3(zr[0], zr[kZ], z[0].x, z[1].x, z[2].x);
+      split3(zr[8], zr[kZ + 8], z[0].y, z[1].y, z[2].y);
+      split3(zr[8 * kZ], zr[9 * kZ], z[0].z, z[1].z, z[2].z);
+      split3(zr[8 * kZ + 8], zr[9 * kZ + 8], z[0].w, z[1].w, z[2].w);
+#pragma unroll
+      for (int j = 0; j < 2; ++j) {
+        auto b0 = [&](int i) { return j == 0 ? B[i].x : B[i].z; };
+        auto b1 = [&](int i) { return j == 0 ? B[i].y : B[i].w; };
+        float c[4] = {0.f, 0.f, 0.f, 0.f}, e[4] = {0.f, 0.f, 0.f, 0.f}, f[4] = {0.f, 0.f, 0.f, 0.f};
+        mma(c, V, b0(2), b1(2));
+        mma(e, z[2], b0(3), b1(3));
+        mma(f, z[1], b0(3), b1(3));
+        mma(c, V, b0(1), b1(1));
+        mma(e, z[0], b0(5), b1(5));
+        mma(f, z[0], b0(4), b1(4));
+        mma(c, V, b0(0), b1(0));
+        mma(e, z[1], b0(4), b1(4));
+        mma(f, z[0], b0(3), b1(3));
+#pragma unroll
+        for (int i = 0; i < 4; ++i) c[i] += e[i] + f[i];
+        S[j][0] = fmaf(D[j].x, S[j][0], c[0]); S[j][1] = fmaf(D[j].y, S[j][1], c[1]);
+        S[j][2] = fmaf(D[j].x, S[j][2], c[2]); S[j][3] = fmaf(D[j].y, S[j][3], c[3]);
+      }
+    }
+    if (more) load_b(src + per);
+  }
+  if (own != nullptr) {
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int n = warp * 16 + 8 * j + 2 * t4 + (e & 1), col = c0 + g + 8 * (e >> 1);
+        if (n < p.d && col < p.dv) own[(size_t)n * p.dv + col] = S[j][e];
+      }
+  }
+}
+
+template <int KP>
+static int chunks_mma_launch(const DeltaParams& p, const float* scratch, cudaStream_t stream) {
+  const size_t smem = sizeof(float) * ((size_t)KP / 16 * 2 * kChunk * 24 + kChunk * (kCols + 1));
+  static OncePerDevice once;
+  if (smem > 48 * 1024 && once.first() &&
+      cudaFuncSetAttribute(delta_chunks_mma_kernel<KP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+    once.forget();
+    return fail("delta_chunks: cannot reserve %zu bytes of shared memory", smem);
+  }
+  ilb::launch(delta_chunks_mma_kernel<KP>, dim3(p.heads, padded_cols(p.dv) / kCols, p.n_seqs), dim3(KP * 2), smem, stream, p, scratch);
+  return check_launch("delta_chunks");
+}
+
 // Floats of scratch that `n_blocks` chunks need.
-ILB_EXPORT long long ilb_delta_chunk_floats(int n_blocks, int heads, int d, int dv) {
-  return (long long)n_blocks * heads * chunk_floats(padded_rows(d), padded_cols(dv));
+ILB_EXPORT long long ilb_delta_chunk_floats(int n_blocks, int heads, int d, int dv, int dtype) {
+  const int KP = padded_rows(d), DP = padded_cols(dv);
+  return (long long)n_blocks * heads * (dtype == kF32 ? chunk_floats(KP, DP) : chunk_floats_mma(KP, DP));
 }
 
 template <int RH>
@@ -592,12 +854,15 @@ ILB_EXPORT int ilb_delta_chunks(const void* proj, int dtype, int ld, int col_r, 
   const DeltaParams p{proj, ld, col_r, col_k, col_v, col_a, low, w0, ab, state, y, cu_q, slots, n_seqs, heads, d, dv, log_decay, unit_eps};
   if (int rc = check_sizes(p, dtype)) return rc;
   ILB_REQUIRE(log_decay >= 0.f && log_decay * kChunk <= 40.f, "delta_chunks: a decay of exp(-%f) a token leaves a chunk's range", (double)log_decay);
-  ILB_REQUIRE(scratch != nullptr && (uintptr_t)scratch % 16 == 0 && ilb_delta_chunk_floats(n_blocks, heads, d, dv) <= scratch_floats,
+  ILB_REQUIRE(scratch != nullptr && (uintptr_t)scratch % 16 == 0 && ilb_delta_chunk_floats(n_blocks, heads, d, dv, dtype) <= scratch_floats,
               "delta_chunks: scratch too small");
   ILB_REQUIRE(heads <= 65535, "delta_chunks: too many heads");
   if (n_seqs == 0 || n_blocks <= 0) return 0;
   if (int rc = dtype == kF32 ? prep_launch<float>(p, scratch, n_blocks, stream) : prep_launch<__nv_bfloat16>(p, scratch, n_blocks, stream)) return rc;
   const int rows = padded_rows(d);
+  if (dtype == kBF16)
+    return rows == 64 ? chunks_mma_launch<64>(p, scratch, stream) : rows == 128 ? chunks_mma_launch<128>(p, scratch, stream)
+                                                                                : chunks_mma_launch<256>(p, scratch, stream);
   return rows == 64 ? chunks_launch<4>(p, scratch, stream) : rows == 128 ? chunks_launch<8>(p, scratch, stream) : chunks_launch<16>(p, scratch, stream);
 }
 

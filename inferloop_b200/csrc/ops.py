@@ -504,7 +504,7 @@ def delta_scan(proj: torch.Tensor, col_r: int, col_k: int, col_v: int, col_a: in
         chunks = step.max_q_len >= DELTA_CHUNK_FROM and workspace is not None and log_decay * DELTA_CHUNK <= 40.0
     if chunks:
         n_blocks = sum(-(-n // DELTA_CHUNK) for n in step.h_q_len) + (step.n_seqs - len(step.h_q_len))
-        scratch = workspace.buffer("delta.chunks", (delta_chunk_floats(n_blocks, heads, d, dv),), torch.float32)
+        scratch = workspace.buffer("delta.chunks", (delta_chunk_floats(n_blocks, heads, d, dv, proj.dtype),), torch.float32)
         _call("delta", "ilb_delta_chunks", _ptr(proj), _i(_code(proj)), _i(proj.stride(0)), _i(col_r), _i(col_k), _i(col_v), _i(col_a), _ptr(low),
               _ptr(w0), _ptr(ab), _f(log_decay), _f(unit_eps), _ptr(state), _ptr(y), _ptr(step.cu_q), _ptr(step.slots), _i(step.n_seqs),
               _i(heads), _i(d), _i(dv), _ptr(scratch), ctypes.c_longlong(scratch.numel()), _i(n_blocks), _stream(y))
@@ -514,10 +514,12 @@ def delta_scan(proj: torch.Tensor, col_r: int, col_k: int, col_v: int, col_a: in
           _i(heads), _i(d), _i(dv), _stream(y))
 
 
-def delta_chunk_floats(n_blocks: int, heads: int, d: int, dv: int) -> int:
+def delta_chunk_floats(n_blocks: int, heads: int, d: int, dv: int, dtype: torch.dtype) -> int:
     """32-bit elements of scratch that so many chunks of 16 tokens need (the layout is delta.cu's)."""
     rows = 64 if d <= 64 else 128 if d <= 128 else 256
     cols = -(-dv // 16) * 16
+    if dtype == torch.bfloat16:
+        return n_blocks * heads * (97 * rows + 40 * cols)
     return n_blocks * heads * (4 * DELTA_CHUNK * rows + rows + 3 * DELTA_CHUNK * cols)
 
 

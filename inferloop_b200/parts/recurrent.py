@@ -263,7 +263,7 @@ class GeneralDelta(Mixer):
     def scratch_bytes(self, tokens: int) -> int:
         size = torch.empty((), dtype=self.ctx.dtype).element_size()
         wide = -(-self.rank // 8) * 8
-        chunks = ops.delta_chunk_floats(-(-tokens // ops.DELTA_CHUNK) + 1, self.heads, self.d, self.dv) * 4
+        chunks = ops.delta_chunk_floats(-(-tokens // ops.DELTA_CHUNK) + 1, self.heads, self.d, self.dv, self.ctx.dtype) * 4
         return tokens * ((self.col_low + 2 * wide + self.inner_v) * size + (self.inner_k + self.inner_v) * 4) + chunks
 
     def forward(self, x: torch.Tensor, residual: torch.Tensor, step, cache) -> None:
