@@ -623,13 +623,20 @@ delta_chunks_kernel(const DeltaParams p, const float* __restrict__ scratch) {
   }
 }
 
+// 16 bytes from global memory, requested where it is written: the request is not moved down to the first use.
+__device__ __forceinline__ uint4 load_here(const uint4* p) {
+  uint4 v;
+  asm volatile("ld.global.v4.u32 {%0, %1, %2, %3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
+  return v;
+}
+
 // The same walk on the tensor cores (mma.sync m16n8k16, 32-bit accumulation), for projections stored in bfloat16: every 32-bit
 // operand is three exact bfloat16 pieces, and of the nine products of two such operands the six that reach 32-bit precision
 // are added, smallest first.  A warp owns 16 rows of the state and the block's 16 columns, transposed in the layout of an
 // accumulator, which is the layout of the operand that the two thin products read; the sums over the warps meet in shared
 // memory.  What a chunk adds to the state is formed apart and joins it with one rounding.
 template <int KP>
-__global__ void __launch_bounds__(KP * 2)
+__global__ void __launch_bounds__(KP * 2, 1)
 delta_chunks_mma_kernel(const DeltaParams p, const float* __restrict__ scratch) {
   ilb::pdl_launch_dependents();
   ilb::pdl_wait();
@@ -656,16 +663,16 @@ delta_chunks_mma_kernel(const DeltaParams p, const float* __restrict__ scratch) 
   auto load_a = [&](const float* at) {
     const uint4* f = reinterpret_cast<const uint4*>(at) + (size_t)warp * 6 * 32 + lane;
 #pragma unroll
-    for (int i = 0; i < 6; ++i) A[i] = __ldg(f + 32 * i);
+    for (int i = 0; i < 6; ++i) A[i] = load_here(f + 32 * i);
   };
   auto load_b = [&](const float* at) {
     const uint4* f = reinterpret_cast<const uint4*>(at) + (size_t)(kWarps * 6 + warp * 6) * 32 + lane;
 #pragma unroll
-    for (int i = 0; i < 6; ++i) B[i] = __ldg(f + 32 * i);
+    for (int i = 0; i < 6; ++i) B[i] = load_here(f + 32 * i);
     const float* d = at + kWarps * 12 * kFragFloats;
     D[0] = *reinterpret_cast<const float2*>(d + warp * 16 + 2 * t4);
     D[1] = *reinterpret_cast<const float2*>(d + warp * 16 + 8 + 2 * t4);
-    V = __ldg(reinterpret_cast<const uint4*>(d + KP + 2 * kChunk * DP) + cb * 32 + lane);
+    V = load_here(reinterpret_cast<const uint4*>(d + KP + 2 * kChunk * DP) + cb * 32 + lane);
   };
   // this thread's elements of U and Y: pairs of columns, dealt out by number
   constexpr int kAdd = (2 * kChunk * 8 + KP * 2 - 1) / (KP * 2);
@@ -678,21 +685,9 @@ delta_chunks_mma_kernel(const DeltaParams p, const float* __restrict__ scratch) 
       if (e < 2 * kChunk * 8) add[i] = *reinterpret_cast<const float2*>(uy + (size_t)(e >> 3) * DP + (e & 7) * 2);
     }
   };
-  // The chunks two and three ahead are asked into L2, each block of a head its share of the lines.
-  const int lines = (int)((chunk_floats_mma(KP, DP) * 4 + 127) / 128), share = (lines + (int)gridDim.y - 1) / (int)gridDim.y;
-  auto ahead = [&](int ci) {
-    if (ci >= n_chunks) return;
-    const char* at = reinterpret_cast<const char*>(scratch + (size_t)first * per + (size_t)ci * per + (size_t)h * chunk_floats_mma(KP, DP));
-    for (int i = tid; i < share; i += KP * 2) {
-      const int line = cb * share + i;
-      if (line < lines) asm volatile("prefetch.global.L2 [%0];" ::"l"(at + (size_t)line * 128));
-    }
-  };
   load_a(src);
   load_b(src);
   load_uy(src);
-  ahead(1);
-  ahead(2);
   // S[j][0, 1]: rows 16 warp + 8 j + 2 t4 (+ 1), column g; [2, 3]: column g + 8
   float S[2][4];
 #pragma unroll
@@ -733,7 +728,6 @@ delta_chunks_mma_kernel(const DeltaParams p, const float* __restrict__ scratch) 
     }
     const bool more = ci + 1 < n_chunks;
     if (more) load_a(src + per);
-    ahead(ci + 3);
     __syncthreads();
 #pragma unroll
     for (int i = 0; i < kAdd; ++i) {
