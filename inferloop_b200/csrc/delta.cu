@@ -247,11 +247,11 @@ __host__ __device__ __forceinline__ long long chunk_floats(int KP, int DP) { ret
 // lanes of a warp hold the operands of mma.m16n8k16, 16 bytes a lane:
 //   per 16 rows of the state: W, X (A operands, 16 tokens x 16 rows), pieces hi mid lo each       6 x 512 bytes
 //   then per 16 rows:         D m, - D q (B operands, 16 tokens x 2 x 8 rows), hi mid lo each      6 x 512 bytes
-//   then D [KP], U, Y [16][DP] in 32-bit, and per 16 columns V transposed (A operand, 16 columns x 16 tokens; exact)   512 bytes
+//   then D [KP]; then per 16 columns: U, Y [16][16] in 32-bit, and V transposed (A operand, 16 columns x 16 tokens; exact), 512 bytes
 constexpr int kFragFloats = 128;                         // 512 bytes
-__host__ __device__ __forceinline__ long long chunk_floats_mma(int KP, int DP) {
-  return (long long)(KP / 16) * 12 * kFragFloats + KP + (long long)2 * kChunk * DP + (long long)(DP / 16) * kFragFloats;
-}
+constexpr int kColFloats = 2 * kChunk * kCols + kFragFloats;
+__host__ __device__ constexpr int row_floats_mma(int KP) { return (KP / 16) * 12 * kFragFloats + KP; }
+__host__ __device__ __forceinline__ long long chunk_floats_mma(int KP, int DP) { return row_floats_mma(KP) + (long long)(DP / kCols) * kColFloats; }
 __host__ __device__ __forceinline__ int padded_cols(int dv) { return (dv + kCols - 1) / kCols * kCols; }
 static inline int padded_rows(int d) { return d <= 64 ? 64 : (d <= 128 ? 128 : 256); }
 
@@ -438,8 +438,13 @@ delta_prep_kernel(const DeltaParams p, float* __restrict__ scratch, int KP) {
       unpack2(ac[t], zero, c);
       unpack2(be[t], zero, e);
       unpack2(sy, u[t], y);
-      outU[t * DP + c0] = u[t];
-      outY[t * DP + c0] = fmaf(c, u[t], fmaf(e, v[t], y));
+      y = fmaf(c, u[t], fmaf(e, v[t], y));
+      if constexpr (FAST) {
+        float* uy = outU + (c0 / kCols) * kColFloats + t * kCols + c0 % kCols;
+        uy[0] = u[t]; uy[kChunk * kCols] = y;
+      } else {
+        outU[t * DP + c0] = u[t]; outY[t * DP + c0] = y;
+      }
     }
   }
   if constexpr (FAST) {
@@ -474,11 +479,10 @@ delta_prep_kernel(const DeltaParams p, float* __restrict__ scratch, int KP) {
         emit((size_t)(slices * 6 + (ks * 2 + what - 2) * 3) * 32 + ln, x);
       }
     }
-    uint4* vfrag = reinterpret_cast<uint4*>(outY + kChunk * DP);
     for (int i = tid; i < DP / 16 * 32; i += kPrepThreads) {
       const int ln = i & 31, g = ln >> 2, t4 = ln & 3;
       const float* m = V + (i >> 5) * 16 + g;
-      vfrag[i] = make_uint4(pack_bf16(m[2 * t4 * DP], m[(2 * t4 + 1) * DP]), pack_bf16(m[2 * t4 * DP + 8], m[(2 * t4 + 1) * DP + 8]),
+      reinterpret_cast<uint4*>(outU + (i >> 5) * kColFloats + 2 * kChunk * kCols)[ln] = make_uint4(pack_bf16(m[2 * t4 * DP], m[(2 * t4 + 1) * DP]), pack_bf16(m[2 * t4 * DP + 8], m[(2 * t4 + 1) * DP + 8]),
                             pack_bf16(m[(2 * t4 + 8) * DP], m[(2 * t4 + 9) * DP]), pack_bf16(m[(2 * t4 + 8) * DP + 8], m[(2 * t4 + 9) * DP + 8]));
     }
   }
@@ -630,21 +634,45 @@ __device__ __forceinline__ uint4 load_here(const uint4* p) {
   return v;
 }
 
+// `bytes` (a multiple of 16, both addresses on 16-byte boundaries) from global to this block's shared memory, counted on `bar`.
+__device__ __forceinline__ void bulk_load(uint32_t dst, const float* src, uint32_t bytes, uint32_t bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];"
+               ::"r"(dst), "l"(src), "r"(bytes), "r"(bar) : "memory");
+}
+
 // The same walk on the tensor cores (mma.sync m16n8k16, 32-bit accumulation), for projections stored in bfloat16: every 32-bit
 // operand is three exact bfloat16 pieces, and of the nine products of two such operands the six that reach 32-bit precision
 // are added, smallest first.  A warp owns 16 rows of the state and the block's 16 columns, transposed in the layout of an
 // accumulator, which is the layout of the operand that the two thin products read; the sums over the warps meet in shared
 // memory.  What a chunk adds to the state is formed apart and joins it with one rounding.
-template <int KP>
+// RING > 0: the chunks' operands come through a ring of that many stages in shared memory, two bulk copies a chunk (the rows'
+// part, which all blocks of the head read, and the block's columns' part); 0: straight into registers, a chunk ahead.
+// Waits are bounded; on expiry a flag is raised and the walk goes on without waiting.
+template <int KP, int RING>
+struct ChunksMma {
+  static constexpr int kWarps = KP / 16, kLd = 20, kZ = kCols + 1;      // kLd: floats from one row of a warp's sums to the next
+  static constexpr int kStage = row_floats_mma(KP) + kColFloats;        // floats
+  static constexpr size_t kSmem = sizeof(float) * ((size_t)RING * kStage + (size_t)kWarps * 2 * kChunk * kLd + kChunk * kZ) + 8 * (RING + 2);
+};
+
+template <int KP, int RING>
 __global__ void __launch_bounds__(KP * 2, 1)
-delta_chunks_mma_kernel(const DeltaParams p, const float* __restrict__ scratch) {
+delta_chunks_mma_kernel(const DeltaParams p, const float* __restrict__ scratch, int* error_flag) {
   ilb::pdl_launch_dependents();
+  using C = ChunksMma<KP, RING>;
+  constexpr int kWarps = C::kWarps, kLd = C::kLd, kZ = C::kZ, kRow = row_floats_mma(KP);
+  extern __shared__ __align__(128) float sm[];
+  float* red = sm + RING * C::kStage;                    // [warps][32][kLd]
+  const uint32_t bar0 = smem_u32(red + kWarps * 2 * kChunk * kLd);      // one mbarrier a stage
+  float* zs = red + kWarps * 2 * kChunk * kLd + 2 * (RING + 1);         // [16][kZ]
+  if (RING > 0) {
+    if (threadIdx.x == 0) {
+      for (int i = 0; i < RING; ++i) mbar_init(bar0 + 8 * i, 1);
+      asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    }
+    __syncthreads();
+  }
   ilb::pdl_wait();
-  constexpr int kWarps = KP / 16, kLd = 24;              // kLd: floats from one row of a warp's sums to the next
-  extern __shared__ __align__(16) float sm[];
-  float* red = sm;                                       // [warps][32][kLd]
-  float* zs = red + kWarps * 2 * kChunk * kLd;           // [16][kCols + 1]
-  constexpr int kZ = kCols + 1;
   const int h = blockIdx.x, cb = blockIdx.y, c0 = cb * kCols, seq = blockIdx.z;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
   const int DP = padded_cols(p.dv);
@@ -656,38 +684,52 @@ delta_chunks_mma_kernel(const DeltaParams p, const float* __restrict__ scratch) 
   float* own = slot >= 0 ? p.state + ((size_t)slot * p.heads + h) * p.d * p.dv : nullptr;
   const int inner_v = p.heads * p.dv;
   const size_t per = (size_t)p.heads * chunk_floats_mma(KP, DP);        // from one chunk to the next
-  const float* src = scratch + ((size_t)first * p.heads + h) * chunk_floats_mma(KP, DP);
+  const float* src0 = scratch + ((size_t)first * p.heads + h) * chunk_floats_mma(KP, DP);
+
+  // One thread asks for a chunk's operands; a stage is asked for again once every thread is past the barrier that follows its
+  // last read.
+  bool ok = true;
+  auto ask = [&](int ci) {
+    const uint32_t dst = smem_u32(sm) + (uint32_t)(ci % (RING > 0 ? RING : 1)) * C::kStage * 4u, bar = bar0 + 8 * (ci % (RING > 0 ? RING : 1));
+    const float* at = src0 + (size_t)ci * per;
+    mbar_expect_tx(bar, C::kStage * 4u);
+    bulk_load(dst, at, kRow * 4u, bar);
+    bulk_load(dst + kRow * 4u, at + kRow + cb * kColFloats, kColFloats * 4u, bar);
+  };
+  if (RING > 0 && tid == 0)
+    for (int i = 0; i < RING && i < n_chunks; ++i) ask(i);
 
   uint4 A[6], B[6], V;                                   // W hi mid lo, X hi mid lo;  D m hi mid lo, - D q hi mid lo
   float2 D[2];
-  auto load_a = [&](const float* at) {
-    const uint4* f = reinterpret_cast<const uint4*>(at) + (size_t)warp * 6 * 32 + lane;
+  constexpr int kAdd = (2 * kChunk * 8 + KP * 2 - 1) / (KP * 2);
+  float2 add[kAdd];                                      // this thread's elements of U and Y: pairs of columns, dealt out by number
+  auto take = [](const uint4* at) { return RING > 0 ? *at : load_here(at); };
+  auto load_a = [&](const float* rows) {
+    const uint4* f = reinterpret_cast<const uint4*>(rows) + (size_t)warp * 6 * 32 + lane;
 #pragma unroll
-    for (int i = 0; i < 6; ++i) A[i] = load_here(f + 32 * i);
+    for (int i = 0; i < 6; ++i) A[i] = take(f + 32 * i);
   };
-  auto load_b = [&](const float* at) {
-    const uint4* f = reinterpret_cast<const uint4*>(at) + (size_t)(kWarps * 6 + warp * 6) * 32 + lane;
+  auto load_b = [&](const float* rows, const float* cols) {
+    const uint4* f = reinterpret_cast<const uint4*>(rows) + (size_t)(kWarps * 6 + warp * 6) * 32 + lane;
 #pragma unroll
-    for (int i = 0; i < 6; ++i) B[i] = load_here(f + 32 * i);
-    const float* d = at + kWarps * 12 * kFragFloats;
+    for (int i = 0; i < 6; ++i) B[i] = take(f + 32 * i);
+    const float* d = rows + kWarps * 12 * kFragFloats;
     D[0] = *reinterpret_cast<const float2*>(d + warp * 16 + 2 * t4);
     D[1] = *reinterpret_cast<const float2*>(d + warp * 16 + 8 + 2 * t4);
-    V = load_here(reinterpret_cast<const uint4*>(d + KP + 2 * kChunk * DP) + cb * 32 + lane);
+    V = take(reinterpret_cast<const uint4*>(cols + 2 * kChunk * kCols) + lane);
   };
-  // this thread's elements of U and Y: pairs of columns, dealt out by number
-  constexpr int kAdd = (2 * kChunk * 8 + KP * 2 - 1) / (KP * 2);
-  float2 add[kAdd];
-  auto load_uy = [&](const float* at) {
-    const float* uy = at + kWarps * 12 * kFragFloats + KP + c0;
+  auto load_uy = [&](const float* cols) {
 #pragma unroll
     for (int i = 0; i < kAdd; ++i) {
       const int e = tid + i * KP * 2;
-      if (e < 2 * kChunk * 8) add[i] = *reinterpret_cast<const float2*>(uy + (size_t)(e >> 3) * DP + (e & 7) * 2);
+      if (e < 2 * kChunk * 8) add[i] = *reinterpret_cast<const float2*>(cols + 2 * e);
     }
   };
-  load_a(src);
-  load_b(src);
-  load_uy(src);
+  if (RING == 0) {
+    load_a(src0);
+    load_b(src0, src0 + kRow + cb * kColFloats);
+    load_uy(src0 + kRow + cb * kColFloats);
+  }
   // S[j][0, 1]: rows 16 warp + 8 j + 2 t4 (+ 1), column g; [2, 3]: column g + 8
   float S[2][4];
 #pragma unroll
@@ -701,7 +743,17 @@ delta_chunks_mma_kernel(const DeltaParams p, const float* __restrict__ scratch) 
     const uint32_t aa[4] = {a.x, a.y, a.z, a.w};
     mma_16816(c, aa, b0, b1);
   };
-  for (int ci = 0; ci < n_chunks; ++ci, src += per) {
+  for (int ci = 0; ci < n_chunks; ++ci) {
+    const float* stage = sm + (ci % (RING > 0 ? RING : 1)) * C::kStage;      // (RING > 0)
+    const float* next = src0 + (size_t)(ci + 1) * per;                     // (RING == 0)
+    const bool more = ci + 1 < n_chunks;
+    if (RING > 0) {
+      if (ok && !mbar_wait(bar0 + 8 * (ci % (RING > 0 ? RING : 1)), (ci / (RING > 0 ? RING : 1)) & 1)) {
+        ok = false;
+        if (error_flag != nullptr) *error_flag = 1;
+      }
+      load_a(stage);
+    }
     {
       uint32_t b[3][2][2];                               // pieces of the state: [piece][columns 8 jj + g][rows 2 t4, 2 t4 + 8]
 #pragma unroll
@@ -726,9 +778,10 @@ delta_chunks_mma_kernel(const DeltaParams p, const float* __restrict__ scratch) 
           *reinterpret_cast<float2*>(r + 8 * kLd) = make_float2(c[2], c[3]);
         }
     }
-    const bool more = ci + 1 < n_chunks;
-    if (more) load_a(src + per);
+    if (RING > 0) load_uy(stage + kRow);
+    else if (more) load_a(next);
     __syncthreads();
+    if (RING > 0 && tid == 0 && ci > 0 && ci - 1 + RING < n_chunks) ask(ci - 1 + RING);      // (everyone is done with the chunk before)
 #pragma unroll
     for (int i = 0; i < kAdd; ++i) {
       const int e = tid + i * KP * 2;
@@ -752,7 +805,8 @@ delta_chunks_mma_kernel(const DeltaParams p, const float* __restrict__ scratch) 
         }
       }
     }
-    if (more) load_uy(src + per);
+    if (RING > 0) load_b(stage, stage + kRow);
+    else if (more) load_uy(next + kRow + cb * kColFloats);
     __syncthreads();
     {
       uint4 z[3];                                        // pieces of Z transposed: columns g, g + 8, tokens 2 t4 (+ 1), + 8
@@ -781,8 +835,10 @@ delta_chunks_mma_kernel(const DeltaParams p, const float* __restrict__ scratch) 
         S[j][2] = fmaf(D[j].x, S[j][2], c[2]); S[j][3] = fmaf(D[j].y, S[j][3], c[3]);
       }
     }
-    if (more) load_b(src + per);
+    if (RING == 0 && more) load_b(next, next + kRow + cb * kColFloats);
   }
+  if (RING > 0 && !ok)                                   // copies that may still be on their way land before the block ends
+    for (int i = 0; i < (RING > 0 ? RING : 1); ++i) mbar_wait(bar0 + 8 * i, 0);
   if (own != nullptr) {
 #pragma unroll
     for (int j = 0; j < 2; ++j)
@@ -794,16 +850,17 @@ delta_chunks_mma_kernel(const DeltaParams p, const float* __restrict__ scratch) 
   }
 }
 
-template <int KP>
-static int chunks_mma_launch(const DeltaParams& p, const float* scratch, cudaStream_t stream) {
-  const size_t smem = sizeof(float) * ((size_t)KP / 16 * 2 * kChunk * 24 + kChunk * (kCols + 1));
+template <int KP, int RING>
+static int chunks_mma_launch(const DeltaParams& p, const float* scratch, int* error_flag, cudaStream_t stream) {
+  constexpr size_t smem = ChunksMma<KP, RING>::kSmem;
+  static_assert(smem <= 227 * 1024, "the ring does not fit shared memory");
   static OncePerDevice once;
   if (smem > 48 * 1024 && once.first() &&
-      cudaFuncSetAttribute(delta_chunks_mma_kernel<KP>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
+      cudaFuncSetAttribute(delta_chunks_mma_kernel<KP, RING>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) {
     once.forget();
     return fail("delta_chunks: cannot reserve %zu bytes of shared memory", smem);
   }
-  ilb::launch(delta_chunks_mma_kernel<KP>, dim3(p.heads, padded_cols(p.dv) / kCols, p.n_seqs), dim3(KP * 2), smem, stream, p, scratch);
+  ilb::launch(delta_chunks_mma_kernel<KP, RING>, dim3(p.heads, padded_cols(p.dv) / kCols, p.n_seqs), dim3(KP * 2), smem, stream, p, scratch, error_flag);
   return check_launch("delta_chunks");
 }
 
@@ -844,7 +901,7 @@ static int prep_launch(const DeltaParams& p, float* scratch, int n_blocks, cudaS
 ILB_EXPORT int ilb_delta_chunks(const void* proj, int dtype, int ld, int col_r, int col_k, int col_v, int col_a, const float* low,
                                 const float* w0, const float* ab, float log_decay, float unit_eps, float* state, float* y,
                                 const int* cu_q, const int* slots, int n_seqs, int heads, int d, int dv, float* scratch,
-                                long long scratch_floats, int n_blocks, cudaStream_t stream) {
+                                long long scratch_floats, int n_blocks, int* error_flag, cudaStream_t stream) {
   const DeltaParams p{proj, ld, col_r, col_k, col_v, col_a, low, w0, ab, state, y, cu_q, slots, n_seqs, heads, d, dv, log_decay, unit_eps};
   if (int rc = check_sizes(p, dtype)) return rc;
   ILB_REQUIRE(log_decay >= 0.f && log_decay * kChunk <= 40.f, "delta_chunks: a decay of exp(-%f) a token leaves a chunk's range", (double)log_decay);
@@ -855,8 +912,8 @@ ILB_EXPORT int ilb_delta_chunks(const void* proj, int dtype, int ld, int col_r, 
   if (int rc = dtype == kF32 ? prep_launch<float>(p, scratch, n_blocks, stream) : prep_launch<__nv_bfloat16>(p, scratch, n_blocks, stream)) return rc;
   const int rows = padded_rows(d);
   if (dtype == kBF16)
-    return rows == 64 ? chunks_mma_launch<64>(p, scratch, stream) : rows == 128 ? chunks_mma_launch<128>(p, scratch, stream)
-                                                                                : chunks_mma_launch<256>(p, scratch, stream);
+    return rows == 64 ? chunks_mma_launch<64, 4>(p, scratch, error_flag, stream)
+                      : rows == 128 ? chunks_mma_launch<128, 4>(p, scratch, error_flag, stream) : chunks_mma_launch<256, 0>(p, scratch, error_flag, stream);
   return rows == 64 ? chunks_launch<4>(p, scratch, stream) : rows == 128 ? chunks_launch<8>(p, scratch, stream) : chunks_launch<16>(p, scratch, stream);
 }
 

@@ -507,7 +507,8 @@ def delta_scan(proj: torch.Tensor, col_r: int, col_k: int, col_v: int, col_a: in
         scratch = workspace.buffer("delta.chunks", (delta_chunk_floats(n_blocks, heads, d, dv, proj.dtype),), torch.float32)
         _call("delta", "ilb_delta_chunks", _ptr(proj), _i(_code(proj)), _i(proj.stride(0)), _i(col_r), _i(col_k), _i(col_v), _i(col_a), _ptr(low),
               _ptr(w0), _ptr(ab), _f(log_decay), _f(unit_eps), _ptr(state), _ptr(y), _ptr(step.cu_q), _ptr(step.slots), _i(step.n_seqs),
-              _i(heads), _i(d), _i(dv), _ptr(scratch), ctypes.c_longlong(scratch.numel()), _i(n_blocks), _stream(y))
+              _i(heads), _i(d), _i(dv), _ptr(scratch), ctypes.c_longlong(scratch.numel()), _i(n_blocks),
+              _ptr(_tc_state(y.device).error if proj.dtype == torch.bfloat16 else None), _stream(y))
         return
     _call("delta", "ilb_delta_scan", _ptr(proj), _i(_code(proj)), _i(proj.stride(0)), _i(col_r), _i(col_k), _i(col_v), _i(col_a), _ptr(low),
           _ptr(w0), _ptr(ab), _f(log_decay), _f(unit_eps), _ptr(state), _ptr(y), _ptr(step.cu_q), _ptr(step.slots), _i(step.n_seqs),
@@ -519,7 +520,7 @@ def delta_chunk_floats(n_blocks: int, heads: int, d: int, dv: int, dtype: torch.
     rows = 64 if d <= 64 else 128 if d <= 128 else 256
     cols = -(-dv // 16) * 16
     if dtype == torch.bfloat16:
-        return n_blocks * heads * (97 * rows + 40 * cols)
+        return n_blocks * heads * (97 * rows + 40 * cols)      # (96 + 1 a row, 640 for 16 columns)
     return n_blocks * heads * (4 * DELTA_CHUNK * rows + rows + 3 * DELTA_CHUNK * cols)
 
 
