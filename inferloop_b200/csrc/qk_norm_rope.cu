@@ -420,6 +420,21 @@ template <> struct RowUnit<__nv_bfloat16, 8> {
   __device__ static __forceinline__ void store(__nv_bfloat16* p, const float* x) { *reinterpret_cast<uint4*>(p) = pack8(x); }
 };
 
+// N consecutive 32-bit numbers; in fours (from a 16-byte boundary) where N is a multiple of eight.
+template <int N>
+__device__ __forceinline__ void load_f32(const float* p, float* x) {
+  if constexpr (N % 8 == 0) {
+#pragma unroll
+    for (int i = 0; i < N / 4; ++i) {
+      const float4 v = __ldg(reinterpret_cast<const float4*>(p) + i);
+      x[4 * i] = v.x; x[4 * i + 1] = v.y; x[4 * i + 2] = v.z; x[4 * i + 3] = v.w;
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < N; ++i) x[i] = p[i];
+  }
+}
+
 struct RowsParams {
   const float* q_weight; const float* k_weight;
   const float2* rope; const float2* v_rope;
@@ -442,16 +457,37 @@ rows_norm_rope_kernel(const TQ* __restrict__ qkv, TQ* __restrict__ q_out, TC* k_
   const TQ* row = qkv + (size_t)t * p.qkv_stride;
   const int nqd = p.nq * p.d, nkd = p.nkv * p.d, nvd = p.nkv * p.dv;
   float x[VEC], y[VEC];
-  float sums[2] = {0.f, 0.f};
-  for (int e = threadIdx.x * VEC; e < nqd + nkd; e += kRowsThreads * VEC) {
-    RowUnit<TQ, VEC>::load(row + e, x);
-    float ss = 0.f;
+  float sum_q = 0.f, sum_k = 0.f;
+  constexpr int kFlight = 4;                               // units whose loads are in flight together
+  for (int e0 = threadIdx.x * VEC; e0 < nqd + nkd; e0 += kFlight * kRowsThreads * VEC) {
+    float v[kFlight][VEC];
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) ss = fmaf(x[i], x[i], ss);
-    sums[e < nqd ? 0 : 1] += ss;
+    for (int f = 0; f < kFlight; ++f) {
+      const int e = e0 + f * kRowsThreads * VEC;
+      if (e < nqd + nkd) RowUnit<TQ, VEC>::load(row + e, v[f]);
+      else {
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) v[f][i] = 0.f;
+      }
+    }
+#pragma unroll
+    for (int f = 0; f < kFlight; ++f) {
+      float ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) ss = fmaf(v[f][i], v[f][i], ss);
+      if (e0 + f * kRowsThreads * VEC < nqd) sum_q += ss; else sum_k += ss;
+    }
   }
-  const float inv_q = 1.0f / sqrtf(block_sum(sums[0], scratch) / (float)nqd + p.eps);
-  const float inv_k = 1.0f / sqrtf(block_sum(sums[1], scratch) / (float)nkd + p.eps);
+  // both sums over the block in one exchange
+  sum_q = warp_sum(sum_q);
+  sum_k = warp_sum(sum_k);
+  if ((threadIdx.x & 31) == 0) { scratch[threadIdx.x >> 5] = sum_q; scratch[16 + (threadIdx.x >> 5)] = sum_k; }
+  __syncthreads();
+  sum_q = 0.f; sum_k = 0.f;
+#pragma unroll
+  for (int w = 0; w < kRowsThreads / 32; ++w) { sum_q += scratch[w]; sum_k += scratch[16 + w]; }
+  const float inv_q = 1.0f / sqrtf(sum_q / (float)nqd + p.eps);
+  const float inv_k = 1.0f / sqrtf(sum_k / (float)nkd + p.eps);
   // where this token's key and value go
   long long place = -1;
   if (k_cache != nullptr) {
@@ -492,18 +528,23 @@ rows_norm_rope_kernel(const TQ* __restrict__ qkv, TQ* __restrict__ q_out, TC* k_
     if (kind != 2) {
       const float inv = kind == 0 ? inv_q : inv_k;
       const float* w = (kind == 0 ? p.q_weight : p.k_weight) + e;
+      float wv[VEC];
+      load_f32<VEC>(w, wv);
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) {
-        x[i] = x[i] * inv * w[i];
-        if (pair) y[i] = y[i] * inv * w[half + i];
+      for (int i = 0; i < VEC; ++i) x[i] = x[i] * inv * wv[i];
+      if (pair) {
+        load_f32<VEC>(w + half, wv);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) y[i] = y[i] * inv * wv[i];
       }
     }
     if (pair) {
-      const float2* cs = table + (size_t)t * half + c;
+      float cs[2 * VEC];
+      load_f32<2 * VEC>(reinterpret_cast<const float*>(table + (size_t)t * half + c), cs);
 #pragma unroll
       for (int i = 0; i < VEC; ++i) {
         const float a = x[i], b = y[i];
-        const float2 w = cs[i];
+        const float2 w = make_float2(cs[2 * i], cs[2 * i + 1]);
         x[i] = __fsub_rn(__fmul_rn(a, w.x), __fmul_rn(b, w.y));
         y[i] = __fadd_rn(__fmul_rn(a, w.y), __fmul_rn(b, w.x));
       }
@@ -576,7 +617,7 @@ ILB_EXPORT int ilb_rows_norm_rope_cache(
                      page_size, num_pages, nq, nkv, d, dv, rope != nullptr ? rotary_dim : 0, qkv_stride, q_out_stride, eps, p_table, p_num_pages, pool};
   auto a16 = [](const void* x) { return (uintptr_t)x % 16 == 0; };
   const bool vec = dtype == kBF16 && d % 8 == 0 && dv % 8 == 0 && (rope == nullptr || rotary_dim % 16 == 0) && (v_rope == nullptr || dv % 16 == 0) &&
-                   qkv_stride % 8 == 0 && q_out_stride % 8 == 0 && a16(qkv) && a16(q_out) && a16(k_cache) && a16(v_cache) && a16(pk_cache) && a16(pv_cache);
+                   qkv_stride % 8 == 0 && q_out_stride % 8 == 0 && a16(qkv) && a16(q_out) && a16(k_cache) && a16(v_cache) && a16(pk_cache) && a16(pv_cache) && a16(q_weight) && a16(k_weight) && a16(rope) && a16(v_rope);
   const int units = ((nq + nkv) * d + nkv * dv) / (vec ? 8 : 1);
   int ny = 1;
   while (n_tokens * ny < 296 && ny * kRowsThreads < units) ++ny;
