@@ -3,7 +3,8 @@
 
     python bench.py [--gpus 1] [--steps K] [--warmup W] [--batch 8] [--impl ours|reference]
                     [--config 8b|14b-mixed|32b-long] [--breakdown] [--kernels [attention|products]] [--further]
-                    [--sufolix [dense|moe]] [--mamevik [latent|ssd|mixed]]
+                    [--sufolix [dense|moe]] [--mamevik [latent|ssd|mixed]] [--dalavik [latent|heads|mixed]]
+                    [--zebivik [parallel|rglru|mixed]] [--sapanex [attention|delta|mixed]]
 
 One JSON line on stdout.  The default (`--config 8b`) is the headline: Qwen3-8B layer sizes,
 36 layers, batch 8, 1,024-token prompts; a "step" is one decode step of the whole batch.
@@ -34,6 +35,7 @@ decode at --batch, one 2,048-token prompt, and the per-op-class device time of b
 `--mamevik` measures the Mamevik decoder (attention over a cached latent with a sink, state-space recurrences, a looped span
 of layers, clamped gated experts) the same way, in three arrangements of its layers, beside a Sufolix model with routed
 experts of the same width, layers and experts.
+`--dalavik`, `--zebivik` and `--sapanex` measure those decoders the same way, each beside the closest models of equal size.
 Peaks come from MEASURED_PEAKS.json beside this file when present, else the fallback
 figures 6.65 TB/s and 1.59 PFLOP/s.  Weights (15 GB and more) exceed L2 (126 MB), so every
 step reads them from HBM: no L2 flush is needed between timed steps.
