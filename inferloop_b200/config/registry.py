@@ -104,12 +104,14 @@ def default_registry() -> ArchitectureRegistry:
         from ..models.dalavik import ARCHITECTURE as DALAVIK
         from ..models.zebivik import ARCHITECTURE as ZEBIVIK
         from ..models.sapanex import ARCHITECTURE as SAPANEX
+        from ..models.tamovik import ARCHITECTURE as TAMOVIK
         _DEFAULT.register(ARCHITECTURE)
         _DEFAULT.register(SUFOLIX)
         _DEFAULT.register(MAMEVIK)
         _DEFAULT.register(DALAVIK)
         _DEFAULT.register(ZEBIVIK)
         _DEFAULT.register(SAPANEX)
+        _DEFAULT.register(TAMOVIK)
     return _DEFAULT
 
 

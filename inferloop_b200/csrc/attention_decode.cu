@@ -544,7 +544,7 @@ decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__
   const int tok = p.cu_q[seq];
   if (p.cu_q[seq + 1] - tok != 1) return;                  // the whole cluster leaves together
   const int pos = p.positions[tok];
-  const int lo = (p.window > 0 && pos + 1 > p.window) ? pos + 1 - p.window : 0;
+  const int lo = first_key(pos, p.window);
   const int hi = pos + 1;
   const int kSplit = p.split;
   const int n_pooled = kPool ? lo / p.pool : 0, pool_tiles = (n_pooled + kKeys - 1) / kKeys;      // pooled rows this token sees, and their tiles
@@ -1102,7 +1102,7 @@ int decode_common(const void* q, const void* qkv, int qkv_stride, const float* q
                   float* scratch, long long scratch_floats, int* counters, long long n_counters, int* error_flag, cudaStream_t stream) {
   ILB_REQUIRE(ilb_attention_decode_tma_supported(nq, nkv, d, page_size),
               "attention decode: heads %d/%d, head size %d, page size %d are not built", nq, nkv, d, page_size);
-  ILB_REQUIRE(n_seqs > 0 && n_seqs <= 65535 && nkv <= 65535 && max_blocks > 0 && num_pages > 0 && window >= 0,
+  ILB_REQUIRE(n_seqs > 0 && n_seqs <= 65535 && nkv <= 65535 && max_blocks > 0 && num_pages > 0,
               "attention decode: bad sizes");
   ILB_REQUIRE(((uintptr_t)k_cache % 16 == 0) && ((uintptr_t)v_cache % 16 == 0), "attention decode: misaligned cache");
   if (qkv != nullptr)

@@ -256,14 +256,13 @@ prefill_kernel(const PrefillParams p) {
     tok[r] = tok0 + (live[r] ? tl : 0);
     head[r] = kvh * G + row % G;
     pos[r] = live[r] ? p.positions[tok[r]] : -1;
-    lo[r] = (live[r] && p.window > 0 && pos[r] + 1 > p.window) ? pos[r] + 1 - p.window : 0;
-    if (!live[r]) lo[r] = 0;
+    lo[r] = live[r] ? first_key(pos[r], p.window) : 0;
   }
   // keys the whole CTA needs: from the smallest window start to the largest position
   const int first_tl = (tile * 64) / G;
   const int last_tl = min(q_len - 1, (tile * 64 + 63) / G);
   const int pos_first = p.positions[tok0 + first_tl], pos_last = p.positions[tok0 + last_tl];
-  const int key_lo = (p.window > 0 && pos_first + 1 > p.window) ? pos_first + 1 - p.window : 0;
+  const int key_lo = first_key(pos_first, p.window);
   const int hi = pos_last + 1;
 
   uint32_t q[D / 16][4];
@@ -340,7 +339,7 @@ decode_kernel(const DecodeParams p) {
   const int tok = p.cu_q[seq];
   if (p.cu_q[seq + 1] - tok != 1) return;          // decode handles one token per sequence
   const int pos = p.positions[tok];
-  const int lo = (p.window > 0 && pos + 1 > p.window) ? pos + 1 - p.window : 0;
+  const int lo = first_key(pos, p.window);
   const int hi = pos + 1;
   const int c_lo = lo / p.chunk, c_hi = pos / p.chunk;
   // the grid's third index counts from the first chunk this token reads: with a window the records of a
@@ -562,7 +561,7 @@ ILB_EXPORT int ilb_attention_prefill(const void* q, void* out, const void* k_cac
   ILB_REQUIRE(ilb_attention_flash_supported(d), "attention prefill: head size %d is not built (32, 64, 96, 128 are)", d);
   ILB_REQUIRE(nq > 0 && nkv > 0 && nq % nkv == 0, "attention prefill: %d query heads are not a multiple of %d kv heads", nq, nkv);
   ILB_REQUIRE(n_seqs > 0 && n_tiles > 0 && nkv <= 65535, "attention prefill: bad grid");
-  ILB_REQUIRE(page_size > 0 && max_blocks > 0 && num_pages > 0 && window >= 0, "attention prefill: bad cache geometry");
+  ILB_REQUIRE(page_size > 0 && max_blocks > 0 && num_pages > 0, "attention prefill: bad cache geometry");
   ILB_REQUIRE(q_stride % 2 == 0 && out_stride % 2 == 0 && ((uintptr_t)q % 4 == 0) && ((uintptr_t)out % 4 == 0) &&
               ((uintptr_t)k_cache % 16 == 0) && ((uintptr_t)v_cache % 16 == 0), "attention prefill: misaligned operands");
   PrefillParams p{(const __nv_bfloat16*)q, (__nv_bfloat16*)out,
@@ -587,7 +586,7 @@ ILB_EXPORT int ilb_attention_decode(const void* q, void* out, const void* k_cach
   ILB_REQUIRE(nq > 0 && nkv > 0 && nq % nkv == 0, "attention decode: %d query heads are not a multiple of %d kv heads", nq, nkv);
   ILB_REQUIRE(n_seqs > 0 && n_seqs <= 65535 && max_chunks > 0 && max_chunks <= 65535, "attention decode: bad grid");
   ILB_REQUIRE(chunk > 0 && chunk % (kWarps * kTileKeys) == 0, "attention decode: chunk %d must be a multiple of %d", chunk, kWarps * kTileKeys);
-  ILB_REQUIRE(page_size > 0 && max_blocks > 0 && num_pages > 0 && window >= 0, "attention decode: bad cache geometry");
+  ILB_REQUIRE(page_size > 0 && max_blocks > 0 && num_pages > 0, "attention decode: bad cache geometry");
   const int G = nq / nkv, rows16 = (G + 15) / 16 * 16;
   ILB_REQUIRE((long long)n_seqs * nkv * max_chunks * G * (d + 2) <= scratch_floats, "attention decode: scratch too small");
   // Every key the block tables can name must fall into one of the chunks: a sequence longer
@@ -595,7 +594,7 @@ ILB_EXPORT int ilb_attention_decode(const void* q, void* out, const void* k_cach
   // would never be written.
   // (With a window a token reads at most (window - 1) / chunk + 2 chunks, and the grid counts from its first.)
   ILB_REQUIRE((long long)max_chunks * chunk >= (long long)max_blocks * page_size ||
-              (window > 0 && max_chunks >= (window - 1) / chunk + 2),
+              (window != 0 && max_chunks >= (abs(window) - 1) / chunk + 2),
               "attention decode: %d chunks of %d keys do not cover the %d x %d keys the block tables can name",
               max_chunks, chunk, max_blocks, page_size);
   // The last chunk's merge keeps one weight per (head of the group, chunk) in the shared

@@ -54,7 +54,7 @@ attention_mix_kernel(const TQ* __restrict__ q, TQ* __restrict__ out, const TC* _
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int per = nq / nkv;
   const int p = a.positions[t];
-  const int lo = (a.window > 0 && p + 1 > a.window) ? p + 1 - a.window : 0;
+  const int lo = first_key(p, a.window);
   const int* table = a.block_table + (size_t)a.seq_of_token[t] * a.max_blocks;
   float temp = 1.0f;
   if (a.temp_coef != 0.f) temp = 1.0f + a.temp_coef * logf((float)((p + 1) / a.temp_every) + 1.0f);
@@ -170,7 +170,7 @@ ILB_EXPORT int ilb_attention_mix(
   ILB_REQUIRE((long long)nq * dv <= (long long)kMixThreads * kMixAcc, "attention_mix: %d heads of %d values exceed %d outputs a token",
               nq, dv, kMixThreads * kMixAcc);
   ILB_REQUIRE(page_size > 0 && max_blocks > 0 && num_pages > 0, "attention_mix: bad cache geometry");
-  ILB_REQUIRE(window >= 0 && softcap >= 0.f, "attention_mix: negative window or cap");
+  ILB_REQUIRE(softcap >= 0.f, "attention_mix: negative cap");
   ILB_REQUIRE((r1 == nullptr) == (r2 == nullptr), "attention_mix: the distance term needs both of its vectors");
   ILB_REQUIRE(temp_coef == 0.f || temp_every > 0, "attention_mix: the query temperature needs a positive period");
   ILB_REQUIRE(q_stride >= nq * d && out_stride >= nq * dv, "attention_mix: strides too small");
@@ -288,7 +288,7 @@ attention_mix_tc_kernel(const MixTcParams a) {
   const int n_rows = min(kTcRows, a.cu_q[seq + 1] - t0);
   const int p0 = a.positions[t0];                 // the rows' positions are p0, p0 + 1, ...
   const int p_last = p0 + n_rows - 1;
-  int key_lo = (a.window > 0 && p0 + 1 > a.window) ? p0 + 1 - a.window : 0, key_hi = p_last + 1;
+  int key_lo = first_key(p0, a.window), key_hi = p_last + 1;
   const int chunk = a.per_token ? blockIdx.y : 0;
   if (a.per_token) {                              // few blocks with many keys: block (16 tokens, chunk of keys) leaves records
     key_lo = max(key_lo, chunk * a.split_chunk);
@@ -361,7 +361,7 @@ attention_mix_tc_kernel(const MixTcParams a) {
       bad = row < 0;
     }
     // a tile on which some (row, key) pair is not read: the diagonal's, a window's edge, a key without a page
-    const bool edge = __syncthreads_or(bad) != 0 || j0 + kTcKeys - 1 > p0 || (a.window > 0 && j0 <= p_last - a.window);
+    const bool edge = __syncthreads_or(bad) != 0 || j0 + kTcKeys - 1 > p0 || j0 < first_key(p_last, a.window);
     {
       for (int r = warp; r < G * kTcKeys; r += kTcWarps) {        // a warp a (kv head, key): its key row and its value row
         const int g = r / kTcKeys, jj = r % kTcKeys, row = row_s[jj];
@@ -442,7 +442,7 @@ attention_mix_tc_kernel(const MixTcParams a) {
           for (int e = 0; e < 4; ++e) {
             const int c = nt * 8 + 2 * tq + (e & 1), j = j0 + c;
             const int pr = (e < 2) ? pr0 : pr1;
-            const bool seen = j <= pr && pr <= p_last && row_s[c] >= 0 && (a.window == 0 || j > pr - a.window);
+            const bool seen = j <= pr && pr <= p_last && row_s[c] >= 0 && j >= first_key(pr, a.window);
             if (!seen) s[nt][e] = -INFINITY;
           }
       }
@@ -532,7 +532,7 @@ attention_mix_merge_kernel(const MixTcParams a) {
   const int t = a.per_token ? blockIdx.x : a.cu_q[blockIdx.x];       // the token, and whose records these are
   const int seq = a.per_token ? t : blockIdx.x;
   const int p = a.positions[t];
-  const int lo = (a.window > 0 && p + 1 > a.window) ? p + 1 - a.window : 0;
+  const int lo = first_key(p, a.window);
   const int c_lo = lo / a.split_chunk, c_hi = p / a.split_chunk;
   const int e = blockIdx.y * blockDim.x + threadIdx.x;            // a thread an output element
   if (e >= H * dv) return;
@@ -591,7 +591,7 @@ attention_mix_heads_kernel(const MixTcParams a) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gq = lane >> 2, tq = lane & 3;
   const int seq = blockIdx.x, chunk = blockIdx.y;
   const int t = a.cu_q[seq], p = a.positions[t];
-  int key_lo = (a.window > 0 && p + 1 > a.window) ? p + 1 - a.window : 0;
+  int key_lo = first_key(p, a.window);
   key_lo = max(key_lo, chunk * a.split_chunk);
   const int key_hi = min(p + 1, (chunk + 1) * a.split_chunk);
   if (key_lo >= key_hi) return;
@@ -814,7 +814,7 @@ ILB_EXPORT int ilb_attention_mix_tc(
     const float* r2, float softcap, float temp_coef, int temp_every, int split_chunk, int max_chunks, float* scratch,
     long long scratch_floats, int per_token, int n_tokens, cudaStream_t stream) {
   ILB_REQUIRE(ilb_attention_mix_tc_supported(nq, nkv, d, dv), "attention_mix_tc: %d / %d heads of %d / %d are not served", nq, nkv, d, dv);
-  ILB_REQUIRE(page_size > 0 && max_blocks > 0 && num_pages > 0 && window >= 0 && softcap >= 0.f, "attention_mix_tc: bad arguments");
+  ILB_REQUIRE(page_size > 0 && max_blocks > 0 && num_pages > 0 && softcap >= 0.f, "attention_mix_tc: bad arguments");
   ILB_REQUIRE((r1 == nullptr) == (r2 == nullptr), "attention_mix_tc: the distance term needs both of its vectors");
   ILB_REQUIRE(temp_coef == 0.f || temp_every > 0, "attention_mix_tc: the query temperature needs a positive period");
   ILB_REQUIRE(q_stride >= nq * d && out_stride >= nq * dv && q_stride % 8 == 0 && out_stride % 2 == 0 && ((uintptr_t)q % 16 == 0) &&

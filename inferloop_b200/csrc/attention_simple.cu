@@ -2,7 +2,8 @@
 //
 // One block per (token, query head).  The token at position p of sequence s reads the keys
 // of positions lo..p of that sequence from the cache (this step's own keys are already
-// there), lo = max(0, p - window + 1) with a window, else 0.  Scores, the running maximum,
+// there), lo = max(0, p - window + 1) with a window, the start of p's aligned chunk of -window
+// positions with a negative one, else 0.  Scores, the running maximum,
 // exponentials, sums and the weighted value sum are all 32-bit; the split of the keys over
 // the block's warps depends on lo and p alone, so the result at a position never depends
 // on what else is in the batch or on how the tokens were cut into steps.
@@ -26,7 +27,7 @@
 using namespace ilb;
 
 constexpr int kWarps = 4;
-constexpr int kMaxHeadDim = 512;
+constexpr int kMaxHeadDim = 640;
 
 template <typename TQ, typename TC>
 __global__ void __launch_bounds__(kWarps * 32)
@@ -48,7 +49,7 @@ paged_attention_simple_kernel(const TQ* __restrict__ q, TQ* __restrict__ out,
   const int kvh = h / (nq / nkv);
   const int p = positions[t];
   const int seq = seq_of_token[t];
-  const int lo = (window > 0 && p + 1 > window) ? p + 1 - window : 0;
+  const int lo = first_key(p, window);
   const int* table = block_table + (size_t)seq * max_blocks;
   const int* ptable = p_table + (size_t)seq * max_blocks;      // (not read without pooled rows)
   const int n_pooled = pool > 0 ? lo / pool : 0;
@@ -141,7 +142,6 @@ ILB_EXPORT int ilb_paged_attention_simple(
   ILB_REQUIRE(dv > 0 && d <= kMaxHeadDim && dv <= kMaxHeadDim, "attention: head size %d / %d exceeds %d", d, dv, kMaxHeadDim);
   ILB_REQUIRE(nq <= 65535, "attention: too many heads");
   ILB_REQUIRE(page_size > 0 && max_blocks > 0 && num_pages > 0, "attention: bad cache geometry");
-  ILB_REQUIRE(window >= 0, "attention: negative window");
   ILB_REQUIRE(pool == 0 || (pool > 0 && window > 0 && pk_cache != nullptr && pv_cache != nullptr && p_table != nullptr && p_num_pages > 0),
               "attention: pooled blocks need a window and pages of their own");
   ILB_REQUIRE(q_stride >= nq * d && out_stride >= nq * dv, "attention: strides too small");

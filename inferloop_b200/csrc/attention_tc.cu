@@ -229,7 +229,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
   const int t_last = min(q_len, t_first + tokens_per_cta) - 1;
   // positions are written by the step's staging copy, an earlier operation in the stream
   const int pos_first = p.positions[tok0 + t_first], pos_last = p.positions[tok0 + t_last];
-  const int key_lo = (p.window > 0 && pos_first + 1 > p.window) ? pos_first + 1 - p.window : 0;
+  const int key_lo = first_key(pos_first, p.window);
   const int first_tile = key_lo / kKeys;
   // pooled rows that the CTA's last row sees (earlier rows see no more), and their tiles: they come first
   int n_pooled = 0, pool_tiles = 0;
@@ -452,7 +452,7 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
     const bool live = row < tokens_per_block * G && tl < q_len;     // rows past the last whole token hold no query
     const int head = kvh * G + row % G;
     const int pos = live ? p.positions[tok0 + tl] : -1;
-    const int lo = (live && p.window > 0 && pos + 1 > p.window) ? pos + 1 - p.window : 0;
+    const int lo = live ? first_key(pos, p.window) : 0;
     const int row_pooled = POOL ? lo / p.pool : 0;     // pooled rows this row sees
     constexpr int kOCols = DV / 2;                     // columns of O this thread owns
     float m_used = -1e30f, l = 0.f;
@@ -649,7 +649,7 @@ ILB_EXPORT int ilb_attention_prefill_tc(const void* q, void* out, const void* k_
   ILB_REQUIRE(row_blocks == 1 || row_blocks == 2, "attention (tensor cores): %d row blocks per CTA (1 or 2)", row_blocks);
   ILB_REQUIRE(ilb_attention_tc_supported(nq, nkv, d, page_size),
               "attention (tensor cores): heads %d/%d, head size %d, page size %d are not built", nq, nkv, d, page_size);
-  ILB_REQUIRE(n_tokens > 0 && n_seqs > 0 && n_tiles > 0 && n_tiles <= 65535 && max_blocks > 0 && num_pages > 0 && window >= 0,
+  ILB_REQUIRE(n_tokens > 0 && n_seqs > 0 && n_tiles > 0 && n_tiles <= 65535 && max_blocks > 0 && num_pages > 0,
               "attention (tensor cores): bad sizes");
   ILB_REQUIRE(q_stride % 8 == 0 && out_stride % 8 == 0 && ((uintptr_t)q % 16 == 0) && ((uintptr_t)out % 16 == 0) &&
               ((uintptr_t)k_cache % 16 == 0) && ((uintptr_t)v_cache % 16 == 0), "attention (tensor cores): misaligned operands");

@@ -47,6 +47,7 @@ MODULES: Dict[str, List[str]] = {
     "attention_mix": [],
     "recurrent": [],
     "delta": [],
+    "mlstm": [],
 }
 
 _LOCK = threading.Lock()

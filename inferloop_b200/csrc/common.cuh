@@ -65,6 +65,13 @@ template <> __device__ __forceinline__ __nv_bfloat16 from_float<__nv_bfloat16>(f
   return __float2bfloat16_rn(v);
 }
 
+// The first key that the token at position `pos` reads: window > 0: the last `window` positions, itself included; window < 0:
+// its aligned chunk of -window positions, counted from position 0; 0: everything.
+__device__ __forceinline__ int first_key(int pos, int window) {
+  if (window > 0) return pos + 1 > window ? pos + 1 - window : 0;
+  return window < 0 ? pos - pos % -window : 0;
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);

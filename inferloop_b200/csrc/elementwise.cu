@@ -150,8 +150,12 @@ __device__ __forceinline__ float sigmoid_stable(float x) {
   return e / (1.0f + e);
 }
 
-// What the gate passes through before it multiplies the other half: 0 silu, 1 relu.
-__device__ __forceinline__ float gate_act(float g, int act) { return act == 1 ? fmaxf(g, 0.f) : g * sigmoid_stable(g); }
+// What the gate passes through before it multiplies the other half: 0 silu, 1 relu, 2 gelu in its tanh form.
+__device__ __forceinline__ float gate_act(float g, int act) {
+  if (act == 1) return fmaxf(g, 0.f);
+  if (act == 2) return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
+  return g * sigmoid_stable(g);
+}
 
 template <typename T>
 __global__ void silu_mul_kernel(const T* __restrict__ gate, const T* __restrict__ up,
@@ -195,7 +199,7 @@ __global__ void silu_mul_bf16x8_kernel(const __nv_bfloat16* __restrict__ gate, c
 ILB_EXPORT int ilb_silu_mul(const void* in, void* out, int dtype, int rows, int width,
                             int in_stride, int act, cudaStream_t stream) {
   ILB_REQUIRE(rows >= 0 && width > 0 && in_stride >= 2 * width, "silu_mul: bad sizes");
-  ILB_REQUIRE(act == 0 || act == 1, "silu_mul: unknown activation %d", act);
+  ILB_REQUIRE(act >= 0 && act <= 2, "silu_mul: unknown activation %d", act);
   if (rows == 0) return 0;
   const int threads = 256;
   if (dtype == kBF16 && width % 8 == 0 && in_stride % 8 == 0 && ((uintptr_t)in % 16 == 0) && ((uintptr_t)out % 16 == 0)) {

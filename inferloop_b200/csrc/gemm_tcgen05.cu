@@ -66,12 +66,18 @@ enum Epilogue : int { kStore = 0, kAccumulate = 1, kSwiGLU = 2 };
 // silu(g) * u with the fast reciprocal: the quotient is within 2 ulp, far inside what the
 // bfloat16 result keeps, and an epilogue thread has 128 of these per tile.
 __device__ __forceinline__ float silu_mul(float g, float u) { return __fdividef(g, 1.0f + __expf(-g)) * u; }
-// The gated unit's epilogue: act(gate) * up with act = silu (gate_relu 0) or relu (1); or (2) the clamped unit
-// a(min(gate, L)) * (clamp(up, -L, L) + offset) with a(g) = g * sigmoid(sharpness * g).
+// gelu in its tanh form times u: z (1 + tanh(w)) / 2 = z / (1 + exp(-2 w)), w = sqrt(2 / pi) (z + 0.044715 z^3).
+__device__ __forceinline__ float gelu_mul(float g, float u) {
+  const float w = 0.7978845608028654f * fmaf(0.044715f * g * g, g, g);
+  return __fdividef(g, 1.0f + __expf(-2.0f * w)) * u;
+}
+// The gated unit's epilogue: act(gate) * up with act = silu (gate_relu 0), relu (1) or gelu's tanh form (3); or (2) the clamped
+// unit a(min(gate, L)) * (clamp(up, -L, L) + offset) with a(g) = g * sigmoid(sharpness * g).
 template <typename P>
 __device__ __forceinline__ float gate_mul(const P& p, float g, float u) {
   if (p.gate_relu == 0) return silu_mul(g, u);
   if (p.gate_relu == 1) return fmaxf(g, 0.f) * u;
+  if (p.gate_relu == 3) return gelu_mul(g, u);
   g = fminf(g, p.act_limit);
   u = fminf(fmaxf(u, -p.act_limit), p.act_limit);
   return __fdividef(g, 1.0f + __expf(-p.act_sharp * g)) * (u + p.act_offset);
@@ -112,7 +118,7 @@ struct Params {
   int tma_out;               // many tokens: the result leaves through shared memory and TMA stores (adds, when accumulating)
   int red_out;               // few tokens, accumulating: the K ranges of a tile are separate CTAs whose shares meet in memory (red.add)
   int relu2;                 // a plain bfloat16 result leaves as relu(result)^2
-  int gate_relu;             // the gated epilogue's activation: 0 silu, 1 relu, 2 the clamped unit with the constants below
+  int gate_relu;             // the gated epilogue's activation: 0 silu, 1 relu, 2 the clamped unit with the constants below, 3 gelu (tanh form)
   float act_limit, act_sharp, act_offset;
 };
 
@@ -923,7 +929,7 @@ struct PairParams {
   int n_items;               // n_whole + rest * split
   int epilogue, out_f32;
   int relu2;                 // a plain bfloat16 result leaves as relu(result)^2
-  int gate_relu;             // the gated epilogue's activation: 0 silu, 1 relu, 2 the clamped unit with the constants below
+  int gate_relu;             // the gated epilogue's activation: 0 silu, 1 relu, 2 the clamped unit with the constants below, 3 gelu (tanh form)
   float act_limit, act_sharp, act_offset;
 };
 
@@ -1595,11 +1601,11 @@ ILB_EXPORT int ilb_gemm_tc(const void* A, const void* W, const float* bias, void
               "gemm_tc: K (%d) and the leading dimensions (%d, %d) must be multiples of 8", K, lda, ldw);
   ILB_REQUIRE(((uintptr_t)A % 16 == 0) && ((uintptr_t)W % 16 == 0), "gemm_tc: operands must be 16-byte aligned");
   // 3 from the caller: the gated epilogue with relu as the gate's activation (else silu); 4: the clamped gated unit
-  // 5: a plain product whose bfloat16 result leaves as relu(result)^2
+  // 5: a plain product whose bfloat16 result leaves as relu(result)^2; 6: the gated epilogue with gelu's tanh form
   const int relu2 = accumulate == 5 ? 1 : 0;
   if (relu2) accumulate = kStore;
   ILB_REQUIRE(!relu2 || !out_f32, "gemm_tc: relu squared belongs to a bfloat16 result");
-  const int gate_relu = accumulate == 3 ? 1 : (accumulate == 4 ? 2 : 0);
+  const int gate_relu = accumulate == 3 ? 1 : (accumulate == 4 ? 2 : (accumulate == 6 ? 3 : 0));
   if (gate_relu) accumulate = kSwiGLU;
   ILB_REQUIRE(gate_relu != 2 || act_limit > 0.f, "gemm_tc: the clamped unit needs a positive limit");
   ILB_REQUIRE(accumulate >= 0 && accumulate <= 2, "gemm_tc: unknown epilogue %d", accumulate);

@@ -10,7 +10,7 @@
 //                  into the token's place of its page (dummy rows and released pages are skipped)
 //
 // A layer may keep a ROTATED KEY PART beside the latent: `tail` more columns of the projection, shared by all
-// heads, turned by the token's position in pairs of neighbours (the first `rot` of them; the rest pass) and stored
+// heads, turned by the token's position in pairs (of neighbours, or of elements rot / 2 apart; the first `rot` of them, the rest pass) and stored
 // behind the latent in the same cache row (row = rank + tail).  Every head's query then ends in `tail` columns of
 // its own that are turned the same way and copied behind the head's mapped query, so that one dot product over
 // rank + tail elements gives q_a . k_a + q_r . k_r.  The same launch does both; a layer that reads another layer's
@@ -31,6 +31,7 @@ struct LatentWrite {
   // the rotated part (tail 0: none): cos/sin per token [tokens][rot / 2][2]
   int tail, rot;
   const float* angles;
+  int apart;           // a pair's two elements: neighbours (0), or rot / 2 apart (1)
 };
 
 // The queries' tails of token t: head i's columns [qcol0 + i * qhs, + tail) of `qsrc` turned into columns
@@ -40,12 +41,19 @@ struct QueryTails {
   int ld_src, ld_dst, heads, col0, head_stride;
 };
 
+// Unit i of a part of `tail` elements: the elements ea and eb (eb == tail: there is none).  Neighbours 2i and 2i + 1; or,
+// `apart`, i and i + rot / 2 inside the turned elements and neighbours behind them.
+__device__ __forceinline__ void pair_places(int i, int tail, int rot, int apart, int& ea, int& eb) {
+  ea = 2 * i;
+  eb = 2 * i + 1;
+  if (apart && eb < rot) { ea = i; eb = i + rot / 2; }
+}
+
 template <typename T>
-__device__ __forceinline__ void turn_pair(const T* __restrict__ src, int i, int tail, int rot, const float* __restrict__ cs,
+__device__ __forceinline__ void turn_pair(const T* __restrict__ src, int i, int ea, int eb, int tail, int rot, const float* __restrict__ cs,
                                           float& a, float& b) {
-  // elements 2i and 2i + 1 (b unused when 2i + 1 == tail)
-  const float u = to_float(src[2 * i]);
-  const float v = 2 * i + 1 < tail ? to_float(src[2 * i + 1]) : 0.f;
+  const float u = to_float(src[ea]);
+  const float v = eb < tail ? to_float(src[eb]) : 0.f;
   if (2 * i + 1 < rot) {
     const float c = cs[2 * i], s = cs[2 * i + 1];
     a = u * c - v * s;
@@ -68,10 +76,12 @@ __device__ __forceinline__ void latent_write_token(const TI* __restrict__ proj, 
     for (int e = threadIdx.x; e < qt->heads * pairs; e += blockDim.x) {
       const int h = e / pairs, i = e % pairs;
       float u, v;
-      turn_pair<TQ>(qsrc + (size_t)h * qt->head_stride, i, tail, rot, cs, u, v);
+      int ea, eb;
+      pair_places(i, tail, rot, a.apart, ea, eb);
+      turn_pair<TQ>(qsrc + (size_t)h * qt->head_stride, i, ea, eb, tail, rot, cs, u, v);
       TQ* o = qdst + (size_t)h * (rank + tail);
-      o[2 * i] = from_float<TQ>(u);
-      if (2 * i + 1 < tail) o[2 * i + 1] = from_float<TQ>(v);
+      o[ea] = from_float<TQ>(u);
+      if (eb < tail) o[eb] = from_float<TQ>(v);
     }
   }
   if (cache == nullptr) return;
@@ -96,9 +106,11 @@ __device__ __forceinline__ void latent_write_token(const TI* __restrict__ proj, 
     dst[i] = from_float<TC>(to_float(row[i]) * inv * w[i]);
   for (int i = threadIdx.x; i < pairs; i += blockDim.x) {
     float u, v;
-    turn_pair<TI>(row + rank, i, tail, rot, cs, u, v);
-    dst[rank + 2 * i] = from_float<TC>(u);
-    if (2 * i + 1 < tail) dst[rank + 2 * i + 1] = from_float<TC>(v);
+    int ea, eb;
+    pair_places(i, tail, rot, a.apart, ea, eb);
+    turn_pair<TI>(row + rank, i, ea, eb, tail, rot, cs, u, v);
+    dst[rank + ea] = from_float<TC>(u);
+    if (eb < tail) dst[rank + eb] = from_float<TC>(v);
   }
 }
 
@@ -117,7 +129,7 @@ ILB_EXPORT int ilb_latent_write(const void* proj, int dtype, int ld, int col0, i
   ILB_REQUIRE(rank > 0 && ld >= col0 + rank && n_tokens >= 0 && eps > 0.f, "latent_write: bad sizes");
   ILB_REQUIRE(page_size > 0 && max_blocks > 0 && num_pages > 0, "latent_write: bad cache geometry");
   if (n_tokens == 0) return 0;
-  const LatentWrite a{w, eps, positions, seq_of_token, block_table, col0, rank, max_blocks, page_size, num_pages, 0, 0, nullptr};
+  const LatentWrite a{w, eps, positions, seq_of_token, block_table, col0, rank, max_blocks, page_size, num_pages, 0, 0, nullptr, 0};
 #define ILB_LW(TI, TC) ilb::launch(latent_write_kernel<TI, TC>, dim3(n_tokens), dim3(128), 0, stream, (const TI*)proj, ld, a, (TC*)cache)
   if (dtype == kF32 && cache_dtype == kF32) ILB_LW(float, float);
   else if (dtype == kBF16 && cache_dtype == kBF16) ILB_LW(__nv_bfloat16, __nv_bfloat16);
@@ -144,7 +156,7 @@ latent_write_rot_kernel(const TI* __restrict__ proj, int ld, const LatentWrite a
 ILB_EXPORT int ilb_latent_write_rot(const void* proj, int dtype, int ld, int col0, int rank, int tail, int rot, const float* angles,
                                     const float* w, float eps, const int* positions, const int* seq_of_token, const int* block_table,
                                     int max_blocks, int page_size, int num_pages, void* cache, int cache_dtype, const void* q_src,
-                                    void* q_dst, int q_dtype, int ld_q, int q_col0, int q_head_stride, int heads, int n_tokens,
+                                    void* q_dst, int q_dtype, int ld_q, int q_col0, int q_head_stride, int heads, int n_tokens, int apart,
                                     cudaStream_t stream) {
   ILB_REQUIRE(rank > 0 && tail >= 0 && n_tokens >= 0, "latent_write_rot: bad sizes");
   ILB_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= tail && (rot == 0 || angles != nullptr), "latent_write_rot: %d of %d elements cannot turn in pairs", rot, tail);
@@ -154,7 +166,7 @@ ILB_EXPORT int ilb_latent_write_rot(const void* proj, int dtype, int ld, int col
               "latent_write_rot: the queries' rows are too short");
   ILB_REQUIRE(cache != nullptr || q_src != nullptr, "latent_write_rot: nothing to do");
   if (n_tokens == 0) return 0;
-  const LatentWrite a{w, eps, positions, seq_of_token, block_table, col0, rank, max_blocks, page_size, num_pages, tail, rot, angles};
+  const LatentWrite a{w, eps, positions, seq_of_token, block_table, col0, rank, max_blocks, page_size, num_pages, tail, rot, angles, apart};
   const QueryTails qt{q_src, q_dst, ld_q, heads * (rank + tail), heads, q_col0, q_head_stride};
 #define ILB_LW(TI, TC, TQ) ilb::launch(latent_write_rot_kernel<TI, TC, TQ>, dim3(n_tokens), dim3(128), 0, stream, (const TI*)proj, ld, a, (TC*)cache, qt)
   const int cd = cache != nullptr ? cache_dtype : q_dtype;
@@ -455,7 +467,7 @@ ILB_EXPORT int ilb_latent_input(const void* proj, int dtype, int ld, const void*
   const long long rows = (long long)heads * ((N + 31) / 32) + kHeadTokens;
   ILB_REQUIRE(rows <= 65535, "latent_input: too many heads");
   if (n_tokens == 0) return 0;
-  const LatentWrite a{norm_w, eps, positions, seq_of_token, block_table, col0, rank, max_blocks, page_size, num_pages, 0, 0, nullptr};
+  const LatentWrite a{norm_w, eps, positions, seq_of_token, block_table, col0, rank, max_blocks, page_size, num_pages, 0, 0, nullptr, 0};
   const dim3 grid((n_tokens + kHeadTokens - 1) / kHeadTokens, (unsigned)rows);
 #define ILB_LI(TI, TC, TO) ilb::launch(latent_input_kernel<TI, TC, TO>, grid, dim3(128), smem, stream, (const TI*)proj, ld, (const TI*)w, \
                                         (TO*)q_out, ldo, n_tokens, heads, K, N, a, (TC*)cache)

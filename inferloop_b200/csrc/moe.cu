@@ -131,7 +131,7 @@ ILB_EXPORT int ilb_moe_logits(const void* x, const void* w, int dtype, float* ou
 __global__ void __launch_bounds__(128)
 moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bias, int ld, int n_tokens, int experts, int top,
                  int softmax, int renormalize, int* __restrict__ choice, float* __restrict__ weight,
-                 const float* __restrict__ correction, int groups, int keep, float out_scale, float renorm_eps) {
+                 const float* __restrict__ correction, int groups, int keep, int best_two, float out_scale, float renorm_eps) {
   ilb::pdl_launch_dependents();
   ilb::pdl_wait();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -166,7 +166,7 @@ moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bia
   }
   // What the experts are ranked by: the scores, or the scores plus a stored correction (the weights below are the
   // scores themselves either way).  With groups, only experts of the `keep` groups of neighbours whose best ranked
-  // member is largest can be chosen (ties to the lower group).
+  // member (`best_two`: whose two best together) is largest can be chosen (ties to the lower group).
   float c[kMaxExpertsPerLane];
 #pragma unroll
   for (int i = 0; i < kMaxExpertsPerLane; ++i) {
@@ -184,6 +184,24 @@ moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bia
         if (e < experts && e / per == g) m = fmaxf(m, c[i]);
       }
       m = warp_max(m);
+      if (best_two) {
+        // the second best: the largest of the others, the best one itself being the group's first member of that value
+        int who = 0x7fffffff;
+#pragma unroll
+        for (int i = 0; i < kMaxExpertsPerLane; ++i) {
+          const int e = lane + 32 * i;
+          if (e < experts && e / per == g && c[i] == m) who = min(who, e);
+        }
+        who = (int)__reduce_min_sync(0xffffffffu, (unsigned)who);
+        float second = -INFINITY;
+#pragma unroll
+        for (int i = 0; i < kMaxExpertsPerLane; ++i) {
+          const int e = lane + 32 * i;
+          if (e < experts && e / per == g && e != who) second = fmaxf(second, c[i]);
+        }
+        second = warp_max(second);
+        if (per > 1) m += second;
+      }
       if (lane == g) mine = m;
     }
     unsigned allowed = 0u;
@@ -247,7 +265,7 @@ ILB_EXPORT int ilb_moe_max_top() { return kMaxTop; }
 // alone, or null.  groups > 1 with keep < groups: only the best `keep` of `groups` equal groups of neighbouring
 // experts can be chosen.  Weights: the chosen scores (divided by their sum + renorm_eps when renormalize) * out_scale.
 ILB_EXPORT int ilb_moe_route(const float* logits, const float* bias, int ld, int n_tokens, int experts, int top, int softmax,
-                             int renormalize, int* choice, float* weight, const float* correction, int groups, int keep,
+                             int renormalize, int* choice, float* weight, const float* correction, int groups, int keep, int best_two,
                              float out_scale, float renorm_eps, cudaStream_t stream) {
   ILB_REQUIRE(groups >= 1 && groups <= 32 && experts % groups == 0 && keep >= 1 && keep <= groups,
               "moe_route: %d groups (at most 32, dividing %d experts), %d kept", groups, experts, keep);
@@ -258,7 +276,7 @@ ILB_EXPORT int ilb_moe_route(const float* logits, const float* bias, int ld, int
   ILB_REQUIRE(ld >= experts, "moe_route: row stride too small");
   if (n_tokens == 0) return 0;
   ilb::launch(moe_route_kernel, dim3((n_tokens + 3) / 4), dim3(128), 0, stream, logits, bias, ld, n_tokens, experts, top, softmax,
-              renormalize, choice, weight, correction, groups, keep, out_scale, renorm_eps);
+              renormalize, choice, weight, correction, groups, keep, best_two, out_scale, renorm_eps);
   return check_launch("moe_route");
 }
 

@@ -115,11 +115,11 @@ def rmsnorm(x: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor
           _i(rows), _i(width), _f(eps), _stream(x))
 
 
-GATE_ACTIVATIONS = {"silu": 0, "relu": 1}
+GATE_ACTIVATIONS = {"silu": 0, "relu": 1, "gelu_tanh": 2}
 
 
 def silu_mul(gate_up: torch.Tensor, out: torch.Tensor, activation: str = "silu") -> None:
-    """out = act(gate_up[:, :I]) * gate_up[:, I:2I], act = silu (default) or relu."""
+    """out = act(gate_up[:, :I]) * gate_up[:, I:2I], act = silu (default), relu or gelu in its tanh form."""
     _need(gate_up, "silu_mul in"); _need(out, "silu_mul out", gate_up.dtype)
     rows, width = out.shape
     if gate_up.shape[0] != rows or gate_up.shape[1] != 2 * width:
@@ -318,9 +318,10 @@ def head_matmul_split(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> No
 def latent_write_rot(proj: torch.Tensor, col0: int, rank: int, tail: int, rot: int, angles: Optional[torch.Tensor],
                      weight: Optional[torch.Tensor], eps: float, step, block_table: Optional[torch.Tensor],
                      cache: Optional[torch.Tensor], q_src: Optional[torch.Tensor] = None, q_dst: Optional[torch.Tensor] = None,
-                     q_col0: int = 0, q_head_stride: int = 0, heads: int = 0) -> None:
+                     q_col0: int = 0, q_head_stride: int = 0, heads: int = 0, half_split: bool = False) -> None:
     """A latent with a rotated part behind it: cache row of token t = [rms(proj[t, col0 : col0 + rank]) * weight |
-    turn(proj[t, col0 + rank : + tail])], the first `rot` elements of the part turned in neighbouring pairs by
+    turn(proj[t, col0 + rank : + tail])], the first `rot` elements of the part turned in neighbouring pairs (or, `half_split`, in
+    pairs rot / 2 apart) by
     `angles` [T, rot / 2, 2] (cos, sin); cache is [pages, 1, page_size, rank + tail] (None: nothing stored).  With
     `q_src` [T, >= q_col0 + heads * q_head_stride]: head i's `tail` columns from q_col0 + i * q_head_stride are
     turned the same way into q_dst[t, i, rank:], q_dst [T, heads * (rank + tail)]."""
@@ -341,7 +342,7 @@ def latent_write_rot(proj: torch.Tensor, col0: int, rank: int, tail: int, rot: i
           _i(0 if block_table is None else block_table.shape[1]), _i(0 if cache is None else cache.shape[2]),
           _i(0 if cache is None else cache.shape[0]), _ptr(cache), _i(_code(ref)), _ptr(q_src), _ptr(q_dst),
           _i(_code(ref if q_src is None else q_src)), _i(0 if q_src is None else q_src.stride(0)), _i(q_col0), _i(q_head_stride),
-          _i(heads), _i(T), _stream(ref))
+          _i(heads), _i(T), _i(1 if half_split else 0), _stream(ref))
 
 
 # --------------------------------------------------------------------------- norm on a sublayer's output
@@ -377,6 +378,29 @@ def group_norm_add(y: torch.Tensor, weight: torch.Tensor, eps: float, groups: in
         raise KernelError("group_norm_add: shapes do not agree")
     _call("sublayer_norm", "ilb_group_norm_add", _ptr(y), _i(y.stride(0)), _ptr(weight), _f(eps), _i(groups), _i(rows), _i(width),
           _ptr(x), _ptr(out), _i(F32 if out is None else _code(out)), _i(1 if zero else 0), _stream(y))
+
+
+def branch_norms_add(rows, weights, eps: float, mult: float, y: Optional[torch.Tensor] = None, norm=None, x: Optional[torch.Tensor] = None,
+                     out: Optional[torch.Tensor] = None) -> None:
+    """z = mult * (rms(rows[0]) * weights[0] + rms(rows[1]) * weights[1]), each row divided by its own sqrt(mean^2 + eps).  With
+    `y`: y += z.  With `norm` = (weight, eps) and `x`: x += rms(z) * weight, and `out` (if given) = the new x in its dtype."""
+    a, b = rows
+    for t, w in ((a, "branch rows"), (b, "branch rows"), (weights[0], "branch norm weight"), (weights[1], "branch norm weight"), (y, "branch sum"), (x, "stream")):
+        _need(t, w, torch.float32)
+    _need(out, "branch out")
+    n, width = a.shape
+    if b.shape != a.shape or weights[0].numel() != width or weights[1].numel() != width or (y is None) == (norm is None) or (norm is None) != (x is None):
+        raise KernelError("branch_norms_add: shapes do not agree, or not one of a sum and a norm")
+    for t in (y, x, out):
+        if t is not None and t.shape != a.shape:
+            raise KernelError("branch_norms_add: shapes do not agree")
+    if norm is not None:
+        _need(norm[0], "norm weight", torch.float32)
+        if norm[0].numel() != width:
+            raise KernelError("branch_norms_add: the norm does not fit the rows")
+    _call("sublayer_norm", "ilb_branch_norms_add", _ptr(a), _ptr(b), _ptr(weights[0]), _ptr(weights[1]), _f(eps), _f(mult), _ptr(y),
+          _ptr(None if norm is None else norm[0]), _f(0.0 if norm is None else norm[1]), _ptr(x), _ptr(out), _i(F32 if out is None else _code(out)),
+          _i(n), _i(width), _stream(a))
 
 
 def dyt(x: torch.Tensor, alpha: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor, out: torch.Tensor) -> None:
@@ -456,18 +480,18 @@ def silu_rows(x: torch.Tensor, width: int, out: torch.Tensor) -> None:
 
 
 def rms_gate(y: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor, scale: float = 1.0,
-             groups: int = 1) -> None:
+             groups: int = 1, divisor: Optional[torch.Tensor] = None) -> None:
     """out = y / sqrt(mean(y^2) + eps) * weight * sigmoid(gate) * scale over whole rows, or over each of `groups` equal parts
     of them; y 32-bit, gate [T, >= width] (its first `width` columns) and out [T, width] (rows of any stride) in the compute
-    dtype."""
+    dtype.  `divisor` [T, groups] 32-bit: a part's y is divided by its number first."""
     _need(y, "rms_gate y", torch.float32); _need(gate, "rms_gate gate", contiguous=False); _need(weight, "rms_gate weight", torch.float32)
-    _need(out, "rms_gate out", gate.dtype, contiguous=False)
+    _need(out, "rms_gate out", gate.dtype, contiguous=False); _need(divisor, "rms_gate divisor", torch.float32)
     T, width = y.shape
     if gate.shape[0] != T or gate.shape[1] < width or gate.stride(1) != 1 or weight.numel() != width or out.shape != y.shape \
-            or out.stride(1) != 1:
+            or out.stride(1) != 1 or (divisor is not None and tuple(divisor.shape) != (T, groups)):
         raise KernelError("rms_gate: shapes do not agree")
     _call("recurrent", "ilb_rms_gate", _ptr(y), _ptr(gate), _i(_code(gate)), _i(gate.stride(0)), _ptr(weight), _ptr(out), _i(out.stride(0)),
-          _i(T), _i(width), _i(groups), _f(eps), _f(scale), _stream(out))
+          _i(T), _i(width), _i(groups), _f(eps), _f(scale), _ptr(divisor), _stream(out))
 
 
 ACTIVATIONS = {"tanh": 0, "relu2": 1}
@@ -558,6 +582,100 @@ def head_gate(o: torch.Tensor, gate: torch.Tensor, heads: int, scale: float = 1.
           _i(width // heads), _f(scale), _stream(o))
 
 
+def gate_rows(o: torch.Tensor, gate: torch.Tensor, out: torch.Tensor) -> None:
+    """out = o * sigmoid(gate), element by element; all [rows, >= width] of one dtype, rows of any stride, width = o's."""
+    _need(o, "gate_rows o", contiguous=False); _need(gate, "gate_rows gate", o.dtype, contiguous=False); _need(out, "gate_rows out", o.dtype, contiguous=False)
+    rows, width = o.shape
+    if gate.shape[0] != rows or gate.shape[1] < width or out.shape != o.shape or any(t.stride(1) != 1 for t in (o, gate, out)):
+        raise KernelError("gate_rows: shapes do not agree")
+    _call("recurrent", "ilb_gate_rows", _ptr(o), _i(o.stride(0)), _ptr(gate), _i(gate.stride(0)), _ptr(out), _i(out.stride(0)), _i(_code(o)),
+          _i(rows), _i(width), _stream(out))
+
+
+# --------------------------------------------------------------------------- matrix memory (mLSTM)
+MLSTM_CHUNK = 64           # tokens a chunk of a long portion holds
+MLSTM_CHUNK_FROM = 16      # portions of bfloat16 projections from this many tokens on run in chunks
+MLSTM_MAX_ROWS = 256       # key channels a head
+
+
+class MatrixMemory:
+    """What the mLSTM kernels take beside the step: columns of the projection, constants, biases of the gates."""
+
+    def __init__(self, heads: int, d: int, dv: int, col_q: int, col_k: int, col_v: int, col_g: int, cap: float, q_scale: float, eps: float,
+                 bias_i: torch.Tensor, bias_f: torch.Tensor) -> None:
+        self.heads, self.d, self.dv = heads, d, dv
+        self.col_q, self.col_k, self.col_v, self.col_g = col_q, col_k, col_v, col_g
+        self.cap, self.q_scale, self.eps = cap, q_scale, eps
+        self.bias_i, self.bias_f = bias_i, bias_f
+
+    def check(self, proj: torch.Tensor, state) -> None:
+        _need(proj, "mlstm projection", contiguous=False)
+        for t, w, shape in ((state["state"], "state", (self.heads, self.d, self.dv)), (state["norm"], "normaliser", (self.heads, self.d)),
+                            (state["max"], "maximum", (self.heads,))):
+            _need(t, "mlstm " + w, torch.float32)
+            if tuple(t.shape[1:]) != shape:
+                raise KernelError(f"mlstm: the {w}'s slots are {tuple(t.shape[1:])}, not {shape}")
+        for t in (self.bias_i, self.bias_f):
+            _need(t, "mlstm gate bias", torch.float32)
+            if t.numel() != self.heads:
+                raise KernelError("mlstm: one gate bias a head")
+        need = max(self.col_q + self.heads * self.d, self.col_k + self.heads * self.d, self.col_v + self.heads * self.dv, self.col_g + self.heads * self.dv)
+        if proj.stride(1) != 1 or proj.shape[1] < need:
+            raise KernelError("mlstm: the projection's rows are too short")
+
+
+def mlstm_scan(m: MatrixMemory, proj: torch.Tensor, gates: torch.Tensor, state, y: torch.Tensor, step, workspace,
+               chunks: Optional[bool] = None) -> Optional[torch.Tensor]:
+    """The matrix memory over the step's tokens, from and to `state` (slots "state", "norm", "max"; see mlstm.cu); gates
+    [T, 2 heads] 32-bit logits, y [T, heads * dv] 32-bit.  Returns what y still has to be divided by, [T, heads], or None.
+    `chunks`: whether the portions run 64 tokens at a time (None: by the longest portion; bfloat16 projections only)."""
+    m.check(proj, state)
+    _need(gates, "mlstm gates", torch.float32, contiguous=False); _need(y, "mlstm y", torch.float32)
+    T = proj.shape[0]
+    if gates.shape[0] != T or gates.shape[1] < 2 * m.heads or gates.stride(1) != 1 or tuple(y.shape) != (T, m.heads * m.dv):
+        raise KernelError("mlstm_scan: shapes do not agree")
+    if chunks is None:
+        chunks = proj.dtype == torch.bfloat16 and step.max_q_len >= MLSTM_CHUNK_FROM
+    if chunks:
+        _need(proj, "mlstm projection", torch.bfloat16, contiguous=False)
+        n_chunks = sum(-(-n // MLSTM_CHUNK) for n in step.h_q_len) + (step.n_seqs - len(step.h_q_len))
+        scratch = workspace.buffer("mlstm.chunks", (mlstm_chunk_floats(n_chunks, m.heads, m.d, m.dv),), torch.float32)
+        _call("mlstm", "ilb_mlstm_chunks", _ptr(proj), _i(proj.stride(0)), _i(m.col_q), _i(m.col_k), _i(m.col_v), _ptr(gates), _i(gates.stride(0)),
+              _ptr(m.bias_i), _ptr(m.bias_f), _f(m.cap), _f(m.q_scale), _f(m.eps), _ptr(state["state"]), _ptr(state["norm"]), _ptr(state["max"]),
+              _ptr(scratch), ctypes.c_longlong(scratch.numel()), _ptr(y), _ptr(step.cu_q), _ptr(step.slots), _i(step.n_seqs), _i(n_chunks),
+              _i(m.heads), _i(m.d), _i(m.dv), _stream(y))
+        return None
+    scratch = workspace.buffer("mlstm.gates", (3 * T * m.heads,), torch.float32)
+    den = workspace.buffer("mlstm.den", (T, m.heads), torch.float32)
+    _call("mlstm", "ilb_mlstm_scan", _ptr(proj), _i(_code(proj)), _i(proj.stride(0)), _i(m.col_q), _i(m.col_k), _i(m.col_v), _ptr(gates),
+          _i(gates.stride(0)), _ptr(m.bias_i), _ptr(m.bias_f), _f(m.cap), _f(m.q_scale), _f(m.eps), _ptr(state["state"]), _ptr(state["norm"]),
+          _ptr(state["max"]), _ptr(scratch), _ptr(y), _ptr(den), _ptr(step.cu_q), _ptr(step.slots), _i(step.n_seqs), _i(T), _i(m.heads), _i(m.d),
+          _i(m.dv), _stream(y))
+    return den
+
+
+def mlstm_chunk_floats(n_chunks: int, heads: int, d: int, dv: int) -> int:
+    """32-bit elements of scratch that so many chunks of 64 tokens need (the layout is mlstm.cu's)."""
+    return n_chunks * heads * (d * dv + d + 4)
+
+
+def mlstm_step(m: MatrixMemory, proj: torch.Tensor, x: torch.Tensor, w_gates: torch.Tensor, norm_w: torch.Tensor, norm_eps: float, state,
+               out: torch.Tensor, step) -> None:
+    """A step of single tokens: the gates' dot products with x, the recurrence, the read-out, the RMS norm of each head and the
+    output gate, in one launch; out [T, heads * dv] (rows of any stride) in proj's dtype."""
+    m.check(proj, state)
+    _need(x, "mlstm x", proj.dtype); _need(w_gates, "mlstm gate matrix", proj.dtype); _need(norm_w, "mlstm norm weight", torch.float32)
+    _need(out, "mlstm out", proj.dtype, contiguous=False)
+    T = proj.shape[0]
+    if tuple(w_gates.shape) != (2 * m.heads, x.shape[1]) or x.shape[0] != T or T != step.n_seqs or norm_w.numel() != m.heads * m.dv \
+            or tuple(out.shape) != (T, m.heads * m.dv) or out.stride(1) != 1:
+        raise KernelError("mlstm_step: shapes do not agree")
+    _call("mlstm", "ilb_mlstm_step", _ptr(proj), _i(_code(proj)), _i(proj.stride(0)), _i(m.col_q), _i(m.col_k), _i(m.col_v), _i(m.col_g), _ptr(x),
+          _i(x.shape[1]), _ptr(w_gates), _ptr(m.bias_i), _ptr(m.bias_f), _f(m.cap), _f(m.q_scale), _f(m.eps), _ptr(norm_w), _f(norm_eps),
+          _ptr(state["state"]), _ptr(state["norm"]), _ptr(state["max"]), _ptr(out), _i(out.stride(0)), _ptr(step.cu_q), _ptr(step.slots),
+          _i(step.n_seqs), _i(m.heads), _i(m.d), _i(m.dv), _stream(out))
+
+
 def gated_rows(a: torch.Tensor, table: torch.Tensor, col0: int, tokens: torch.Tensor, out: torch.Tensor) -> None:
     """out[t, k] = gelu_tanh(a[t, k]) * table[tokens[t], col0 + k]."""
     _need(a, "gated_rows a"); _need(table, "gated_rows table", a.dtype); _need(out, "gated_rows out", a.dtype)
@@ -634,11 +752,11 @@ def moe_logits(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
 def moe_route(logits: torch.Tensor, experts: int, top: int, softmax: bool, renormalize: bool,
               choice: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] = None,
               correction: Optional[torch.Tensor] = None, groups: int = 1, keep: int = 1, scale: float = 1.0,
-              renorm_eps: float = 0.0) -> None:
+              renorm_eps: float = 0.0, group_best_two: bool = False) -> None:
     """The `top` experts with the largest scores of every token and their weights; `bias` [experts]
     is added to the logits first.  `correction` [experts] is added to the scores for the ranking alone (the
     weights stay the scores); with `groups` > 1 the experts form that many equal groups of neighbours, a group
-    ranks by its best member, and only the best `keep` groups' experts can be chosen.  The weights are divided by
+    ranks by its best member (`group_best_two`: by its two best together), and only the best `keep` groups' experts can be chosen.  The weights are divided by
     their sum + `renorm_eps` when `renormalize`, then multiplied by `scale`."""
     _need(logits, "router logits", torch.float32); _need(choice, "moe choice", torch.int32); _need(weight, "moe weight", torch.float32)
     _need(bias, "router bias", torch.float32); _need(correction, "router correction", torch.float32)
@@ -647,7 +765,8 @@ def moe_route(logits: torch.Tensor, experts: int, top: int, softmax: bool, renor
             or (correction is not None and correction.numel() != experts):
         raise KernelError("moe_route: shapes do not agree")
     _call("moe", "ilb_moe_route", _ptr(logits), _ptr(bias), _i(logits.stride(0)), _i(T), _i(experts), _i(top), _i(1 if softmax else 0),
-          _i(1 if renormalize else 0), _ptr(choice), _ptr(weight), _ptr(correction), _i(groups), _i(keep), _f(scale), _f(renorm_eps),
+          _i(1 if renormalize else 0), _ptr(choice), _ptr(weight), _ptr(correction), _i(groups), _i(keep), _i(1 if group_best_two else 0), _f(scale),
+          _f(renorm_eps),
           _stream(logits))
 
 
@@ -873,6 +992,34 @@ def rows_norm_rope_cache(qkv: torch.Tensor, q_out: torch.Tensor, q_weight: torch
           _i(0 if pooled is None else pooled.k.shape[0]), _i(0 if pooled is None else pooled.pool), _stream(qkv))
 
 
+def conv_rows_norm_cache(qkv: torch.Tensor, q_out: torch.Tensor, conv_w: torch.Tensor, conv_state: torch.Tensor, q_weight: torch.Tensor,
+                         k_weight: torch.Tensor, eps: float, rope: Optional[torch.Tensor], rotary_dim: int, step, block_table: torch.Tensor,
+                         k_cache: Optional[torch.Tensor], v_cache: Optional[torch.Tensor], nq: int, nkv: int, d: int, dv: int,
+                         values_are_keys: bool = False) -> None:
+    """`rows_norm_rope_cache` for queries and keys that pass a causal convolution per channel first: conv_w
+    [taps, (nq + nkv) d] 32-bit, conv_state [slots, taps - 1, (nq + nkv) d] 32-bit (the last raw inputs, brought up to date).
+    `values_are_keys`: the values are the convolved keys before their norm, and qkv holds no columns for them."""
+    _need(qkv, "qkv", contiguous=False); _need(q_out, "q_out", qkv.dtype); _need(conv_w, "conv weight", torch.float32)
+    _need(conv_state, "conv state", torch.float32); _need(q_weight, "q norm weight", torch.float32); _need(k_weight, "k norm weight", torch.float32)
+    _need(rope, "rope table", torch.float32); _need(k_cache, "k cache", qkv.dtype); _need(v_cache, "v cache", qkv.dtype)
+    _need(block_table, "block table", torch.int32)
+    T, width, taps = qkv.shape[0], (nq + nkv) * d, conv_w.shape[0]
+    if qkv.stride(1) != 1 or qkv.shape[1] < width + (0 if values_are_keys else nkv * dv) or conv_w.shape[1] != width \
+            or tuple(conv_state.shape[1:]) != (taps - 1, width) or q_weight.numel() != nq * d or k_weight.numel() != nkv * d \
+            or (rope is not None and tuple(rope.shape) != (T, rotary_dim // 2, 2)) or (values_are_keys and dv != d) \
+            or tuple(q_out.shape) != (T, nq * d):
+        raise KernelError("conv_rows_norm_cache: shapes do not agree")
+    page_size = num_pages = 0
+    if k_cache is not None:
+        num_pages, page_size = k_cache.shape[0], k_cache.shape[2]
+        if tuple(k_cache.shape[1:]) != (nkv, page_size, d) or tuple(v_cache.shape) != (num_pages, nkv, page_size, dv):
+            raise KernelError("conv_rows_norm_cache: cache shapes do not match the heads")
+    _call("qk_norm_rope", "ilb_conv_rows_norm_cache", _ptr(qkv), _ptr(q_out), _i(_code(qkv)), _ptr(conv_w), _i(taps), _ptr(conv_state), _ptr(q_weight),
+          _ptr(k_weight), _f(eps), _ptr(rope), _i(rotary_dim), _ptr(step.positions), _ptr(step.seq_of_token), _ptr(step.cu_q), _ptr(step.slots),
+          _i(step.n_seqs), _i(0 if step.decode_only else 1), _ptr(block_table), _i(block_table.shape[1]), _i(page_size), _i(num_pages), _ptr(k_cache),
+          _ptr(v_cache), _i(T), _i(nq), _i(nkv), _i(d), _i(dv), _i(qkv.stride(0)), _i(q_out.shape[1]), _i(1 if values_are_keys else 0), _stream(qkv))
+
+
 class PooledRows:
     """What attention over a window sees before it: the means of aligned blocks of `pool` tokens, in pages of their own
     (`k`, `v` [pages, nkv, page_size, d / dv], block table `table`)."""
@@ -1095,12 +1242,12 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[
             accumulate: bool = False, max_ctas: int = 0, swiglu: bool = False, gate: str = "silu", glu=None, relu2: bool = False) -> None:
     """out (+)= a @ w.T (+ bias) on tcgen05 tensor cores (see gemm_tcgen05.cu).  With
     `swiglu`, `w` holds blocks of 64 gate rows followed by their 64 up rows and `out` is
-    [M, N/2] = act(gate) * up, act = `gate` ("silu" or "relu"); or, with `glu` = (limit, sharpness, up_offset), the
+    [M, N/2] = act(gate) * up, act = `gate` ("silu", "relu" or "gelu_tanh"); or, with `glu` = (limit, sharpness, up_offset), the
     clamped unit a(min(gate, limit)) * (clamp(up, -limit, limit) + up_offset), a(g) = g * sigmoid(sharpness * g).
     With `relu2` a bfloat16 `out` receives relu(result)^2."""
     if relu2 and (swiglu or accumulate or out.dtype != torch.bfloat16):
         raise KernelError("gemm: relu squared belongs to a plain product with a bfloat16 result")
-    if gate not in ("silu", "relu"):
+    if gate not in GATE_ACTIVATIONS:
         raise KernelError(f"gemm: the gated epilogue has no activation {gate!r}")
     if glu is not None and (not swiglu or float(glu[0]) <= 0):
         raise KernelError("gemm: the clamped gated unit belongs to the gated epilogue and needs a positive limit")
@@ -1114,7 +1261,7 @@ def gemm_tc(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: Optional[
     if accumulate and (out.dtype != torch.float32 or swiglu):
         raise KernelError("gemm: accumulation needs a 32-bit output and no SwiGLU epilogue")
     st = _tc_state(a.device)
-    mode = (4 if glu is not None else 3 if gate == "relu" else 2) if swiglu else (1 if accumulate else 5 if relu2 else 0)
+    mode = (4 if glu is not None else {"silu": 2, "relu": 3, "gelu_tanh": 6}[gate]) if swiglu else (1 if accumulate else 5 if relu2 else 0)
     limit, sharp, offset = glu if glu is not None else (0.0, 1.0, 0.0)
     _call("gemm_tcgen05", "ilb_gemm_tc", _ptr(a), _ptr(w), _ptr(bias), _ptr(out),
           _i(1 if out.dtype == torch.float32 else 0), _i(M), _i(N), _i(K), _i(a.stride(0)), _i(w.stride(0)),
@@ -1341,7 +1488,8 @@ def attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache
     tensor-core kernels for a bfloat16 cache and a head size they are built for (split-KV
     when every sequence brings one token), else the exact kernel.  `sink` [nq] 32-bit: a logit
     per query head that joins the softmax's denominator (no key, no value, no scale).  `pooled`: rows
-    that stand for whole blocks of tokens before the window, in the same softmax.  `turn` [T, dv / 2, 2]: the heads'
+    that stand for whole blocks of tokens before the window, in the same softmax.  `window`: 0 for all keys, n > 0 for the last n,
+    n < 0 for those of the token's aligned chunk of -n positions.  `turn` [T, dv / 2, 2]: the heads'
     outputs are turned back by these angles (see `turn_back`)."""
     dv = d if dv is None else int(dv)
     _need(sink, "attention sink", torch.float32)
@@ -1368,7 +1516,7 @@ def attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache
         capacity = block_table.shape[1] * page_size
         max_chunks = max(1, -(-capacity // decode_chunk))
         if window:                       # a token reads the chunks its window touches, counted from the first of them
-            max_chunks = min(max_chunks, (window - 1) // decode_chunk + 2)
+            max_chunks = min(max_chunks, (abs(window) - 1) // decode_chunk + 2)
         scratch = workspace.buffer("attn.decode_scratch", (step.n_seqs * nkv * max_chunks * G * (d + 2),), torch.float32)
         tickets = workspace.zeroed("attn.decode_tickets", (max(step.n_seqs * nkv, 4096),), torch.int32)
         attention_decode(q, out, k_cache, v_cache, step.positions, step.cu_q, block_table, window, scale,

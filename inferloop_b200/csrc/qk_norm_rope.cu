@@ -631,6 +631,187 @@ ILB_EXPORT int ilb_rows_norm_rope_cache(
   return check_launch("rows_norm_rope_cache");
 }
 
+// ---------------------------------------------------------------- short convolutions, then norms over whole rows
+// The same input stage for queries and keys that pass a causal convolution per channel first:
+//   u_t = sum_j w[j, c] raw_{t - (taps - 1) + j},   q <- turn(u_q / sqrt(mean(u_q^2) + eps) * wq),   k likewise
+// and values that are either columns of their own behind q | k, as they are, or (values_are_keys) u_k before its norm.
+// The raw inputs ahead of the step come from state [slots, taps - 1, (nq + nkv) d] 32-bit; zeros before the sequence's start.
+// A block a token: the convolved row waits in shared memory for its sums.  A sequence of one token is one block, which also
+// moves the state on; the state of the others is moved on by a second launch, when nobody reads the old one any more.
+struct ConvRowsParams {
+  RowsParams r;
+  const float* conv_w;               // [taps, (nq + nkv) d]
+  float* state;
+  const int* cu_q; const int* slots;
+  int taps, values_are_keys;
+};
+
+template <typename T, int VEC>
+__global__ void __launch_bounds__(kRowsThreads)
+conv_rows_norm_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* k_cache, T* v_cache, const ConvRowsParams c) {
+  ilb::pdl_launch_dependents();
+  ilb::pdl_wait();
+  const RowsParams& p = c.r;
+  extern __shared__ __align__(16) float u[];             // [(nq + nkv) d]
+  __shared__ float scratch[33];
+  const int t = blockIdx.x, seq = p.seq_of_token[t];
+  const int tok0 = c.cu_q[seq], lt = t - tok0, slot = c.slots[seq];
+  const bool alone = c.cu_q[seq + 1] - tok0 == 1;
+  const int nqd = p.nq * p.d, nkd = p.nkv * p.d, width = nqd + nkd, before = c.taps - 1;
+  float* own = slot >= 0 ? c.state + (size_t)slot * before * width : nullptr;
+  float sum_q = 0.f, sum_k = 0.f;
+  for (int e = threadIdx.x * VEC; e < width; e += kRowsThreads * VEC) {
+    float acc[VEC];
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) acc[i] = 0.f;
+    for (int j = 0; j < c.taps; ++j) {
+      const int back = before - j;
+      float x[VEC], w[VEC];
+      if (lt >= back) RowUnit<T, VEC>::load(qkv + (size_t)(t - back) * p.qkv_stride + e, x);
+      else if (own != nullptr) {                           // (plain loads: this launch may write the slot)
+        const float* s = own + (size_t)(before + lt - back) * width + e;
+        if constexpr (VEC == 8) {
+          const float4 a = *reinterpret_cast<const float4*>(s), b = *reinterpret_cast<const float4*>(s + 4);
+          x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w; x[4] = b.x; x[5] = b.y; x[6] = b.z; x[7] = b.w;
+        } else {
+          x[0] = *s;
+        }
+      } else {
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) x[i] = 0.f;
+      }
+      load_f32<VEC>(c.conv_w + (size_t)j * width + e, w);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) acc[i] = fmaf(w[i], x[i], acc[i]);
+      if (alone && j > 0 && own != nullptr) {
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) own[(size_t)(j - 1) * width + e + i] = x[i];
+      }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) { u[e + i] = acc[i]; ss = fmaf(acc[i], acc[i], ss); }
+    if (e < nqd) sum_q += ss; else sum_k += ss;
+  }
+  sum_q = warp_sum(sum_q);
+  sum_k = warp_sum(sum_k);
+  if ((threadIdx.x & 31) == 0) { scratch[threadIdx.x >> 5] = sum_q; scratch[16 + (threadIdx.x >> 5)] = sum_k; }
+  __syncthreads();
+  sum_q = 0.f; sum_k = 0.f;
+#pragma unroll
+  for (int w = 0; w < kRowsThreads / 32; ++w) { sum_q += scratch[w]; sum_k += scratch[16 + w]; }
+  const float inv_q = 1.0f / sqrtf(sum_q / (float)nqd + p.eps);
+  const float inv_k = 1.0f / sqrtf(sum_k / (float)nkd + p.eps);
+  long long place = -1;
+  if (k_cache != nullptr) {
+    const int pos = p.positions[t], blk = pos / p.page_size;
+    if (blk >= 0 && blk < p.max_blocks) {
+      const int page = p.block_table[(size_t)seq * p.max_blocks + blk];
+      if (page >= 0 && page < p.num_pages) place = (long long)page * p.nkv * p.page_size + pos % p.page_size;      // never write outside the pool
+    }
+  }
+  const int half = p.rotary_dim / 2;
+  for (int e = threadIdx.x * VEC; e < width; e += kRowsThreads * VEC) {
+    const bool is_q = e < nqd;
+    if (!is_q && place < 0) continue;
+    const int r = is_q ? e : e - nqd, h = r / p.d, ch = r % p.d;
+    const float inv = is_q ? inv_q : inv_k;
+    float x[VEC], w[VEC];
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) x[i] = u[e + i];
+    if (!is_q && c.values_are_keys) RowUnit<T, VEC>::store(v_cache + ((size_t)place + (size_t)h * p.page_size) * p.dv + ch, x);
+    load_f32<VEC>((is_q ? p.q_weight : p.k_weight) + r, w);
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) x[i] = x[i] * inv * w[i];
+    if (p.rope != nullptr && ch < 2 * half) {
+      const int o = ch < half ? half : -half;            // the pair's other member
+      float y[VEC], cs[2 * VEC];
+      load_f32<VEC>((is_q ? p.q_weight : p.k_weight) + r + o, w);
+      load_f32<2 * VEC>(reinterpret_cast<const float*>(p.rope + (size_t)t * half + (ch < half ? ch : ch - half)), cs);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) {
+        y[i] = u[e + o + i] * inv * w[i];
+        x[i] = __fadd_rn(__fmul_rn(x[i], cs[2 * i]), __fmul_rn(y[i], ch < half ? -cs[2 * i + 1] : cs[2 * i + 1]));
+      }
+    }
+    if (is_q) RowUnit<T, VEC>::store(q_out + (size_t)t * p.q_out_stride + r, x);
+    else RowUnit<T, VEC>::store(k_cache + ((size_t)place + (size_t)h * p.page_size) * p.d + ch, x);
+  }
+  if (c.values_are_keys || place < 0) return;
+  for (int e = threadIdx.x * VEC; e < p.nkv * p.dv; e += kRowsThreads * VEC) {
+    float x[VEC];
+    RowUnit<T, VEC>::load(qkv + (size_t)t * p.qkv_stride + width + e, x);
+    RowUnit<T, VEC>::store(v_cache + ((size_t)place + (size_t)(e / p.dv) * p.page_size) * p.dv + e % p.dv, x);
+  }
+}
+
+// The sequences that bring several tokens: state <- their last taps - 1 raw inputs.
+template <typename T>
+__global__ void __launch_bounds__(256)
+conv_rows_state_kernel(const T* __restrict__ qkv, int ld, int width, int before, float* __restrict__ state, const int* __restrict__ cu_q,
+                       const int* __restrict__ slots) {
+  ilb::pdl_launch_dependents();
+  ilb::pdl_wait();
+  const int seq = blockIdx.y, e = blockIdx.x * 256 + threadIdx.x;
+  const int tok0 = cu_q[seq], n = cu_q[seq + 1] - tok0, slot = slots[seq];
+  if (e >= width || n <= 1 || slot < 0) return;
+  float* own = state + (size_t)slot * before * width + e;
+  for (int j = 0; j < before; ++j) {                     // (rows behind j are still the old ones)
+    const int at = n - before + j;
+    own[(size_t)j * width] = at >= 0 ? to_float(qkv[(size_t)(tok0 + at) * ld + e]) : own[(size_t)(j + n) * width];
+  }
+}
+
+// qkv [T, qkv_stride] of `dtype`: raw q | k (| v); n_several: whether a sequence of the step brings more than one token.
+ILB_EXPORT int ilb_conv_rows_norm_cache(
+    const void* qkv, void* q_out, int dtype, const float* conv_w, int taps, float* state, const float* q_weight, const float* k_weight,
+    float eps, const float* rope, int rotary_dim, const int* positions, const int* seq_of_token, const int* cu_q, const int* slots,
+    int n_seqs, int n_several, const int* block_table, int max_blocks, int page_size, int num_pages, void* k_cache, void* v_cache,
+    int n_tokens, int nq, int nkv, int d, int dv, int qkv_stride, int q_out_stride, int values_are_keys, cudaStream_t stream) {
+  ILB_REQUIRE(n_tokens >= 0 && nq > 0 && nkv > 0 && d > 0 && dv > 0 && eps > 0.f && n_seqs >= 0 && n_seqs <= 65535, "conv_rows_norm: bad sizes");
+  ILB_REQUIRE(conv_w != nullptr && taps >= 1 && (taps == 1 || state != nullptr), "conv_rows_norm: %d taps need weights and a state", taps);
+  ILB_REQUIRE(q_weight != nullptr && k_weight != nullptr, "conv_rows_norm: the norms' weights are missing");
+  ILB_REQUIRE(rope == nullptr || (rotary_dim > 0 && rotary_dim % 2 == 0 && rotary_dim <= d),
+              "conv_rows_norm: rotary dimension %d must be even and at most the head size %d", rotary_dim, d);
+  ILB_REQUIRE(!values_are_keys || dv == d, "conv_rows_norm: values that are keys have the keys' head size, found %d and %d", dv, d);
+  const int width = (nq + nkv) * d;
+  ILB_REQUIRE(qkv_stride >= width + (values_are_keys ? 0 : nkv * dv) && q_out_stride >= nq * d, "conv_rows_norm: strides too small");
+  ILB_REQUIRE((k_cache == nullptr) == (v_cache == nullptr), "conv_rows_norm: need both caches or none");
+  ILB_REQUIRE(k_cache == nullptr || (page_size > 0 && max_blocks > 0 && num_pages > 0), "conv_rows_norm: bad cache geometry");
+  ILB_REQUIRE(dtype == kF32 || dtype == kBF16, "conv_rows_norm: unknown dtype %d", dtype);
+  const size_t smem = sizeof(float) * width;
+  constexpr int kMost = 200 * 1024;
+  ILB_REQUIRE(smem <= kMost, "conv_rows_norm: rows of %d channels do not fit shared memory", width);
+  if (n_tokens == 0) return 0;
+  ConvRowsParams c{};
+  c.r.q_weight = q_weight; c.r.k_weight = k_weight; c.r.rope = (const float2*)rope; c.r.positions = positions; c.r.seq_of_token = seq_of_token;
+  c.r.block_table = block_table; c.r.max_blocks = max_blocks; c.r.page_size = page_size; c.r.num_pages = num_pages; c.r.nq = nq; c.r.nkv = nkv;
+  c.r.d = d; c.r.dv = dv; c.r.rotary_dim = rope != nullptr ? rotary_dim : 0; c.r.qkv_stride = qkv_stride; c.r.q_out_stride = q_out_stride; c.r.eps = eps;
+  c.conv_w = conv_w; c.state = state; c.cu_q = cu_q; c.slots = slots; c.taps = taps; c.values_are_keys = values_are_keys;
+  auto a16 = [](const void* x) { return (uintptr_t)x % 16 == 0; };
+  const bool vec = dtype == kBF16 && d % 8 == 0 && dv % 8 == 0 && (rope == nullptr || rotary_dim % 16 == 0) && qkv_stride % 8 == 0 && q_out_stride % 8 == 0 &&
+                   a16(qkv) && a16(q_out) && a16(k_cache) && a16(v_cache) && a16(q_weight) && a16(k_weight) && a16(conv_w) && a16(state) && a16(rope);
+  static OncePerDevice once;
+  if (smem > 48 * 1024 && once.first() &&
+      (cudaFuncSetAttribute(conv_rows_norm_kernel<__nv_bfloat16, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMost) != cudaSuccess ||
+       cudaFuncSetAttribute(conv_rows_norm_kernel<__nv_bfloat16, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMost) != cudaSuccess ||
+       cudaFuncSetAttribute(conv_rows_norm_kernel<float, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMost) != cudaSuccess)) {
+    once.forget();
+    return fail("conv_rows_norm: cannot reserve %d bytes of shared memory", kMost);
+  }
+#define ILB_CR(T, V) ilb::launch(conv_rows_norm_kernel<T, V>, dim3(n_tokens), dim3(kRowsThreads), smem, stream, (const T*)qkv, (T*)q_out, (T*)k_cache, (T*)v_cache, c)
+  if (vec) ILB_CR(__nv_bfloat16, 8);
+  else if (dtype == kBF16) ILB_CR(__nv_bfloat16, 1);
+  else ILB_CR(float, 1);
+#undef ILB_CR
+  if (int rc = check_launch("conv_rows_norm")) return rc;
+  if (!n_several || taps == 1 || n_seqs == 0) return 0;
+  const dim3 grid((width + 255) / 256, n_seqs);
+  if (dtype == kF32) ilb::launch(conv_rows_state_kernel<float>, grid, dim3(256), 0, stream, (const float*)qkv, qkv_stride, width, taps - 1, state, cu_q, slots);
+  else ilb::launch(conv_rows_state_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, (const __nv_bfloat16*)qkv, qkv_stride, width, taps - 1, state, cu_q, slots);
+  return check_launch("conv_rows_state");
+}
+
 // ---------------------------------------------------------------- means of blocks of cached rows
 // The token at position p completes block b = p / pool if (p + 1) % pool == 0: row b of the second set of pages becomes the
 // mean (32-bit sum) of the block's `pool` keys and of its values as the cache holds them.  One block of threads per block of

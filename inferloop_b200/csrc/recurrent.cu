@@ -13,9 +13,10 @@
 //   silu_rows   out = silu(x) of the leading columns of a projection, widened to 32-bit: the inputs of a linear
 //               attention whose queries, keys and values pass silu.
 //   rms_gate    out = y / sqrt(mean(y^2) + eps) * w * sigmoid(gate) * scale over a whole row, or over each of `groups`
-//               equal consecutive parts of it (one block a part).
+//               equal consecutive parts of it (one block a part); with `divisor` a part's y is divided by its own number first.
 //   head_gate   dst[t, h, :] = o[t, h, :] * sigmoid(g[t, h]) * scale: one gate a head on an attention's output (in place, or into
 //               the columns of a wider matrix).
+//   gate_rows   dst = o * sigmoid(g) element by element, rows of any stride.
 //
 // All arithmetic is 32-bit; the compute dtype is the storage type of the projections that come in and of the rows
 // that go to the next product.  A sequence whose slot is negative (a dummy row that pads a recorded launch) starts
@@ -267,7 +268,7 @@ ILB_EXPORT int ilb_silu_rows(const void* x, int dtype, int ld, float* out, int r
 template <typename TI>
 __global__ void __launch_bounds__(256)
 rms_gate_kernel(const float* __restrict__ y, const TI* __restrict__ gate, int ld_gate, const float* __restrict__ w,
-                TI* __restrict__ out, int ld_out, int width, float eps, float scale) {
+                TI* __restrict__ out, int ld_out, int width, float eps, float scale, const float* __restrict__ divisor) {
   ilb::pdl_launch_dependents();
   ilb::pdl_wait();
   __shared__ float scratch[33];
@@ -279,7 +280,8 @@ rms_gate_kernel(const float* __restrict__ y, const TI* __restrict__ gate, int ld
   float ss = 0.f;
   for (int i = threadIdx.x; i < width; i += blockDim.x) ss = fmaf(yr[i], yr[i], ss);
   ss = block_sum(ss, scratch);
-  const float inv = scale / sqrtf(ss / (float)width + eps);
+  const float by = divisor != nullptr ? 1.0f / divisor[(size_t)t * gridDim.y + part] : 1.0f;
+  const float inv = scale * by / sqrtf(ss * by * by / (float)width + eps);
   for (int i = threadIdx.x; i < width; i += blockDim.x)
     out[(size_t)t * ld_out + i] = from_float<TI>(yr[i] * inv * w[i] * sigmoid_f(to_float(gr[i])));
 }
@@ -290,7 +292,7 @@ constexpr int kGateKeep = 4;
 
 __global__ void __launch_bounds__(256)
 rms_gate_vec_kernel(const float* __restrict__ y, const __nv_bfloat16* __restrict__ gate, int ld_gate, const float* __restrict__ w,
-                    __nv_bfloat16* __restrict__ out, int ld_out, int width, float eps, float scale) {
+                    __nv_bfloat16* __restrict__ out, int ld_out, int width, float eps, float scale, const float* __restrict__ divisor) {
   ilb::pdl_launch_dependents();
   ilb::pdl_wait();
   __shared__ float scratch[33];
@@ -315,7 +317,8 @@ rms_gate_vec_kernel(const float* __restrict__ y, const __nv_bfloat16* __restrict
     ss = fmaf(v.x, v.x, ss); ss = fmaf(v.y, v.y, ss); ss = fmaf(v.z, v.z, ss); ss = fmaf(v.w, v.w, ss);
   }
   ss = block_sum(ss, scratch);
-  const float inv = scale / sqrtf(ss / (float)width + eps);
+  const float by = divisor != nullptr ? 1.0f / divisor[(size_t)t * gridDim.y + part] : 1.0f;
+  const float inv = scale * by / sqrtf(ss * by * by / (float)width + eps);
   auto write = [&](int i, const float4 v) {
     const uint2 g = gr[i];
     const float4 wv = wr[i];
@@ -342,7 +345,8 @@ constexpr int kPartWarps = 8, kPartKeep = 8;
 
 __global__ void __launch_bounds__(kPartWarps * 32)
 rms_gate_parts_kernel(const float* __restrict__ y, const __nv_bfloat16* __restrict__ gate, int ld_gate, const float* __restrict__ w,
-                      __nv_bfloat16* __restrict__ out, int ld_out, int rows, int groups, int part_width, float eps, float scale) {
+                      __nv_bfloat16* __restrict__ out, int ld_out, int rows, int groups, int part_width, float eps, float scale,
+                      const float* __restrict__ divisor) {
   ilb::pdl_launch_dependents();
   ilb::pdl_wait();
   const long long id = (long long)blockIdx.x * kPartWarps + (threadIdx.x >> 5);
@@ -364,7 +368,8 @@ rms_gate_parts_kernel(const float* __restrict__ y, const __nv_bfloat16* __restri
       ss = fmaf(keep[j].z, keep[j].z, ss); ss = fmaf(keep[j].w, keep[j].w, ss);
     }
   }
-  const float inv = scale / sqrtf(warp_sum(ss) / (float)part_width + eps);
+  const float by = divisor != nullptr ? 1.0f / divisor[id] : 1.0f;
+  const float inv = scale * by / sqrtf(warp_sum(ss) * by * by / (float)part_width + eps);
 #pragma unroll
   for (int j = 0; j < kPartKeep; ++j) {
     const int i = lane + 32 * j;
@@ -381,9 +386,9 @@ rms_gate_parts_kernel(const float* __restrict__ y, const __nv_bfloat16* __restri
 }
 
 // y: [rows, width] 32-bit; gate: [rows, ld_gate] of `dtype` (its first `width` columns from the pointer given);
-// out: [rows, ld_out] of `dtype` (its first `width` columns).
+// out: [rows, ld_out] of `dtype` (its first `width` columns); divisor: [rows, groups] or null.
 ILB_EXPORT int ilb_rms_gate(const float* y, const void* gate, int dtype, int ld_gate, const float* w, void* out, int ld_out, int rows,
-                            int width, int groups, float eps, float scale, cudaStream_t stream) {
+                            int width, int groups, float eps, float scale, const float* divisor, cudaStream_t stream) {
   ILB_REQUIRE(rows >= 0 && width > 0 && ld_gate >= width && ld_out >= width && eps > 0.f, "rms_gate: bad sizes");
   ILB_REQUIRE(groups > 0 && groups <= 65535 && width % groups == 0, "rms_gate: %d groups do not cut a row of %d", groups, width);
   if (rows == 0) return 0;
@@ -393,20 +398,20 @@ ILB_EXPORT int ilb_rms_gate(const float* y, const void* gate, int dtype, int ld_
     if (groups > 1 && part <= 4 * 32 * kPartKeep) {
       const long long blocks = ((long long)rows * groups + kPartWarps - 1) / kPartWarps;
       ilb::launch(rms_gate_parts_kernel, dim3((unsigned)blocks), dim3(kPartWarps * 32), 0, stream, y, (const __nv_bfloat16*)gate, ld_gate, w,
-                  (__nv_bfloat16*)out, ld_out, rows, groups, part, eps, scale);
+                  (__nv_bfloat16*)out, ld_out, rows, groups, part, eps, scale, divisor);
       return check_launch("rms_gate");
     }
     const int per = part / 4, vthreads = per >= 1024 ? 256 : (per >= 256 ? 128 : (per > 32 ? 64 : 32));
     ilb::launch(rms_gate_vec_kernel, dim3(rows, groups), dim3(vthreads), 0, stream, y, (const __nv_bfloat16*)gate, ld_gate, w, (__nv_bfloat16*)out, ld_out,
-                part, eps, scale);
+                part, eps, scale, divisor);
     return check_launch("rms_gate");
   }
   const int threads = part >= 1024 ? 256 : (part >= 256 ? 128 : 64);
   if (dtype == kF32)
-    ilb::launch(rms_gate_kernel<float>, dim3(rows, groups), dim3(threads), 0, stream, y, (const float*)gate, ld_gate, w, (float*)out, ld_out, part, eps, scale);
+    ilb::launch(rms_gate_kernel<float>, dim3(rows, groups), dim3(threads), 0, stream, y, (const float*)gate, ld_gate, w, (float*)out, ld_out, part, eps, scale, divisor);
   else if (dtype == kBF16)
     ilb::launch(rms_gate_kernel<__nv_bfloat16>, dim3(rows, groups), dim3(threads), 0, stream, y, (const __nv_bfloat16*)gate, ld_gate, w,
-                (__nv_bfloat16*)out, ld_out, part, eps, scale);
+                (__nv_bfloat16*)out, ld_out, part, eps, scale, divisor);
   else return fail("rms_gate: unknown dtype %d", dtype);
   return check_launch("rms_gate");
 }
@@ -469,6 +474,52 @@ ILB_EXPORT int ilb_head_gate(const void* o, void* dst, int ld_dst, const void* g
                 rows, heads, dv, scale);
   else return fail("head_gate: unknown dtype %d", dtype);
   return check_launch("head_gate");
+}
+
+// ---------------------------------------------------------------- a gate an element
+template <typename TI, int VEC>
+__global__ void __launch_bounds__(256)
+gate_rows_kernel(const TI* o, int ld_o, const TI* __restrict__ gate, int ld_gate, TI* dst, int ld_dst, int rows, int units) {
+  ilb::pdl_launch_dependents();
+  ilb::pdl_wait();
+  const size_t n = (size_t)rows * units;
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
+    const size_t r = i / units, c = (i % units) * VEC;
+    if constexpr (VEC == 8) {
+      const uint4 a = *reinterpret_cast<const uint4*>(o + r * ld_o + c), b = *reinterpret_cast<const uint4*>(gate + r * ld_gate + c);
+      const uint32_t av[4] = {a.x, a.y, a.z, a.w}, bv[4] = {b.x, b.y, b.z, b.w};
+      uint32_t w[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const __nv_bfloat162 v = __floats2bfloat162_rn(__uint_as_float(av[j] << 16) * sigmoid_t<true>(__uint_as_float(bv[j] << 16)),
+                                                       __uint_as_float(av[j] & 0xFFFF0000u) * sigmoid_t<true>(__uint_as_float(bv[j] & 0xFFFF0000u)));
+        w[j] = *reinterpret_cast<const uint32_t*>(&v);
+      }
+      *reinterpret_cast<uint4*>(dst + r * ld_dst + c) = make_uint4(w[0], w[1], w[2], w[3]);
+    } else {
+      dst[r * ld_dst + c] = from_float<TI>(to_float(o[r * ld_o + c]) * sigmoid_f(to_float(gate[r * ld_gate + c])));
+    }
+  }
+}
+
+// o [rows, ld_o], gate [rows, ld_gate], dst [rows, ld_dst] (it may be o), all of `dtype`, their first `width` columns.
+ILB_EXPORT int ilb_gate_rows(const void* o, int ld_o, const void* gate, int ld_gate, void* dst, int ld_dst, int dtype, int rows, int width,
+                             cudaStream_t stream) {
+  ILB_REQUIRE(rows >= 0 && width > 0 && ld_o >= width && ld_gate >= width && ld_dst >= width, "gate_rows: bad sizes");
+  ILB_REQUIRE(dtype == kF32 || dtype == kBF16, "gate_rows: unknown dtype %d", dtype);
+  if (rows == 0) return 0;
+  const bool vec = dtype == kBF16 && width % 8 == 0 && ld_o % 8 == 0 && ld_gate % 8 == 0 && ld_dst % 8 == 0 && ((uintptr_t)o % 16 == 0) &&
+                   ((uintptr_t)gate % 16 == 0) && ((uintptr_t)dst % 16 == 0);
+  const int units = vec ? width / 8 : width;
+  const size_t n = (size_t)rows * units;
+  const int blocks = (int)((n + 255) / 256 < 148 * 16 ? (n + 255) / 256 : 148 * 16);
+  if (vec) ilb::launch(gate_rows_kernel<__nv_bfloat16, 8>, dim3(blocks), dim3(256), 0, stream, (const __nv_bfloat16*)o, ld_o, (const __nv_bfloat16*)gate, ld_gate,
+                       (__nv_bfloat16*)dst, ld_dst, rows, units);
+  else if (dtype == kBF16)
+    ilb::launch(gate_rows_kernel<__nv_bfloat16, 1>, dim3(blocks), dim3(256), 0, stream, (const __nv_bfloat16*)o, ld_o, (const __nv_bfloat16*)gate, ld_gate,
+                (__nv_bfloat16*)dst, ld_dst, rows, units);
+  else ilb::launch(gate_rows_kernel<float, 1>, dim3(blocks), dim3(256), 0, stream, (const float*)o, ld_o, (const float*)gate, ld_gate, (float*)dst, ld_dst, rows, units);
+  return check_launch("gate_rows");
 }
 
 ILB_DEFINE_LAST_ERROR()

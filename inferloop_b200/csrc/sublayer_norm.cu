@@ -8,6 +8,8 @@
 //   gated_rows       out[t, k] = gelu_tanh(a[t, k]) * table[token[t], col0 + k]: a gate on a slice of a
 //                    per-token row of a table
 //
+//   branch_norms_add two sublayers side by side, each output normed by itself, their sum (times a constant) added, or normed again
+//                    and added to the stream (below)
 //   sum_norm         the other arrangement, x <- norm(keep * x + sublayer(x)) * g: y already holds the sum (below)
 //
 // Everything is 32-bit but what is stored in the compute dtype.  One block a token row.  The sum of squares of a
@@ -407,6 +409,121 @@ ILB_EXPORT int ilb_dyt_add(float* y, const float* alpha1, const float* g1, const
                 (__nv_bfloat16*)out, zero, total, width);
   else return fail("dyt_add: unknown dtype %d", out_dtype);
   return check_launch("dyt_add");
+}
+
+// ---------------------------------------------------------------- two branches, each normed, then the norm of their sum
+// z = mult (rms(a) wa + rms(b) wb); then y += z, or (w given) x += rms(z) w and out = the new x.  One block a row.  VEC: rows of
+// multiples of four that fit kBranchKeep vectors a thread stay in registers from the first read to the last write.
+constexpr int kBranchKeep = 4;
+
+__device__ __forceinline__ void block_sum2(float& u, float& v, float (&s)[2 * kNormWarps]) {
+  u = warp_sum(u);
+  v = warp_sum(v);
+  __syncthreads();
+  if ((threadIdx.x & 31) == 0) { s[threadIdx.x >> 5] = u; s[kNormWarps + (threadIdx.x >> 5)] = v; }
+  __syncthreads();
+  u = 0.f; v = 0.f;
+#pragma unroll
+  for (int i = 0; i < kNormWarps; ++i) { u += s[i]; v += s[kNormWarps + i]; }
+}
+
+template <typename TO, bool VEC>
+__global__ void __launch_bounds__(kNormThreads)
+branch_norms_add_kernel(const float* __restrict__ a, const float* __restrict__ b, const float* __restrict__ wa, const float* __restrict__ wb,
+                        float eps, float mult, float* __restrict__ y, const float* __restrict__ w, float w_eps, float* __restrict__ x,
+                        TO* __restrict__ out, int width) {
+  ilb::pdl_launch_dependents();
+  ilb::pdl_wait();
+  __shared__ float s[2 * kNormWarps];
+  const size_t at = (size_t)blockIdx.x * width;
+  float sa = 0.f, sb = 0.f;
+  if constexpr (VEC) {
+    const int n4 = width / 4;
+    const float4 *a4 = reinterpret_cast<const float4*>(a + at), *b4 = reinterpret_cast<const float4*>(b + at);
+    const float4 *wa4 = reinterpret_cast<const float4*>(wa), *wb4 = reinterpret_cast<const float4*>(wb), *w4 = reinterpret_cast<const float4*>(w);
+    float4 va[kBranchKeep], vb[kBranchKeep], old[kBranchKeep];
+    float4* into = reinterpret_cast<float4*>((w != nullptr ? x : y) + at);
+#pragma unroll
+    for (int k = 0; k < kBranchKeep; ++k) {
+      const int i = threadIdx.x + k * kNormThreads;
+      const bool on = i < n4;
+      va[k] = on ? a4[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+      vb[k] = on ? b4[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+      old[k] = on ? into[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+      sa = fmaf(va[k].x, va[k].x, sa); sa = fmaf(va[k].y, va[k].y, sa); sa = fmaf(va[k].z, va[k].z, sa); sa = fmaf(va[k].w, va[k].w, sa);
+      sb = fmaf(vb[k].x, vb[k].x, sb); sb = fmaf(vb[k].y, vb[k].y, sb); sb = fmaf(vb[k].z, vb[k].z, sb); sb = fmaf(vb[k].w, vb[k].w, sb);
+    }
+    block_sum2(sa, sb, s);
+    const float ia = mult / sqrtf(sa / (float)width + eps), ib = mult / sqrtf(sb / (float)width + eps);
+    float ss = 0.f, unused = 0.f;
+#pragma unroll
+    for (int k = 0; k < kBranchKeep; ++k) {
+      const int i = threadIdx.x + k * kNormThreads;
+      if (i < n4) {
+        const float4 p = wa4[i], q = wb4[i];
+        va[k] = make_float4(fmaf(va[k].x * ia, p.x, vb[k].x * ib * q.x), fmaf(va[k].y * ia, p.y, vb[k].y * ib * q.y),
+                            fmaf(va[k].z * ia, p.z, vb[k].z * ib * q.z), fmaf(va[k].w * ia, p.w, vb[k].w * ib * q.w));
+        ss = fmaf(va[k].x, va[k].x, ss); ss = fmaf(va[k].y, va[k].y, ss); ss = fmaf(va[k].z, va[k].z, ss); ss = fmaf(va[k].w, va[k].w, ss);
+      }
+    }
+    float inv = 1.f;
+    if (w != nullptr) {
+      block_sum2(ss, unused, s);
+      inv = 1.0f / sqrtf(ss / (float)width + w_eps);
+    }
+#pragma unroll
+    for (int k = 0; k < kBranchKeep; ++k) {
+      const int i = threadIdx.x + k * kNormThreads;
+      if (i < n4) {
+        const float4 g = w != nullptr ? w4[i] : make_float4(1.f, 1.f, 1.f, 1.f);
+        const float4 r = make_float4(fmaf(va[k].x * inv, g.x, old[k].x), fmaf(va[k].y * inv, g.y, old[k].y), fmaf(va[k].z * inv, g.z, old[k].z),
+                                     fmaf(va[k].w * inv, g.w, old[k].w));
+        into[i] = r;
+        if (out != nullptr) {
+          if constexpr (sizeof(TO) == 4) {
+            reinterpret_cast<float4*>(out + at)[i] = r;
+          } else {
+            __nv_bfloat162 lo = __floats2bfloat162_rn(r.x, r.y), hi = __floats2bfloat162_rn(r.z, r.w);
+            reinterpret_cast<uint2*>(out + at)[i] = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
+          }
+        }
+      }
+    }
+  } else {
+    for (int i = threadIdx.x; i < width; i += kNormThreads) { sa = fmaf(a[at + i], a[at + i], sa); sb = fmaf(b[at + i], b[at + i], sb); }
+    block_sum2(sa, sb, s);
+    const float ia = mult / sqrtf(sa / (float)width + eps), ib = mult / sqrtf(sb / (float)width + eps);
+    auto z = [&](int i) { return fmaf(a[at + i] * ia, wa[i], b[at + i] * ib * wb[i]); };
+    float inv = 1.f;
+    if (w != nullptr) {
+      float ss = 0.f, unused = 0.f;
+      for (int i = threadIdx.x; i < width; i += kNormThreads) { const float v = z(i); ss = fmaf(v, v, ss); }
+      block_sum2(ss, unused, s);
+      inv = 1.0f / sqrtf(ss / (float)width + w_eps);
+    }
+    float* into = (w != nullptr ? x : y) + at;
+    for (int i = threadIdx.x; i < width; i += kNormThreads) {
+      const float r = fmaf(z(i) * inv, w != nullptr ? w[i] : 1.f, into[i]);
+      into[i] = r;
+      if (out != nullptr) out[at + i] = from_float<TO>(r);
+    }
+  }
+}
+
+// a, b, y, x: [rows, width] 32-bit; out [rows, width] of `dtype` or null.  Either y (the sum is added into it), or w and x.
+ILB_EXPORT int ilb_branch_norms_add(const float* a, const float* b, const float* wa, const float* wb, float eps, float mult, float* y,
+                                    const float* w, float w_eps, float* x, void* out, int dtype, int rows, int width, cudaStream_t stream) {
+  ILB_REQUIRE(rows >= 0 && width > 0 && eps > 0.f && wa != nullptr && wb != nullptr, "branch_norms_add: bad sizes");
+  ILB_REQUIRE((w != nullptr) == (x != nullptr) && (w != nullptr) == (y == nullptr) && (w == nullptr || w_eps > 0.f), "branch_norms_add: a sum, or a norm and a stream");
+  ILB_REQUIRE(dtype == kF32 || dtype == kBF16, "branch_norms_add: unknown dtype %d", dtype);
+  if (rows == 0) return 0;
+  auto a16 = [](const void* p) { return (uintptr_t)p % 16 == 0; };
+  const bool vec = width % 4 == 0 && width / 4 <= kBranchKeep * kNormThreads && a16(a) && a16(b) && a16(wa) && a16(wb) && a16(y) && a16(w) && a16(x) && a16(out);
+#define ILB_BN(TO, V) ilb::launch(branch_norms_add_kernel<TO, V>, dim3(rows), dim3(kNormThreads), 0, stream, a, b, wa, wb, eps, mult, y, w, w_eps, x, (TO*)out, width)
+  if (dtype == kF32) { if (vec) ILB_BN(float, true); else ILB_BN(float, false); }
+  else { if (vec) ILB_BN(__nv_bfloat16, true); else ILB_BN(__nv_bfloat16, false); }
+#undef ILB_BN
+  return check_launch("branch_norms_add");
 }
 
 ILB_DEFINE_LAST_ERROR()

@@ -36,8 +36,14 @@ window's tokens a position sees, in the same softmax, the mean key and the mean 
 lies wholly before its window.  The means are rows of a second set of pages (one row per P tokens), made as soon as a block's
 last token is cached; the tokens' own pages go when both the window and their block are done with them.
 
+`chunk` = n: a position sees the earlier ones of its own aligned chunk of n positions (counted from the sequence's start).
+`conv` = taps (with norms over whole rows): queries and keys pass a causal convolution over time per channel (weights
+[channels, taps], no bias) between the projection and the norm; the last taps - 1 projected values are state of the request.
+`values` = "keys" (with `conv`): there is no value matrix, the values are the keys as they leave the convolution, before their norm.
+
 `output_gate` = "head": head h's output is multiplied by sigmoid((W_g x)_h), one number a head from a matrix
-[heads, hidden] whose rows ride behind q|k|v in the one projection.  `out_scale`: a constant on the whole mixer's
+[heads, hidden] whose rows ride behind q|k|v in the one projection; "element": every element of the heads' outputs by its own
+sigmoid, from a matrix [heads * v_head_dim, hidden].  `out_scale`: a constant on the whole mixer's
 output (a mixer that runs beside another one), applied in 32-bit to what the output projection reads and to its bias.
 """
 from __future__ import annotations
@@ -50,7 +56,7 @@ import torch
 from ..csrc import ops
 from ..weights.decl import WeightDecl
 from . import registry
-from .base import CacheNeeds, Mixer, PagedKVNeed
+from .base import CacheNeeds, Mixer, PagedKVNeed, SlotStateNeed
 from .linear import linear
 
 
@@ -83,6 +89,15 @@ class GQAttention(Mixer):
         self.bias = bool(bias)                               # q, k, v
         self.out_bias = bias is True
         self.window = spec.get("window")
+        chunk = spec.get("chunk")
+        if chunk and self.window:
+            raise ValueError("attention: keys are limited by a window or by aligned chunks, not both")
+        self.chunk = int(chunk or 0)
+        self.seen = -self.chunk if self.chunk else int(self.window or 0)      # as the attention kernels take it
+        self.taps = int(spec.get("conv") or 0)
+        self.values_are_keys = spec.get("values") == "keys"
+        if spec.get("values") not in (None, "keys"):
+            raise ValueError(f"values must be None or 'keys', found {spec.get('values')!r}")
         self.scale = float(spec["scale"]) if spec.get("scale") is not None else 1.0 / math.sqrt(self.d)
         self.value_mix = spec.get("value_mix")
         if self.value_mix not in (None, "first", "mixed"):
@@ -99,12 +114,16 @@ class GQAttention(Mixer):
         self.head_mix = bool(spec.get("head_mix", False))
         self.has_sink = bool(spec.get("sink", False))
         self.output_gate = spec.get("output_gate")
-        if self.output_gate not in (None, "head"):
-            raise ValueError(f"output_gate must be None or 'head', found {self.output_gate!r}")
+        if self.output_gate not in (None, "head", "element"):
+            raise ValueError(f"output_gate must be None, 'head' or 'element', found {self.output_gate!r}")
         self.out_scale = float(spec.get("out_scale", 1.0))
-        if self.out_scale != 1.0 and not self.output_gate:
-            raise ValueError("attention: a constant on the output is applied by the gate's kernel (output_gate)")
-        self.gate_rows = -(-self.nq // 8) * 8 if self.output_gate else 0      # (padded: the projection's rows stay multiples of 16 bytes)
+        if self.out_scale != 1.0 and self.output_gate != "head":
+            raise ValueError("attention: a constant on the output is applied by the heads' gates (output_gate='head')")
+        self.n_gates = {None: 0, "head": self.nq, "element": self.nq * self.dv}[self.output_gate]
+        self.v_cols = 0 if self.values_are_keys else self.nkv * self.dv
+        # (padded: the projection's rows stay multiples of 16 bytes)
+        self.gate_rows = self.n_gates + -((self.nq + self.nkv) * self.d + self.v_cols + self.n_gates) % 8 if self.output_gate == "element" \
+            else -(-self.nq // 8) * 8 if self.output_gate else 0
         self.shaped = bool(self.temp_coef or self.softcap or self.distance_bias or self.head_mix)
         if self.shaped and self.value_mix is not None:
             raise ValueError("attention: reshaped scores and mixed values are not served together")
@@ -122,11 +141,16 @@ class GQAttention(Mixer):
                                   or getattr(self.position, "interleaved", False)):
             raise ValueError("attention: norms over whole rows are served before a half-split rotation, with a plain softmax and unmixed values")
         self.rotary_dim = int(spec["position"].get("rotary_dim", 0))
+        if (self.taps or self.values_are_keys) and (not self.taps or not self.qk_norm_rows or self.value_position is not None or self.pool or self.bias):
+            raise ValueError("attention: convolutions (and values that are keys behind one) are served with norms over whole rows, without biases, "
+                             "turned values and pooled blocks")
+        if self.values_are_keys and self.dv != self.d:
+            raise ValueError(f"attention: values that are keys have the keys' head size, found {self.dv} and {self.d}")
         p = prefix
         names = {"q": "q_proj.weight", "k": "k_proj.weight", "v": "v_proj.weight", "o": "o_proj.weight",
                  "qb": "q_proj.bias", "kb": "k_proj.bias", "vb": "v_proj.bias", "ob": "o_proj.bias",
                  "qn": "q_norm.weight", "kn": "k_norm.weight", "vmix": "v_mix",
-                 "r1": "r1", "r2": "r2", "head_mix": "talk", "sink": "sink", "g": "gate.weight"}
+                 "r1": "r1", "r2": "r2", "head_mix": "talk", "sink": "sink", "g": "gate.weight", "qc": "q_conv.weight", "kc": "k_conv.weight"}
         for role, name in spec.get("names", ()):
             if role not in names:
                 raise ValueError(f"attention has no tensor role {role!r}")
@@ -136,13 +160,17 @@ class GQAttention(Mixer):
                      | (ops.NORM_AFTER_ROTATION if self.qk_norm_after else 0)
                      | (ops.NORM_UNWEIGHTED if self.qk_norm_unweighted else 0))
         self.w_qkv = self.b_qkv = self.w_o = self.b_o = self.q_norm = self.k_norm = self.v_lambda = None
-        self.r1 = self.r2 = self.mix = self.sink = None
+        self.r1 = self.r2 = self.mix = self.sink = self.conv_w = None
 
     # ------------------------------------------------------------------ weights
     def declare_weights(self) -> List[WeightDecl]:
         n, d, dv, H = self.names, self.d, self.dv, self.hidden
-        out = [WeightDecl(n["q"], (self.nq * d, H)), WeightDecl(n["k"], (self.nkv * d, H)),
-               WeightDecl(n["v"], (self.nkv * dv, H)), WeightDecl(n["o"], (H, self.nq * dv))]
+        out = [WeightDecl(n["q"], (self.nq * d, H)), WeightDecl(n["k"], (self.nkv * d, H))]
+        if not self.values_are_keys:
+            out.append(WeightDecl(n["v"], (self.nkv * dv, H)))
+        out.append(WeightDecl(n["o"], (H, self.nq * dv)))
+        if self.taps:
+            out += [WeightDecl(n["qc"], (self.nq * d, self.taps), "vector", "mix"), WeightDecl(n["kc"], (self.nkv * d, self.taps), "vector", "mix")]
         if self.bias:
             out += [WeightDecl(n["qb"], (self.nq * d,), "vector", "bias"),
                     WeightDecl(n["kb"], (self.nkv * d,), "vector", "bias"),
@@ -160,7 +188,7 @@ class GQAttention(Mixer):
         if self.has_sink:
             out.append(WeightDecl(n["sink"], (self.nq,), "vector", "around_zero"))
         if self.output_gate:
-            out.append(WeightDecl(n["g"], (self.nq, H)))
+            out.append(WeightDecl(n["g"], (self.n_gates, H)))
         if self.value_mix == "mixed":
             out.append(WeightDecl(n["vmix"], (), "vector", "mix"))
         elif bool(self.spec.get("value_mix_tensor_unused", False)):
@@ -169,10 +197,10 @@ class GQAttention(Mixer):
 
     def bind(self, tensors: Mapping[str, torch.Tensor]) -> None:
         n = self.names
-        rows = [tensors[n["q"]], tensors[n["k"]], tensors[n["v"]]]
+        rows = [tensors[n["q"]], tensors[n["k"]]] + ([] if self.values_are_keys else [tensors[n["v"]]])
         if self.output_gate:
             g = tensors[n["g"]]
-            rows += [g, g.new_zeros(self.gate_rows - self.nq, self.hidden)]
+            rows += [g, g.new_zeros(self.gate_rows - self.n_gates, self.hidden)]
         self.w_qkv = torch.cat(rows, dim=0).contiguous()
         self.w_o = tensors[n["o"]].contiguous()
         if self.bias:
@@ -182,6 +210,8 @@ class GQAttention(Mixer):
             self.b_qkv = torch.cat(biases).contiguous()
         if self.out_bias:
             self.b_o = (tensors[n["ob"]] * self.out_scale).contiguous() if self.out_scale != 1.0 else tensors[n["ob"]].contiguous()
+        if self.taps:          # [taps, channels]: a tap's weights side by side
+            self.conv_w = torch.cat([tensors[n["qc"]], tensors[n["kc"]]], dim=0).t().contiguous()
         if self.value_mix == "mixed":
             self.v_lambda = tensors[n["vmix"]].reshape(1).contiguous()
         if self.qk_norm or self.qk_norm_rows:
@@ -197,14 +227,16 @@ class GQAttention(Mixer):
     def cache_needs(self) -> CacheNeeds:
         v_dim = self.dv if self.dv != self.d else None
         if not self.pool:
-            return CacheNeeds(paged=PagedKVNeed(self.nkv, self.d, self.window, v_dim))
+            # (no token looks back beyond its own chunk)
+            slots = (SlotStateNeed("conv", (self.taps - 1, (self.nq + self.nkv) * self.d), torch.float32),) if self.taps else ()
+            return CacheNeeds(paged=PagedKVNeed(self.nkv, self.d, self.chunk or self.window, v_dim), slots=slots)
         # a token is read while it is in the window, and until its block is complete
         return CacheNeeds(paged=PagedKVNeed(self.nkv, self.d, max(self.window, self.pool), v_dim),
                           pooled=PagedKVNeed(self.nkv, self.d, None, v_dim, self.pool))
 
     def scratch_bytes(self, tokens: int) -> int:
         size = torch.empty((), dtype=self.ctx.dtype).element_size()
-        width = (self.nq + self.nkv) * self.d + self.nkv * self.dv + self.gate_rows
+        width = (self.nq + self.nkv) * self.d + self.v_cols + self.gate_rows
         kept = self.nkv * self.dv if self.value_mix else 0
         return tokens * ((width + self.nq * (self.d + self.dv) + kept) * size + self.rotary_dim * 4)
 
@@ -221,7 +253,7 @@ class GQAttention(Mixer):
     def forward(self, x: torch.Tensor, residual: torch.Tensor, step, cache) -> None:
         T = x.shape[0]
         ws, dt = self.ctx.workspace, self.ctx.dtype
-        width = (self.nq + self.nkv) * self.d + self.nkv * self.dv + self.gate_rows
+        width = (self.nq + self.nkv) * self.d + self.v_cols + self.gate_rows
         qkv = ws.buffer("attn.qkv", (T, width), dt)
         ops.scope("attention.qkv_projection")
         linear(x, self.w_qkv, qkv, self.b_qkv)
@@ -239,7 +271,7 @@ class GQAttention(Mixer):
         the caller."""
         T = qkv.shape[0]
         ws, dt = self.ctx.workspace, self.ctx.dtype
-        gate_col0 = (self.nq + self.nkv) * self.d + self.nkv * self.dv      # the heads' gate logits ride behind q | k | v
+        gate_col0 = (self.nq + self.nkv) * self.d + self.v_cols      # the gates' logits ride behind q | k | v
         table = step.block_tables[cache.group]
         ops.scope("attention.position_table")
         rope = self.position.table(step)
@@ -260,7 +292,7 @@ class GQAttention(Mixer):
             o = ws.buffer("attn.o", (T, self.nq * self.d), dt)
             ops.scope("attention.decode (q/k norm, rotation, cache write inside)")
             ops.attention_decode_fused(qkv, o, self.q_norm, self.k_norm, self.qk_norm_eps, rope, cache.k, cache.v,
-                                       cache.writable, step.positions, step.cu_q, table, self.window or 0, self.scale,
+                                       cache.writable, step.positions, step.cu_q, table, self.seen, self.scale,
                                        step.n_seqs, self.nq, self.nkv, self.d,
                                        long_context=step.max_kv_len >= ops.DECODE_LONG_CONTEXT, mode=self.mode,
                                        rotary_dim=self.rotary_dim or None, v_first=v_first,
@@ -279,12 +311,12 @@ class GQAttention(Mixer):
         o = ws.buffer("attn.o", (T, self.nq * self.dv), dt)
         ops.scope("attention.attention")
         if self.shaped:
-            ops.attention_mixed_heads(q, o, cache.k, cache.v, step, table, self.window or 0, self.scale, self.nq, self.nkv,
+            ops.attention_mixed_heads(q, o, cache.k, cache.v, step, table, self.seen, self.scale, self.nq, self.nkv,
                                       self.d, self.dv, sink=self.sink, head_mix=self.mix, dist_r1=self.r1, dist_r2=self.r2,
                                       softcap=self.softcap, temp_coef=self.temp_coef, temp_every=self.temp_every,
                                       workspace=ws, decode_chunk=ops.DECODE_CHUNK_MIN)
         else:
-            ops.attention(q, o, cache.k, cache.v, step, table, self.window or 0, self.scale,
+            ops.attention(q, o, cache.k, cache.v, step, table, self.seen, self.scale,
                           self.nq, self.nkv, self.d, workspace=ws, decode_chunk=self.decode_chunk, dv=self.dv, sink=self.sink)
         self._finish(o, qkv, gate_col0, residual, out)
 
@@ -300,22 +332,31 @@ class GQAttention(Mixer):
             pooled = ops.PooledRows(self.pool, cache.pooled.k, cache.pooled.v, step.block_tables[cache.pooled.group])
         # (a step of single tokens: a block's other rows are cached already, and the input stage makes its mean too)
         inside = pooled is not None and cache.writable and step.decode_only
-        ops.rows_norm_rope_cache(qkv, q, self.q_norm, self.k_norm, self.qk_norm_eps, rope, self.rotary_dim, v_rope, step, table,
-                                 cache.k if cache.writable else None, cache.v if cache.writable else None, self.nq, self.nkv, self.d, self.dv,
-                                 pooled=pooled if inside else None)
+        if self.taps:
+            ops.conv_rows_norm_cache(qkv, q, self.conv_w, cache.state["conv"], self.q_norm, self.k_norm, self.qk_norm_eps, rope, self.rotary_dim,
+                                     step, table, cache.k if cache.writable else None, cache.v if cache.writable else None, self.nq, self.nkv,
+                                     self.d, self.dv, values_are_keys=self.values_are_keys)
+        else:
+            ops.rows_norm_rope_cache(qkv, q, self.q_norm, self.k_norm, self.qk_norm_eps, rope, self.rotary_dim, v_rope, step, table,
+                                     cache.k if cache.writable else None, cache.v if cache.writable else None, self.nq, self.nkv, self.d, self.dv,
+                                     pooled=pooled if inside else None)
         if pooled is not None and cache.writable and not inside:
             ops.scope("attention.block_means")
             ops.pool_means(cache.k, cache.v, pooled, step, table)
         o = ws.buffer("attn.o", (T, self.nq * self.dv), dt)
         ops.scope("attention.attention")
-        ops.attention(q, o, cache.k, cache.v, step, table, self.window or 0, self.scale, self.nq, self.nkv, self.d, workspace=ws,
+        ops.attention(q, o, cache.k, cache.v, step, table, self.seen, self.scale, self.nq, self.nkv, self.d, workspace=ws,
                       decode_chunk=self.decode_chunk, dv=self.dv, pooled=pooled, turn=v_rope)
         self._finish(o, qkv, gate_col0, residual, out)
 
     def _finish(self, o: torch.Tensor, qkv: torch.Tensor, gate_col0: int, residual: torch.Tensor, out: Optional[torch.Tensor]) -> None:
         """The gate a head and the mixer's constant on what the output product reads, then that product (or, with `out`,
         the gated rows into the caller's matrix)."""
-        if self.output_gate:
+        if self.output_gate == "element":
+            ops.scope("attention.output_gate")
+            gated = out if out is not None else o
+            ops.gate_rows(o, qkv[:, gate_col0:], gated)
+        elif self.output_gate:
             ops.scope("attention.output_gate")
             ops.head_gate(o, qkv[:, gate_col0:], self.nq, self.out_scale, out=out)
         elif out is not None:

@@ -156,8 +156,16 @@ class OutputNormBlock(Block):
         if memo is None or memo.pop(self.PREPARED, None) != prepared:
             ops.scope("norm")
             ops.cast_zero(hidden, x, y)
+        branches = getattr(self.mixer, "normed_branches", False)
         for i, (norm, run) in enumerate(subs):
             ops.scope("mixer" if i == 0 else "feed_forward")
+            if i == 0 and branches and norm.groups == 1:
+                # the branches' norms, their sum, its norm and the stream's sum in one launch; nothing was added into y
+                outputs, weights, eps, mult = self.mixer.forward_branches(x, step, cache)
+                ops.scope("norm")
+                ops.branch_norms_add(outputs, weights, eps, mult, norm=(norm.weight, norm.eps), x=hidden,
+                                     out=x if len(subs) > 1 or memo is not None else None)
+                continue
             run(x, y, step, cache)
             ops.scope("norm")
             if i + 1 < len(subs) or memo is not None:

@@ -21,7 +21,8 @@ What a description may add (all spec parameters; absent, the layer is the one ab
                     s_ij = scale * (qa_i . Uk c_j + qr_i . kr_j).  The cache row is [c | rotated kr]: the score
                     stays one dot product over rank + t elements between [Uk^T qa | rotated qr] and the row,
                     and the kernels' output keeps only its first `rank` columns for Uv.  `position` names the
-                    rotation (pairs of neighbours over the first `rotary_dim` of the t elements).
+                    rotation (pairs of neighbours, or of elements half of it apart, over the first `rotary_dim` of
+                    the t elements).
   `own_cache` = False   the layer has no W_dkv: the run order lets it read another layer's rows, written
                     (normed and rotated) by that layer; its own Uk, Uv, queries and everything else.
 """
@@ -57,8 +58,7 @@ class LatentAttention(Mixer):
         self.own_cache = bool(spec.get("own_cache", True))
         self.position = registry.build("position", spec["position"], ctx) if spec.get("position") is not None else None
         self.rot = int(spec["position"].get("rotary_dim", 0)) if self.position is not None and self.tail else 0
-        if self.tail and self.position is not None and not getattr(self.position, "interleaved", False) and self.rot:
-            raise ValueError("latent attention: the rotated part turns in pairs of neighbours (position kind rope_interleaved)")
+        self.half_split = bool(self.rot) and not getattr(self.position, "interleaved", False)
         if self.rot > self.tail:
             raise ValueError(f"latent attention: {self.rot} rotated elements in a part of {self.tail}")
         self.general = bool(self.q_rank or self.tail or not self.own_cache)
@@ -149,7 +149,8 @@ class LatentAttention(Mixer):
         if write or tail:
             ops.latent_write_rot(proj, q_cols, r, tail, self.rot, angles, self.latent_norm if write else None, self.eps, step,
                                  table if write else None, cache.k if write else None,
-                                 q_src if tail else None, q if tail else None, q_col0=d, q_head_stride=qh, heads=H)
+                                 q_src if tail else None, q if tail else None, q_col0=d, q_head_stride=qh, heads=H,
+                                 half_split=self.half_split)
         ops.scope("attention.queries_to_latent")
         ops.head_matmul(q_src, self.up_k, q, x_head_stride=qh, out_head_stride=row)
         ops.scope("attention.attention")

@@ -36,7 +36,7 @@ class SwiGLU(FeedForward):
                 raise ValueError(f"swiglu has no tensor role {role!r}")
             names[role] = name
         self.names = {k: prefix + v for k, v in names.items()}
-        # what the gate passes through: "silu" (SwiGLU) or "relu"; or a PartSpec of kind "clamped_glu" (limit, sharpness,
+        # what the gate passes through: "silu" (SwiGLU), "relu" or "gelu_tanh"; or a PartSpec of kind "clamped_glu" (limit, sharpness,
         # up_offset): a(min(gate, limit)) * (clamp(up, -limit, limit) + up_offset) with a(g) = g * sigmoid(sharpness * g)
         act = spec.get("activation", "silu")
         self.glu = None

@@ -9,8 +9,8 @@
   y += sigmoid(W_gate x) * shared(x)    when the description has a shared expert (`shared_inter`;
   `shared_gate` False leaves the multiplier out)
   (`correction`: the experts are ranked by s + c with a stored vector c, the weights stay s;  `groups` = (count, keep):
-  the experts form `count` equal groups of neighbours, a group ranks by its best member, and only experts of the best
-  `keep` groups can be chosen;  `renorm_eps` joins the sum that `renormalize` divides by;  `route_scale` multiplies the weights)
+  the experts form `count` equal groups of neighbours, a group ranks by its best member (`group_rank` "best_two": by its two
+  best together), and only experts of the best `keep` groups can be chosen;  `renorm_eps` joins the sum that `renormalize` divides by;  `route_scale` multiplies the weights)
 
 The experts' matrices are stacked at load into [experts, 2 I, H] (gate rows, then up rows) and
 [experts, H, I].  A step sorts its (token, choice) pairs by expert on the device into rows
@@ -54,6 +54,10 @@ class RoutedExperts(FeedForward):
         self.correction = bool(spec.get("correction", False))         # a vector added to the scores for the ranking alone
         groups = spec.get("groups")
         self.groups, self.keep = (int(groups[0]), int(groups[1])) if groups else (1, 1)
+        group_rank = str(spec.get("group_rank", "best"))
+        if group_rank not in ("best", "best_two"):
+            raise ValueError(f"group_rank must be 'best' or 'best_two', found {group_rank!r}")
+        self.group_best_two = group_rank == "best_two"
         self.route_scale = float(spec.get("route_scale", 1.0))
         self.renorm_eps = float(spec.get("renorm_eps", 0.0))
         if self.groups < 1 or self.experts % self.groups or not 1 <= self.keep <= self.groups or self.groups > 32:
@@ -166,7 +170,8 @@ class RoutedExperts(FeedForward):
         choice = ws.buffer("moe.choice", (T * K,), torch.int32)
         weight = ws.buffer("moe.weight", (T * K,), torch.float32)
         ops.moe_route(logits, E, K, self.score == "softmax", self.renormalize, choice, weight, bias=self.b_router,
-                      correction=self.c_router, groups=self.groups, keep=self.keep, scale=self.route_scale, renorm_eps=self.renorm_eps)
+                      correction=self.c_router, groups=self.groups, keep=self.keep, scale=self.route_scale, renorm_eps=self.renorm_eps,
+                      group_best_two=self.group_best_two)
         pos = ws.buffer("moe.pos", (T * K,), torch.int32)
         block_expert = ws.buffer("moe.block_expert", (rows // block,), torch.int32)
         ops.moe_plan(choice, E, block, pos, block_expert)

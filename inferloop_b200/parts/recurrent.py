@@ -26,8 +26,19 @@ w = exp(-c sigmoid(W_2 tanh(W_1 h) + w0)), a = sigmoid(a + ab), u = k / sqrt(sum
 each head's o is RMS-normed by itself, the heads together are multiplied by a weight and by sigmoid(g), and projected.  State
 per request: S [heads, dim, vdim] in 32-bit.  All projections of h are one product; the kernels are csrc/delta.cu.
 
+`mlstm` (the matrix memory of xLSTM): q, k, v, g = projections of h and two gate logits a head,
+
+    i = cap tanh((W_i h + b_i) / cap),  f = logsigmoid(cap tanh((W_f h + b_f) / cap)),  m_t = max(f + m_{t-1}, i)
+    S_t = exp(f + m_{t-1} - m_t) S_{t-1} + exp(i - m_t) k v^T,  n_t likewise with k alone
+    o_t = S_t^T q / sqrt(dim) / (max(|n_t . q| / sqrt(dim), exp(-m_t)) + den_eps)
+
+each head's o is RMS-normed by itself, the heads together are multiplied by a weight and by sigmoid(g), and projected.  State
+per request: S [heads, dim, vdim], n [heads, dim] and m [heads] in 32-bit, all zero at the start.  The gates' logits are 32-bit
+dot products with the mixer's input; the kernels are csrc/mlstm.cu.
+
 `parallel`: several mixers read the same input and add into the same output, each with its own tensors under its
-own prefix, its own cache (at most one of them paged) and its own constant on its output.
+own prefix, its own cache (at most one of them paged) and its own constant on its output.  With `out_norms` every branch's
+output is RMS-normed over its whole row first, with a weight of its own, and the sum of the normed rows times `out_mult` is added.
 """
 from __future__ import annotations
 
@@ -294,6 +305,105 @@ class GeneralDelta(Mixer):
         linear(gated, self.w_o, residual, accumulate=True)
 
 
+class MatrixMemory(Mixer):
+    """spec: hidden_size, heads, head_dim, v_head_dim, eps (the norm of a head), gate_cap, den_eps, names."""
+    graph_safe = True
+    reads_input = True                       # `forward_projected` needs the mixer's input too (the gates' dot products)
+
+    def __init__(self, spec, ctx, prefix: str = "") -> None:
+        super().__init__(spec, ctx, prefix)
+        self.hidden = int(spec["hidden_size"])
+        self.heads = int(spec["heads"])
+        self.d = int(spec["head_dim"])
+        self.dv = int(spec["v_head_dim"])
+        self.eps = float(spec["eps"])
+        self.cap = float(spec["gate_cap"])
+        self.den_eps = float(spec.get("den_eps", 1e-6))
+        if self.cap <= 0:
+            raise ValueError("mlstm: gate_cap must be positive")
+        if self.d > ops.MLSTM_MAX_ROWS:
+            raise ValueError(f"mlstm: a state of {self.d} rows exceeds {ops.MLSTM_MAX_ROWS}")
+        self.inner_k, self.inner_v = self.heads * self.d, self.heads * self.dv
+        self.names = _names({"q": "q", "k": "k", "v": "v", "g": "g", "i": "i", "ib": "i.b", "f": "f", "fb": "f.b", "norm": "norm", "o": "o"},
+                            spec, prefix, "the matrix memory")
+        # columns of the one projection: every part starts on a 16-byte boundary of a bfloat16 row
+        up = lambda n: -(-n // 8) * 8
+        self.col_q, self.col_k = 0, up(self.inner_k)
+        self.col_v = self.col_k + up(self.inner_k)
+        self.col_g = self.col_v + up(self.inner_v)
+        self.columns = self.col_g + up(self.inner_v)
+        self.w_in = self.w_gates = self.norm_w = self.w_o = self.memory = None
+
+    def declare_weights(self) -> List[WeightDecl]:
+        n, H = self.names, self.hidden
+        return [WeightDecl(n["q"], (self.inner_k, H)), WeightDecl(n["k"], (self.inner_k, H)), WeightDecl(n["v"], (self.inner_v, H)),
+                WeightDecl(n["g"], (self.inner_v, H)), WeightDecl(n["i"], (self.heads, H)), WeightDecl(n["ib"], (self.heads,), "vector", "bias"),
+                WeightDecl(n["f"], (self.heads, H)), WeightDecl(n["fb"], (self.heads,), "vector", "bias"),
+                WeightDecl(n["norm"], (self.inner_v,), "vector", "norm"), WeightDecl(n["o"], (H, self.inner_v))]
+
+    def bind(self, tensors: Mapping[str, torch.Tensor]) -> None:
+        n = self.names
+        rows = []
+        for role, at in (("q", self.col_k), ("k", self.col_v), ("v", self.col_g), ("g", self.columns)):
+            w = tensors[n[role]]
+            rows += [w, w.new_zeros(at - sum(r.shape[0] for r in rows) - w.shape[0], self.hidden)]
+        self.w_in = torch.cat(rows, dim=0).contiguous()
+        self.w_gates = torch.cat([tensors[n["i"]], tensors[n["f"]]], dim=0).contiguous()
+        self.norm_w, self.w_o = tensors[n["norm"]].contiguous(), tensors[n["o"]].contiguous()
+        self.memory = ops.MatrixMemory(self.heads, self.d, self.dv, self.col_q, self.col_k, self.col_v, self.col_g, self.cap,
+                                       self.d ** -0.5, self.den_eps, tensors[n["ib"]].contiguous(), tensors[n["fb"]].contiguous())
+
+    def cache_needs(self) -> CacheNeeds:
+        return CacheNeeds(slots=(SlotStateNeed("state", (self.heads, self.d, self.dv), torch.float32),
+                                 SlotStateNeed("norm", (self.heads, self.d), torch.float32),
+                                 SlotStateNeed("max", (self.heads,), torch.float32)))
+
+    def scratch_bytes(self, tokens: int) -> int:
+        size = torch.empty((), dtype=self.ctx.dtype).element_size()
+        chunks = ops.mlstm_chunk_floats(-(-tokens // ops.MLSTM_CHUNK) + 1, self.heads, self.d, self.dv) * 4
+        return tokens * ((self.columns + self.inner_v) * size + (6 * self.heads + self.inner_v) * 4) + chunks
+
+    def input_rows(self):
+        """(matrix, bias or None) of the one product this mixer starts with (see `forward_projected`)."""
+        return self.w_in, None
+
+    def take_input_rows(self, rows: torch.Tensor) -> None:
+        """The same matrix as a view of the stacked one: no second copy is kept."""
+        self.w_in = rows
+
+    def output_rows(self):
+        """(matrix [hidden, heads * v_head_dim], bias or None) of the product this mixer ends with."""
+        return self.w_o, None
+
+    def forward(self, x: torch.Tensor, residual: torch.Tensor, step, cache) -> None:
+        proj = self.ctx.workspace.buffer("mlstm.proj", (x.shape[0], self.columns), self.ctx.dtype)
+        ops.scope("mlstm.in_projection")
+        linear(x, self.w_in, proj)
+        self.forward_projected(proj, residual, step, cache, x=x)
+
+    def forward_projected(self, proj: torch.Tensor, residual: torch.Tensor, step, cache, out=None, x=None) -> None:
+        """The mixer from its projection's output on: `proj` [T, q | k | v | gate], rows of any stride; `x` the mixer's input.  With
+        `out` [T, heads * v_head_dim] (rows of any stride) the normed, gated rows go there and the output product is left to the
+        caller."""
+        T, ws, dt = proj.shape[0], self.ctx.workspace, self.ctx.dtype
+        gated = out if out is not None else ws.buffer("mlstm.gated", (T, self.inner_v), dt)
+        if step.decode_only:
+            ops.scope("mlstm.step (gates, recurrence, norm and output gate inside)")
+            ops.mlstm_step(self.memory, proj, x, self.w_gates, self.norm_w, self.eps, cache.state, gated, step)
+        else:
+            ops.scope("mlstm.gates")
+            gates = ws.buffer("mlstm.logits", (T, 2 * self.heads), torch.float32)
+            linear(x, self.w_gates, gates)
+            ops.scope("mlstm.scan")
+            y = ws.buffer("mlstm.y", (T, self.inner_v), torch.float32)
+            den = ops.mlstm_scan(self.memory, proj, gates, cache.state, y, step, ws)
+            ops.scope("mlstm.norm_gate")
+            ops.rms_gate(y, proj[:, self.col_g:], self.norm_w, self.eps, gated, groups=self.heads, divisor=den)
+        if out is None:
+            ops.scope("mlstm.out_projection")
+            linear(gated, self.w_o, residual, accumulate=True)
+
+
 class ParallelMixers(Mixer):
     """spec: `branches` = ((sub-prefix, PartSpec of role mixer), ...).  Every branch reads the block's input and adds
     into the block's output; a branch's constant on its output is its own parameter (`out_scale`).  Branches that start
@@ -301,7 +411,10 @@ class ParallelMixers(Mixer):
     stacked at load (each branch keeps a view of its rows) and every branch reads its columns of the result.  Branches
     that also end with one product each (`output_rows`) share that too: every branch writes what its product would read
     into its columns of one matrix, and one product with the branches' matrices side by side adds all of them into the
-    block's output (the sum over a row of the stacked matrix is the sum of the branches' products)."""
+    block's output (the sum over a row of the stacked matrix is the sum of the branches' products).
+
+    `out_norms` (optional): a name under the prefix per branch; that branch's output passes an RMS norm over its whole row with
+    the named weight (`norm_eps`), and the normed rows' sum times `out_mult` (default 1) is what is added."""
 
     def __init__(self, spec, ctx, prefix: str = "") -> None:
         super().__init__(spec, ctx, prefix)
@@ -311,6 +424,15 @@ class ParallelMixers(Mixer):
         self.parts = [registry.build("mixer", part, ctx, prefix + sub) for sub, part in branches]
         self.w_all = self.b_all = self.w_out = self.b_out = None
         self.columns, self.out_columns = [], []
+        self.out_names = [prefix + str(n) for n in spec.get("out_norms", ())]
+        self.out_mult = float(spec.get("out_mult", 1.0))
+        self.norm_eps = float(spec.get("norm_eps", 0.0))
+        self.hidden = int(spec.get("hidden_size", 0))
+        self.out_norms: List[torch.Tensor] = []
+        if self.out_names and (len(self.out_names) != len(self.parts) or len(self.parts) != 2 or self.norm_eps <= 0 or self.hidden <= 0):
+            raise ValueError("parallel: norms of the branches' outputs need two branches, a name for each, norm_eps and hidden_size")
+        if not self.out_names and self.out_mult != 1.0:
+            raise ValueError("parallel: a common constant comes with norms of the branches' outputs")
         if sum(1 for p in self.parts if p.cache_needs().paged is not None) > 1:
             raise ValueError("parallel: at most one branch may keep keys and values in pages")
 
@@ -319,13 +441,17 @@ class ParallelMixers(Mixer):
         return all(p.graph_safe for p in self.parts)
 
     def declare_weights(self) -> List[WeightDecl]:
-        return [d for p in self.parts for d in p.declare_weights()]
+        return [d for p in self.parts for d in p.declare_weights()] + [WeightDecl(n, (self.hidden,), "vector", "norm") for n in self.out_names]
 
     def bind(self, tensors: Mapping[str, torch.Tensor]) -> None:
         for p in self.parts:
             p.bind(tensors)
+        self.out_norms = [tensors[n].contiguous() for n in self.out_names]
         self.w_all = self.b_all = self.w_out = self.b_out = None
         self.columns, self.out_columns = [], []
+        if self.out_norms and any(getattr(p, "output_rows", lambda: None)() is None or not hasattr(p, "forward_projected") or p.input_rows()[0].shape[0] % 8
+                                  for p in self.parts):
+            raise ValueError("parallel: norms of the branches' outputs need branches that give up their first and last product")
         if len(self.parts) < 2 or not all(hasattr(p, "input_rows") and hasattr(p, "forward_projected") for p in self.parts):
             return
         rows = [p.input_rows() for p in self.parts]
@@ -342,6 +468,8 @@ class ParallelMixers(Mixer):
             if hasattr(p, "take_input_rows"):
                 p.take_input_rows(self.w_all[at:at + w.shape[0]])
             at += w.shape[0]
+        if self.out_norms:              # (each output is normed by itself: the products stay apart)
+            return
         outs = [p.output_rows() if hasattr(p, "output_rows") else None for p in self.parts]
         if any(o is None for o in outs) or any(w.shape[1] % 8 for w, _ in outs) or len({(w.dtype, w.shape[0]) for w, _ in outs}) != 1:
             return
@@ -362,9 +490,46 @@ class ParallelMixers(Mixer):
         return CacheNeeds(paged=paged, slots=tuple(slots))
 
     def scratch_bytes(self, tokens: int) -> int:
-        return sum(p.scratch_bytes(tokens) for p in self.parts)          # (the shared matrices are the branches' own, side by side)
+        normed = tokens * self.hidden * 4 * len(self.out_names)
+        return normed + sum(p.scratch_bytes(tokens) for p in self.parts)          # (the shared matrices are the branches' own, side by side)
+
+    @property
+    def normed_branches(self) -> bool:
+        """Whether the branches' outputs are normed: a block may then take them as they are (`forward_branches`) and norm, add up
+        and go on in one launch."""
+        return bool(self.out_names)
+
+    def forward_branches(self, x: torch.Tensor, step, cache):
+        """(the branches' outputs, 32-bit rows each; their norms' weights; eps; the constant on the normed rows' sum)."""
+        T, ws = x.shape[0], self.ctx.workspace
+        outputs = list(ws.buffer("parallel.outputs", (len(self.parts), T, self.hidden), torch.float32).unbind(0))
+        pre = [ws.buffer(f"parallel.pre/{i}", (T, p.output_rows()[0].shape[1]), self.ctx.dtype) for i, p in enumerate(self.parts)]
+        proj = ws.buffer("parallel.proj", (T, self.w_all.shape[0]), self.ctx.dtype)
+        ops.scope("parallel.in_projection")
+        linear(x, self.w_all, proj, self.b_all)
+        for i, p in enumerate(self.parts):
+            a, b = self.columns[i]
+            p.forward_projected(proj[:, a:b], None, step, self._own(cache, i), out=pre[i], **self._extra(p, x))
+        ops.scope("parallel.out_projection")
+        for p, rows, out in zip(self.parts, pre, outputs):
+            linear(rows, p.output_rows()[0], out, p.output_rows()[1])
+        return outputs, self.out_norms, self.norm_eps, self.out_mult
+
+    @staticmethod
+    def _own(cache, i: int):
+        tag = f"{i}."
+        return dataclasses.replace(cache, state={k[len(tag):]: v for k, v in cache.state.items() if k.startswith(tag)})
+
+    @staticmethod
+    def _extra(part, x: torch.Tensor) -> dict:
+        return dict(x=x) if getattr(part, "reads_input", False) else {}
 
     def forward(self, x: torch.Tensor, residual: torch.Tensor, step, cache) -> None:
+        if self.out_norms:
+            outputs, weights, eps, mult = self.forward_branches(x, step, cache)
+            ops.scope("parallel.output_norms")
+            ops.branch_norms_add(outputs, weights, eps, mult, y=residual)
+            return
         proj = None
         if self.w_all is not None:
             proj = self.ctx.workspace.buffer("parallel.proj", (x.shape[0], self.w_all.shape[0]), self.ctx.dtype)
@@ -374,14 +539,13 @@ class ParallelMixers(Mixer):
         if self.w_out is not None:
             pre = self.ctx.workspace.buffer("parallel.pre", (x.shape[0], self.w_out.shape[1]), self.ctx.dtype)
         for i, p in enumerate(self.parts):
-            tag = f"{i}."
-            own = dataclasses.replace(cache, state={k[len(tag):]: v for k, v in cache.state.items() if k.startswith(tag)})
+            own, extra = self._own(cache, i), self._extra(p, x)
             if pre is not None:
                 (a, b), (c, d) = self.columns[i], self.out_columns[i]
-                p.forward_projected(proj[:, a:b], residual, step, own, out=pre[:, c:d])
+                p.forward_projected(proj[:, a:b], residual, step, own, out=pre[:, c:d], **extra)
             elif proj is not None:
                 a, b = self.columns[i]
-                p.forward_projected(proj[:, a:b], residual, step, own)
+                p.forward_projected(proj[:, a:b], residual, step, own, **extra)
             else:
                 p.forward(x, residual, step, own)
         if pre is not None:
@@ -392,4 +556,5 @@ class ParallelMixers(Mixer):
 registry.register("mixer", "gated_linear_recurrence", GatedLinearRecurrence)
 registry.register("mixer", "decayed_linear_attention", DecayedLinearAttention)
 registry.register("mixer", "general_delta", GeneralDelta)
+registry.register("mixer", "mlstm", MatrixMemory)
 registry.register("mixer", "parallel", ParallelMixers)
