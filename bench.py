@@ -5,6 +5,7 @@
                     [--config 8b|14b-mixed|32b-long] [--breakdown] [--kernels [attention|products]] [--further]
                     [--sufolix [dense|moe]] [--mamevik [latent|ssd|mixed]] [--dalavik [latent|heads|mixed]]
                     [--zebivik [parallel|rglru|mixed]] [--sapanex [attention|delta|mixed]]
+                    [--tamovik [latent|parallel|mixed]]
 
 One JSON line on stdout.  The default (`--config 8b`) is the headline: Qwen3-8B layer sizes,
 36 layers, batch 8, 1,024-token prompts; a "step" is one decode step of the whole batch.
@@ -35,7 +36,7 @@ decode at --batch, one 2,048-token prompt, and the per-op-class device time of b
 `--mamevik` measures the Mamevik decoder (attention over a cached latent with a sink, state-space recurrences, a looped span
 of layers, clamped gated experts) the same way, in three arrangements of its layers, beside a Sufolix model with routed
 experts of the same width, layers and experts.
-`--dalavik`, `--zebivik` and `--sapanex` measure those decoders the same way, each beside the closest models of equal size.
+`--dalavik`, `--zebivik`, `--sapanex` and `--tamovik` measure those decoders the same way, each beside the closest models of equal size.
 Peaks come from MEASURED_PEAKS.json beside this file when present, else the fallback
 figures 6.65 TB/s and 1.59 PFLOP/s.  Weights (15 GB and more) exceed L2 (126 MB), so every
 step reads them from HBM: no L2 flush is needed between timed steps.
@@ -280,8 +281,38 @@ def sapanex_numbers(cfg: dict):
             "state_bytes_per_seq": state}
 
 
+def tamovik_numbers(cfg: dict):
+    """The same for a Tamovik configuration: a latent layer's cache row is the latent with the shared rotated key part; a
+    parallel layer counts both of its mixers (a position of its chunked side reads its own chunk's keys: the bytes and flops
+    per key of context hold up to that many)."""
+    W, V, L = cfg["width"], cfg["vocab"], len(cfg["layers"])
+    params, kv, attn, state = 0, 0, 0, 0
+    for layer in cfg["layers"]:
+        m, f = layer["mixer"], layer["mlp"]
+        if layer["type"] == "latent_attention":
+            row, H = m["kv_rank"] + m["rot_dim"], m["heads"]
+            params += (H * (m["dim"] + m["rot_dim"]) + row + H * m["vdim"]) * W + H * (m["dim"] + m["vdim"]) * m["kv_rank"]
+            kv += row * 2
+            attn += 4 * H * row
+        else:
+            a, b = m["left"], m["right"]
+            params += (3 * a["heads"] + a["kv_heads"]) * a["dim"] * W
+            params += (2 * b["heads"] * b["dim"] + 3 * b["heads"] * b["vdim"] + 2 * b["heads"]) * W
+            kv += 2 * a["kv_heads"] * a["dim"] * 2
+            attn += 4 * a["heads"] * a["dim"]
+            state += 2 * 4 * (b["heads"] * b["dim"] * (b["vdim"] + 1) + (a["conv"] - 1) * (a["heads"] + a["kv_heads"]) * a["dim"])
+        if f is not None and f["kind"] == "dense":
+            params += 3 * W * f["ff"]
+        elif f is not None:
+            params += 3 * W * f["router"]["top"] * f["expert"]["ff"] + W * f["router"]["experts"]
+    return {"layer_params": params / L, "head_params": V * W, "kv_bytes_per_token": kv, "attn_flops_per_pair": attn, "layers": L,
+            "state_bytes_per_seq": state}
+
+
 def model_numbers(cfg: dict):
     """Parameters the matrix products of one token touch, and bytes of cache per token."""
+    if cfg.get("architecture") == "Tamovik":
+        return tamovik_numbers(cfg)
     if cfg.get("architecture") == "Sapanex":
         return sapanex_numbers(cfg)
     if cfg.get("architecture") == "Zebivik":
@@ -1083,6 +1114,70 @@ def run_sapanex(args) -> dict:
     return out
 
 
+# ----------------------------------------------------------------------------- the Tamovik decoder beside Mamevik and Zebivik
+def tamovik_config(kind: str, layers: int, width: int, vocab: int, experts: int, top: int, expert_ff: int) -> dict:
+    """`kind`: "latent" (every layer attends over a cached latent with a rotated key part), "parallel" (every layer is attention
+    in aligned chunks beside a matrix memory) or "mixed" (two latent layers, one parallel layer, in turn; the first layer's
+    feed-forward is the dense unit)."""
+    lat = {"type": "latent_attention", "mixer": {"heads": 16, "dim": 96, "rot_dim": 32, "vdim": 128, "kv_rank": 96, "scale": 128 ** -0.5,
+                                                 "rot": {"base": 500000.0, "dims": 32,
+                                                         "scaling": {"factor": 8.0, "original": 8192, "fast": 32.0, "slow": 1.0}}}}
+    par = {"type": "parallel", "mixer": {
+        "left": {"heads": 16, "kv_heads": 4, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "conv": 4, "mask": {"size": 8192}},
+        "right": {"heads": 8, "dim": 128, "vdim": 128, "gate_cap": 15.0}}}
+    mlp = {"kind": "moe", "router": {"experts": experts, "top": top, "groups": {"count": 4, "keep": 2}}, "expert": {"ff": expert_ff, "limit": 7.0}}
+    pick = {"latent": lambda i: lat, "parallel": lambda i: par, "mixed": lambda i: par if i % 3 == 2 else lat}[kind]
+    out = [dict(pick(i), mlp=json.loads(json.dumps(mlp))) for i in range(layers)]
+    if kind == "mixed":
+        out[0]["mlp"] = {"kind": "dense", "ff": top * expert_ff}
+    return {"architecture": "Tamovik", "vocab": vocab, "width": width, "norm": {"eps": 1e-6},
+            "embedding": {"bigram": {"buckets": 65521, "mul_prev": 131, "mul_cur": 17}}, "layers": out}
+
+
+def run_tamovik(args) -> dict:
+    """Decode and prefill of the Tamovik decoder at layer sizes of a real model (latent layers, parallel layers, both in turn),
+    beside the closest models the engine has at the same width, layers and experts: the Mamevik decoder with attention over a
+    latent whose cached rows are as wide (the latent layers' relative) and the Zebivik decoder with softmax attention beside a
+    linear attention of the same heads (the parallel layers' relative); with the device time of every op class."""
+    import torch
+    L, W, V = args.layers if args.layers != FULL_LAYERS else 8, 2048, 32768
+    E, TOP, EFF = 16, 2, 1408
+    which = ["latent", "parallel", "mixed"] if args.tamovik == "all" else [args.tamovik]
+    out = {"metric": "tamovik_vs_mamevik_and_zebivik_equal_size", "unit": "tokens/s", "n_gpus": 1, "dtype": "bf16", "data": "synthetic",
+           "steps": args.steps, "warmup": args.warmup, "batch": args.batch, "peaks": peaks(), "cases": {}}
+    arms = {kind: tamovik_config(kind, L, W, V, E, TOP, EFF) for kind in which}
+    arms["mamevik"] = mamevik_config("latent", L, W, V, E, TOP, EFF)
+    arms["zebivik"] = zebivik_config("parallel", L, W, V, E, TOP, EFF)
+    for arm, cfg in arms.items():
+        pages = (args.batch * (PROMPT_LEN + args.steps + args.warmup + 64) + PREFILL_LEN) // PAGE + 64
+        bench = Bench(cfg, SEED, pages, max(args.batch, 8), 8192, PREFILL_LEN)
+        with ClockSampler() as clocks:
+            tps, ms, kernels, ctx = bench.decode_device(args.batch, args.steps, args.warmup, arm, PROMPT_LEN)
+        routed = sum(1 for l in cfg["layers"] if l["mlp"] is not None and l["mlp"]["kind"] == "moe")
+        touched = bench.weight_bytes - routed * 3 * W * EFF * 2 * max(0, E - min(E, args.batch * TOP))
+        if "bigram" in cfg.get("embedding", {}):      # of the table of pairs a step reads one row a token
+            touched -= (cfg["embedding"]["bigram"]["buckets"] + 1) * W * 2
+        step_bytes = touched + args.batch * (ctx * bench.nums["kv_bytes_per_token"] + bench.nums.get("state_bytes_per_seq", 0))
+        r = {"decode_tokens_per_s": round(tps, 1), "decode_ms_per_step": round(ms, 4), "kernels_per_step": kernels,
+             "decode_frac_of_hbm": round(step_bytes / (ms / 1e3) / 1e9 / bench.pk["hbm_gbs"], 4),
+             "weights_gb": round(bench.weight_bytes / 1e9, 3), "clocks": clocks.summary(),
+             "prefill": bench.prefill_timed(PREFILL_LEN, 3, PREFILL_SAMPLES)}
+        if args.breakdown:
+            r["breakdown"] = bench.breakdown(args.batch, PROMPT_LEN, PREFILL_LEN)
+        out["cases"][arm] = r
+        del bench
+        torch.cuda.empty_cache()
+    out["sizes"] = {"layers": L, "width": W, "vocab": V, "experts": E, "top": TOP, "expert_ff": EFF,
+                    "mixers": {kind: sorted({json.dumps(l["mixer"], sort_keys=True) for l in arms[kind]["layers"]}) for kind in which}}
+    for kind in which:
+        c = out["cases"][kind]
+        for other in ("mamevik", "zebivik"):
+            base = out["cases"][other]
+            c[f"decode_ms_per_step_over_{other}"] = round(c["decode_ms_per_step"] / base["decode_ms_per_step"], 4)
+            c[f"prefill_ms_over_{other}"] = round(c["prefill"]["ms"] / base["prefill"]["ms"], 4)
+    return out
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1107,6 +1202,8 @@ def main() -> int:
                     help="the Zebivik decoder beside a Mamevik and a Sufolix model of equal size (decode, prefill, op classes with --breakdown)")
     ap.add_argument("--sapanex", nargs="?", const="all", default=None, choices=["all", "attention", "delta", "mixed"],
                     help="the Sapanex decoder beside a Sufolix and a Mamevik model of equal size (decode, prefill, op classes with --breakdown)")
+    ap.add_argument("--tamovik", nargs="?", const="all", default=None, choices=["all", "latent", "parallel", "mixed"],
+                    help="the Tamovik decoder beside a Mamevik and a Zebivik model of equal size (decode, prefill, op classes with --breakdown)")
     args = ap.parse_args()
 
     if args.impl == "reference":
@@ -1139,6 +1236,9 @@ def main() -> int:
         return 0
     if args.sapanex:
         print(json.dumps(run_sapanex(args)))
+        return 0
+    if args.tamovik:
+        print(json.dumps(run_tamovik(args)))
         return 0
     result = {"8b": run_8b, "14b-mixed": run_14b_mixed, "32b-long": run_32b_long}[args.config](args)
     print(json.dumps(result))

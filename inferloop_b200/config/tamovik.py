@@ -95,6 +95,8 @@ class ChunkedBranch:
         out = cls(heads, kv, dim, _int(d, "conv", what), _num(d, "scale", what), chunk)
         if dim > 512:
             raise UnsupportedConfig(f"config.json: {what}: head sizes beyond 512 are not served")
+        if out.conv > 16:
+            raise UnsupportedConfig(f"config.json: {what}.conv: more than 16 taps are not served")
         if (heads + kv) * dim > 51200:
             raise UnsupportedConfig(f"config.json: {what}: more than 51,200 channels of queries and keys are not served")
         return out

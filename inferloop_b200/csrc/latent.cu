@@ -253,7 +253,7 @@ head_matmul_kernel(const TI* __restrict__ x, int ldx, const TW* __restrict__ w, 
 template <typename TI, typename TC, typename TO>
 __global__ void __launch_bounds__(128)
 latent_input_kernel(const TI* __restrict__ proj, int ld, const TI* __restrict__ w, TO* __restrict__ q_out, int ldo, int n_tokens,
-                    int heads, int K, int N, const LatentWrite a, TC* __restrict__ cache) {
+                    int heads, int K, int N, int xhs, int ohs, const LatentWrite a, TC* __restrict__ cache, const QueryTails qt) {
   ilb::pdl_launch_dependents();
   ilb::pdl_wait();
   extern __shared__ __align__(16) float xs[];
@@ -261,10 +261,10 @@ latent_input_kernel(const TI* __restrict__ proj, int ld, const TI* __restrict__ 
   const int n_blocks = (N + 31) / 32, t0 = blockIdx.x * kHeadTokens;
   const int y = blockIdx.y;
   if (y < heads * n_blocks) {
-    head_matmul_block<TI, TI, TO, 4>(proj, ld, w, q_out, ldo, n_tokens, K, N, K, N, t0, y / n_blocks, y % n_blocks, xs);
+    head_matmul_block<TI, TI, TO, 4>(proj, ld, w, q_out, ldo, n_tokens, K, N, xhs, ohs, t0, y / n_blocks, y % n_blocks, xs);
   } else {
     const int t = t0 + (y - heads * n_blocks);
-    if (t < n_tokens) latent_write_token<TI, TC>(proj, ld, a, cache, t, scratch);
+    if (t < n_tokens) latent_write_token<TI, TC>(proj, ld, a, cache, t, scratch, qt.src != nullptr ? &qt : nullptr);
   }
 }
 
@@ -454,23 +454,27 @@ ILB_EXPORT int ilb_head_matmul(const void* x, int dtype, int ldx, const void* w,
   return check_launch("head_matmul");
 }
 
-// ilb_latent_write and ilb_head_matmul (queries: heads x K at the row's start) of a step of few tokens as one launch.
+// ilb_latent_write (or, with a rotated part of `tail` elements, ilb_latent_write_rot for the latent and the queries' tails) and
+// ilb_head_matmul (queries: heads x (K + tail) at the row's start) of a step of few tokens as one launch.
 ILB_EXPORT int ilb_latent_input(const void* proj, int dtype, int ld, const void* w, void* q_out, int out_dtype, int ldo, int n_tokens,
                                 int heads, int K, int N, int col0, int rank, const float* norm_w, float eps, const int* positions,
                                 const int* seq_of_token, const int* block_table, int max_blocks, int page_size, int num_pages,
-                                void* cache, int cache_dtype, cudaStream_t stream) {
-  ILB_REQUIRE(n_tokens >= 0 && heads > 0 && K > 0 && N > 0 && rank > 0 && eps > 0.f, "latent_input: bad sizes");
-  ILB_REQUIRE(ld >= heads * K && ld >= col0 + rank && ldo >= heads * N, "latent_input: strides too small");
+                                void* cache, int cache_dtype, int tail, int rot, const float* angles, int apart, cudaStream_t stream) {
+  ILB_REQUIRE(n_tokens >= 0 && heads > 0 && K > 0 && N > 0 && rank > 0 && eps > 0.f && tail >= 0, "latent_input: bad sizes");
+  ILB_REQUIRE(ld >= heads * (K + tail) && ld >= col0 + rank + tail && ldo >= heads * (N + tail), "latent_input: strides too small");
+  ILB_REQUIRE(rot >= 0 && rot % 2 == 0 && rot <= tail && (rot == 0 || angles != nullptr) && (tail == 0 || N == rank),
+              "latent_input: %d of %d elements cannot turn in pairs", rot, tail);
   ILB_REQUIRE(page_size > 0 && max_blocks > 0 && num_pages > 0, "latent_input: bad cache geometry");
   const size_t smem = sizeof(float) * kHeadTokens * ((size_t)K + 128);
   ILB_REQUIRE(smem <= 48 * 1024, "latent_input: inner size %d exceeds %d", K, 48 * 1024 / 4 / kHeadTokens - 128);
   const long long rows = (long long)heads * ((N + 31) / 32) + kHeadTokens;
   ILB_REQUIRE(rows <= 65535, "latent_input: too many heads");
   if (n_tokens == 0) return 0;
-  const LatentWrite a{norm_w, eps, positions, seq_of_token, block_table, col0, rank, max_blocks, page_size, num_pages, 0, 0, nullptr, 0};
+  const LatentWrite a{norm_w, eps, positions, seq_of_token, block_table, col0, rank, max_blocks, page_size, num_pages, tail, rot, angles, apart};
+  const QueryTails qt{tail > 0 ? proj : nullptr, q_out, ld, ldo, heads, K, K + tail};
   const dim3 grid((n_tokens + kHeadTokens - 1) / kHeadTokens, (unsigned)rows);
 #define ILB_LI(TI, TC, TO) ilb::launch(latent_input_kernel<TI, TC, TO>, grid, dim3(128), smem, stream, (const TI*)proj, ld, (const TI*)w, \
-                                        (TO*)q_out, ldo, n_tokens, heads, K, N, a, (TC*)cache)
+                                        (TO*)q_out, ldo, n_tokens, heads, K, N, K + tail, N + tail, a, (TC*)cache, qt)
   if (dtype == kF32 && cache_dtype == kF32 && out_dtype == kF32) ILB_LI(float, float, float);
   else if (dtype == kBF16 && cache_dtype == kBF16 && out_dtype == kBF16) ILB_LI(__nv_bfloat16, __nv_bfloat16, __nv_bfloat16);
   else return fail("latent_input: unsupported dtypes %d/%d/%d", dtype, cache_dtype, out_dtype);

@@ -127,7 +127,8 @@ ILB_EXPORT int ilb_moe_logits(const void* x, const void* w, int dtype, float* ou
   return check_launch("moe_logits");
 }
 
-// One warp per token.
+// One warp per token; a lane holds EPL experts (lane, lane + 32, ...).
+template <int EPL>
 __global__ void __launch_bounds__(128)
 moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bias, int ld, int n_tokens, int experts, int top,
                  int softmax, int renormalize, int* __restrict__ choice, float* __restrict__ weight,
@@ -138,10 +139,10 @@ moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bia
   const int t = blockIdx.x * 4 + warp;
   if (t >= n_tokens) return;
   const float* z = logits + (size_t)t * ld;
-  float s[kMaxExpertsPerLane];
+  float s[EPL];
   float zmax = -INFINITY;
 #pragma unroll
-  for (int i = 0; i < kMaxExpertsPerLane; ++i) {
+  for (int i = 0; i < EPL; ++i) {
     const int e = lane + 32 * i;
     s[i] = e < experts ? (bias != nullptr ? z[e] + bias[e] : z[e]) : -INFINITY;
     zmax = fmaxf(zmax, s[i]);
@@ -150,26 +151,26 @@ moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bia
     zmax = warp_max(zmax);
     float sum = 0.f;
 #pragma unroll
-    for (int i = 0; i < kMaxExpertsPerLane; ++i) {
+    for (int i = 0; i < EPL; ++i) {
       const int e = lane + 32 * i;
       s[i] = e < experts ? expf(s[i] - zmax) : -INFINITY;
       if (e < experts) sum += s[i];
     }
     sum = warp_sum(sum);
 #pragma unroll
-    for (int i = 0; i < kMaxExpertsPerLane; ++i)
+    for (int i = 0; i < EPL; ++i)
       if (lane + 32 * i < experts) s[i] = s[i] / sum;
   } else {
 #pragma unroll
-    for (int i = 0; i < kMaxExpertsPerLane; ++i)
+    for (int i = 0; i < EPL; ++i)
       if (lane + 32 * i < experts) s[i] = sigmoid_stable(s[i]);
   }
   // What the experts are ranked by: the scores, or the scores plus a stored correction (the weights below are the
   // scores themselves either way).  With groups, only experts of the `keep` groups of neighbours whose best ranked
   // member (`best_two`: whose two best together) is largest can be chosen (ties to the lower group).
-  float c[kMaxExpertsPerLane];
+  float c[EPL];
 #pragma unroll
-  for (int i = 0; i < kMaxExpertsPerLane; ++i) {
+  for (int i = 0; i < EPL; ++i) {
     const int e = lane + 32 * i;
     c[i] = (e < experts && correction != nullptr) ? s[i] + correction[e] : s[i];
   }
@@ -179,7 +180,7 @@ moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bia
     for (int g = 0; g < groups; ++g) {
       float m = -INFINITY;
 #pragma unroll
-      for (int i = 0; i < kMaxExpertsPerLane; ++i) {
+      for (int i = 0; i < EPL; ++i) {
         const int e = lane + 32 * i;
         if (e < experts && e / per == g) m = fmaxf(m, c[i]);
       }
@@ -188,14 +189,14 @@ moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bia
         // the second best: the largest of the others, the best one itself being the group's first member of that value
         int who = 0x7fffffff;
 #pragma unroll
-        for (int i = 0; i < kMaxExpertsPerLane; ++i) {
+        for (int i = 0; i < EPL; ++i) {
           const int e = lane + 32 * i;
           if (e < experts && e / per == g && c[i] == m) who = min(who, e);
         }
         who = (int)__reduce_min_sync(0xffffffffu, (unsigned)who);
         float second = -INFINITY;
 #pragma unroll
-        for (int i = 0; i < kMaxExpertsPerLane; ++i) {
+        for (int i = 0; i < EPL; ++i) {
           const int e = lane + 32 * i;
           if (e < experts && e / per == g && e != who) second = fmaxf(second, c[i]);
         }
@@ -220,7 +221,7 @@ moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bia
       if (lane == best_g) mine = -INFINITY;
     }
 #pragma unroll
-    for (int i = 0; i < kMaxExpertsPerLane; ++i) {
+    for (int i = 0; i < EPL; ++i) {
       const int e = lane + 32 * i;
       if (e < experts && !((allowed >> (e / per)) & 1u)) c[i] = -INFINITY;
     }
@@ -231,7 +232,7 @@ moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bia
     float best = -INFINITY;
     int best_e = 0x7fffffff;
 #pragma unroll
-    for (int i = 0; i < kMaxExpertsPerLane; ++i) {
+    for (int i = 0; i < EPL; ++i) {
       const int e = lane + 32 * i;
       if (e < experts && (c[i] > best || (c[i] == best && e < best_e)) && c[i] != -INFINITY) { best = c[i]; best_e = e; }
     }
@@ -244,7 +245,7 @@ moe_route_kernel(const float* __restrict__ logits, const float* __restrict__ bia
     if (best_e == 0x7fffffff) { best_e = 0; best = 0.f; }      // (non-finite logits: keep the indices in range)
     float score = 0.f;                                          // the winner's score, from the lane that holds it
 #pragma unroll
-    for (int i = 0; i < kMaxExpertsPerLane; ++i)
+    for (int i = 0; i < EPL; ++i)
       if (lane + 32 * i == best_e) { score = s[i]; c[i] = -INFINITY; }      // taken
     score = __shfl_sync(0xffffffffu, score, best_e & 31);
     if (score == -INFINITY) score = 0.f;
@@ -275,8 +276,13 @@ ILB_EXPORT int ilb_moe_route(const float* logits, const float* bias, int ld, int
   ILB_REQUIRE(top > 0 && top <= experts && top <= kMaxTop, "moe_route: top %d of %d experts (at most %d)", top, experts, kMaxTop);
   ILB_REQUIRE(ld >= experts, "moe_route: row stride too small");
   if (n_tokens == 0) return 0;
-  ilb::launch(moe_route_kernel, dim3((n_tokens + 3) / 4), dim3(128), 0, stream, logits, bias, ld, n_tokens, experts, top, softmax,
-              renormalize, choice, weight, correction, groups, keep, best_two, out_scale, renorm_eps);
+#define ILB_ROUTE(EPL) ilb::launch(moe_route_kernel<EPL>, dim3((n_tokens + 3) / 4), dim3(128), 0, stream, logits, bias, ld, n_tokens, experts, top, softmax, \
+                                   renormalize, choice, weight, correction, groups, keep, best_two, out_scale, renorm_eps)
+  if (experts <= 32) ILB_ROUTE(1);
+  else if (experts <= 64) ILB_ROUTE(2);
+  else if (experts <= 128) ILB_ROUTE(4);
+  else ILB_ROUTE(kMaxExpertsPerLane);
+#undef ILB_ROUTE
   return check_launch("moe_route");
 }
 

@@ -269,19 +269,23 @@ LATENT_INPUT_TOKENS = 16      # steps of up to this many tokens run the latent w
 
 
 def latent_input(proj: torch.Tensor, w: torch.Tensor, q_out: torch.Tensor, col0: int, rank: int, weight: torch.Tensor, eps: float,
-                 step, block_table: torch.Tensor, cache: torch.Tensor) -> None:
-    """`latent_write` and `head_matmul(proj, w, q_out)` of a step of few tokens in one launch (see latent.cu)."""
+                 step, block_table: torch.Tensor, cache: torch.Tensor, tail: int = 0, rot: int = 0, angles: Optional[torch.Tensor] = None,
+                 half_split: bool = False) -> None:
+    """`latent_write` (with `tail`: `latent_write_rot`, the queries' tails included) and `head_matmul` of a step of few tokens in one
+    launch (see latent.cu): head i's query is [K | tail] columns of proj, its mapped query [N | tail] columns of q_out."""
     _need(proj, "latent projection"); _need(w, "head_matmul w", proj.dtype); _need(q_out, "mapped queries", proj.dtype)
     _need(weight, "latent norm weight", torch.float32); _need(cache, "latent cache", proj.dtype); _need(block_table, "block table", torch.int32)
     heads, K, N = w.shape
-    if cache.dim() != 4 or cache.shape[1] != 1 or cache.shape[3] != rank or weight.numel() != rank:
-        raise KernelError("latent_input: cache must be [pages, 1, page_size, rank]")
-    if proj.shape[0] != step.n_tokens or proj.shape[1] < max(heads * K, col0 + rank) or tuple(q_out.shape) != (proj.shape[0], heads * N):
+    _need(angles, "rotation table", torch.float32)
+    if cache.dim() != 4 or cache.shape[1] != 1 or cache.shape[3] != rank + tail or weight.numel() != rank:
+        raise KernelError("latent_input: cache must be [pages, 1, page_size, rank + tail]")
+    if proj.shape[0] != step.n_tokens or proj.shape[1] < max(heads * (K + tail), col0 + rank + tail) \
+            or tuple(q_out.shape) != (proj.shape[0], heads * (N + tail)) or (angles is not None and tuple(angles.shape) != (proj.shape[0], rot // 2, 2)):
         raise KernelError("latent_input: shapes do not agree")
     _call("latent", "ilb_latent_input", _ptr(proj), _i(_code(proj)), _i(proj.stride(0)), _ptr(w), _ptr(q_out), _i(_code(q_out)),
           _i(q_out.stride(0)), _i(proj.shape[0]), _i(heads), _i(K), _i(N), _i(col0), _i(rank), _ptr(weight), _f(eps), _ptr(step.positions),
           _ptr(step.seq_of_token), _ptr(block_table), _i(block_table.shape[1]), _i(cache.shape[2]), _i(cache.shape[0]), _ptr(cache),
-          _i(_code(cache)), _stream(cache))
+          _i(_code(cache)), _i(tail), _i(rot), _ptr(angles), _i(1 if half_split else 0), _stream(cache))
 
 
 def head_matmul(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, x_head_stride: Optional[int] = None,

@@ -638,6 +638,8 @@ ILB_EXPORT int ilb_rows_norm_rope_cache(
 // The raw inputs ahead of the step come from state [slots, taps - 1, (nq + nkv) d] 32-bit; zeros before the sequence's start.
 // A block a token: the convolved row waits in shared memory for its sums.  A sequence of one token is one block, which also
 // moves the state on; the state of the others is moved on by a second launch, when nobody reads the old one any more.
+constexpr int kMostTaps = 16;
+
 struct ConvRowsParams {
   RowsParams r;
   const float* conv_w;               // [taps, (nq + nkv) d]
@@ -646,7 +648,8 @@ struct ConvRowsParams {
   int taps, values_are_keys;
 };
 
-template <typename T, int VEC>
+// MT: the most taps this form holds in flight (taps <= MT).
+template <typename T, int VEC, int MT>
 __global__ void __launch_bounds__(kRowsThreads)
 conv_rows_norm_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* k_cache, T* v_cache, const ConvRowsParams c) {
   ilb::pdl_launch_dependents();
@@ -661,31 +664,42 @@ conv_rows_norm_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* k_cac
   float* own = slot >= 0 ? c.state + (size_t)slot * before * width : nullptr;
   float sum_q = 0.f, sum_k = 0.f;
   for (int e = threadIdx.x * VEC; e < width; e += kRowsThreads * VEC) {
-    float acc[VEC];
+    float acc[VEC], x[MT][VEC];
 #pragma unroll
     for (int i = 0; i < VEC; ++i) acc[i] = 0.f;
-    for (int j = 0; j < c.taps; ++j) {
+#pragma unroll
+    for (int j = 0; j < MT; ++j) {                         // every tap's inputs are asked for before the first is used
       const int back = before - j;
-      float x[VEC], w[VEC];
-      if (lt >= back) RowUnit<T, VEC>::load(qkv + (size_t)(t - back) * p.qkv_stride + e, x);
-      else if (own != nullptr) {                           // (plain loads: this launch may write the slot)
+      if (j < c.taps && lt >= back) RowUnit<T, VEC>::load(qkv + (size_t)(t - back) * p.qkv_stride + e, x[j]);
+      else if (j < c.taps && own != nullptr) {             // (plain loads: this launch may write the slot)
         const float* s = own + (size_t)(before + lt - back) * width + e;
         if constexpr (VEC == 8) {
           const float4 a = *reinterpret_cast<const float4*>(s), b = *reinterpret_cast<const float4*>(s + 4);
-          x[0] = a.x; x[1] = a.y; x[2] = a.z; x[3] = a.w; x[4] = b.x; x[5] = b.y; x[6] = b.z; x[7] = b.w;
+          x[j][0] = a.x; x[j][1] = a.y; x[j][2] = a.z; x[j][3] = a.w; x[j][4] = b.x; x[j][5] = b.y; x[j][6] = b.z; x[j][7] = b.w;
         } else {
-          x[0] = *s;
+          x[j][0] = *s;
         }
       } else {
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) x[i] = 0.f;
+        for (int i = 0; i < VEC; ++i) x[j][i] = 0.f;
       }
-      load_f32<VEC>(c.conv_w + (size_t)j * width + e, w);
+    }
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) acc[i] = fmaf(w[i], x[i], acc[i]);
-      if (alone && j > 0 && own != nullptr) {
+    for (int j = 0; j < MT; ++j) {
+      if (j < c.taps) {
+        float w[VEC];
+        load_f32<VEC>(c.conv_w + (size_t)j * width + e, w);
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) own[(size_t)(j - 1) * width + e + i] = x[i];
+        for (int i = 0; i < VEC; ++i) acc[i] = fmaf(w[i], x[j][i], acc[i]);
+        if (alone && j > 0 && own != nullptr) {
+          float* s = own + (size_t)(j - 1) * width + e;
+          if constexpr (VEC == 8) {
+            reinterpret_cast<float4*>(s)[0] = make_float4(x[j][0], x[j][1], x[j][2], x[j][3]);
+            reinterpret_cast<float4*>(s)[1] = make_float4(x[j][4], x[j][5], x[j][6], x[j][7]);
+          } else {
+            *s = x[j][0];
+          }
+        }
       }
     }
     float ss = 0.f;
@@ -769,7 +783,7 @@ ILB_EXPORT int ilb_conv_rows_norm_cache(
     int n_seqs, int n_several, const int* block_table, int max_blocks, int page_size, int num_pages, void* k_cache, void* v_cache,
     int n_tokens, int nq, int nkv, int d, int dv, int qkv_stride, int q_out_stride, int values_are_keys, cudaStream_t stream) {
   ILB_REQUIRE(n_tokens >= 0 && nq > 0 && nkv > 0 && d > 0 && dv > 0 && eps > 0.f && n_seqs >= 0 && n_seqs <= 65535, "conv_rows_norm: bad sizes");
-  ILB_REQUIRE(conv_w != nullptr && taps >= 1 && (taps == 1 || state != nullptr), "conv_rows_norm: %d taps need weights and a state", taps);
+  ILB_REQUIRE(conv_w != nullptr && taps >= 1 && taps <= kMostTaps && (taps == 1 || state != nullptr), "conv_rows_norm: %d taps (at most %d) need weights and a state", taps, kMostTaps);
   ILB_REQUIRE(q_weight != nullptr && k_weight != nullptr, "conv_rows_norm: the norms' weights are missing");
   ILB_REQUIRE(rope == nullptr || (rotary_dim > 0 && rotary_dim % 2 == 0 && rotary_dim <= d),
               "conv_rows_norm: rotary dimension %d must be even and at most the head size %d", rotary_dim, d);
@@ -793,16 +807,16 @@ ILB_EXPORT int ilb_conv_rows_norm_cache(
                    a16(qkv) && a16(q_out) && a16(k_cache) && a16(v_cache) && a16(q_weight) && a16(k_weight) && a16(conv_w) && a16(state) && a16(rope);
   static OncePerDevice once;
   if (smem > 48 * 1024 && once.first() &&
-      (cudaFuncSetAttribute(conv_rows_norm_kernel<__nv_bfloat16, 8>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMost) != cudaSuccess ||
-       cudaFuncSetAttribute(conv_rows_norm_kernel<__nv_bfloat16, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMost) != cudaSuccess ||
-       cudaFuncSetAttribute(conv_rows_norm_kernel<float, 1>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMost) != cudaSuccess)) {
+      (cudaFuncSetAttribute(conv_rows_norm_kernel<__nv_bfloat16, 8, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMost) != cudaSuccess ||
+       cudaFuncSetAttribute(conv_rows_norm_kernel<__nv_bfloat16, 1, kMostTaps>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMost) != cudaSuccess ||
+       cudaFuncSetAttribute(conv_rows_norm_kernel<float, 1, kMostTaps>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMost) != cudaSuccess)) {
     once.forget();
     return fail("conv_rows_norm: cannot reserve %d bytes of shared memory", kMost);
   }
-#define ILB_CR(T, V) ilb::launch(conv_rows_norm_kernel<T, V>, dim3(n_tokens), dim3(kRowsThreads), smem, stream, (const T*)qkv, (T*)q_out, (T*)k_cache, (T*)v_cache, c)
-  if (vec) ILB_CR(__nv_bfloat16, 8);
-  else if (dtype == kBF16) ILB_CR(__nv_bfloat16, 1);
-  else ILB_CR(float, 1);
+#define ILB_CR(T, V, MT) ilb::launch(conv_rows_norm_kernel<T, V, MT>, dim3(n_tokens), dim3(kRowsThreads), smem, stream, (const T*)qkv, (T*)q_out, (T*)k_cache, (T*)v_cache, c)
+  if (vec && taps <= 4) ILB_CR(__nv_bfloat16, 8, 4);
+  else if (dtype == kBF16) ILB_CR(__nv_bfloat16, 1, kMostTaps);
+  else ILB_CR(float, 1, kMostTaps);
 #undef ILB_CR
   if (int rc = check_launch("conv_rows_norm")) return rc;
   if (!n_several || taps == 1 || n_seqs == 0) return 0;

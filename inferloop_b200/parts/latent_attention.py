@@ -122,7 +122,7 @@ class LatentAttention(Mixer):
     def _forward_general(self, x: torch.Tensor, residual: torch.Tensor, step, cache) -> None:
         """The layer with any of: queries through a latent, a rotated part, another layer's cache."""
         T, ws, dt = x.shape[0], self.ctx.workspace, self.ctx.dtype
-        H, d, dv, r, tail = self.heads, self.d, self.dv, self.rank, self.tail
+        H, d, r, tail = self.heads, self.d, self.rank, self.tail
         row, qh = r + tail, d + tail
         q_cols = self.q_rank or H * qh
         # a latent that is normed next is kept in 32-bit; queries that are used as they are, in the compute dtype
@@ -145,6 +145,11 @@ class LatentAttention(Mixer):
             angles = self.position.table(step)
         q = ws.buffer("latent.q", (T, H * row), dt)
         write = cache.writable and self.own_cache
+        if T <= ops.LATENT_INPUT_TOKENS and write and not self.q_rank and cache.k.dtype == dt:
+            ops.scope("attention.input_stage (latent norm, rotations, cache write, queries to latent)")
+            ops.latent_input(proj, self.up_k, q, q_cols, r, self.latent_norm, self.eps, step, table, cache.k, tail, self.rot, angles, self.half_split)
+            self._attend(q, residual, step, cache, table, row)
+            return
         ops.scope("attention.latent_norm_cache_write")
         if write or tail:
             ops.latent_write_rot(proj, q_cols, r, tail, self.rot, angles, self.latent_norm if write else None, self.eps, step,
@@ -153,6 +158,11 @@ class LatentAttention(Mixer):
                                  half_split=self.half_split)
         ops.scope("attention.queries_to_latent")
         ops.head_matmul(q_src, self.up_k, q, x_head_stride=qh, out_head_stride=row)
+        self._attend(q, residual, step, cache, table, row)
+
+    def _attend(self, q: torch.Tensor, residual: torch.Tensor, step, cache, table, row: int) -> None:
+        """From the mapped queries [T, heads * row] on: attention over the cached rows, values, output product."""
+        T, ws, dt, H, dv = q.shape[0], self.ctx.workspace, self.ctx.dtype, self.heads, self.dv
         ops.scope("attention.attention")
         o = ws.buffer("latent.o", (T, H * row), dt)
         ops.attention(q, o, cache.k, cache.k, step, table, self.window or 0, self.scale, H, 1, row, workspace=ws,
@@ -167,7 +177,7 @@ class LatentAttention(Mixer):
         if self.general:
             return self._forward_general(x, residual, step, cache)
         T, ws, dt = x.shape[0], self.ctx.workspace, self.ctx.dtype
-        H, d, dv, r = self.heads, self.d, self.dv, self.rank
+        H, d, r = self.heads, self.d, self.rank
         proj = ws.buffer("latent.proj", (T, H * d + r), dt)
         ops.scope("attention.qkv_projection")
         linear(x, self.w_in, proj)
@@ -182,15 +192,7 @@ class LatentAttention(Mixer):
                 ops.latent_write(proj, H * d, r, self.latent_norm, self.eps, step, table, cache.k)
             ops.scope("attention.queries_to_latent")
             ops.head_matmul(proj, self.up_k, q)
-        ops.scope("attention.attention")
-        o = ws.buffer("latent.o", (T, H * r), dt)
-        ops.attention(q, o, cache.k, cache.k, step, table, self.window or 0, self.scale, H, 1, r, workspace=ws,
-                      decode_chunk=self.decode_chunk, sink=self.sink)
-        ops.scope("attention.latent_to_values")
-        v = ws.buffer("latent.v", (T, H * dv), dt)
-        ops.head_matmul(o, self.up_v, v)
-        ops.scope("attention.o_projection")
-        linear(v, self.w_o, residual, accumulate=True)
+        self._attend(q, residual, step, cache, table, r)
 
 
 registry.register("mixer", "latent_attention", LatentAttention)

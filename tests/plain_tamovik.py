@@ -145,12 +145,14 @@ def mlstm_gates(w, p, m, h):
     return i, f
 
 
-def matrix_memory(q, k, v, i, f):
-    """q, k [T, H, d], v [T, H, dv], log gates i, f [T, H] -> o [T, H, dv], token by token from zero."""
+def matrix_memory(q, k, v, i, f, terms=None):
+    """q, k [T, H, d], v [T, H, dv], log gates i, f [T, H] -> o [T, H, dv], token by token from zero.  `terms` collects, per
+    token, what the read-out's two sums are made of: (sum of |k||q||v| weighted, sum of |k||q| weighted, denominator)."""
     T, H, d = q.shape
     S, n = torch.zeros(H, d, v.shape[2], dtype=q.dtype), torch.zeros(H, d, dtype=q.dtype)
     m = torch.zeros(H, dtype=q.dtype)
     out = []
+    Sa, na = S.clone(), n.clone()
     for t in range(T):
         new = torch.maximum(f[t] + m, i[t])
         keep, add = torch.exp(f[t] + m - new), torch.exp(i[t] - new)
@@ -159,6 +161,10 @@ def matrix_memory(q, k, v, i, f):
         m = new
         den = torch.maximum((n * q[t]).sum(-1).abs(), torch.exp(-m)) + DENOMINATOR_EPS
         out.append(torch.einsum("hde,hd->he", S, q[t]) / den[:, None])
+        if terms is not None:
+            Sa = keep[:, None, None] * Sa + add[:, None, None] * (k[t][:, :, None] * v[t][:, None, :]).abs()
+            na = keep[:, None] * na + add[:, None] * k[t].abs()
+            terms.append((torch.einsum("hde,hd->he", Sa, q[t].abs()), (na * q[t].abs()).sum(-1), den))
     return torch.stack(out)
 
 
