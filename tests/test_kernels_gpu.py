@@ -295,8 +295,8 @@ def test_kernels_refuse_what_they_cannot_do():
     o = ops()
     with pytest.raises(KernelError, match="CUDA only"):
         o.rmsnorm(torch.randn(2, 8), torch.ones(8), 1e-6, torch.empty(2, 8))
-    q = torch.randn(1, 2 * 528, device="cuda")
-    kc = torch.zeros(2, 1, 16, 528, device="cuda")
+    q = torch.randn(1, 2 * 656, device="cuda")
+    kc = torch.zeros(2, 1, 16, 656, device="cuda")
     with pytest.raises(KernelError, match="head size"):
         o.paged_attention_simple(q, torch.empty_like(q), kc, kc, torch.zeros(1, dtype=torch.int32, device="cuda"),
                                  torch.zeros(1, dtype=torch.int32, device="cuda"),
