@@ -300,7 +300,7 @@ def test_kernels_refuse_what_they_cannot_do():
     with pytest.raises(KernelError, match="head size"):
         o.paged_attention_simple(q, torch.empty_like(q), kc, kc, torch.zeros(1, dtype=torch.int32, device="cuda"),
                                  torch.zeros(1, dtype=torch.int32, device="cuda"),
-                                 torch.zeros(1, 1, dtype=torch.int32, device="cuda"), 0, 1.0, 2, 1, 528)
+                                 torch.zeros(1, 1, dtype=torch.int32, device="cuda"), 0, 1.0, 2, 1, 656)
     with pytest.raises(KernelError, match="multiple"):
         kc = torch.zeros(2, 2, 16, 16, device="cuda")
         q = torch.randn(1, 3 * 16, device="cuda")
