@@ -379,7 +379,8 @@ ILB_EXPORT int ilb_mlstm_step(const void* proj, int dtype, int ld, int col_q, in
 // ---------------------------------------------------------------- long portions, 64 tokens at a time
 constexpr int kChunk = 64;            // tokens of a chunk
 constexpr int kTileCols = 64;         // value columns per block
-constexpr int kChunkThreads = 128;    // four warps
+constexpr int kHalfCols = 32;         // ... and per warp
+constexpr int kChunkThreads = 256;    // eight warps
 constexpr int kLdV = kTileCols + 8;   // row stride of tiles with 64 columns in shared memory (elements)
 
 // a = hi + mid + lo exactly, each a bfloat16 (8 + 8 + 8 significant bits); two numbers at a time
@@ -438,20 +439,29 @@ __device__ __forceinline__ void chunk_gates(const MlstmParams& p, int h, int t0,
 __device__ __forceinline__ void load_tile(const __nv_bfloat16* __restrict__ proj, int ld, int t0, int n, int col, int width, int padded,
                                           __nv_bfloat16* dst, int ld_dst, bool vec) {
   const int p8 = padded / 8;
-  for (int u = threadIdx.x; u < kChunk * p8; u += kChunkThreads) {
-    const int r = u / p8, c = (u % p8) * 8;
-    uint4 v = make_uint4(0u, 0u, 0u, 0u);
-    if (r < n && c < width) {
-      const __nv_bfloat16* src = proj + (size_t)(t0 + r) * ld + col + c;
-      if (vec && c + 8 <= width) v = __ldg(reinterpret_cast<const uint4*>(src));
-      else {
-        __nv_bfloat16 e[8];
+  constexpr int kFlight = 4;                             // units whose loads are in flight together
+  for (int u0 = threadIdx.x; u0 < kChunk * p8; u0 += kFlight * kChunkThreads) {
+    uint4 v[kFlight];
 #pragma unroll
-        for (int j = 0; j < 8; ++j) e[j] = c + j < width ? src[j] : __float2bfloat16_rn(0.f);
-        v = *reinterpret_cast<const uint4*>(e);
+    for (int f = 0; f < kFlight; ++f) {
+      const int u = u0 + f * kChunkThreads, r = u / p8, c = (u % p8) * 8;
+      v[f] = make_uint4(0u, 0u, 0u, 0u);
+      if (r < n && c < width) {
+        const __nv_bfloat16* src = proj + (size_t)(t0 + r) * ld + col + c;
+        if (vec && c + 8 <= width) v[f] = __ldg(reinterpret_cast<const uint4*>(src));
+        else {
+          __align__(16) __nv_bfloat16 e[8];
+#pragma unroll
+          for (int j = 0; j < 8; ++j) e[j] = c + j < width ? src[j] : __float2bfloat16_rn(0.f);
+          v[f] = *reinterpret_cast<const uint4*>(e);
+        }
       }
     }
-    *reinterpret_cast<uint4*>(dst + r * ld_dst + c) = v;
+#pragma unroll
+    for (int f = 0; f < kFlight; ++f) {
+      const int u = u0 + f * kChunkThreads;
+      if (u < kChunk * p8) *reinterpret_cast<uint4*>(dst + (u / p8) * ld_dst + (u % p8) * 8) = v[f];
+    }
   }
 }
 
@@ -460,7 +470,7 @@ static inline size_t local_smem(int d) { return (size_t)2 * kChunk * (padded16(d
 static inline size_t out_smem(int d) { return (size_t)2 * (2 * kChunk * (padded16(d) + 8) + kChunk * kLdV + 3 * padded16(d) * kLdV); }
 
 // (1) chunk_state = sum_s (w_s k_s) v_s^T with w_s = exp(F_L - F_s + i_s - m), m = max_s (F_L - F_s + i_s); chunk_norm the same
-// with k alone.  A block per (chunk, head, 64 columns); warp w takes rows 16 w, 16 w + 64, ...
+// with k alone.  A block per (chunk, head, 64 columns); a warp takes 16 rows and 32 of the columns at a time.
 __global__ void __launch_bounds__(kChunkThreads)
 mlstm_local_kernel(const MlstmParams p, const ChunkScratch s, int vec) {
   ilb::pdl_launch_dependents();
@@ -500,10 +510,12 @@ mlstm_local_kernel(const MlstmParams p, const ChunkScratch s, int vec) {
     wt[kb][2] = w[16 * kb + 2 * t4 + 8]; wt[kb][3] = w[16 * kb + 2 * t4 + 9];
   }
   float* dst = s.state + at * p.d * p.dv;
-  for (int r0 = warp * 16; r0 < DP; r0 += 64) {
-    float acc[kTileCols / 8][4];
+  for (int unit = warp; unit < DP / 8; unit += kChunkThreads / 32) {
+    const int r0 = (unit >> 1) * 16, n0 = (unit & 1) * kHalfCols;
+    if (c0 + n0 >= p.dv) continue;
+    float acc[kHalfCols / 8][4];
 #pragma unroll
-    for (int i = 0; i < kTileCols / 8; ++i)
+    for (int i = 0; i < kHalfCols / 8; ++i)
 #pragma unroll
       for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
 #pragma unroll
@@ -518,9 +530,9 @@ mlstm_local_kernel(const MlstmParams p, const ChunkScratch s, int vec) {
         split3(__uint_as_float(k[e] << 16) * wa, __uint_as_float(k[e] & 0xFFFF0000u) * wb, hi[e], mid[e], lo[e]);
       }
 #pragma unroll
-      for (int nd = 0; nd < kTileCols / 16; ++nd) {
+      for (int nd = 0; nd < kHalfCols / 16; ++nd) {
         uint32_t b0, b1, b2, b3;
-        ldmatrix_x4_trans(smem_u32(Vs + (16 * kb + (lane & 7) + ((lane >> 3) & 1) * 8) * kLdV + nd * 16 + (lane >> 4) * 8), b0, b1, b2, b3);
+        ldmatrix_x4_trans(smem_u32(Vs + (16 * kb + (lane & 7) + ((lane >> 3) & 1) * 8) * kLdV + n0 + nd * 16 + (lane >> 4) * 8), b0, b1, b2, b3);
         mma_16816(acc[2 * nd], lo, b0, b1);
         mma_16816(acc[2 * nd + 1], lo, b2, b3);
         mma_16816(acc[2 * nd], mid, b0, b1);
@@ -531,8 +543,8 @@ mlstm_local_kernel(const MlstmParams p, const ChunkScratch s, int vec) {
     }
     const int ra = r0 + (lane >> 2), rb = ra + 8;
 #pragma unroll
-    for (int i = 0; i < kTileCols / 8; ++i) {
-      const int c = c0 + i * 8 + 2 * t4;
+    for (int i = 0; i < kHalfCols / 8; ++i) {
+      const int c = c0 + n0 + i * 8 + 2 * t4;
       if (p.dv % 2 == 0) {
         if (c < p.dv) {
           if (ra < p.d) *reinterpret_cast<float2*>(dst + (size_t)ra * p.dv + c) = make_float2(acc[i][0], acc[i][1]);
@@ -552,13 +564,15 @@ mlstm_local_kernel(const MlstmParams p, const ChunkScratch s, int vec) {
 // (2) The chunks of a sequence one after the other: afterwards chunk_state, chunk_norm and chunk_max hold what comes INTO the
 // chunk, and the slot holds state and normaliser after the last one (m stays: every block here reads it).  A thread owns an
 // element (blocks beyond the state's: of the normaliser).
-constexpr int kCarryBatch = 4;
+constexpr int kCarryBatch = 16;       // chunks whose loads are in flight together
+constexpr int kCarryTile = 32;        // chunks whose factors are in shared memory at a time
 
 __global__ void __launch_bounds__(256)
 mlstm_carry_kernel(const MlstmParams p, const ChunkScratch s, float* __restrict__ max_in, int state_blocks) {
   ilb::pdl_launch_dependents();
   ilb::pdl_wait();
-  const int h = blockIdx.y, seq = blockIdx.z;
+  __shared__ float keep[kCarryTile], add[kCarryTile];
+  const int h = blockIdx.y, seq = blockIdx.z, lane = threadIdx.x & 31;
   const bool is_norm = (int)blockIdx.x >= state_blocks;
   const int size = is_norm ? p.d : p.d * p.dv;
   const int e = ((int)blockIdx.x - (is_norm ? state_blocks : 0)) * 256 + threadIdx.x;
@@ -566,36 +580,48 @@ mlstm_carry_kernel(const MlstmParams p, const ChunkScratch s, float* __restrict_
   for (int i = 0; i < seq; ++i) first += (p.cu_q[i + 1] - p.cu_q[i] + kChunk - 1) / kChunk;
   const int n = (p.cu_q[seq + 1] - p.cu_q[seq] + kChunk - 1) / kChunk;
   const int slot = p.slots[seq];
-  float m = slot >= 0 ? p.max[(size_t)slot * p.heads + h] : 0.f;
+  float m = slot >= 0 ? p.max[(size_t)slot * p.heads + h] : 0.f;      // (kept by the first warp)
   float* own = slot >= 0 ? (is_norm ? p.norm : p.state) + ((size_t)slot * p.heads + h) * size + e : nullptr;
   float* at = (is_norm ? s.norm : s.state) + e;
   const bool live = e < size;
   float run = own != nullptr && live ? *own : 0.f;
-  for (int c0 = first; c0 < first + n; c0 += kCarryBatch) {
-    float local[kCarryBatch], lm[kCarryBatch], ls[kCarryBatch];
-#pragma unroll
-    for (int j = 0; j < kCarryBatch; ++j) {
-      const size_t c = (size_t)min(c0 + j, first + n - 1) * p.heads + h;
-      local[j] = live ? at[c * size] : 0.f;
-      lm[j] = s.max[c];
-      ls[j] = s.sum[c];
-    }
-#pragma unroll
-    for (int j = 0; j < kCarryBatch; ++j) {
-      if (c0 + j < first + n) {
-        const size_t c = (size_t)(c0 + j) * p.heads + h;
-        if (live) at[c * size] = run;
-        if (blockIdx.x == 0 && threadIdx.x == 0) max_in[c] = m;
-        const float next = fmaxf(ls[j] + m, lm[j]);
-        run = fmaf(expf(ls[j] + m - next), run, expf(lm[j] - next) * local[j]);
+  for (int t0 = 0; t0 < n; t0 += kCarryTile) {
+    const int tn = min(kCarryTile, n - t0);
+    __syncthreads();                                     // everyone is done with the tile before
+    if (threadIdx.x < 32) {
+      const size_t c = (size_t)(first + t0 + min(lane, tn - 1)) * p.heads + h;
+      const float lm = s.max[c], ls = s.sum[c];
+      float before = m, after = m;
+      for (int j = 0; j < tn; ++j) {
+        const float next = fmaxf(__shfl_sync(0xffffffffu, ls, j) + m, __shfl_sync(0xffffffffu, lm, j));
+        if (lane == j) { before = m; after = next; }
         m = next;
+      }
+      if (lane < tn) {
+        keep[lane] = expf(ls + before - after);
+        add[lane] = expf(lm - after);
+        if (blockIdx.x == 0) max_in[c] = before;
+      }
+    }
+    __syncthreads();
+    for (int c0 = 0; c0 < tn; c0 += kCarryBatch) {
+      float local[kCarryBatch];
+#pragma unroll
+      for (int j = 0; j < kCarryBatch; ++j)
+        local[j] = live && c0 + j < tn ? at[((size_t)(first + t0 + c0 + j) * p.heads + h) * size] : 0.f;
+#pragma unroll
+      for (int j = 0; j < kCarryBatch; ++j) {
+        if (c0 + j < tn) {
+          if (live) at[((size_t)(first + t0 + c0 + j) * p.heads + h) * size] = run;
+          run = fmaf(keep[c0 + j], run, add[c0 + j] * local[j]);
+        }
       }
     }
   }
   if (own != nullptr && live && n > 0) *own = run;
 }
 
-// (3) A block per (chunk, head, 64 columns); warp w owns tokens 16 w .. 16 w + 15 of the chunk.
+// (3) A block per (chunk, head, 64 columns); warp w owns tokens 16 (w % 4) .. + 15 of the chunk and 32 of the columns.
 __global__ void __launch_bounds__(kChunkThreads)
 mlstm_out_kernel(const MlstmParams p, const ChunkScratch s, const float* __restrict__ max_in, float* __restrict__ y, int vec) {
   ilb::pdl_launch_dependents();
@@ -612,7 +638,8 @@ mlstm_out_kernel(const MlstmParams p, const ChunkScratch s, const float* __restr
   if (!find_tile(p.cu_q, p.n_seqs, kChunk, blockIdx.x, seq, ci)) return;
   const int h = blockIdx.y, c0 = blockIdx.z * kTileCols;
   const int tok0 = p.cu_q[seq], q_len = p.cu_q[seq + 1] - tok0, t0 = tok0 + ci * kChunk, n = min(kChunk, q_len - ci * kChunk);
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g8 = lane >> 2, t4 = lane & 3;
+  const int tid = threadIdx.x, lane = tid & 31, g8 = lane >> 2, t4 = lane & 3;
+  const int warp = (tid >> 5) & 3, n0 = (tid >> 7) * kHalfCols;      // rows and columns of this warp
   const __nv_bfloat16* proj = reinterpret_cast<const __nv_bfloat16*>(p.proj);
   const size_t at = (size_t)blockIdx.x * p.heads + h;
   const float m_in = max_in[at];
@@ -622,41 +649,65 @@ mlstm_out_kernel(const MlstmParams p, const ChunkScratch s, const float* __restr
   {
     const float* S = s.state + at * p.d * p.dv;
     const int plane = DP * kLdV;
-    const bool pairs = p.dv % 2 == 0;
-    for (int u = tid; u < DP * (kTileCols / 2); u += kChunkThreads) {
-      const int r = u / (kTileCols / 2), c = (u % (kTileCols / 2)) * 2;
-      float2 v = make_float2(0.f, 0.f);
-      if (r < p.d && c0 + c < p.dv) {
-        const float* src = S + (size_t)r * p.dv + c0 + c;
-        if (pairs) v = *reinterpret_cast<const float2*>(src);
-        else { v.x = src[0]; v.y = c0 + c + 1 < p.dv ? src[1] : 0.f; }
+    const bool fours = p.dv % 4 == 0;
+    constexpr int kFlight = 8;                           // units of four columns whose loads are in flight together
+    for (int u0 = tid; u0 < DP * (kTileCols / 4); u0 += kFlight * kChunkThreads) {
+      float4 v[kFlight];
+#pragma unroll
+      for (int f = 0; f < kFlight; ++f) {
+        const int u = u0 + f * kChunkThreads, r = u / (kTileCols / 4), c = c0 + (u % (kTileCols / 4)) * 4;
+        v[f] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (r < p.d && c < p.dv) {
+          const float* src = S + (size_t)r * p.dv + c;
+          if (fours) v[f] = *reinterpret_cast<const float4*>(src);
+          else {
+            v[f].x = src[0];
+            if (c + 1 < p.dv) v[f].y = src[1];
+            if (c + 2 < p.dv) v[f].z = src[2];
+            if (c + 3 < p.dv) v[f].w = src[3];
+          }
+        }
       }
-      uint32_t hi, mid, lo;
-      split3(v.x, v.y, hi, mid, lo);
-      *reinterpret_cast<uint32_t*>(Ss + r * kLdV + c) = hi;
-      *reinterpret_cast<uint32_t*>(Ss + plane + r * kLdV + c) = mid;
-      *reinterpret_cast<uint32_t*>(Ss + 2 * plane + r * kLdV + c) = lo;
+#pragma unroll
+      for (int f = 0; f < kFlight; ++f) {
+        const int u = u0 + f * kChunkThreads;
+        if (u < DP * (kTileCols / 4)) {
+          uint2 hi, mid, lo;
+          split3(v[f].x, v[f].y, hi.x, mid.x, lo.x);
+          split3(v[f].z, v[f].w, hi.y, mid.y, lo.y);
+          __nv_bfloat16* at = Ss + (u / (kTileCols / 4)) * kLdV + (u % (kTileCols / 4)) * 4;
+          *reinterpret_cast<uint2*>(at) = hi;
+          *reinterpret_cast<uint2*>(at + plane) = mid;
+          *reinterpret_cast<uint2*>(at + 2 * plane) = lo;
+        }
+      }
     }
   }
-  if (warp == 0) chunk_gates(p, h, t0, n, g);
+  if (tid < 32) chunk_gates(p, h, t0, n, g);
   __syncthreads();
   if (tid < kChunk) ms[tid] = g.F[tid] + fmaxf(m_in, g.M[tid]);
-  {   // n_in . q: two threads a token
-    const int t = tid >> 1, half = tid & 1;
+  {   // n_in . q: four threads a token
+    const int t = tid >> 2, part = tid & 3;
     const float* nin = s.norm + at * p.d;
     float v = 0.f;
-    for (int r = half; r < p.d; r += 2) v = fmaf(nin[r], __bfloat162float(Qs[t * ldk + r]), v);
+#pragma unroll 8
+    for (int r = part; r < p.d; r += 4) v = fmaf(nin[r], __bfloat162float(Qs[t * ldk + r]), v);
     v += __shfl_xor_sync(0xffffffffu, v, 1);
-    if (half == 0) nq[t] = v;
+    v += __shfl_xor_sync(0xffffffffu, v, 2);
+    if (part == 0) nq[t] = v;
   }
   __syncthreads();
   const int ra = warp * 16 + g8, rb = ra + 8;            // this lane's two tokens
-  if (warp * 16 < n) {
-    float P[kChunk / 8][4], O[kTileCols / 8][4];
+  if (warp * 16 < n && c0 + n0 < p.dv) {
+    float P[kChunk / 8][4], O[kHalfCols / 8][4];
 #pragma unroll
     for (int i = 0; i < kChunk / 8; ++i)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) { P[i][e] = 0.f; O[i][e] = 0.f; }
+      for (int e = 0; e < 4; ++e) P[i][e] = 0.f;
+#pragma unroll
+    for (int i = 0; i < kHalfCols / 8; ++i)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) O[i][e] = 0.f;
     for (int kb = 0; kb < DP / 16; ++kb) {
       uint32_t a[4];
       ldmatrix_x4(smem_u32(Qs + (warp * 16 + (lane & 15)) * ldk + kb * 16 + (lane >> 4) * 8), a[0], a[1], a[2], a[3]);
@@ -673,9 +724,9 @@ mlstm_out_kernel(const MlstmParams p, const ChunkScratch s, const float* __restr
       // the incoming state's read-out
 #pragma unroll
       for (int piece = 2; piece >= 0; --piece) {
-        const __nv_bfloat16* S = Ss + piece * DP * kLdV;
+        const __nv_bfloat16* S = Ss + piece * DP * kLdV + n0;
 #pragma unroll
-        for (int nd = 0; nd < kTileCols / 16; ++nd) {
+        for (int nd = 0; nd < kHalfCols / 16; ++nd) {
           uint32_t b0, b1, b2, b3;
           ldmatrix_x4_trans(smem_u32(S + (kb * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * kLdV + nd * 16 + (lane >> 4) * 8), b0, b1, b2, b3);
           mma_16816(O[2 * nd], a, b0, b1);
@@ -686,7 +737,7 @@ mlstm_out_kernel(const MlstmParams p, const ChunkScratch s, const float* __restr
     const float ma = ms[ra], mb = ms[rb], Fa = g.F[ra] - ma, Fb = g.F[rb] - mb;
     const float ga = __expf(Fa + m_in) * p.q_scale, gb = __expf(Fb + m_in) * p.q_scale;
 #pragma unroll
-    for (int i = 0; i < kTileCols / 8; ++i) { O[i][0] *= ga; O[i][1] *= ga; O[i][2] *= gb; O[i][3] *= gb; }
+    for (int i = 0; i < kHalfCols / 8; ++i) { O[i][0] *= ga; O[i][1] *= ga; O[i][2] *= gb; O[i][3] *= gb; }
     float suma = 0.f, sumb = 0.f;
 #pragma unroll
     for (int i = 0; i < kChunk / 8; ++i) {
@@ -711,9 +762,9 @@ mlstm_out_kernel(const MlstmParams p, const ChunkScratch s, const float* __restr
         split3(P[2 * kb + 1][0], P[2 * kb + 1][1], hi[2], mid[2], lo[2]);
         split3(P[2 * kb + 1][2], P[2 * kb + 1][3], hi[3], mid[3], lo[3]);
 #pragma unroll
-        for (int nd = 0; nd < kTileCols / 16; ++nd) {
+        for (int nd = 0; nd < kHalfCols / 16; ++nd) {
           uint32_t b0, b1, b2, b3;
-          ldmatrix_x4_trans(smem_u32(Vs + (16 * kb + (lane & 7) + ((lane >> 3) & 1) * 8) * kLdV + nd * 16 + (lane >> 4) * 8), b0, b1, b2, b3);
+          ldmatrix_x4_trans(smem_u32(Vs + (16 * kb + (lane & 7) + ((lane >> 3) & 1) * 8) * kLdV + n0 + nd * 16 + (lane >> 4) * 8), b0, b1, b2, b3);
           mma_16816(O[2 * nd], lo, b0, b1);
           mma_16816(O[2 * nd + 1], lo, b2, b3);
           mma_16816(O[2 * nd], mid, b0, b1);
@@ -729,8 +780,8 @@ mlstm_out_kernel(const MlstmParams p, const ChunkScratch s, const float* __restr
     float* ya = y + (size_t)(t0 + ra) * inner + (size_t)h * p.dv;
     float* yb = y + (size_t)(t0 + rb) * inner + (size_t)h * p.dv;
 #pragma unroll
-    for (int i = 0; i < kTileCols / 8; ++i) {
-      const int c = c0 + i * 8 + 2 * t4;
+    for (int i = 0; i < kHalfCols / 8; ++i) {
+      const int c = c0 + n0 + i * 8 + 2 * t4;
       if (p.dv % 2 == 0) {
         if (c < p.dv) {
           if (ra < n) *reinterpret_cast<float2*>(ya + c) = make_float2(O[i][0] * da, O[i][1] * da);

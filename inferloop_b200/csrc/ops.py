@@ -996,6 +996,9 @@ def rows_norm_rope_cache(qkv: torch.Tensor, q_out: torch.Tensor, q_weight: torch
           _i(0 if pooled is None else pooled.k.shape[0]), _i(0 if pooled is None else pooled.pool), _stream(qkv))
 
 
+CONV_TILE = 4              # tokens of a sequence per block of the convolved input stage
+
+
 def conv_rows_norm_cache(qkv: torch.Tensor, q_out: torch.Tensor, conv_w: torch.Tensor, conv_state: torch.Tensor, q_weight: torch.Tensor,
                          k_weight: torch.Tensor, eps: float, rope: Optional[torch.Tensor], rotary_dim: int, step, block_table: torch.Tensor,
                          k_cache: Optional[torch.Tensor], v_cache: Optional[torch.Tensor], nq: int, nkv: int, d: int, dv: int,
@@ -1020,7 +1023,7 @@ def conv_rows_norm_cache(qkv: torch.Tensor, q_out: torch.Tensor, conv_w: torch.T
             raise KernelError("conv_rows_norm_cache: cache shapes do not match the heads")
     _call("qk_norm_rope", "ilb_conv_rows_norm_cache", _ptr(qkv), _ptr(q_out), _i(_code(qkv)), _ptr(conv_w), _i(taps), _ptr(conv_state), _ptr(q_weight),
           _ptr(k_weight), _f(eps), _ptr(rope), _i(rotary_dim), _ptr(step.positions), _ptr(step.seq_of_token), _ptr(step.cu_q), _ptr(step.slots),
-          _i(step.n_seqs), _i(0 if step.decode_only else 1), _ptr(block_table), _i(block_table.shape[1]), _i(page_size), _i(num_pages), _ptr(k_cache),
+          _i(step.n_seqs), _i(sum(-(-n // CONV_TILE) for n in step.h_q_len) + (step.n_seqs - len(step.h_q_len))), _i(0 if step.decode_only else 1), _ptr(block_table), _i(block_table.shape[1]), _i(page_size), _i(num_pages), _ptr(k_cache),
           _ptr(v_cache), _i(T), _i(nq), _i(nkv), _i(d), _i(dv), _i(qkv.stride(0)), _i(q_out.shape[1]), _i(1 if values_are_keys else 0), _stream(qkv))
 
 

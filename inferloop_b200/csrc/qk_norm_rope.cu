@@ -636,126 +636,183 @@ ILB_EXPORT int ilb_rows_norm_rope_cache(
 //   u_t = sum_j w[j, c] raw_{t - (taps - 1) + j},   q <- turn(u_q / sqrt(mean(u_q^2) + eps) * wq),   k likewise
 // and values that are either columns of their own behind q | k, as they are, or (values_are_keys) u_k before its norm.
 // The raw inputs ahead of the step come from state [slots, taps - 1, (nq + nkv) d] 32-bit; zeros before the sequence's start.
-// A block a token: the convolved row waits in shared memory for its sums.  A sequence of one token is one block, which also
-// moves the state on; the state of the others is moved on by a second launch, when nobody reads the old one any more.
+// A block takes up to TT consecutive tokens of a sequence: a thread owns units of VEC channels, has the raw inputs of all its
+// taps and tokens in flight together, and the convolved rows wait in shared memory for their sums.  A sequence of one token is
+// one block, which also moves the state on; the state of the others is moved on by a second launch, when nobody reads the old
+// one any more.
 constexpr int kMostTaps = 16;
+constexpr int kConvTile = 4;                             // tokens of a sequence per block (1 for rows that would not fit shared memory so often)
 
 struct ConvRowsParams {
   RowsParams r;
   const float* conv_w;               // [taps, (nq + nkv) d]
   float* state;
   const int* cu_q; const int* slots;
-  int taps, values_are_keys;
+  int n_seqs, taps, values_are_keys;
 };
 
-// MT: the most taps this form holds in flight (taps <= MT).
-template <typename T, int VEC, int MT>
-__global__ void __launch_bounds__(kRowsThreads)
+// VEC raw inputs as they are stored.  (The state keeps them widened: a bfloat16 input comes back from there without loss.)
+template <typename T, int VEC> struct RawUnit;
+template <typename T> struct RawUnit<T, 1> {
+  float v;
+  __device__ __forceinline__ void zero() { v = 0.f; }
+  __device__ __forceinline__ void load(const T* p) { v = to_float(*p); }
+  __device__ __forceinline__ void load_state(const float* p) { v = *p; }
+  __device__ __forceinline__ void get(float* x) const { x[0] = v; }
+  __device__ __forceinline__ void store_state(float* p) const { *p = v; }
+};
+template <> struct RawUnit<__nv_bfloat16, 8> {
+  uint4 v;
+  __device__ __forceinline__ void zero() { v = make_uint4(0u, 0u, 0u, 0u); }
+  __device__ __forceinline__ void load(const __nv_bfloat16* p) { v = *reinterpret_cast<const uint4*>(p); }
+  __device__ __forceinline__ void load_state(const float* p) {      // (plain loads: this launch may write the slot)
+    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+    const float x[8] = {a.x, a.y, a.z, a.w, b.x, b.y, b.z, b.w};
+    v = pack8(x);
+  }
+  __device__ __forceinline__ void get(float* x) const { unpack8(v, x); }
+  __device__ __forceinline__ void store_state(float* p) const {
+    float x[8];
+    unpack8(v, x);
+    reinterpret_cast<float4*>(p)[0] = make_float4(x[0], x[1], x[2], x[3]);
+    reinterpret_cast<float4*>(p)[1] = make_float4(x[4], x[5], x[6], x[7]);
+  }
+};
+
+// MT: the most taps (taps <= MT; the taps are aligned to its end).
+template <typename T, int VEC, int MT, int TT>
+__global__ void __launch_bounds__(512)
 conv_rows_norm_kernel(const T* __restrict__ qkv, T* __restrict__ q_out, T* k_cache, T* v_cache, const ConvRowsParams c) {
   ilb::pdl_launch_dependents();
   ilb::pdl_wait();
   const RowsParams& p = c.r;
-  extern __shared__ __align__(16) float u[];             // [(nq + nkv) d]
-  __shared__ float scratch[33];
-  const int t = blockIdx.x, seq = p.seq_of_token[t];
-  const int tok0 = c.cu_q[seq], lt = t - tok0, slot = c.slots[seq];
-  const bool alone = c.cu_q[seq + 1] - tok0 == 1;
-  const int nqd = p.nq * p.d, nkd = p.nkv * p.d, width = nqd + nkd, before = c.taps - 1;
+  extern __shared__ __align__(16) float u[];             // [TT][(nq + nkv) d]
+  __shared__ float scratch[2 * TT * 16];
+  __shared__ long long places[TT];
+  __shared__ float inv[2 * TT];
+  int seq = 0, tile = blockIdx.x;
+  for (; seq < c.n_seqs; ++seq) {
+    const int n = (c.cu_q[seq + 1] - c.cu_q[seq] + TT - 1) / TT;
+    if (tile < n) break;
+    tile -= n;
+  }
+  if (seq >= c.n_seqs) return;
+  const int tok0 = c.cu_q[seq], q_len = c.cu_q[seq + 1] - tok0, slot = c.slots[seq];
+  const int lt0 = tile * TT, ts = min(TT, q_len - lt0), t0 = tok0 + lt0;
+  const int nqd = p.nq * p.d, nkd = p.nkv * p.d, width = nqd + nkd, before = c.taps - 1, skip = MT - c.taps;
   float* own = slot >= 0 ? c.state + (size_t)slot * before * width : nullptr;
-  float sum_q = 0.f, sum_k = 0.f;
-  for (int e = threadIdx.x * VEC; e < width; e += kRowsThreads * VEC) {
-    float acc[VEC], x[MT][VEC];
-#pragma unroll
-    for (int i = 0; i < VEC; ++i) acc[i] = 0.f;
-#pragma unroll
-    for (int j = 0; j < MT; ++j) {                         // every tap's inputs are asked for before the first is used
-      const int back = before - j;
-      if (j < c.taps && lt >= back) RowUnit<T, VEC>::load(qkv + (size_t)(t - back) * p.qkv_stride + e, x[j]);
-      else if (j < c.taps && own != nullptr) {             // (plain loads: this launch may write the slot)
-        const float* s = own + (size_t)(before + lt - back) * width + e;
-        if constexpr (VEC == 8) {
-          const float4 a = *reinterpret_cast<const float4*>(s), b = *reinterpret_cast<const float4*>(s + 4);
-          x[j][0] = a.x; x[j][1] = a.y; x[j][2] = a.z; x[j][3] = a.w; x[j][4] = b.x; x[j][5] = b.y; x[j][6] = b.z; x[j][7] = b.w;
-        } else {
-          x[j][0] = *s;
-        }
-      } else {
-#pragma unroll
-        for (int i = 0; i < VEC; ++i) x[j][i] = 0.f;
+  const int warps = blockDim.x / 32, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (threadIdx.x < ts) {                                // where each token's key and value go
+    long long place = -1;
+    if (k_cache != nullptr) {
+      const int pos = p.positions[t0 + threadIdx.x], blk = pos / p.page_size;
+      if (blk >= 0 && blk < p.max_blocks) {
+        const int page = p.block_table[(size_t)seq * p.max_blocks + blk];
+        if (page >= 0 && page < p.num_pages) place = (long long)page * p.nkv * p.page_size + pos % p.page_size;      // never write outside the pool
       }
     }
+    places[threadIdx.x] = place;
+  }
+  float sum_q[TT], sum_k[TT];
+#pragma unroll
+  for (int tt = 0; tt < TT; ++tt) { sum_q[tt] = 0.f; sum_k[tt] = 0.f; }
+  for (int e = threadIdx.x * VEC; e < width; e += blockDim.x * VEC) {
+    RawUnit<T, VEC> raw[MT + TT - 1];                    // row r: the token r - (MT - 1) places from the tile's first
+#pragma unroll
+    for (int r = 0; r < MT + TT - 1; ++r) {
+      const int lt = lt0 + r - (MT - 1);
+      raw[r].zero();
+      if (r >= skip && lt < q_len) {
+        if (lt >= 0) raw[r].load(qkv + (size_t)(tok0 + lt) * p.qkv_stride + e);
+        else if (own != nullptr) raw[r].load_state(own + (size_t)(before + lt) * width + e);
+      }
+    }
+    float acc[TT][VEC];
+#pragma unroll
+    for (int tt = 0; tt < TT; ++tt)
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) acc[tt][i] = 0.f;
 #pragma unroll
     for (int j = 0; j < MT; ++j) {
-      if (j < c.taps) {
+      if (j >= skip) {
         float w[VEC];
-        load_f32<VEC>(c.conv_w + (size_t)j * width + e, w);
+        load_f32<VEC>(c.conv_w + (size_t)(j - skip) * width + e, w);
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) acc[i] = fmaf(w[i], x[j][i], acc[i]);
-        if (alone && j > 0 && own != nullptr) {
-          float* s = own + (size_t)(j - 1) * width + e;
-          if constexpr (VEC == 8) {
-            reinterpret_cast<float4*>(s)[0] = make_float4(x[j][0], x[j][1], x[j][2], x[j][3]);
-            reinterpret_cast<float4*>(s)[1] = make_float4(x[j][4], x[j][5], x[j][6], x[j][7]);
-          } else {
-            *s = x[j][0];
-          }
+        for (int tt = 0; tt < TT; ++tt) {
+          float x[VEC];
+          raw[j + tt].get(x);
+#pragma unroll
+          for (int i = 0; i < VEC; ++i) acc[tt][i] = fmaf(w[i], x[i], acc[tt][i]);
         }
       }
     }
-    float ss = 0.f;
+    if (q_len == 1 && own != nullptr) {
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) { u[e + i] = acc[i]; ss = fmaf(acc[i], acc[i], ss); }
-    if (e < nqd) sum_q += ss; else sum_k += ss;
+      for (int r = 1; r < MT; ++r)
+        if (r > skip) raw[r].store_state(own + (size_t)(r - skip - 1) * width + e);
+    }
+#pragma unroll
+    for (int tt = 0; tt < TT; ++tt) {
+      float ss = 0.f;
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) { u[(size_t)tt * width + e + i] = acc[tt][i]; ss = fmaf(acc[tt][i], acc[tt][i], ss); }
+      if (e < nqd) sum_q[tt] += ss; else sum_k[tt] += ss;
+    }
   }
-  sum_q = warp_sum(sum_q);
-  sum_k = warp_sum(sum_k);
-  if ((threadIdx.x & 31) == 0) { scratch[threadIdx.x >> 5] = sum_q; scratch[16 + (threadIdx.x >> 5)] = sum_k; }
+#pragma unroll
+  for (int tt = 0; tt < TT; ++tt) {
+    const float a = warp_sum(sum_q[tt]), b = warp_sum(sum_k[tt]);
+    if (lane == 0) { scratch[(2 * tt) * 16 + warp] = a; scratch[(2 * tt + 1) * 16 + warp] = b; }
+  }
   __syncthreads();
-  sum_q = 0.f; sum_k = 0.f;
-#pragma unroll
-  for (int w = 0; w < kRowsThreads / 32; ++w) { sum_q += scratch[w]; sum_k += scratch[16 + w]; }
-  const float inv_q = 1.0f / sqrtf(sum_q / (float)nqd + p.eps);
-  const float inv_k = 1.0f / sqrtf(sum_k / (float)nkd + p.eps);
-  long long place = -1;
-  if (k_cache != nullptr) {
-    const int pos = p.positions[t], blk = pos / p.page_size;
-    if (blk >= 0 && blk < p.max_blocks) {
-      const int page = p.block_table[(size_t)seq * p.max_blocks + blk];
-      if (page >= 0 && page < p.num_pages) place = (long long)page * p.nkv * p.page_size + pos % p.page_size;      // never write outside the pool
-    }
+  if (threadIdx.x < 2 * TT) {
+    float a = 0.f;
+    for (int w = 0; w < warps; ++w) a += scratch[threadIdx.x * 16 + w];
+    inv[threadIdx.x] = 1.0f / sqrtf(a / (float)((threadIdx.x & 1) ? nkd : nqd) + p.eps);
   }
+  __syncthreads();
   const int half = p.rotary_dim / 2;
-  for (int e = threadIdx.x * VEC; e < width; e += kRowsThreads * VEC) {
+  for (int e = threadIdx.x * VEC; e < width; e += blockDim.x * VEC) {
     const bool is_q = e < nqd;
-    if (!is_q && place < 0) continue;
     const int r = is_q ? e : e - nqd, h = r / p.d, ch = r % p.d;
-    const float inv = is_q ? inv_q : inv_k;
-    float x[VEC], w[VEC];
-#pragma unroll
-    for (int i = 0; i < VEC; ++i) x[i] = u[e + i];
-    if (!is_q && c.values_are_keys) RowUnit<T, VEC>::store(v_cache + ((size_t)place + (size_t)h * p.page_size) * p.dv + ch, x);
+    const bool turned = p.rope != nullptr && ch < 2 * half;
+    const int o = ch < half ? half : -half;              // the pair's other member
+    float w[VEC], w2[VEC];
     load_f32<VEC>((is_q ? p.q_weight : p.k_weight) + r, w);
+    if (turned) load_f32<VEC>((is_q ? p.q_weight : p.k_weight) + r + o, w2);
 #pragma unroll
-    for (int i = 0; i < VEC; ++i) x[i] = x[i] * inv * w[i];
-    if (p.rope != nullptr && ch < 2 * half) {
-      const int o = ch < half ? half : -half;            // the pair's other member
-      float y[VEC], cs[2 * VEC];
-      load_f32<VEC>((is_q ? p.q_weight : p.k_weight) + r + o, w);
-      load_f32<2 * VEC>(reinterpret_cast<const float*>(p.rope + (size_t)t * half + (ch < half ? ch : ch - half)), cs);
+    for (int tt = 0; tt < TT; ++tt) {
+      if (tt >= ts) break;
+      const long long place = places[tt];
+      if (!is_q && place < 0) continue;
+      const float f = inv[2 * tt + (is_q ? 0 : 1)];
+      const float* ut = u + (size_t)tt * width + e;
+      float x[VEC];
 #pragma unroll
-      for (int i = 0; i < VEC; ++i) {
-        y[i] = u[e + o + i] * inv * w[i];
-        x[i] = __fadd_rn(__fmul_rn(x[i], cs[2 * i]), __fmul_rn(y[i], ch < half ? -cs[2 * i + 1] : cs[2 * i + 1]));
+      for (int i = 0; i < VEC; ++i) x[i] = ut[i];
+      if (!is_q && c.values_are_keys) RowUnit<T, VEC>::store(v_cache + ((size_t)place + (size_t)h * p.page_size) * p.dv + ch, x);
+#pragma unroll
+      for (int i = 0; i < VEC; ++i) x[i] = x[i] * f * w[i];
+      if (turned) {
+        float cs[2 * VEC];
+        load_f32<2 * VEC>(reinterpret_cast<const float*>(p.rope + (size_t)(t0 + tt) * half + (ch < half ? ch : ch - half)), cs);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) {
+          const float y = ut[o + i] * f * w2[i];
+          x[i] = __fadd_rn(__fmul_rn(x[i], cs[2 * i]), __fmul_rn(y, ch < half ? -cs[2 * i + 1] : cs[2 * i + 1]));
+        }
       }
+      if (is_q) RowUnit<T, VEC>::store(q_out + (size_t)(t0 + tt) * p.q_out_stride + r, x);
+      else RowUnit<T, VEC>::store(k_cache + ((size_t)place + (size_t)h * p.page_size) * p.d + ch, x);
     }
-    if (is_q) RowUnit<T, VEC>::store(q_out + (size_t)t * p.q_out_stride + r, x);
-    else RowUnit<T, VEC>::store(k_cache + ((size_t)place + (size_t)h * p.page_size) * p.d + ch, x);
   }
-  if (c.values_are_keys || place < 0) return;
-  for (int e = threadIdx.x * VEC; e < p.nkv * p.dv; e += kRowsThreads * VEC) {
+  if (c.values_are_keys) return;
+  for (int e = threadIdx.x * VEC; e < p.nkv * p.dv * ts; e += blockDim.x * VEC) {
+    const int tt = e / (p.nkv * p.dv), r = e % (p.nkv * p.dv);
+    if (places[tt] < 0) continue;
     float x[VEC];
-    RowUnit<T, VEC>::load(qkv + (size_t)t * p.qkv_stride + width + e, x);
-    RowUnit<T, VEC>::store(v_cache + ((size_t)place + (size_t)(e / p.dv) * p.page_size) * p.dv + e % p.dv, x);
+    RowUnit<T, VEC>::load(qkv + (size_t)(t0 + tt) * p.qkv_stride + width + r, x);
+    RowUnit<T, VEC>::store(v_cache + ((size_t)places[tt] + (size_t)(r / p.dv) * p.page_size) * p.dv + r % p.dv, x);
   }
 }
 
@@ -776,11 +833,12 @@ conv_rows_state_kernel(const T* __restrict__ qkv, int ld, int width, int before,
   }
 }
 
-// qkv [T, qkv_stride] of `dtype`: raw q | k (| v); n_several: whether a sequence of the step brings more than one token.
+// qkv [T, qkv_stride] of `dtype`: raw q | k (| v); n_tiles: the sum over the sequences of ceil(tokens / 4); several: whether a
+// sequence of the step brings more than one token.
 ILB_EXPORT int ilb_conv_rows_norm_cache(
     const void* qkv, void* q_out, int dtype, const float* conv_w, int taps, float* state, const float* q_weight, const float* k_weight,
     float eps, const float* rope, int rotary_dim, const int* positions, const int* seq_of_token, const int* cu_q, const int* slots,
-    int n_seqs, int n_several, const int* block_table, int max_blocks, int page_size, int num_pages, void* k_cache, void* v_cache,
+    int n_seqs, int n_tiles, int several, const int* block_table, int max_blocks, int page_size, int num_pages, void* k_cache, void* v_cache,
     int n_tokens, int nq, int nkv, int d, int dv, int qkv_stride, int q_out_stride, int values_are_keys, cudaStream_t stream) {
   ILB_REQUIRE(n_tokens >= 0 && nq > 0 && nkv > 0 && d > 0 && dv > 0 && eps > 0.f && n_seqs >= 0 && n_seqs <= 65535, "conv_rows_norm: bad sizes");
   ILB_REQUIRE(conv_w != nullptr && taps >= 1 && taps <= kMostTaps && (taps == 1 || state != nullptr), "conv_rows_norm: %d taps (at most %d) need weights and a state", taps, kMostTaps);
@@ -793,33 +851,41 @@ ILB_EXPORT int ilb_conv_rows_norm_cache(
   ILB_REQUIRE((k_cache == nullptr) == (v_cache == nullptr), "conv_rows_norm: need both caches or none");
   ILB_REQUIRE(k_cache == nullptr || (page_size > 0 && max_blocks > 0 && num_pages > 0), "conv_rows_norm: bad cache geometry");
   ILB_REQUIRE(dtype == kF32 || dtype == kBF16, "conv_rows_norm: unknown dtype %d", dtype);
-  const size_t smem = sizeof(float) * width;
   constexpr int kMost = 200 * 1024;
+  // (single tokens, and rows of many channels, go a token a block)
+  const int tile = several && (size_t)kConvTile * width * sizeof(float) <= 100 * 1024 ? kConvTile : 1;
+  const size_t smem = sizeof(float) * width * tile;
   ILB_REQUIRE(smem <= kMost, "conv_rows_norm: rows of %d channels do not fit shared memory", width);
   if (n_tokens == 0) return 0;
   ConvRowsParams c{};
   c.r.q_weight = q_weight; c.r.k_weight = k_weight; c.r.rope = (const float2*)rope; c.r.positions = positions; c.r.seq_of_token = seq_of_token;
   c.r.block_table = block_table; c.r.max_blocks = max_blocks; c.r.page_size = page_size; c.r.num_pages = num_pages; c.r.nq = nq; c.r.nkv = nkv;
   c.r.d = d; c.r.dv = dv; c.r.rotary_dim = rope != nullptr ? rotary_dim : 0; c.r.qkv_stride = qkv_stride; c.r.q_out_stride = q_out_stride; c.r.eps = eps;
-  c.conv_w = conv_w; c.state = state; c.cu_q = cu_q; c.slots = slots; c.taps = taps; c.values_are_keys = values_are_keys;
+  c.conv_w = conv_w; c.state = state; c.cu_q = cu_q; c.slots = slots; c.n_seqs = n_seqs; c.taps = taps; c.values_are_keys = values_are_keys;
   auto a16 = [](const void* x) { return (uintptr_t)x % 16 == 0; };
   const bool vec = dtype == kBF16 && d % 8 == 0 && dv % 8 == 0 && (rope == nullptr || rotary_dim % 16 == 0) && qkv_stride % 8 == 0 && q_out_stride % 8 == 0 &&
                    a16(qkv) && a16(q_out) && a16(k_cache) && a16(v_cache) && a16(q_weight) && a16(k_weight) && a16(conv_w) && a16(state) && a16(rope);
-  static OncePerDevice once;
-  if (smem > 48 * 1024 && once.first() &&
-      (cudaFuncSetAttribute(conv_rows_norm_kernel<__nv_bfloat16, 8, 4>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMost) != cudaSuccess ||
-       cudaFuncSetAttribute(conv_rows_norm_kernel<__nv_bfloat16, 1, kMostTaps>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMost) != cudaSuccess ||
-       cudaFuncSetAttribute(conv_rows_norm_kernel<float, 1, kMostTaps>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMost) != cudaSuccess)) {
-    once.forget();
-    return fail("conv_rows_norm: cannot reserve %d bytes of shared memory", kMost);
-  }
-#define ILB_CR(T, V, MT) ilb::launch(conv_rows_norm_kernel<T, V, MT>, dim3(n_tokens), dim3(kRowsThreads), smem, stream, (const T*)qkv, (T*)q_out, (T*)k_cache, (T*)v_cache, c)
-  if (vec && taps <= 4) ILB_CR(__nv_bfloat16, 8, 4);
-  else if (dtype == kBF16) ILB_CR(__nv_bfloat16, 1, kMostTaps);
-  else ILB_CR(float, 1, kMostTaps);
+  const int units = width / (vec ? 8 : 1), threads = units >= 512 ? 512 : (units + 31) / 32 * 32;
+  const int blocks = tile == kConvTile ? n_tiles : n_tokens;
+#define ILB_CR(T, V, MT, TT)                                                                                                        \
+  do {                                                                                                                              \
+    static OncePerDevice once;                                                                                                      \
+    if (smem > 48 * 1024 && once.first() &&                                                                                         \
+        cudaFuncSetAttribute(conv_rows_norm_kernel<T, V, MT, TT>, cudaFuncAttributeMaxDynamicSharedMemorySize, kMost) != cudaSuccess) { \
+      once.forget();                                                                                                                \
+      return fail("conv_rows_norm: cannot reserve %d bytes of shared memory", kMost);                                               \
+    }                                                                                                                               \
+    ilb::launch(conv_rows_norm_kernel<T, V, MT, TT>, dim3(blocks), dim3(threads), smem, stream, (const T*)qkv, (T*)q_out, (T*)k_cache, \
+                (T*)v_cache, c);                                                                                                    \
+  } while (0)
+#define ILB_CRT(T, V, MT) do { if (tile == kConvTile) ILB_CR(T, V, MT, kConvTile); else ILB_CR(T, V, MT, 1); } while (0)
+  if (vec && taps <= 4) ILB_CRT(__nv_bfloat16, 8, 4);
+  else if (dtype == kBF16) ILB_CRT(__nv_bfloat16, 1, kMostTaps);
+  else ILB_CRT(float, 1, kMostTaps);
+#undef ILB_CRT
 #undef ILB_CR
   if (int rc = check_launch("conv_rows_norm")) return rc;
-  if (!n_several || taps == 1 || n_seqs == 0) return 0;
+  if (!several || taps == 1 || n_seqs == 0) return 0;
   const dim3 grid((width + 255) / 256, n_seqs);
   if (dtype == kF32) ilb::launch(conv_rows_state_kernel<float>, grid, dim3(256), 0, stream, (const float*)qkv, qkv_stride, width, taps - 1, state, cu_q, slots);
   else ilb::launch(conv_rows_state_kernel<__nv_bfloat16>, grid, dim3(256), 0, stream, (const __nv_bfloat16*)qkv, qkv_stride, width, taps - 1, state, cu_q, slots);
