@@ -865,7 +865,8 @@ ILB_EXPORT int ilb_conv_rows_norm_cache(
   auto a16 = [](const void* x) { return (uintptr_t)x % 16 == 0; };
   const bool vec = dtype == kBF16 && d % 8 == 0 && dv % 8 == 0 && (rope == nullptr || rotary_dim % 16 == 0) && qkv_stride % 8 == 0 && q_out_stride % 8 == 0 &&
                    a16(qkv) && a16(q_out) && a16(k_cache) && a16(v_cache) && a16(q_weight) && a16(k_weight) && a16(conv_w) && a16(state) && a16(rope);
-  const int units = width / (vec ? 8 : 1), threads = units >= 512 ? 512 : (units + 31) / 32 * 32;
+  // (tiles of several tokens: small blocks, of which enough fit a multiprocessor to hide each other's loads)
+  const int units = width / (vec ? 8 : 1), most = tile == kConvTile ? 128 : 512, threads = units >= most ? most : (units + 31) / 32 * 32;
   const int blocks = tile == kConvTile ? n_tiles : n_tokens;
 #define ILB_CR(T, V, MT, TT)                                                                                                        \
   do {                                                                                                                              \
