@@ -122,6 +122,22 @@ def test_prefill_against_token_by_token_and_portions(root, name, dtype):
     assert all(n == g.pool.num_pages for g, n in zip(r.cache.groups, r.cache.free_pages().values()))
 
 
+@pytest.mark.parametrize("page", [32, 64, 128])
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_larger_pages(root, page, dtype):
+    """The tensor-core sizes over pages that chunks end inside of, two requests side by side."""
+    toks = {k: tokens_for(root, "L", dtype, n, 20 + n) for k, n in (("a", 90), ("b", 64))}
+    ref = {k: reference(root, "L", dtype, v) for k, v in toks.items()}
+    r = runner_for(root, "L", dtype, pages=2 * -(-90 // page), page=page)
+    t = Trace()
+    t.step([("a", toks["a"][:57], list(range(57))), ("b", toks["b"][:2], [0, 1])])
+    t.step([("a", toks["a"][57:70], [0, 12]), ("b", toks["b"][2:50], list(range(48)))])
+    for i in range(14):
+        t.step([("a", toks["a"][70 + i:71 + i], [0]), ("b", toks["b"][50 + i:51 + i], [0])], end=["b"] if i == 13 else [])
+    t.step([("a", toks["a"][84:], list(range(6)))], end=["a"])
+    check_trace(run_trace_inprocess(r, t), t, ref, dtype, f"pages of {page}")
+
+
 @pytest.mark.parametrize("name,dtype", ENGINE_CASES)
 def test_mixed_batches_with_pages_and_slots_used_again(root, name, dtype):
     """Up to four live requests of unequal length, portions beside single tokens, four state slots for seven requests and a
